@@ -35,7 +35,7 @@ _SIGNATURES = {
     "b200_qknorm_mrope_kvwrite": [P, L, P, L, P, P, I, P, P, F, P, P, P, I, I, I, I, L, I, I, P, P],
     "b200_quant_fp8_group128": [P, P, P, L, I, I, P],
     "b200_quant_fp8_per_token": [P, L, P, P, L, I, P],
-    "b200_activation": [P, P, L, I, I, I, F, F, P],
+    "b200_activation": [P, P, L, I, I, I, F, F, I, P],
     "b200_rms_norm_gated": [P, P, P, P, L, I, F, I, P],
     "b200_rms_norm_quant_fp8": [P, P, P, P, P, L, I, F, I, L, P],
     "b200_silu_mul_quant_fp8": [P, P, P, L, I, F, P],
@@ -46,7 +46,7 @@ _SIGNATURES = {
     "b200_attn_decode_tc_lse": [P, L, L, P, P, L, I, P, P, P, I, I, I, I, I, F, I, I, I, P, L, P, I, P, P, P, P],
     "b200_merge_attn_partials": [P, P, L, I, I, I, P, L, P, P],
     "b200_attn_decode_set_l2_prefetch": [I],
-    "b200_mla_preprocess": [P, L, I, I, I, I, P, L, I, P, F, P, P, L, P, P, P, L, P, P, P, P],
+    "b200_mla_preprocess": [P, L, I, I, I, I, P, L, I, P, F, P, P, L, P, P, P, L, P, P, I, P, P],
     "b200_argmax": [P, I, L, I, I, P, P],
     "b200_cast_bf16_f32": [P, L, P, L, I, I, P],
     "b200_apply_penalties": [P, L, I, I, P, I, P, I, P, P, P, P],

@@ -8,7 +8,9 @@ setup (setup.py:74-132): ``MAX_JOBS``, ``CMAKE_BUILD_TYPE``.
 """
 from __future__ import annotations
 
+import fcntl
 import hashlib
+import json
 import os
 import subprocess
 import sys
@@ -18,6 +20,7 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OBJ_DIR = os.path.join(HERE, "csrc", "build")
 LIB_PATH = os.path.join(HERE, "_C.so")
+MANIFEST = os.path.join(OBJ_DIR, "linked.json")
 
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 ARCH_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a"]
@@ -48,50 +51,100 @@ def _headers_digest() -> str:
     return h.hexdigest()
 
 
-def _compile_one(src: str, hdr_digest: str, verbose: bool) -> tuple[str, bool]:
+def _object_path(src: str, hdr_digest: str) -> str:
     with open(src, "rb") as fh:
         digest = hashlib.sha256(fh.read() + hdr_digest.encode()).hexdigest()[:16]
+    return os.path.join(OBJ_DIR, f"{os.path.splitext(os.path.basename(src))[0]}.{digest}.o")
+
+
+def _compile_one(src: str, hdr_digest: str, verbose: bool) -> tuple[str, bool]:
     base = os.path.splitext(os.path.basename(src))[0]
-    obj = os.path.join(OBJ_DIR, f"{base}.{digest}.o")
+    obj = _object_path(src, hdr_digest)
     if os.path.exists(obj):
         return obj, False
     for old in os.listdir(OBJ_DIR):
         if old.startswith(base + ".") and old.endswith(".o"):
             os.remove(os.path.join(OBJ_DIR, old))
-    cmd = [NVCC, *ARCH_FLAGS, *_common_flags(), "-x", "cu", "-c", src, "-o", obj]
+    part = f"{obj}.{os.getpid()}.part.o"        # an interrupted compilation leaves no object
+    cmd = [NVCC, *ARCH_FLAGS, *_common_flags(), "-x", "cu", "-c", src, "-o", part]
     if verbose:
         print(" ".join(cmd), flush=True)
     res = subprocess.run(cmd, capture_output=True, text=True)
     if res.returncode != 0:
         raise RuntimeError(f"nvcc failed for {src}:\n{res.stdout}\n{res.stderr}")
+    os.replace(part, obj)
     if res.stderr.strip() and (verbose or os.environ.get("B200_PTXAS_VERBOSE")):
         print(res.stderr, file=sys.stderr)
     return obj, True
 
 
-def build(verbose: bool = False, force: bool = False) -> str:
-    """Compile and link the native library; returns its path."""
+#: sources a model needs, for builds that compile no more than that (architecture -> names; others: all)
+MODEL_SOURCES = {
+    "Vofelix": ("activations", "attention_decode", "attention_mla_decode", "cache_ops", "gemm_bf16", "gemm_bf16_2cta",
+                "latent_attention", "linear_attention", "mla_preprocess", "sampler", "stream_norm"),
+}
+
+
+def _linked() -> list[str]:
+    """Names of the objects in the present library ([]: unknown)."""
+    try:
+        with open(MANIFEST) as fh:
+            return json.load(fh) if os.path.exists(LIB_PATH) else []
+    except (OSError, ValueError):
+        return []
+
+
+def build(verbose: bool = False, force: bool = False, sources=None) -> str:
+    """Compile and link the native library; returns its path.  ``sources`` (names without suffix)
+    limits the compilation to these files: the library then holds them and whatever else has an
+    up-to-date object, and a later call without the limit adds the rest."""
     os.makedirs(OBJ_DIR, exist_ok=True)
+    with open(os.path.join(OBJ_DIR, ".lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return _build_locked(verbose, force, sources)
+
+
+def _build_locked(verbose: bool, force: bool, sources) -> str:
     if force:
         for f in os.listdir(OBJ_DIR):
-            os.remove(os.path.join(OBJ_DIR, f))
+            if f != ".lock":
+                os.remove(os.path.join(OBJ_DIR, f))
     hdr = _headers_digest()
     srcs = _sources()
+    if sources is not None:
+        names = set(sources)
+        known = {os.path.splitext(os.path.basename(s))[0] for s in srcs}
+        if names - known:
+            raise ValueError(f"no such source: {sorted(names - known)}")
+        wanted = [s for s in srcs if os.path.splitext(os.path.basename(s))[0] in names]
+    else:
+        wanted = srcs
     jobs = int(os.environ.get("MAX_JOBS", os.cpu_count() or 4))
     with ThreadPoolExecutor(max_workers=jobs) as ex:
-        results = list(ex.map(lambda s: _compile_one(s, hdr, verbose), srcs))
+        results = list(ex.map(lambda s: _compile_one(s, hdr, verbose), wanted))
     objs = [o for o, _ in results]
-    changed = any(c for _, c in results)
-    if changed or not os.path.exists(LIB_PATH):
-        cmd = [NVCC, *ARCH_FLAGS, "-shared", "-o", LIB_PATH + ".tmp", *objs,
-               "-cudart", "static", "-Xlinker", "--no-undefined", "-lpthread", "-ldl", "-lrt"]
-        if verbose:
-            print(" ".join(cmd), flush=True)
-        res = subprocess.run(cmd, capture_output=True, text=True)
-        if res.returncode != 0:
-            raise RuntimeError(f"link failed:\n{res.stdout}\n{res.stderr}")
-        os.replace(LIB_PATH + ".tmp", LIB_PATH)
+    linked = _linked()
+    if set(map(os.path.basename, objs)) <= set(linked):
+        return LIB_PATH
+    objs += [o for o in (_object_path(s, hdr) for s in srcs if s not in wanted) if os.path.exists(o)]
+    # linked under another name first: a library that is loaded somewhere is replaced, not written over
+    tmp = f"{LIB_PATH}.{os.getpid()}.tmp"
+    cmd = [NVCC, *ARCH_FLAGS, "-shared", "-o", tmp, *objs,
+           "-cudart", "static", "-Xlinker", "--no-undefined", "-lpthread", "-ldl", "-lrt"]
+    if verbose:
+        print(" ".join(cmd), flush=True)
+    res = subprocess.run(cmd, capture_output=True, text=True)
+    if res.returncode != 0:
+        raise RuntimeError(f"link failed:\n{res.stdout}\n{res.stderr}")
+    os.replace(tmp, LIB_PATH)
+    with open(MANIFEST, "w") as fh:
+        json.dump(sorted(map(os.path.basename, objs)), fh)
     return LIB_PATH
+
+
+def ensure(architecture: str) -> str:
+    """Library with everything ``architecture`` needs, compiled from the present sources."""
+    return build(sources=MODEL_SOURCES.get(architecture))
 
 
 if __name__ == "__main__":

@@ -10,10 +10,12 @@ from __future__ import annotations
 
 import json
 import os
-from dataclasses import dataclass, field, asdict
+from dataclasses import dataclass, field, asdict, replace
 from typing import Any, Optional
 
 import torch
+
+from .layer_plan import PLAN_FORMATS
 
 
 @dataclass
@@ -107,6 +109,12 @@ class ModelConfig:
     qk_nope_head_dim: int = 0
     qk_rope_head_dim: int = 0
     v_head_dim: int = 0
+    # ---- decoders described layer by layer (layer_plan.py) ----
+    layer_plan: Optional[list] = None        # per layer {"mixer", "mlp", "over": fields of this layer}
+    layer_loop: Optional[tuple] = None       # (start, stop, times): layers start..stop-1 run times in a row
+    norm_type: str = "rms"                   # "rms" | "layer" (weight and bias)
+    token_side_dim: int = 0                  # per-layer token input: width of a layer's slice of the table
+    attention_sink: bool = False             # a learned logit per head in the softmax denominator
     # ---- numerics / quantization ----
     dtype: str = "bfloat16"
     quantization: Optional[str] = None   # None | "fp8" (128x128 block) | "w8a8_dynamic"
@@ -137,6 +145,10 @@ class ModelConfig:
     @property
     def is_hybrid(self) -> bool:
         return self.full_attention_interval > 0
+
+    def layer_config(self, layer_idx: int) -> "ModelConfig":
+        """The configuration as layer ``layer_idx`` sees it: its own sizes where the model has a plan."""
+        return replace(self, **self.layer_plan[layer_idx]["over"]) if self.layer_plan else self
 
     def is_linear_layer(self, layer_idx: int) -> bool:
         if self.layer_types and layer_idx < len(self.layer_types):
@@ -169,6 +181,8 @@ class ModelConfig:
     # ------------------------------------------------------------------
     @classmethod
     def from_hf_dict(cls, d: dict, **over) -> "ModelConfig":
+        if d.get("architecture") in PLAN_FORMATS:
+            return cls(**{"architecture": d["architecture"], **PLAN_FORMATS[d["architecture"]](d), **over})
         arch = (d.get("architectures") or ["LlamaForCausalLM"])[0]
         top = d
         if "text_config" in d and "hidden_size" not in d:      # nested multimodal layout
@@ -464,6 +478,16 @@ PRESETS: dict[str, Any] = {
         head_dim=32, rope_theta=1e6, qk_norm=True, dtype="float32", full_attention_interval=2,
         linear_num_key_heads=2, linear_num_value_heads=4, linear_key_head_dim=32,
         linear_value_head_dim=32, linear_conv_kernel_dim=4),
+    "tiny-vofelix": lambda: ModelConfig.from_hf_dict({
+        "architecture": "Vofelix", "vocab": 320, "width": 96, "norm": {"eps": 1e-5}, "embedding": {"scale": 8.0},
+        "token_side": {"dim": 16}, "loop": {"start": 1, "stop": 3, "times": 2}, "layers": [
+            {"type": "delta", "mixer": {"heads": 4, "kv_heads": 2, "dim": 16, "vdim": 24, "conv": 3}, "mlp": None},
+            {"type": "latent_attention", "mlp": {"kind": "dense", "ff": 160}, "mixer": {
+                "heads": 4, "dim": 24, "rot_dim": 8, "vdim": 16, "kv_rank": 40, "scale": 0.2, "mask": {"size": 24},
+                "rot": {"base": 10000.0, "dims": 8,
+                        "scaling": {"factor": 2.0, "original": 256, "fast": 16.0, "slow": 1.0}}}},
+            {"type": "delta", "mixer": {"heads": 2, "kv_heads": 2, "dim": 32, "vdim": 32, "conv": 4}, "mlp": None},
+        ]}, dtype="float32", name="tiny-vofelix"),
     "tiny-deepseek": lambda: _preset(
         name="tiny-deepseek", architecture="DeepseekV3ForCausalLM", vocab_size=512,
         hidden_size=128, intermediate_size=256, num_hidden_layers=3, num_attention_heads=4,

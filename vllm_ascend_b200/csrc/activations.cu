@@ -5,7 +5,7 @@
 // The reference routes these through vendor ops and small Triton kernels
 // (vllm_ascend/ops/activation.py:35-86, ops/layernorm.py:110-197).
 #include "common.cuh"
-#include <cuda_bf16.h>
+#include "dtypes.cuh"
 
 namespace b200 {
 
@@ -63,6 +63,30 @@ __global__ void act_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* _
   }
 }
 
+// any width, bf16 or fp32: one element per thread (fp32 activations, widths that are no multiple of 8)
+template <typename T>
+__global__ void act_scalar_kernel(const T* __restrict__ x, T* __restrict__ out, long T_rows, int I, int kind, int gated,
+                                  float alpha, float limit) {
+  const long total = T_rows * I;
+  for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
+    const long row = i / I;
+    const int c = (int)(i - row * I);
+    const T* xr = x + row * (gated ? 2L * I : (long)I);
+    float g = to_f(xr[c]), u = gated ? to_f(xr[I + c]) : 1.f;
+    float r;
+    if (kind == ACT_SWIGLU_OAI) {
+      g = fminf(g, limit);
+      u = fminf(fmaxf(u, -limit), limit);
+      r = g / (1.f + expf(-alpha * g)) * (u + 1.f);
+    } else if (kind == ACT_QUICK_GELU) {
+      r = g / (1.f + expf(-1.702f * g)) * u;
+    } else {
+      r = act_fn(g, kind) * u;
+    }
+    out[i] = from_f<T>(r);
+  }
+}
+
 // one warp per row group of `group` columns (group = H for a plain gated norm, or the per-head
 // size when the norm is applied per head); H % group == 0, group % 8 == 0
 __global__ void rms_norm_gated_kernel(const __nv_bfloat16* __restrict__ x,
@@ -102,14 +126,24 @@ __global__ void rms_norm_gated_kernel(const __nv_bfloat16* __restrict__ x,
 using namespace b200;
 
 B200_API int b200_activation(const void* x, void* out, long T, int I, int kind, int gated, float alpha,
-                             float limit, cudaStream_t stream) {
+                             float limit, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (I & 7) return 9100;
   if (kind < ACT_GELU || kind > ACT_SWIGLU_OAI || (kind == ACT_SWIGLU_OAI && !gated)) return 9600;
-  const long total = T * (I >> 3);
+  const bool scalar = dtype != 0 || (I & 7);
+  const long total = T * (scalar ? I : I >> 3);
   long blocks = (total + 255) / 256;
   const long cap = (long)num_sms() * 16;
   if (blocks > cap) blocks = cap;
+  if (dtype) {
+    act_scalar_kernel<float><<<(unsigned)blocks, 256, 0, stream>>>((const float*)x, (float*)out, T, I, kind, gated,
+                                                                   alpha, limit);
+    return B200_CHECK_LAUNCH();
+  }
+  if (scalar) {
+    act_scalar_kernel<__nv_bfloat16><<<(unsigned)blocks, 256, 0, stream>>>(
+        (const __nv_bfloat16*)x, (__nv_bfloat16*)out, T, I, kind, gated, alpha, limit);
+    return B200_CHECK_LAUNCH();
+  }
   act_kernel<<<(unsigned)blocks, 256, 0, stream>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)out, T, I, kind,
                                                    gated, alpha, limit);
   return B200_CHECK_LAUNCH();

@@ -150,7 +150,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, long q_stride,
 __global__ void merge_splits_kernel(const float* __restrict__ partial_o,
                                     const float* __restrict__ partial_lse, int num_splits, int D,
                                     int Hq, __nv_bfloat16* __restrict__ out, long out_stride,
-                                    float* __restrict__ lse_out) {
+                                    long out_head, float* __restrict__ lse_out) {
   const long t = blockIdx.x;
   const int hq = blockIdx.y;
   const long base = (t * Hq + hq) * num_splits;
@@ -171,17 +171,17 @@ __global__ void merge_splits_kernel(const float* __restrict__ partial_o,
         acc += w * partial_o[(base + s) * D + d];
       }
     }
-    out[t * out_stride + (long)hq * D + d] = __float2bfloat16(L > 0.f ? acc / L : 0.f);
+    out[t * out_stride + hq * out_head + d] = __float2bfloat16(L > 0.f ? acc / L : 0.f);
   }
 }
 
 int launch_merge_splits(const float* partial_o, const float* partial_lse, long T, int Hq,
                         int num_splits, int D, void* out, long out_stride, cudaStream_t stream,
-                        float* lse_out) {
+                        float* lse_out, long out_head) {
   if (T <= 0) return 0;
   dim3 grid((unsigned)T, (unsigned)Hq);
   merge_splits_kernel<<<grid, D >= 128 ? 128 : 64, 0, stream>>>(
-      partial_o, partial_lse, num_splits, D, Hq, (__nv_bfloat16*)out, out_stride, lse_out);
+      partial_o, partial_lse, num_splits, D, Hq, (__nv_bfloat16*)out, out_stride, out_head ? out_head : D, lse_out);
   return B200_CHECK_LAUNCH();
 }
 

@@ -1,0 +1,292 @@
+// Kernels around an fp32 residual stream (decoders that normalise a sub-layer's input and its output):
+//   stream_norm      one pass over a token's row between two sub-layers:
+//                      r  = scale * embed[id]                    (start of the stream), or
+//                      r += norm_post(y) (+ scale * embed[id])   (a sub-layer's output joins; a looped
+//                                                                 stack is fed the embedding again)
+//                      x  = norm_next(r), or r rounded to the activation type
+//   side_gate        g = gelu_tanh(a) * side_embed[id, slice]    (per-layer token input)
+//   gated_head_norm  o = rms_norm(o) * w * silu(z) per head      (delta-rule read-out)
+// Either norm is a layer norm (weight, bias) or an RMS norm, statistics in fp32.  Activations, weights and
+// tables are bf16 or fp32.  The reference fuses add + norm the same way on a 16-bit residual
+// (vllm_ascend/ops/layernorm.py:63-85).
+#include "common.cuh"
+#include "dtypes.cuh"
+
+namespace b200 {
+
+enum : int { NORM_NONE = 0, NORM_LAYER = 1, NORM_RMS = 2, NORM_PLAIN = 3 };
+enum : int { EMB_NONE = 0, EMB_SET = 1, EMB_ADD = 2 };
+
+struct StreamParams {
+  float* r;               // [T, W]
+  const void* y;          // [T, W] sub-layer output (post != NONE)
+  long y_stride;
+  int post;
+  const void *post_w, *post_b;
+  int emb;
+  const long* ids;        // [T]; null: row t of the table
+  const void* table;      // [rows, W]
+  long table_rows;
+  float emb_scale;
+  int next;
+  const void *next_w, *next_b;
+  void* x;                // [T, W]
+  int W;
+  float eps;
+  int* status;
+};
+
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_reduce_sum(v);
+  const int warps = (blockDim.x + 31) >> 5;
+  if (warps == 1) return v;
+  __syncthreads();                     // the previous use of red is over
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = (threadIdx.x & 31) < warps ? red[threadIdx.x & 31] : 0.f;
+  return warp_reduce_sum(t);
+}
+
+template <typename T, int VEC, int PER>
+__device__ __forceinline__ void row_norm(float (&v)[PER][VEC], int kind, const T* w, const T* b, int W, float eps,
+                                         float* red) {
+  const int nvec = W / VEC;
+  float mean = 0.f;
+  if (kind == NORM_LAYER) {
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; i++)
+#pragma unroll
+      for (int e = 0; e < VEC; e++) s += v[i][e];      // slots beyond the row hold zero
+    mean = block_sum(s, red) / (float)W;
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < PER; i++)
+    if ((int)threadIdx.x + i * (int)blockDim.x < nvec)
+#pragma unroll
+      for (int e = 0; e < VEC; e++) {
+        const float d = v[i][e] - mean;
+        ss += d * d;
+      }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
+#pragma unroll
+  for (int i = 0; i < PER; i++) {
+    const int c = (int)threadIdx.x + i * (int)blockDim.x;
+    if (c >= nvec) continue;
+    float wv[VEC], bv[VEC];
+    load_vec<T, VEC>(w + (long)c * VEC, wv);
+#pragma unroll
+    for (int e = 0; e < VEC; e++) bv[e] = 0.f;
+    if (b) load_vec<T, VEC>(b + (long)c * VEC, bv);
+#pragma unroll
+    for (int e = 0; e < VEC; e++) v[i][e] = (v[i][e] - mean) * inv * wv[e] + bv[e];
+  }
+}
+
+template <typename T, int VEC, int PER>
+__global__ void stream_norm_kernel(const StreamParams p) {
+  __shared__ float red[32];
+  const long t = blockIdx.x;
+  const int nvec = p.W / VEC;
+  float v[PER][VEC];
+  float* rrow = p.r + t * p.W;
+  if (p.post != NORM_NONE) {
+    const T* yrow = (const T*)p.y + t * p.y_stride;
+#pragma unroll
+    for (int i = 0; i < PER; i++) {
+      const int c = (int)threadIdx.x + i * (int)blockDim.x;
+      if (c < nvec) load_vec<T, VEC>(yrow + (long)c * VEC, v[i]);
+      else
+#pragma unroll
+        for (int e = 0; e < VEC; e++) v[i][e] = 0.f;
+    }
+    if (p.post != NORM_PLAIN)
+      row_norm<T, VEC, PER>(v, p.post, (const T*)p.post_w, (const T*)p.post_b, p.W, p.eps, red);
+  } else {
+#pragma unroll
+    for (int i = 0; i < PER; i++)
+#pragma unroll
+      for (int e = 0; e < VEC; e++) v[i][e] = 0.f;
+  }
+  const T* erow = nullptr;
+  if (p.emb != EMB_NONE) {
+    const long id = p.ids ? p.ids[t] : t;
+    if (id >= 0 && id < p.table_rows) erow = (const T*)p.table + id * p.W;
+    else if (threadIdx.x == 0 && p.status) atomicCAS(p.status, 0, B200_BAD_INDEX);
+  }
+#pragma unroll
+  for (int i = 0; i < PER; i++) {
+    const int c = (int)threadIdx.x + i * (int)blockDim.x;
+    if (c >= nvec) continue;
+    if (p.emb != EMB_SET) {
+      float rv[VEC];
+      load_vec<float, VEC>(rrow + (long)c * VEC, rv);
+#pragma unroll
+      for (int e = 0; e < VEC; e++) v[i][e] += rv[e];
+    }
+    if (erow) {
+      float ev[VEC];
+      load_vec<T, VEC>(erow + (long)c * VEC, ev);
+#pragma unroll
+      for (int e = 0; e < VEC; e++) v[i][e] += ev[e] * p.emb_scale;
+    }
+    if (p.post != NORM_NONE || p.emb != EMB_NONE) store_vec<float, VEC>(rrow + (long)c * VEC, v[i]);
+  }
+  if (p.next == NORM_NONE) return;
+  if (p.next != NORM_PLAIN)
+    row_norm<T, VEC, PER>(v, p.next, (const T*)p.next_w, (const T*)p.next_b, p.W, p.eps, red);
+  T* xrow = (T*)p.x + t * p.W;
+#pragma unroll
+  for (int i = 0; i < PER; i++) {
+    const int c = (int)threadIdx.x + i * (int)blockDim.x;
+    if (c < nvec) store_vec<T, VEC>(xrow + (long)c * VEC, v[i]);
+  }
+}
+
+// a [T, D] -> out [T, D]; the table row holds one D-wide slice per layer
+template <typename T, int VEC>
+__global__ void side_gate_kernel(const T* __restrict__ a, long a_stride, const long* __restrict__ ids,
+                                 const T* __restrict__ table, long table_stride, long table_rows, long offset,
+                                 T* __restrict__ out, long tokens, int D, int* status) {
+  const int nvec = D / VEC;
+  const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= tokens * nvec) return;
+  const long t = i / nvec;
+  const int c = (int)(i - t * nvec) * VEC;
+  const long id = ids[t];
+  float av[VEC], ev[VEC];
+  load_vec<T, VEC>(a + t * a_stride + c, av);
+  if (id >= 0 && id < table_rows) load_vec<T, VEC>(table + id * table_stride + offset + c, ev);
+  else {
+#pragma unroll
+    for (int e = 0; e < VEC; e++) ev[e] = 0.f;
+    if (c == 0 && status) atomicCAS(status, 0, B200_BAD_INDEX);
+  }
+#pragma unroll
+  for (int e = 0; e < VEC; e++) av[e] = gelu_tanh_f(av[e]) * ev[e];
+  store_vec<T, VEC>(out + t * D + c, av);
+}
+
+// one warp per (token, head): o [T, H, D] dense, z rows with a stride, out dense
+template <typename T, int VEC>
+__global__ void gated_head_norm_kernel(const T* __restrict__ o, const T* __restrict__ z, long z_stride,
+                                       const T* __restrict__ w, T* __restrict__ out, long rows, int H, int D,
+                                       float eps) {
+  const long r = (long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (r >= rows) return;
+  const int lane = threadIdx.x & 31;
+  const long t = r / H;
+  const int h = (int)(r - t * H);
+  const T* orow = o + r * D;
+  const T* zrow = z + t * z_stride + (long)h * D;
+  float ss = 0.f;
+  for (int c = lane * VEC; c < D; c += 32 * VEC) {
+    float v[VEC];
+    load_vec<T, VEC>(orow + c, v);
+#pragma unroll
+    for (int e = 0; e < VEC; e++) ss += v[e] * v[e];
+  }
+  const float inv = 1.f / sqrtf(warp_reduce_sum(ss) / (float)D + eps);
+  for (int c = lane * VEC; c < D; c += 32 * VEC) {
+    float v[VEC], zv[VEC], wv[VEC];
+    load_vec<T, VEC>(orow + c, v);
+    load_vec<T, VEC>(zrow + c, zv);
+    load_vec<T, VEC>(w + c, wv);
+#pragma unroll
+    for (int e = 0; e < VEC; e++) v[e] = v[e] * inv * wv[e] * silu_f<T>(zv[e]);
+    store_vec<T, VEC>(out + r * D + c, v);
+  }
+}
+
+template <typename T, int VEC>
+static int launch_stream(const StreamParams& p, long tokens, cudaStream_t stream) {
+  const int nvec = p.W / VEC;
+  int threads = (((nvec + 1) / 2 + 31) / 32) * 32;
+  if (threads > 1024) threads = 1024;
+  const int per = (nvec + threads - 1) / threads;
+  const dim3 grid((unsigned)tokens);
+  if (per <= 1) stream_norm_kernel<T, VEC, 1><<<grid, threads, 0, stream>>>(p);
+  else if (per <= 2) stream_norm_kernel<T, VEC, 2><<<grid, threads, 0, stream>>>(p);
+  else if (per <= 4) stream_norm_kernel<T, VEC, 4><<<grid, threads, 0, stream>>>(p);
+  else if (per <= 8) stream_norm_kernel<T, VEC, 8><<<grid, threads, 0, stream>>>(p);
+  else return 9710;
+  return B200_CHECK_LAUNCH();
+}
+
+template <typename T>
+static int stream_norm_t(const StreamParams& p, long tokens, cudaStream_t stream) {
+  const bool vec = p.W % 4 == 0 && p.y_stride % 4 == 0 && aligned16(p.r) && aligned16(p.y) && aligned16(p.x) &&
+                   aligned16(p.table) && aligned16(p.post_w) && aligned16(p.post_b) && aligned16(p.next_w) &&
+                   aligned16(p.next_b);
+  return vec ? launch_stream<T, 4>(p, tokens, stream) : launch_stream<T, 1>(p, tokens, stream);
+}
+
+template <typename T>
+static int side_gate_t(const void* a, long a_stride, const void* ids, const void* table, long table_stride,
+                       long table_rows, long offset, void* out, long tokens, int D, int* status, cudaStream_t stream) {
+  const bool vec = D % 4 == 0 && a_stride % 4 == 0 && table_stride % 4 == 0 && offset % 4 == 0 && aligned16(a) &&
+                   aligned16(table) && aligned16(out);
+  const long n = tokens * (D / (vec ? 4 : 1));
+  const unsigned blocks = (unsigned)((n + 255) / 256);
+  if (vec)
+    side_gate_kernel<T, 4><<<blocks, 256, 0, stream>>>((const T*)a, a_stride, (const long*)ids, (const T*)table,
+                                                       table_stride, table_rows, offset, (T*)out, tokens, D, status);
+  else
+    side_gate_kernel<T, 1><<<blocks, 256, 0, stream>>>((const T*)a, a_stride, (const long*)ids, (const T*)table,
+                                                       table_stride, table_rows, offset, (T*)out, tokens, D, status);
+  return B200_CHECK_LAUNCH();
+}
+
+template <typename T>
+static int gated_head_norm_t(const void* o, const void* z, long z_stride, const void* w, void* out, long tokens,
+                             int H, int D, float eps, cudaStream_t stream) {
+  const long rows = tokens * H;
+  const bool vec = D % 4 == 0 && z_stride % 4 == 0 && aligned16(o) && aligned16(z) && aligned16(w) && aligned16(out);
+  const unsigned blocks = (unsigned)((rows + 7) / 8);
+  if (vec)
+    gated_head_norm_kernel<T, 4><<<blocks, 256, 0, stream>>>((const T*)o, (const T*)z, z_stride, (const T*)w,
+                                                             (T*)out, rows, H, D, eps);
+  else
+    gated_head_norm_kernel<T, 1><<<blocks, 256, 0, stream>>>((const T*)o, (const T*)z, z_stride, (const T*)w,
+                                                             (T*)out, rows, H, D, eps);
+  return B200_CHECK_LAUNCH();
+}
+
+}  // namespace b200
+
+using namespace b200;
+
+// dtype: 0 bf16, 1 fp32 (y, x, norm weights, table).  Kinds: 0 none, 1 layer norm, 2 RMS norm, 3 plain
+// (post: add y as it is; next: round r to the activation type).  emb: 0 none, 1 set, 2 add.
+B200_API int b200_stream_norm(void* r, const void* y, long y_stride, int post, const void* post_w, const void* post_b,
+                              int emb, const void* ids, const void* table, long table_rows, float emb_scale, int next,
+                              const void* next_w, const void* next_b, void* x, long tokens, int W, float eps, int dtype,
+                              int* status, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (W < 1 || (post != NORM_NONE && !y) || (next != NORM_NONE && !x) || (emb != EMB_NONE && !table)) return 9700;
+  if ((post == NORM_LAYER || post == NORM_RMS) && !post_w) return 9701;
+  if ((next == NORM_LAYER || next == NORM_RMS) && !next_w) return 9702;
+  StreamParams p{(float*)r, y, y_stride, post, post_w, post_b, emb, (const long*)ids, table, table_rows, emb_scale,
+                 next, next_w, next_b, x, W, eps, status};
+  return dtype ? stream_norm_t<float>(p, tokens, stream) : stream_norm_t<__nv_bfloat16>(p, tokens, stream);
+}
+
+B200_API int b200_side_gate(const void* a, long a_stride, const void* ids, const void* table, long table_stride,
+                            long table_rows, long offset, void* out, long tokens, int D, int dtype, int* status,
+                            cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (D < 1 || offset < 0 || offset + D > table_stride) return 9720;
+  return dtype ? side_gate_t<float>(a, a_stride, ids, table, table_stride, table_rows, offset, out, tokens, D, status,
+                                    stream)
+               : side_gate_t<__nv_bfloat16>(a, a_stride, ids, table, table_stride, table_rows, offset, out, tokens, D,
+                                            status, stream);
+}
+
+B200_API int b200_gated_head_norm(const void* o, const void* z, long z_stride, const void* w, void* out, long tokens,
+                                  int H, int D, float eps, int dtype, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (H < 1 || D < 1) return 9730;
+  return dtype ? gated_head_norm_t<float>(o, z, z_stride, w, out, tokens, H, D, eps, stream)
+               : gated_head_norm_t<__nv_bfloat16>(o, z, z_stride, w, out, tokens, H, D, eps, stream);
+}

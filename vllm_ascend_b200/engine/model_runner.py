@@ -181,7 +181,9 @@ class ModelRunner:
         self.loaded_from_peer = bool(loader is not None and loader.load(self.model))
         if self.mcfg.model_path and not self.loaded_from_peer:
             from ..models.transformer import iterate_safetensors
-            self.model.load_weights(iterate_safetensors(self.mcfg.model_path))
+            loaded = self.model.load_weights(iterate_safetensors(self.mcfg.model_path))
+            if hasattr(self.model, "check_loaded"):
+                self.model.check_loaded(loaded)
         self.load_time = time.time() - t0
         if self.mcfg.is_multimodal and self.model.is_first:
             from .mm_runner import MultimodalState
@@ -215,15 +217,17 @@ class ModelRunner:
                 n_s = 1
                 for d in ss:
                     n_s *= d
-                total += n_c * 2 + n_s * 4
+                total += n_c * (4 if self.kv_dtype == torch.float32 else 2) + n_s * 4
         return total
 
     def kv_bytes_per_block(self) -> int:
-        m = self.model
-        n_layers = self._num_kv_layers()
         itemsize = torch.tensor([], dtype=self.kv_dtype).element_size()
-        per_tok = sum(self._cache_widths()) * itemsize
-        return n_layers * self.block_size * per_tok
+        if self.mcfg.layer_plan:             # every layer has sizes of its own
+            per_tok = sum(L.self_attn.dc + L.self_attn.dr for L in self.model.layers
+                          if not getattr(L.self_attn, "is_linear_attention", False))
+        else:
+            per_tok = self._num_kv_layers() * sum(self._cache_widths())
+        return self.block_size * per_tok * itemsize
 
     @property
     def kv_dtype(self) -> torch.dtype:
@@ -258,7 +262,7 @@ class ModelRunner:
         free, total = torch.cuda.mem_get_info(self.device)
         budget = total * cc.gpu_memory_utilization - (total - free) - self.activation_bytes_estimate() \
             - self.state_bytes()
-        n = int(budget // self.kv_bytes_per_block())
+        n = int(budget // max(self.kv_bytes_per_block(), 1))      # a purely recurrent model pages nothing
         if n < 8:
             raise RuntimeError(f"not enough memory for the KV cache ({budget / 2**30:.1f} GiB left)")
         # a block beyond what max_num_seqs full-length sequences can use is wasted
@@ -278,8 +282,8 @@ class ModelRunner:
                 continue
             if c.use_mla:
                 nb_main = 1 if self._offload_cfg().enabled else num_blocks      # host-resident: placeholders
-                shapes = [(nb_main, self.block_size, 1, c.kv_lora_rank),
-                          (nb_main, self.block_size, 1, c.qk_rope_head_dim)]
+                a = layer.self_attn
+                shapes = [(nb_main, self.block_size, 1, a.dc), (nb_main, self.block_size, 1, a.dr)]
                 if c.use_sparse:          # index keys of the lightning indexer
                     shapes.append((num_blocks, self.block_size, 1, c.index_head_dim))
             else:
@@ -740,6 +744,34 @@ class ModelRunner:
             out[r.request_id] = [t]
         return out
 
+    def append_tokens(self, req: Request, tokens) -> None:
+        """Known next tokens of a request that already owns a batch row (its prompt grows)."""
+        at = req.num_computed_tokens
+        self.token_ids_cpu[req.row, at:at + len(tokens)] = tokens
+
+    @torch.inference_mode()
+    def execute_logits(self, so: SchedulerOutput, rows: list) -> Optional[torch.Tensor]:
+        """One step that samples nothing: the logits (fp32, on the host) at the given token rows of the
+        batch (``so.scheduled`` order).  Decode-only batches replay their graph, as in ``execute``."""
+        self.stats["steps"] += 1
+        self._sync_rows(so)
+        gsize = self._graph_size_for(len(so.scheduled)) if all(n == 1 for _, n in so.scheduled) else None
+        meta, T, Tp, _, _ = self._prepare_inputs(so, pad_to=gsize)
+        if gsize is not None:
+            hidden = self.graph_wrapper.replay(self.graphs[(gsize, False)])
+            self.stats["graph_replays"] += 1
+        else:
+            hidden = self._forward(Tp, meta)
+            self.stats["eager_steps"] += 1
+        out = []
+        for a in range(0, len(rows), 1024):            # bounded logits footprint
+            idx = torch.tensor(rows[a:a + 1024], dtype=torch.int64, device=self.device)
+            out.append(self.model.compute_logits(hidden[idx]).float().cpu())
+        if self.is_cuda:
+            torch.cuda.current_stream().synchronize()
+            _native.check_status(self.device)
+        return torch.cat(out) if out else None
+
     def _sample_pcp(self, hidden: torch.Tensor, sel: list, sample_reqs: list) -> dict:
         """Split prefill step: PCP rank 0 holds the last token of every chunk, samples, and sends
         the token ids to the other ranks of the group."""
@@ -1178,6 +1210,11 @@ class ModelRunner:
                     worst = max(worst, s * a.Hq * ns * (a.D + 1) * 4)
             if worst:
                 ops.reserve_attention_scratch(self.device, worst)
+        else:
+            from ..attention.mla import reserve_mla_scratch
+            for a in {id(L.self_attn): L.self_attn for L in self.model.layers}.values():
+                if not getattr(a, "is_linear_attention", False):
+                    reserve_mla_scratch(self.device, self.capture_sizes[-1], a.H, a.dc)
         from ..compilation.cuda_graph import BatchDescriptor, CUDAGraphWrapper, global_graph_pool
         self.graph_pool = global_graph_pool()
 

@@ -317,6 +317,35 @@ class Scheduler:
             out.kv_connector_metadata = self.kv_connector.build_connector_meta(out)
         return out
 
+    def schedule_portions(self, portions: list) -> SchedulerOutput:
+        """A step whose batch is given by the caller: ``portions`` = [(request, number of its next tokens)].
+        A request not seen before takes a batch row (and with it a state slot); every request gets the
+        blocks its tokens need.  Raises when the pool or the rows do not suffice."""
+        self.step_id += 1
+        out = SchedulerOutput(scheduled=[], step_id=self.step_id)
+        out.finished_ids, self.finished_since_last = self.finished_since_last, []
+        decodes, prefills = [], []
+        for req, n in portions:
+            if req.num_computed_tokens + n > self.cfg.max_model_len:
+                raise ValueError(f"request {req.request_id} grows past max_model_len {self.cfg.max_model_len}")
+            if req.row < 0:
+                if not self._free_rows:
+                    raise RuntimeError(f"no free batch row for request {req.request_id}")
+                req.row = self._free_rows.pop()
+                req.status = RequestStatus.RUNNING
+                self.requests[req.request_id] = req
+                self.running.append(req)
+                out.new_block_rows.append(req)
+            need = self._blocks_needed(req, req.num_computed_tokens + n)
+            if need:
+                req.block_ids.extend(self.pool.allocate(need))
+                if req not in out.new_block_rows:
+                    out.new_block_rows.append(req)
+            (decodes if n == 1 and req.num_computed_tokens > 0 else prefills).append((req, n))
+        out.scheduled = decodes + prefills
+        out.num_scheduled_tokens = sum(n for _, n in out.scheduled)
+        return out
+
     # ------------------------------------------------------------------ results
     def advance(self, out: SchedulerOutput) -> None:
         """Asynchronous scheduling: account for a step at launch time instead of at completion.

@@ -28,6 +28,14 @@ for _arch in ("LlamaForCausalLM", "MistralForCausalLM", "Qwen2ForCausalLM", "Qwe
     register_model(_arch, _causal_lm)
 
 
+def _planned_lm(cfg, device, **kw):
+    from .planned import PlannedCausalLM
+    return PlannedCausalLM(cfg, device, **kw)
+
+
+register_model("Vofelix", _planned_lm)
+
+
 def _qwen_vl(cfg, device, **kw):
     from .qwen_vl import QwenVLForConditionalGeneration
     return QwenVLForConditionalGeneration(cfg, device, **kw)

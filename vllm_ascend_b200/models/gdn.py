@@ -1,4 +1,4 @@
-"""Gated DeltaNet linear-attention layer (the recurrent layers of Qwen3-Next style hybrids).
+"""Gated DeltaNet linear-attention layer (the recurrent layers of Qwen3-Next style hybrids and of Vofelix).
 
 Per token: projections to q, k, v, an output gate z and two per-head scalars (b -> write
 strength beta, a -> decay g); a short causal convolution + SiLU over [q | k | v]; the gated
@@ -11,12 +11,11 @@ interleaved per-group layout are re-ordered at load time).
 from __future__ import annotations
 
 import torch
-import torch.nn.functional as F
 
-from .. import ops
 from ..config import ModelConfig
 from ..ops import linear_attn as la
-from .layers import ColumnParallelLinear, ParamFactory, RowParallelLinear, TPComm
+from ..ops.stream import gated_head_norm
+from .layers import ColumnParallelLinear, ParamFactory, RowParallelLinear, TPComm, copy_exact
 
 
 class GatedDeltaNet:
@@ -59,17 +58,48 @@ class GatedDeltaNet:
         mixed = qkvz[:, :2 * kd + vd]
         z = qkvz[:, 2 * kd + vd:]
         cu, slots, has_init = meta.query_start_loc, meta.state_slots, meta.has_initial_state
-        mixed = la.causal_conv1d(mixed, self.conv_weight, None, conv_state, cu, slots, has_init, act=True)
-        q = mixed[:, :kd].reshape(T, self.Hk, self.Dk)
-        k = mixed[:, kd:2 * kd].reshape(T, self.Hk, self.Dk)
-        v = mixed[:, 2 * kd:].reshape(T, self.Hv, self.Dv)
-        beta = torch.sigmoid(ba[:, :self.Hv].float())
-        g = -torch.exp(self.A_log) * F.softplus(ba[:, self.Hv:].float() + self.dt_bias)
+        uniform = meta.max_query_len <= 1
+        # one launch: convolution + SiLU of [q | k | v], write strength and log-decay of every head
+        mixed, beta, g = la.causal_conv1d(mixed, self.conv_weight, None, conv_state, cu, slots, has_init, act=True,
+                                          uniform=uniform, gates=(ba, self.A_log, self.dt_bias))
+        q = mixed[:, :kd].view(T, self.Hk, self.Dk)
+        k = mixed[:, kd:2 * kd].view(T, self.Hk, self.Dk)
+        v = mixed[:, 2 * kd:].view(T, self.Hv, self.Dv)
         o = la.gated_delta_rule(q, k, v, g, beta, ssm_state, cu, slots, has_init, self.scale, l2norm=True,
-                                cu_cpu=None if meta.max_query_len <= 1 else meta.query_start_loc_cpu)
-        o = ops.rms_norm_gated(o.reshape(T, vd), z.contiguous(), self.norm_weight, self.cfg.rms_norm_eps,
-                               group=self.Dv, norm_before_gate=True)
-        return self.out_proj(o)
+                                cu_cpu=None if uniform else meta.query_start_loc_cpu)
+        return self.out_proj(gated_head_norm(o, z, self.norm_weight, self.cfg.rms_norm_eps))
+
+    # parts of the fused projections, in row order: (name, key or value heads)
+    _QKVZ = (("q", "k"), ("k", "k"), ("v", "v"), ("g", "v"))
+
+    def load_part(self, part: str, w: torch.Tensor) -> None:
+        """One un-fused tensor: the projections q, k, v, g (output gate), b (write strength), a (decay), o, the
+        convolutions q.conv, k.conv, v.conv, and A_log, dt_bias, norm."""
+        tp, r = self.out_proj.comm.size, self.out_proj.comm.rank
+        sizes = {"k": self.key_dim, "v": self.value_dim}
+        if part == "o":
+            n = w.shape[1] // tp
+            return copy_exact(self.out_proj.weight, w[:, r * n:(r + 1) * n], part)
+        if part == "norm":
+            return copy_exact(self.norm_weight, w, part)
+        rows = w[r * w.shape[0] // tp:(r + 1) * w.shape[0] // tp]
+        if part in ("A_log", "dt_bias"):
+            return copy_exact(getattr(self, part), rows, part)
+        if part in ("b", "a"):
+            at = 0 if part == "b" else self.Hv
+            return copy_exact(self.in_proj_ba.weight[at:at + self.Hv], rows, part)
+        name, _, conv = part.partition(".")
+        at = 0
+        for p, kind in self._QKVZ:
+            if p == name and conv in ("", "conv") and not (conv and p == "g"):
+                dst = self.conv_weight if conv else self.in_proj_qkvz.weight
+                return copy_exact(dst[at:at + sizes[kind]], rows, part)
+            at += sizes[kind]
+        raise KeyError(part)
+
+    @staticmethod
+    def parts() -> list[str]:
+        return ["q", "k", "v", "g", "b", "a", "o", "q.conv", "k.conv", "v.conv", "A_log", "dt_bias", "norm"]
 
     def load_hf(self, suffix: str, w: torch.Tensor, tp: int, r: int) -> bool:
         """One tensor of a published checkpoint (name relative to ``linear_attn.``).  The checkpoint

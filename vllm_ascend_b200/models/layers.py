@@ -56,6 +56,13 @@ class ParamFactory:
         return torch.zeros(shape, dtype=dtype or self.dtype, device=self.device)
 
 
+def copy_exact(dst: torch.Tensor, src: torch.Tensor, name: str) -> None:
+    """Copy a checkpoint tensor into its place; the shapes must agree (no broadcasting)."""
+    if tuple(dst.shape) != tuple(src.shape):
+        raise ValueError(f"tensor {name}: expected shape {tuple(dst.shape)}, found {tuple(src.shape)}")
+    dst.copy_(src)
+
+
 # ---------------------------------------------------------------- TP communication
 class TPComm:
     """Collective that follows a row-parallel GEMM / precedes a column-parallel one.

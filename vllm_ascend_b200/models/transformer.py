@@ -20,7 +20,7 @@ from ..ops import fused_moe, reference as ref
 from ..parallel import state as pstate
 from .layers import (ColumnParallelLinear, GQAAttention, Linear, ParallelLMHead, ParamFactory,
                      RMSNorm, RowParallelLinear, SwiGLUMLP, TPComm, VocabParallelEmbedding,
-                     get_cos_sin_cache)
+                     copy_exact, get_cos_sin_cache)
 
 
 # ---------------------------------------------------------------- MoE block
@@ -176,7 +176,8 @@ class MLAAttention:
     (qk_rope_head_dim), in two paged tensors.  Scores are
     q_nope·W_UK·latent + q_pe·k_pe; the value path is latent·W_UV — i.e. MQA over a
     576-wide key with the up-projections folded into q and the output
-    (``W_UK_T`` / ``W_UV`` of mla_v1.py:907-971).
+    (``W_UK_T`` / ``W_UV`` of mla_v1.py:907-971).  Options: a sliding window (``sliding_window``), a
+    learned sink per head (``attention_sink``), a score scale of its own (``attention_multiplier``).
     """
 
     def __init__(self, pf: ParamFactory, cfg: ModelConfig, layer_idx: int, comm: TPComm,
@@ -211,9 +212,16 @@ class MLAAttention:
             import math
             m = 0.1 * sc["mscale_all_dim"] * math.log(sc.get("factor", 1.0)) + 1.0
             self.scale *= m * m
-        self.cos_sin = get_cos_sin_cache(self.dr, max_pos, cfg.rope_theta,
-                                         dict(sc, rope_type="deepseek_yarn") if sc else None,
-                                         pf.device)
+        if cfg.attention_multiplier is not None:
+            self.scale = float(cfg.attention_multiplier)
+        if sc and sc.get("rope_type") != "yarn_interp":
+            sc = dict(sc, rope_type="deepseek_yarn")
+        self.cos_sin = get_cos_sin_cache(self.dr, max_pos, cfg.rope_theta, sc or None, pf.device)
+        self.window = int(cfg.sliding_window or 0)
+        self.sink = pf.normal(f"{p}.sink", (cfg.num_attention_heads,), 0, comm.rank, tp, std=1.0,
+                              dtype=torch.float32) if cfg.attention_sink else None
+        if pstate.get_dcp_group().world_size > 1 and (self.window or self.sink is not None):
+            raise NotImplementedError("decode context parallelism does not serve latent attention with a window or sink")
         # lightning indexer (sparse attention): a few small heads score every cached key per query and
         # attention runs over the index_topk best; weights are replicated over TP (every rank needs
         # the full selection).  Names follow the published checkpoints (self_attn.indexer.*).
@@ -279,9 +287,38 @@ class MLAAttention:
             o_lat = mla_attention_dcp(q_lat, q_pe, lat_cache, pe_cache, meta, self.scale, dcp,
                                       getattr(meta, "dcp_interleave", 1))
         else:
-            o_lat = mla_ops.mla_paged_attention(q_lat, q_pe, lat_cache, pe_cache, meta, self.scale)
+            # head-major result: the rows of the per-head value product
+            o_lat = torch.empty((self.H, T, self.dc), dtype=q_lat.dtype, device=q_lat.device).transpose(0, 1)
+            mla_ops.mla_paged_attention(q_lat, q_pe, lat_cache, pe_cache, meta, self.scale, window=self.window,
+                                        sink=self.sink, out=o_lat)
         o = self._per_head_matmul(o_lat, self.W_UV, self.W_UV_nk)
         return self.o_proj(o.reshape(T, self.H * self.dv))
+
+    def load_part(self, part: str, w: torch.Tensor) -> None:
+        """One un-fused tensor: q, dkv (joint down-projection), dkv.norm, uk / uv (key and value
+        up-projections, head by head), sink, o."""
+        tp, r = self.o_proj.comm.size, self.o_proj.comm.rank
+        if part == "dkv":
+            return copy_exact(self.kv_a_proj.weight, w, part)
+        if part == "dkv.norm":
+            return copy_exact(self.kv_a_norm.weight, w, part)
+        if part == "o":
+            n = w.shape[1] // tp
+            return copy_exact(self.o_proj.weight, w[:, r * n:(r + 1) * n], part)
+        rows = w[r * w.shape[0] // tp:(r + 1) * w.shape[0] // tp]
+        if part == "q":
+            return copy_exact(self.q_proj.weight, rows, part)
+        if part == "sink" and self.sink is not None:
+            return copy_exact(self.sink, rows, part)
+        if part in ("uk", "uv"):
+            kv_b = self.kv_b_proj.weight.view(self.H, self.dn + self.dv, self.dc)
+            n = self.dn if part == "uk" else self.dv
+            copy_exact(kv_b[:, :self.dn] if part == "uk" else kv_b[:, self.dn:], rows.reshape(-1, n, w.shape[1]), part)
+            return None
+        raise KeyError(part)
+
+    def parts(self) -> list[str]:
+        return ["q", "dkv", "dkv.norm", "uk", "uv", "o"] + (["sink"] if self.sink is not None else [])
 
     def _per_head_matmul(self, x: torch.Tensor, w_kn: torch.Tensor, w_nk: torch.Tensor) -> torch.Tensor:
         """x [T, H, K] times one [K, N] matrix per head -> [T, H, N] (the two weight absorptions of MLA:

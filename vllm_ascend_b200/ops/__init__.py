@@ -530,10 +530,10 @@ def mla_preprocess(q: torch.Tensor, kv: torch.Tensor, norm_w: torch.Tensor, eps:
     Returns (latent [T, dc], k_pe [T, dr]) when ``want_outputs`` else None."""
     T, H, D = q.shape
     dc = kv.shape[1] - dr
-    native = (_use_native(q) and kv.dtype == _BF16 and q.stride(2) == 1 and q.stride(1) == D and kv.stride(1) == 1
-              and cos_sin.dtype == torch.float32 and cos_sin.shape[1] == dr and dn % 2 == 0 and dr % 2 == 0
-              and q.stride(0) % 2 == 0
-              and (lat_cache is None or (lat_cache.dtype == _BF16 and lat_cache.is_contiguous()
+    native = (q.is_cuda and q.dtype in (_BF16, torch.float32) and kv.dtype == q.dtype == norm_w.dtype
+              and q.stride(2) == 1 and q.stride(1) == D and kv.stride(1) == 1
+              and cos_sin.dtype == torch.float32 and cos_sin.shape[1] == dr and dr % 2 == 0
+              and (lat_cache is None or (lat_cache.dtype == q.dtype and lat_cache.is_contiguous()
                                          and pe_cache.is_contiguous())))
     if not native:
         latent = ref.rms_norm(kv[:, :dc].contiguous(), norm_w, eps)[0]
@@ -554,7 +554,7 @@ def mla_preprocess(q: torch.Tensor, kv: torch.Tensor, norm_w: torch.Tensor, eps:
         q.data_ptr(), q.stride(0), T, H, dn, dr, kv.data_ptr(), kv.stride(0), dc, norm_w.data_ptr(), float(eps),
         positions.data_ptr(), cos_sin.data_ptr(), cos_sin.shape[0], _native.ptr(slot_mapping) if use_slots else None,
         _native.ptr(lat_cache), _native.ptr(pe_cache), num_slots, _native.ptr(latent), _native.ptr(k_pe),
-        _native.status_word(q.device).data_ptr(), _native.stream_ptr())
+        int(q.dtype == torch.float32), _native.status_word(q.device).data_ptr(), _native.stream_ptr())
     _native.check(rc, "mla_preprocess")
     launch_counter[0] += 1
     return (latent, k_pe) if want_outputs else None
@@ -703,12 +703,12 @@ _ACT_KINDS = {"gelu": 1, "gelu_tanh": 2, "quick_gelu": 3, "swiglu_oai": 4}
 def activation(x: torch.Tensor, kind: str, gated: bool = False, alpha: float = 1.702, limit: float = 7.0):
     """GELU (erf / tanh), QuickGELU, and the clamped "swiglu-oai" gate; ``gated`` inputs are [gate | up]."""
     I = x.shape[-1] // 2 if gated else x.shape[-1]
-    if not _use_native(x) or I % 8 or not x.is_contiguous():
+    if not x.is_cuda or x.dtype not in (_BF16, torch.float32) or not x.is_contiguous():
         return ref.activation(x, kind, gated, alpha, limit)
     x2 = x.view(-1, x.shape[-1])
     out = torch.empty((x2.shape[0], I), dtype=x.dtype, device=x.device)
     rc = _native.lib().b200_activation(x2.data_ptr(), out.data_ptr(), x2.shape[0], I, _ACT_KINDS[kind], int(gated),
-                                       alpha, limit, _native.stream_ptr())
+                                       alpha, limit, int(x.dtype == torch.float32), _native.stream_ptr())
     _native.check(rc, "activation")
     launch_counter[0] += 1
     return out.view(*x.shape[:-1], I)

@@ -12,9 +12,11 @@ import torch.nn.functional as F
 from .. import _native
 
 P, I, L, Fl = c_void_p, c_int, c_long, c_float
-_native.register_signature("b200_causal_conv1d", [P, L, P, P, P, P, P, P, P, L, I, I, I, I, L, P, P])
+_native.register_signature("b200_causal_conv1d", [P, L, P, P, P, P, P, P, P, L, L, I, I, I, I, I, L, I, P, L, P, P, I, P, P,
+                                                  P, P])
 _native.register_signature("b200_gated_delta_rule", [P, P, P, L, L, P, P, P, P, P, P, P, L, I, I, I, I, I, Fl, I,
-                                                     L, P, P])
+                                                     L, I, P, P])
+_DTYPES = {torch.bfloat16: 0, torch.float32: 1}
 
 
 def causal_conv1d_ref(x, weight, bias, state, cu, slots, has_init, act=True):
@@ -32,22 +34,43 @@ def causal_conv1d_ref(x, weight, bias, state, cu, slots, has_init, act=True):
         if bias is not None:
             out = out + bias.float()
         y[t0:t1] = (F.silu(out) if act else out).to(x.dtype)
-        state[s] = seq[-(K - 1):].to(state.dtype)
+        state[s] = seq[seq.shape[0] - (K - 1):].to(state.dtype)
     return y
 
 
-def causal_conv1d(x, weight, bias, state, cu, slots, has_init, act=True):
-    if not (x.is_cuda and x.dtype == torch.bfloat16):
-        return causal_conv1d_ref(x, weight, bias, state, cu, slots, has_init, act)
+def delta_gates_ref(ba, A_log, dt_bias):
+    """ba [T, 2H] = raw write strength, raw decay input -> (beta, log-decay) fp32 [T, H]."""
+    H = A_log.shape[0]
+    return torch.sigmoid(ba[:, :H].float()), -torch.exp(A_log) * F.softplus(ba[:, H:].float() + dt_bias)
+
+
+def causal_conv1d(x, weight, bias, state, cu, slots, has_init, act=True, uniform=False, gates=None):
+    """``uniform``: every sequence of the step has exactly one token.  ``gates`` = (ba [T, 2H], A_log [H],
+    dt_bias [H]) adds the two scalars of the gated delta rule to the same launch: the result is then
+    (y, beta, log-decay)."""
+    if not x.is_cuda:
+        y = causal_conv1d_ref(x, weight, bias, state, cu, slots, has_init, act)
+        return y if gates is None else (y, *delta_gates_ref(*gates))
+    if x.dtype not in _DTYPES or weight.dtype != x.dtype or state.dtype != x.dtype or x.stride(1) != 1:
+        raise TypeError("causal_conv1d takes bf16 or fp32 rows with weights and state of the same type")
     T, C = x.shape
     y = torch.empty((T, C), dtype=x.dtype, device=x.device)
+    H, beta, g, ba, A_log, dt_bias = 0, None, None, None, None, None
+    if gates is not None:
+        ba, A_log, dt_bias = gates
+        H = A_log.shape[0]
+        if ba.dtype != x.dtype or ba.stride(1) != 1 or A_log.dtype != torch.float32 or dt_bias.dtype != torch.float32:
+            raise TypeError("delta-rule gates: rows of the activations' type, fp32 A_log and dt_bias")
+        beta, g = torch.empty((2, T, H), dtype=torch.float32, device=x.device).unbind(0)
     rc = _native.lib().b200_causal_conv1d(
         x.data_ptr(), x.stride(0), weight.data_ptr(), _native.ptr(bias), state.data_ptr(), cu.data_ptr(),
-        slots.data_ptr(), has_init.data_ptr(), y.data_ptr(), y.stride(0), cu.numel() - 1, C, weight.shape[1],
-        int(act), state.shape[0], _native.status_word(x.device).data_ptr(), _native.stream_ptr())
+        slots.data_ptr(), has_init.data_ptr(), y.data_ptr(), y.stride(0), T, cu.numel() - 1, C, weight.shape[1],
+        int(act), int(uniform and T == cu.numel() - 1), state.shape[0], _DTYPES[x.dtype], _native.ptr(ba),
+        0 if ba is None else ba.stride(0), _native.ptr(A_log), _native.ptr(dt_bias), H, _native.ptr(beta),
+        _native.ptr(g), _native.status_word(x.device).data_ptr(), _native.stream_ptr())
     _native.check(rc, "causal_conv1d")
     _native.count_launch()
-    return y
+    return y if gates is None else (y, beta, g)
 
 
 def gated_delta_rule_ref(q, k, v, g, beta, state, cu, slots, has_init, scale, l2norm=True):
@@ -210,18 +233,20 @@ def gated_delta_rule(q, k, v, g, beta, state, cu, slots, has_init, scale, l2norm
                                                g[rows_t], beta[rows_t], state, cu_s, slots[sel].contiguous(),
                                                has_init[sel].contiguous(), scale, l2norm)
             return out
-    if not (q.is_cuda and q.dtype == torch.bfloat16):
+    if not q.is_cuda:
         return gated_delta_rule_ref(q, k, v, g, beta, state, cu, slots, has_init, scale, l2norm)
     T, Hv, DV = v.shape
     Hk, DK = q.shape[1], q.shape[2]
-    assert q.stride(0) == k.stride(0) and q.stride(2) == 1 and q.stride(1) == DK and v.stride(1) == DV
+    if q.dtype not in _DTYPES or k.dtype != q.dtype or v.dtype != q.dtype or state.dtype != torch.float32:
+        raise TypeError("gated_delta_rule takes bf16 or fp32 q, k, v of one type and an fp32 state")
+    assert v.stride(2) == 1 and q.stride(0) == k.stride(0) and q.stride(2) == 1 and q.stride(1) == DK and v.stride(1) == DV
     out = torch.empty((T, Hv, DV), dtype=v.dtype, device=v.device)
     g = g.float().contiguous()
     beta = beta.float().contiguous()
     rc = _native.lib().b200_gated_delta_rule(
         q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), v.stride(0), g.data_ptr(), beta.data_ptr(),
         state.data_ptr(), cu.data_ptr(), slots.data_ptr(), has_init.data_ptr(), out.data_ptr(), out.stride(0),
-        cu.numel() - 1, Hk, Hv, DK, DV, scale, int(l2norm), state.shape[0],
+        cu.numel() - 1, Hk, Hv, DK, DV, scale, int(l2norm), state.shape[0], _DTYPES[q.dtype],
         _native.status_word(q.device).data_ptr(), _native.stream_ptr())
     _native.check(rc, "gated_delta_rule")
     _native.count_launch()

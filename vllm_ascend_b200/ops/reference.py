@@ -64,7 +64,7 @@ def build_cos_sin_cache(rot_dim: int, max_pos: int, theta: float,
         factor = float(rope_scaling.get("factor", 1.0))
         if kind == "linear":
             inv_freq = inv_freq / factor
-        elif kind in ("yarn", "deepseek_yarn"):
+        elif kind in ("yarn", "deepseek_yarn", "yarn_interp"):
             orig = rope_scaling.get("original_max_position_embeddings", max_pos)
             beta_fast = rope_scaling.get("beta_fast", 32)
             beta_slow = rope_scaling.get("beta_slow", 1)
@@ -74,7 +74,9 @@ def build_cos_sin_cache(rot_dim: int, max_pos: int, theta: float,
 
             low = max(math.floor(corr_dim(beta_fast)), 0)
             high = min(math.ceil(corr_dim(beta_slow)), rot_dim - 1)
-            if low == high:
+            if kind == "yarn_interp":
+                high = low + max(high - low, 0.001)
+            elif low == high:
                 high += 0.001
             ramp = ((torch.arange(half, dtype=torch.float64) - low) / (high - low)).clamp(0, 1)
             mask = 1 - ramp
@@ -88,6 +90,8 @@ def build_cos_sin_cache(rot_dim: int, max_pos: int, theta: float,
                           yarn_mscale(factor, rope_scaling.get("mscale_all_dim", 0.0) or 1.0)
                           if rope_scaling.get("mscale_all_dim") else
                           yarn_mscale(factor, rope_scaling.get("mscale", 1.0)))
+            elif kind == "yarn_interp":         # the factor on cos and sin, without a floor at 1
+                mscale = 0.1 * math.log(factor) + 1.0
             else:
                 mscale = yarn_mscale(factor)
         elif kind == "llama3":
