@@ -47,7 +47,7 @@ def _headers_digest() -> str:
         if f.endswith((".cuh", ".h", ".hpp")):
             with open(os.path.join(CSRC, f), "rb") as fh:
                 h.update(fh.read())
-    h.update(" ".join(_common_flags()).encode())
+    h.update(" ".join(f for f in _common_flags() if f != CSRC).encode())      # the same wherever the tree lies
     return h.hexdigest()
 
 
@@ -96,8 +96,8 @@ def _linked() -> list[str]:
 
 def build(verbose: bool = False, force: bool = False, sources=None) -> str:
     """Compile and link the native library; returns its path.  ``sources`` (names without suffix)
-    limits the compilation to these files: the library then holds them and whatever else has an
-    up-to-date object, and a later call without the limit adds the rest."""
+    limits the compilation to these files and what a present library holds already; a later call
+    without the limit adds the rest."""
     os.makedirs(OBJ_DIR, exist_ok=True)
     with open(os.path.join(OBJ_DIR, ".lock"), "w") as lock:
         fcntl.flock(lock, fcntl.LOCK_EX)
@@ -116,6 +116,9 @@ def _build_locked(verbose: bool, force: bool, sources) -> str:
         known = {os.path.splitext(os.path.basename(s))[0] for s in srcs}
         if names - known:
             raise ValueError(f"no such source: {sorted(names - known)}")
+        if os.path.exists(LIB_PATH):        # never shrink a library: what it holds is kept up to date as well
+            held = {o.split(".")[0] for o in _linked()}
+            names = names | held if held else known
         wanted = [s for s in srcs if os.path.splitext(os.path.basename(s))[0] in names]
     else:
         wanted = srcs
