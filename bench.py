@@ -26,6 +26,9 @@ Workloads (``--mode``):
 * ``pd``: disaggregated prefill: the first half of the ranks form the prefill engine (TP), the second
   half the decode engine (expert parallel with data-parallel attention for MoE models), KV blocks
   move over NVLink (``ours`` only).
+* ``layers``: prefill and decode throughput of plan-built decoders (Vofelix) beside the closest existing
+  models at equal layer sizes, one GPU (``benchmarks/plan_bench.py``, ``ours`` only); the line's value is the
+  decode rate of the whole design and ``cases`` holds the table.
 
 Rank 0 prints ONE JSON line.  ``value`` is timed with CUDA events (max over ranks); ``e2e.value``
 is the same passes timed by the host clock around ``LLM.generate`` — every engine step inside
@@ -104,7 +107,7 @@ def parse_args():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "vllm"])
     ap.add_argument("--engine", default="native", choices=["native", "vllm"])
     ap.add_argument("--model", default="qwen3-8b", choices=sorted(HF_SHAPES))
-    ap.add_argument("--mode", default="offline", choices=["offline", "serve", "pd"])
+    ap.add_argument("--mode", default="offline", choices=["offline", "serve", "pd", "layers"])
     ap.add_argument("--concurrency", type=int, default=64)
     ap.add_argument("--num-prompts", type=int, default=1024)
     ap.add_argument("--input-len", type=int, default=1024)
@@ -568,6 +571,17 @@ def main():
                                              f"{type(e).__name__}: {e}"[:400]}), flush=True)
             # a non-zero status lets the launcher stop the other ranks instead of leaving them in a collective
             os._exit(0 if world == 1 else 3)
+    elif args.mode == "layers":
+        sys.path.insert(0, REPO)
+        from benchmarks.plan_bench import run_models
+        sampler = ClockSampler(local)
+        sampler.start()
+        cases = run_models()
+        best = cases["whole design"]["decode 256 ctx 2048"]
+        print(json.dumps({"metric": "decode tokens/s", "value": best["tok_s"], "unit": "tok/s", "n_gpus": 1,
+                          "ms_per_step": best["ms"], "higher_is_better": True, "vs_baseline": None, "dtype": "bf16",
+                          "data": "synthetic", "config": {"model": "vofelix-bench", "mode": "layers"}, "cases": cases,
+                          "clocks": sampler.stop()}), flush=True)
     elif args.mode == "pd":
         sys.path.insert(0, REPO)
         from benchmarks.pd_bench import run_pd

@@ -1,0 +1,243 @@
+#!/usr/bin/env python
+"""Prefill and decode throughput of plan-built decoders (Vofelix) beside the closest existing models at equal
+size, random weights, one GPU.
+
+    python bench.py --mode layers                 # or: python benchmarks/plan_bench.py
+    python benchmarks/plan_bench.py --kernels     # the single kernels with their rooflines
+
+Model cases time the engine's own step on the device (CUDA events, median): a prefill step of whole prompts,
+and decode-graph replays of a batch with a given context.  Weights and caches are larger than L2.  Kernel
+cases rewrite a buffer larger than L2 between iterations.  Rooflines are the measured copy bandwidth and
+cuBLAS bf16 rate of MEASURED_PEAKS.json.
+"""
+from __future__ import annotations
+
+import argparse
+import gc
+import json
+import os
+import sys
+
+import numpy as np
+import torch
+
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+sys.path.insert(0, ROOT)
+sys.path.insert(0, os.path.join(ROOT, "benchmarks"))
+
+VOCAB, LAYERS = 32000, 8
+
+
+def _latent(heads, window):
+    return {"type": "latent_attention", "mlp": {"kind": "dense", "ff": 12288}, "mixer": {
+        "heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5,
+        "mask": {"size": window} if window else None, "rot": {"base": 1e4, "dims": 64}}}
+
+
+def _delta(ff=12288):
+    return {"type": "delta", "mlp": {"kind": "dense", "ff": ff} if ff else None,
+            "mixer": {"heads": 32, "kv_heads": 16, "dim": 128, "vdim": 128, "conv": 4}}
+
+
+def _vofelix(layers, side=128, loop=None):
+    from vllm_ascend_b200.config import ModelConfig
+    d = {"architecture": "Vofelix", "vocab": VOCAB, "width": 4096, "norm": {"eps": 1e-6}, "embedding": {"scale": 64.0},
+         "layers": layers}
+    if side:
+        d["token_side"] = {"dim": side}
+    if loop:
+        d["loop"] = loop
+    return ModelConfig.from_hf_dict(d, name="vofelix-bench")
+
+
+def _existing(**kw):
+    from vllm_ascend_b200.config import ModelConfig
+    return ModelConfig(vocab_size=VOCAB, hidden_size=4096, intermediate_size=12288, num_hidden_layers=LAYERS,
+                       hidden_act="gelu_pytorch_tanh", **kw)
+
+
+def _mla(heads):
+    return _existing(name="mla-dense", architecture="DeepseekV2ForCausalLM", num_attention_heads=heads,
+                     num_key_value_heads=heads, head_dim=192, use_mla=True, kv_lora_rank=512, qk_nope_head_dim=128,
+                     qk_rope_head_dim=64, v_head_dim=128, rope_theta=1e4)
+
+
+def _gdn():
+    return _existing(name="gdn-hybrid", architecture="Qwen3NextForCausalLM", num_attention_heads=32,
+                     num_key_value_heads=8, head_dim=128, qk_norm=True, full_attention_interval=LAYERS,
+                     linear_num_key_heads=16, linear_num_value_heads=32, linear_key_head_dim=128,
+                     linear_value_head_dim=128, linear_conv_kernel_dim=4)
+
+
+#: label -> configuration.  The plain Vofelix stacks have the mixers and feed-forward of their neighbour
+MODELS = {
+    "latent w=0 h32": lambda: _vofelix([_latent(32, 0)] * LAYERS, side=0),
+    "existing MLA h32": lambda: _mla(32),
+    "latent w=1024 h32": lambda: _vofelix([_latent(32, 1024)] * LAYERS, side=0),
+    "latent w=1024 h16": lambda: _vofelix([_latent(16, 1024)] * LAYERS, side=0),
+    "existing MLA h16": lambda: _mla(16),
+    "delta": lambda: _vofelix([_delta()] * (LAYERS - 1) + [_latent(32, 1024)], side=0),
+    "existing GDN": lambda: _gdn(),
+    "whole design": lambda: _vofelix([_delta(None), _delta(None), _latent(32, 1024), _latent(32, 1024), _delta(None),
+                                      _delta(None)], loop={"start": 0, "stop": 3, "times": 2}),
+}
+
+
+def peaks():
+    p = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    if os.path.exists(p):
+        d = json.load(open(p))
+        return d["hbm_gbs"], d["bf16_tflops"]
+    return 6650.0, 1590.0
+
+
+def _median_ms(fn, iters=12, warm=4):
+    for _ in range(warm):
+        fn()
+    torch.cuda.synchronize()
+    ts = []
+    for _ in range(iters):
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        fn()
+        b.record()
+        torch.cuda.synchronize()
+        ts.append(a.elapsed_time(b))
+    return float(np.median(ts))
+
+
+def bench_model(cfg, prefill=((4, 2048),), decode=((1, 2048), (64, 2048), (256, 2048))) -> dict:
+    """Tokens/s of prefill steps (sequences, length) and of decode steps (sequences, context)."""
+    from vllm_ascend_b200 import LLM, SamplingParams
+    from vllm_ascend_b200.engine.request import Request
+    B = max(b for b, _ in decode)
+    L = max(n for _, n in decode + tuple(prefill)) + 128
+    llm = LLM(cfg, device="cuda", max_model_len=L, max_num_seqs=B, max_num_batched_tokens=8192, async_scheduling=False,
+              num_gpu_blocks_override=B * (L // 128 + 1) + 2, cudagraph_capture_sizes=sorted({b for b, _ in decode}))
+    eng, run = llm.engine.scheduler, llm.engine.runner
+    rng = np.random.default_rng(0)
+    out = {}
+
+    def requests(n, length):
+        return [Request(f"b{rng.integers(1 << 60)}", rng.integers(0, VOCAB, size=length).astype(np.int32),
+                        SamplingParams(max_tokens=1)) for _ in range(n)]
+
+    def finish(reqs):
+        for r in reqs:
+            eng.abort_request(r.request_id)
+            eng.requests.pop(r.request_id, None)
+    with torch.inference_mode():
+        for b, n in prefill:
+            reqs = requests(b, n)
+            so = eng.schedule_portions([(r, n) for r in reqs])
+            run._sync_rows(so)
+            meta, _, Tp, _, _ = run._prepare_inputs(so)
+            ms = _median_ms(lambda: run._forward(Tp, meta))
+            out[f"prefill {b}x{n}"] = {"ms": round(ms, 3), "tok_s": round(b * n / ms * 1e3)}
+            finish(reqs)
+        for b, n in decode:
+            reqs = requests(b, n + 1)
+            # context: cache contents are whatever is there, lengths and pages are real
+            so = eng.schedule_portions([(r, n) for r in reqs])
+            run._sync_rows(so)
+            for r in reqs:
+                r.num_computed_tokens = n
+            so = eng.schedule_portions([(r, 1) for r in reqs])
+            run._sync_rows(so)
+            run._prepare_inputs(so, pad_to=b)
+            ms = _median_ms(lambda: run.graph_wrapper.replay(run.graphs[(b, False)]), iters=20)
+            out[f"decode {b} ctx {n}"] = {"ms": round(ms, 3), "tok_s": round(b / ms * 1e3)}
+            finish(reqs)
+    run.drop_graphs()
+    del llm, eng, run
+    gc.collect()
+    torch.cuda.empty_cache()
+    return out
+
+
+# ---------------------------------------------------------------- single kernels
+def bench_kernels() -> list[dict]:
+    from kernel_bench import timeit
+    from vllm_ascend_b200 import ops
+    from vllm_ascend_b200.attention import mla
+    from vllm_ascend_b200.ops import linear_attn as la
+    from vllm_ascend_b200.ops import stream as st
+    hbm, tf = peaks()
+    bf, dev = torch.bfloat16, "cuda"
+    res = []
+
+    def rec(name, ms, nbytes=0, flops=0):
+        t_mem, t_fl = nbytes / hbm / 1e6, flops / tf / 1e9
+        res.append({"kernel": name, "ms": round(ms, 4), "GB/s": round(nbytes / ms / 1e6), "TFLOP/s": round(flops / ms / 1e9, 1),
+                    "roofline_frac": round(max(t_mem, t_fl) / ms, 3)})
+
+    def mk(*s, dtype=bf):
+        return torch.randn(*s, device=dev, dtype=dtype)
+    for T in (256, 8192):
+        W = 4096
+        r, y, w, b = mk(T, W, dtype=torch.float32), mk(T, W), mk(W), mk(W)
+        ln = st.NormSpec("layer", w, b)
+        rec(f"stream_norm post+next T={T}", timeit(lambda: st.stream_norm(r, y, ln, ln, 1e-6, bf)), T * W * 12)
+        res_b = mk(T, W)
+        rec(f"[existing] add+rms_norm T={T}", timeit(lambda: ops.rms_norm(y, w, 1e-6, res_b)), T * W * 8)
+    H, Hk, D = 32, 16, 128
+    for B, n in ((256, 1), (4, 2048), (1, 8192)):
+        T = B * n
+        C = (2 * Hk + H) * D
+        cu = torch.arange(0, T + 1, n, dtype=torch.int32, device=dev)
+        slots = torch.arange(B, dtype=torch.int32, device=dev)
+        init = torch.ones(B, dtype=torch.int32, device=dev)
+        x, cw, cs = mk(T, C + H * D), mk(C, 4), mk(B, 3, C)
+        ba, A, dt = mk(T, 2 * H), mk(H, dtype=torch.float32), mk(H, dtype=torch.float32)
+        S = torch.zeros(B, H, D, D, dtype=torch.float32, device=dev)
+        tag = f"{B}x{n}"
+        rec(f"conv+gates {tag}", timeit(lambda: la.causal_conv1d(x[:, :C], cw, None, cs, cu, slots, init, uniform=n == 1,
+                                                                gates=(ba, A, dt))),
+            T * (C * 4 + H * 12) + B * 3 * C * 4)
+        m, be, g = la.causal_conv1d(x[:, :C], cw, None, cs, cu, slots, init, uniform=n == 1, gates=(ba, A, dt))
+        q, k, v = (m[:, :Hk * D].view(T, Hk, D), m[:, Hk * D:2 * Hk * D].view(T, Hk, D), m[:, 2 * Hk * D:].view(T, H, D))
+        rec(f"delta rule {tag}", timeit(lambda: la.gated_delta_rule(q, k, v, g, be, S, cu, slots, init, D ** -0.5)),
+            T * (C + H * D) * 2 + B * H * D * D * 8, 8 * T * H * D * D)
+        o, nw = mk(T, H, D), mk(D)
+        rec(f"gated head norm {tag}", timeit(lambda: st.gated_head_norm(o, x[:, C:], nw, 1e-6)), T * H * D * 6)
+    for H in (16, 32):
+        for B, n, ctx, win in ((256, 1, 2048, 0), (256, 1, 2048, 1024), (4, 2048, 2048, 0), (4, 2048, 2048, 1024)):
+            if n > 1 and win == 0 and H == 32:
+                continue
+            bs, nb = 128, B * ctx // 128 + 1
+            lat, pe = mk(nb, bs, 1, 512), mk(nb, bs, 1, 64)
+            bt = (torch.arange(B * ctx // bs, dtype=torch.int32, device=dev).view(B, -1) + 1).contiguous()
+            T = B * n
+            cu = torch.arange(0, T + 1, n, dtype=torch.int32, device=dev)
+            sl = torch.full((B,), ctx, dtype=torch.int32, device=dev)
+            ql, qp = mk(T, H, 512), mk(T, H, 64)
+            sink = torch.zeros(H, device=dev) if win else None
+            keys = sum(min(win or ctx, ctx - n + i + 1) for i in range(n)) * B
+            reads = B * min(ctx, (win or ctx) + n)
+            rec(f"latent attention H={H} {B}x{n} ctx {ctx} window {win}",
+                timeit(lambda: mla.latent_attention_tc(ql, qp, lat, pe, bt, 0.07, cu=cu, seq_lens=sl, uniform=n == 1,
+                                                       window=win, sink=sink, max_kv_len=ctx)),
+                reads * 1152 + T * H * (576 + 512) * 2, keys * H * (576 + 512) * 2)
+    return res
+
+
+def run_models(names=None) -> dict:
+    return {k: bench_model(MODELS[k]()) for k in MODELS if not names or k in names}
+
+
+def main() -> None:
+    ap = argparse.ArgumentParser()
+    ap.add_argument("--kernels", action="store_true")
+    ap.add_argument("--only", default="", help="model labels with commas between them")
+    args = ap.parse_args()
+    if args.kernels:
+        for row in bench_kernels():
+            print(json.dumps(row))
+        return
+    for k in MODELS:
+        if not args.only or k in args.only.split(","):
+            print(json.dumps({k: bench_model(MODELS[k]())}), flush=True)
+
+
+if __name__ == "__main__":
+    main()

@@ -141,12 +141,35 @@ def alone(name, pieces):
     return [[(name, p, k == len(pieces) - 1)] for k, p in enumerate(pieces)]
 
 
-def error(got, want):
-    """Largest per-position rms difference, relative to the spread of the logits."""
+def errors(got, want):
+    """Per-position rms difference, relative to the spread of the logits."""
     d = got.double() - want.double()
     d = d - d.mean(-1, keepdim=True)
-    return float((d ** 2).mean(-1).sqrt().max() / want.double().std())
+    return (d ** 2).mean(-1).sqrt() / want.double().std()
 
 
-def reference(cfg, w, ids):
-    return vo.forward(cfg, w, ids)
+def error(got, want):
+    return float(errors(got, want).max())
+
+
+_KNOWN = {}
+
+
+def reference(cfg, w, ids, rounded=False):
+    key = (json.dumps(cfg), float(w["embed"].double().sum()), tuple(ids), rounded)
+    if key not in _KNOWN:
+        _KNOWN[key] = vo.forward(cfg, w, ids, rounded=rounded)
+    return _KNOWN[key]
+
+
+def check(got, cfg, w, ids, dtype, note=None):
+    """fp32: every position within 1e-4.  bf16: the errors are those of rounding, i.e. neither their mean nor
+    the largest is far above what rounding the sub-layers' inputs and outputs causes in the definition."""
+    want = reference(cfg, w, ids)
+    e = errors(got, want)
+    if dtype == "float32":
+        assert float(e.max()) < 1e-4, (note, float(e.max()))
+        return
+    r = errors(reference(cfg, w, ids, True), want)
+    assert float(e.mean()) < 2.5 * float(r.mean()) and float(e.max()) < 3 * max(float(r.max()), 0.02), \
+        (note, float(e.mean()), float(r.mean()), float(e.max()), float(r.max()))

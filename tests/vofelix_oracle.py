@@ -149,8 +149,11 @@ def sub(w, prefix):
     return {k[len(prefix):]: t for k, t in w.items() if k.startswith(prefix)}
 
 
-def forward(cfg, w, ids, dtype=torch.float64, collect=None):
-    """Logits [n, vocab] of one sequence; ``collect`` receives the stream after every layer run."""
+def forward(cfg, w, ids, dtype=torch.float64, collect=None, rounded=False):
+    """Logits [n, vocab] of one sequence; ``collect`` receives the stream after every layer run.  ``rounded``:
+    what enters and leaves a sub-layer is rounded to bf16 (the size of the error that rounding causes)."""
+    def cast(t):
+        return t.to(torch.bfloat16).to(dtype) if rounded else t
     w = {k: t.to(dtype) if t.is_floating_point() else t for k, t in w.items()}
     ids = torch.as_tensor(ids, dtype=torch.int64)
     eps = cfg["norm"]["eps"]
@@ -161,7 +164,7 @@ def forward(cfg, w, ids, dtype=torch.float64, collect=None):
         L, p = cfg["layers"][i], sub(w, f"l{i}.")
 
         def norm(name, t):
-            return layer_norm(t, p[name], p[name + ".b"], eps)
+            return cast(layer_norm(cast(t) if name.endswith("b") else t, p[name], p[name + ".b"], eps))
         if run in again:
             x = x + x0
         mixer = {"latent_attention": latent_attention, "delta": delta_mixer}[L["type"]]
@@ -172,4 +175,4 @@ def forward(cfg, w, ids, dtype=torch.float64, collect=None):
             x = token_side(x, ids, i, cfg["token_side"]["dim"], w["side.embed"], sub(p, "side."), eps)
         if collect is not None:
             collect.append(x)
-    return layer_norm(x, w["final.norm"], w["final.norm.b"], eps) @ w["head"].T
+    return cast(layer_norm(x, w["final.norm"], w["final.norm.b"], eps)) @ w["head"].T
