@@ -196,7 +196,8 @@ def bench_kernels() -> list[dict]:
             T * (C * 4 + H * 12) + B * 3 * C * 4)
         m, be, g = la.causal_conv1d(x[:, :C], cw, None, cs, cu, slots, init, uniform=n == 1, gates=(ba, A, dt))
         q, k, v = (m[:, :Hk * D].view(T, Hk, D), m[:, Hk * D:2 * Hk * D].view(T, Hk, D), m[:, 2 * Hk * D:].view(T, H, D))
-        rec(f"delta rule {tag}", timeit(lambda: la.gated_delta_rule(q, k, v, g, be, S, cu, slots, init, D ** -0.5)),
+        rec(f"delta rule {tag}", timeit(lambda: la.gated_delta_rule(q, k, v, g, be, S, cu, slots, init, D ** -0.5,
+                                                                    uniform=n == 1)),
             T * (C + H * D) * 2 + B * H * D * D * 8, 8 * T * H * D * D)
         o, nw = mk(T, H, D), mk(D)
         rec(f"gated head norm {tag}", timeit(lambda: st.gated_head_norm(o, x[:, C:], nw, 1e-6)), T * H * D * 6)

@@ -146,7 +146,8 @@ def test_delta_rule_over_portions(dtype, H, Hk, d, vd):
             part = lambda t: torch.cat([t[i][at[i]:at[i] + pair[i]] for i in todo]).cuda()      # noqa: E731
             o = la.gated_delta_rule(part(q), part(k), part(v), part(logg), part(beta), state, torch.from_numpy(cu).cuda(),
                                     torch.tensor([slots[i] for i in todo], dtype=torch.int32).cuda(),
-                                    torch.tensor([at[i] > 0 for i in todo], dtype=torch.int32).cuda(), d ** -0.5)
+                                    torch.tensor([at[i] > 0 for i in todo], dtype=torch.int32).cuda(), d ** -0.5,
+                                    uniform=all(pair[i] == 1 for i in todo))
             for j, i in enumerate(todo):
                 got[i].append(o[cu[j]:cu[j + 1]].cpu())
                 at[i] += pair[i]
@@ -157,6 +158,31 @@ def test_delta_rule_over_portions(dtype, H, Hk, d, vd):
             close(torch.cat(got[i]), want, dtype)
             close(state[slots[i]], S, torch.float32, 4)
     assert bool((state[1] == 9.0).all())                     # nobody's slot
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,Hk,d,vd", [(4, 2, 12, 20), (6, 2, 40, 48), (4, 4, 128, 128), (2, 2, 200, 72), (3, 1, 33, 130),
+                                       (2, 1, 256, 128), (3, 3, 16, 4)])
+def test_delta_decode_with_the_gated_norm(dtype, H, Hk, d, vd):
+    g = gen(d + vd)
+    B, owner = 5, [h // (H // Hk) for h in range(H)]
+    q, k = (rnd(g, B, Hk, d, dtype=dtype) for _ in range(2))
+    v, z, w = rnd(g, B, H, vd, dtype=dtype), rnd(g, B, 2 * H * vd, dtype=dtype), rnd(g, vd, dtype=dtype)
+    beta, logg = torch.rand(B, H, generator=g), -torch.rand(B, H, generator=g)
+    S0 = torch.randn(B + 1, H, d, vd, generator=g)
+    state, slots, init = S0.cuda(), [3, 0, 5, 1, 2], [1, 0, 1, 1, 0]
+    i32 = lambda t: torch.tensor(t, dtype=torch.int32).cuda()                           # noqa: E731
+    got = la.gated_delta_rule(q.cuda(), k.cuda(), v.cuda(), logg.cuda(), beta.cuda(), state, i32(list(range(B + 1))),
+                              i32(slots), i32(init), d ** -0.5, uniform=True,
+                              gate=(z.cuda()[:, H * vd:], w.cuda(), 1e-5))
+    for b in range(B):
+        o, S = vo.delta_scan(vo.unit(q[b:b + 1].double())[:, owner] * d ** -0.5, vo.unit(k[b:b + 1].double())[:, owner],
+                             v[b:b + 1].double(), beta[b:b + 1].double(), torch.exp(logg[b:b + 1].double()),
+                             S0[slots[b]].double() if init[b] else None)
+        want = vo.rms_norm(o[0], w.double(), 1e-5) * vo.silu(z[b, H * vd:].double()).view(H, vd)
+        close(got[b], want.reshape(-1), dtype, 1.5)
+        close(state[slots[b]], S, torch.float32, 4)
+    assert torch.equal(state[4].cpu(), S0[4])
 
 
 # ---------------------------------------------------------------- latent attention

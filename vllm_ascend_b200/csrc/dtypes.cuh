@@ -55,51 +55,27 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.f + tanhf(u));
 }
 
-// packed pair of fp32 operations
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
-  float2 d;
-  asm("{\n\t.reg .b64 A, B, C, D;\n\t"
-      "mov.b64 A, {%2, %3};\n\tmov.b64 B, {%4, %5};\n\tmov.b64 C, {%6, %7};\n\t"
-      "fma.rn.f32x2 D, A, B, C;\n\tmov.b64 {%0, %1}, D;\n\t}"
-      : "=f"(d.x), "=f"(d.y)
-      : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
+// two fp32 values in one 64-bit register, and the packed operations on them
+using f32x2 = unsigned long long;
+__device__ __forceinline__ f32x2 pack2(float lo, float hi) {
+  f32x2 d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
   return d;
 }
-__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+__device__ __forceinline__ float2 unpack2(f32x2 v) {
   float2 d;
-  asm("{\n\t.reg .b64 A, B, D;\n\t"
-      "mov.b64 A, {%2, %3};\n\tmov.b64 B, {%4, %5};\n\t"
-      "mul.rn.f32x2 D, A, B;\n\tmov.b64 {%0, %1}, D;\n\t}"
-      : "=f"(d.x), "=f"(d.y)
-      : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(v));
   return d;
 }
-
-// R consecutive elements held as they are stored (fetched one token ahead), R even
-template <typename T, int R>
-struct RawSlice {
-  T e[R];
-  // VEC: 16-byte loads, ``left`` (elements up to the end of the row) is a multiple of the vector
-  template <bool VEC>
-  __device__ __forceinline__ void load(const T* p, int left) {
-    constexpr int V = 16 / (int)sizeof(T);
-    if constexpr (VEC && R % V == 0) {
-#pragma unroll
-      for (int i = 0; i < R; i += V) {
-        if (i < left) load_raw<T, V>(p + i, e + i);
-        else
-#pragma unroll
-          for (int j = 0; j < V; j++) e[i + j] = from_f<T>(0.f);
-      }
-    } else {
-#pragma unroll
-      for (int i = 0; i < R; i++) e[i] = i < left ? p[i] : from_f<T>(0.f);
-    }
-  }
-  __device__ __forceinline__ void unpack(float2* v) const {
-#pragma unroll
-    for (int i = 0; i < R / 2; i++) v[i] = make_float2(to_f(e[2 * i]), to_f(e[2 * i + 1]));
-  }
-};
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
 
 }  // namespace b200

@@ -14,7 +14,6 @@ import torch
 
 from ..config import ModelConfig
 from ..ops import linear_attn as la
-from ..ops.stream import gated_head_norm
 from .layers import ColumnParallelLinear, ParamFactory, RowParallelLinear, TPComm, copy_exact
 
 
@@ -66,8 +65,9 @@ class GatedDeltaNet:
         k = mixed[:, kd:2 * kd].view(T, self.Hk, self.Dk)
         v = mixed[:, 2 * kd:].view(T, self.Hv, self.Dv)
         o = la.gated_delta_rule(q, k, v, g, beta, ssm_state, cu, slots, has_init, self.scale, l2norm=True,
-                                cu_cpu=None if uniform else meta.query_start_loc_cpu)
-        return self.out_proj(gated_head_norm(o, z, self.norm_weight, self.cfg.rms_norm_eps))
+                                cu_cpu=None if uniform else meta.query_start_loc_cpu, uniform=uniform,
+                                gate=(z, self.norm_weight, self.cfg.rms_norm_eps))
+        return self.out_proj(o)
 
     # parts of the fused projections, in row order: (name, key or value heads)
     _QKVZ = (("q", "k"), ("k", "k"), ("v", "v"), ("g", "v"))

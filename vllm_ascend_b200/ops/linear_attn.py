@@ -15,7 +15,7 @@ P, I, L, Fl = c_void_p, c_int, c_long, c_float
 _native.register_signature("b200_causal_conv1d", [P, L, P, P, P, P, P, P, P, L, L, I, I, I, I, I, L, I, P, L, P, P, I, P, P,
                                                   P, P])
 _native.register_signature("b200_gated_delta_rule", [P, P, P, L, L, P, P, P, P, P, P, P, L, I, I, I, I, I, Fl, I,
-                                                     L, I, P, P])
+                                                     L, I, I, P, L, P, Fl, P, P])
 _DTYPES = {torch.bfloat16: 0, torch.float32: 1}
 
 
@@ -209,8 +209,11 @@ def _chunk_min(on_cuda: bool = False) -> int:
     return int(envs.VLLM_B200_GDN_CHUNK_MIN)
 
 
-def gated_delta_rule(q, k, v, g, beta, state, cu, slots, has_init, scale, l2norm=True, cu_cpu=None):
-    """``cu_cpu`` (host copy of ``cu``) lets long sequences (>= ``VLLM_B200_GDN_CHUNK_MIN`` new tokens:
+def gated_delta_rule(q, k, v, g, beta, state, cu, slots, has_init, scale, l2norm=True, cu_cpu=None, uniform=False,
+                     gate=None):
+    """``uniform``: every sequence of the step has exactly one token.  ``gate`` = (z [T, Hv * DV], weight [DV],
+    eps): the result is the gated RMS norm of the read-out, [T, Hv * DV] (fused into the decode kernel).
+    ``cu_cpu`` (host copy of ``cu``) lets long sequences (>= ``VLLM_B200_GDN_CHUNK_MIN`` new tokens:
     prefill chunks) take the chunk-parallel form while decode and verification rows stay on the
     per-token recurrence."""
     cmin = _chunk_min(q.is_cuda) if cu_cpu is not None else 0
@@ -232,25 +235,40 @@ def gated_delta_rule(q, k, v, g, beta, state, cu, slots, has_init, scale, l2norm
                 out[rows_t] = gated_delta_rule(q[rows_t].contiguous(), k[rows_t].contiguous(), v[rows_t].contiguous(),
                                                g[rows_t], beta[rows_t], state, cu_s, slots[sel].contiguous(),
                                                has_init[sel].contiguous(), scale, l2norm)
-            return out
+            return _gate(out, gate)
     if not q.is_cuda:
-        return gated_delta_rule_ref(q, k, v, g, beta, state, cu, slots, has_init, scale, l2norm)
+        return _gate(gated_delta_rule_ref(q, k, v, g, beta, state, cu, slots, has_init, scale, l2norm), gate)
     T, Hv, DV = v.shape
     Hk, DK = q.shape[1], q.shape[2]
     if q.dtype not in _DTYPES or k.dtype != q.dtype or v.dtype != q.dtype or state.dtype != torch.float32:
         raise TypeError("gated_delta_rule takes bf16 or fp32 q, k, v of one type and an fp32 state")
-    assert v.stride(2) == 1 and q.stride(0) == k.stride(0) and q.stride(2) == 1 and q.stride(1) == DK and v.stride(1) == DV
+    assert v.stride(2) == 1 and q.stride(0) == k.stride(0) and q.stride(2) == 1 and q.stride(1) == DK \
+        and v.stride(1) == DV
     out = torch.empty((T, Hv, DV), dtype=v.dtype, device=v.device)
     g = g.float().contiguous()
     beta = beta.float().contiguous()
-    rc = _native.lib().b200_gated_delta_rule(
-        q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), v.stride(0), g.data_ptr(), beta.data_ptr(),
-        state.data_ptr(), cu.data_ptr(), slots.data_ptr(), has_init.data_ptr(), out.data_ptr(), out.stride(0),
-        cu.numel() - 1, Hk, Hv, DK, DV, scale, int(l2norm), state.shape[0], _DTYPES[q.dtype],
-        _native.status_word(q.device).data_ptr(), _native.stream_ptr())
+    uniform = bool(uniform and T == cu.numel() - 1)
+    fused = uniform and gate is not None and gate[0].dtype == q.dtype and gate[1].dtype == q.dtype \
+        and gate[0].stride(1) == 1
+    for z in ((gate[0], None) if fused else (None,)):
+        rc = _native.lib().b200_gated_delta_rule(
+            q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), v.stride(0), g.data_ptr(), beta.data_ptr(),
+            state.data_ptr(), cu.data_ptr(), slots.data_ptr(), has_init.data_ptr(), out.data_ptr(), out.stride(0),
+            cu.numel() - 1, Hk, Hv, DK, DV, scale, int(l2norm), state.shape[0], _DTYPES[q.dtype], int(uniform),
+            _native.ptr(z), 0 if z is None else z.stride(0), None if z is None else gate[1].data_ptr(),
+            0.0 if z is None else float(gate[2]), _native.status_word(q.device).data_ptr(), _native.stream_ptr())
+        if rc != -1:                  # -1: these sizes have no fused form, nothing was launched
+            break
     _native.check(rc, "gated_delta_rule")
     _native.count_launch()
-    return out
+    return out.view(T, Hv * DV) if z is not None else _gate(out, gate)
+
+
+def _gate(out, gate):
+    if gate is None:
+        return out
+    from .stream import gated_head_norm
+    return gated_head_norm(out, *gate)
 
 
 # ---------------------------------------------------------------------------- lightning attention
