@@ -211,7 +211,8 @@ def bench_gdn(a):
         cu = torch.arange(0, T + 1, q_len, dtype=torch.int32, device=dev)
         slots = torch.arange(B, dtype=torch.int32, device=dev)
         init = torch.ones(B, dtype=torch.int32, device=dev)
-        ms = timeit(lambda: la.gated_delta_rule(q, k, v, gg, beta, S, cu, slots, init, DK ** -0.5), a.iters)
+        ms = timeit(lambda: la.gated_delta_rule(q, k, v, gg, beta, S, cu, slots, init, DK ** -0.5,
+                                                 uniform=q_len == 1), a.iters)
         state_bytes = 2.0 * B * Hv * DK * DV * 4
         print(f"gated-delta-rule B={B} q_len={q_len} Hv={Hv} {DK}x{DV}: {ms:.4f} ms  state {state_bytes / ms / 1e6:.0f} GB/s "
               f"({state_bytes / ms / 1e6 / hbm:.2f} {tag})  {T / ms * 1e3:.0f} tok/s", flush=True)

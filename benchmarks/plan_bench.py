@@ -78,8 +78,8 @@ MODELS = {
     "existing MLA h16": lambda: _mla(16),
     "delta": lambda: _vofelix([_delta()] * (LAYERS - 1) + [_latent(32, 1024)], side=0),
     "existing GDN": lambda: _gdn(),
-    "whole design": lambda: _vofelix([_delta(None), _delta(None), _latent(32, 1024), _latent(32, 1024), _delta(None),
-                                      _delta(None)], loop={"start": 0, "stop": 3, "times": 2}),
+    "whole design": lambda: _vofelix([_delta(None), _latent(32, 1024), _delta(None), _delta(None), _latent(32, 1024),
+                                      _delta(None)], loop={"start": 1, "stop": 4, "times": 2}),
 }
 
 

@@ -221,8 +221,8 @@ def attend(q_lat, q_pe, lat, pe, first, last, scale, sink):
 
 
 CASES = [  # H, dc, dr, block, window, lens, q_lens
-    (6, 96, 16, 64, 50, [300, 49, 50, 51, 1], [300, 49, 50, 51, 1]),
-    (6, 96, 16, 64, 50, [300, 178, 129, 1, 77], [1, 1, 1, 1, 1]),
+    (7, 104, 24, 64, 50, [300, 49, 50, 51, 1], [300, 49, 50, 51, 1]),
+    (7, 104, 24, 64, 50, [300, 178, 129, 1, 77], [1, 1, 1, 1, 1]),
     (3, 20, 6, 16, 7, [40, 9, 200], [40, 1, 2]),
     (16, 512, 64, 128, 130, [700, 131, 258], [37, 131, 1]),
     (32, 512, 64, 128, 0, [500, 100], [1, 1]),
@@ -299,7 +299,7 @@ def test_a_sink_far_above_or_below_the_scores():
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,dn,dr,dc", [(3, 11, 6, 20), (6, 64, 16, 96), (2, 8, 2, 8)])
+@pytest.mark.parametrize("H,dn,dr,dc", [(3, 11, 6, 20), (5, 56, 24, 120), (2, 8, 2, 8)])
 def test_latent_preprocess(dtype, H, dn, dr, dc):
     g = gen(dc)
     T, base = 13, 5000.0
