@@ -1,0 +1,271 @@
+"""Paged grouped-query attention with options: sliding window that keeps the first tokens of a sequence, capped
+scores, a learned bias by distance, an attention sink, a gate per head on the output, value heads of another
+size than the key heads.  And the pass in front of it: short convolution, q / k norm over all heads, rotary
+positions, cache write.
+
+GPU tensors run the kernels of csrc/qkv_prep.cu and csrc/attention_variant.cu (fp32, odd sizes) or the tcgen05
+kernels of csrc/attention_tc.cu and csrc/attention_decode_tc.cu (bf16); CPU tensors run the PyTorch definitions
+below.  The reference's paged attention has the window and the mask (vllm_ascend/attention/attention_v1.py:1341-1472)."""
+from __future__ import annotations
+
+import ctypes
+import math
+from ctypes import c_float, c_int, c_long, c_void_p
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from .. import _native
+from ..ops import linear_attn as la
+from ..ops import reference as ref
+
+
+def _fields(**kinds):
+    """ctypes fields of the kernels' argument structs: pointers, then 64-bit, then 32-bit members."""
+    ctype = {"pointers": c_void_p, "longs": c_long, "ints": c_int, "floats": c_float}
+    return [(name, ctype[kind]) for kind, names in kinds.items() for name in names.split()]
+
+
+class _PrepArgs(ctypes.Structure):
+    """QkvPrepArgs of csrc/qkv_prep.cu."""
+    _fields_ = _fields(
+        pointers="qkv conv_w state cu slots has_init q_norm k_norm positions cos_sin slot_mapping q_out k_cache v_cache sums",
+        longs="qkv_stride state_rows cache_slots k_block k_tok k_head v_block v_tok v_head tokens",
+        ints="num_seqs taps heads kv_heads dim vdim q_norm_dims k_norm_dims values_from_keys rot cos_rows block_size "
+             "uniform phase dtype", floats="eps")
+
+
+class _AttnArgs(ctypes.Structure):
+    """AttnVariantArgs of csrc/attention.h."""
+    _fields_ = _fields(
+        pointers="q k_cache v_cache out cu seq_lens block_table row_seq row_kv_len bias sink gate scratch",
+        longs="q_stride out_stride gate_stride num_blocks tokens k_block k_tok k_head v_block v_tok v_head",
+        ints="num_seqs max_blocks block_size heads kv_heads dim vdim window keep_first bias_len num_splits dtype",
+        floats="scale softcap")
+
+
+_ENTRY = [c_void_p, c_void_p, c_void_p]
+for _name in ("b200_qkv_prep", "b200_attention_variant", "b200_attention_variant_prefill",
+              "b200_attention_variant_decode"):
+    _native.register_signature(_name, _ENTRY)
+
+
+def _launch(entry: str, args: ctypes.Structure, device, launches: int = 1) -> None:
+    rc = getattr(_native.lib(), entry)(ctypes.addressof(args), _native.status_word(device).data_ptr(), _native.stream_ptr())
+    _native.check(rc, entry[5:])
+    _native.count_launch(launches)
+
+
+@dataclass
+class AttnOptions:
+    scale: float
+    window: int = 0                          # 0: all earlier tokens
+    keep_first: int = 0                      # with a window: the first tokens that stay visible
+    softcap: float = 0.0                     # 0: scores as they are
+    bias: Optional[torch.Tensor] = None      # fp32 [H, n]: added to the score by distance (the last entry from n - 1 on)
+    sink: Optional[torch.Tensor] = None      # fp32 [H]: exp(sink) joins the softmax denominator
+
+    @property
+    def plain(self) -> bool:
+        return not self.keep_first and not self.softcap and self.bias is None and self.sink is None
+
+
+def distance_buckets(rows: int, largest: int, count: int) -> list[int]:
+    """Bucket of every distance 0 .. count - 1 in a table of ``rows`` rows: one bucket each below rows / 2,
+    logarithmic buckets up to ``largest`` from there on."""
+    half = rows // 2
+    out = []
+    for n in range(count):
+        if n < half:
+            out.append(n)
+        elif largest <= half or half == 0:
+            out.append(rows - 1)
+        else:
+            out.append(min(rows - 1, half + math.floor(math.log(n / half) / math.log(largest / half) * (rows - half))))
+    return out
+
+
+def distance_table(rel: torch.Tensor, largest: int, count: int) -> torch.Tensor:
+    """rel [rows, H] -> fp32 [H, n] indexed by distance; from the first distance of the last bucket on (or from
+    ``count`` - 1 on) the bias stays the same."""
+    rows = rel.shape[0]
+    idx = distance_buckets(rows, largest, max(1, min(count, max(largest, rows) + 1)))
+    if rows - 1 in idx:
+        idx = idx[:idx.index(rows - 1) + 1]
+    return rel.float()[torch.tensor(idx, device=rel.device)].T.contiguous()
+
+
+# ---------------------------------------------------------------- q / k / v in front of the attention
+@dataclass
+class PrepSpec:
+    """What happens to the rows [q | k | v | rest] of a fused projection."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    eps: float
+    q_norm: torch.Tensor                     # [heads * dim], [kv_heads * dim]
+    k_norm: torch.Tensor
+    norm_dims: tuple                         # widths the means are over (all ranks' heads)
+    values_from_keys: bool = False           # no v columns: the values are the keys before norm and rotation
+    conv: Optional[torch.Tensor] = None      # [columns of q, k (and v), taps]
+    rot_dims: int = 0
+    cos_sin: Optional[torch.Tensor] = None   # fp32 [positions, rot_dims]
+
+    @property
+    def columns(self) -> int:
+        return self.heads * self.dim + self.kv_heads * self.dim + (0 if self.values_from_keys else self.kv_heads * self.vdim)
+
+
+def _prep_ref(s: PrepSpec, qkv, meta, k_cache, v_cache, state, reduce_sums):
+    T, nq, nk = qkv.shape[0], s.heads * s.dim, s.kv_heads * s.dim
+    x = qkv[:, :s.columns]
+    if s.conv is not None:
+        slots, init = meta.state_slots, meta.has_initial_state
+        if state is None:                    # one tap: nothing is kept
+            x = (x.float() * s.conv.float()[:, 0]).to(x.dtype)
+        else:
+            x = la.causal_conv1d_ref(x, s.conv, None, state, meta.query_start_loc, slots, init, act=False)
+    q, k = x[:, :nq].float(), x[:, nq:nq + nk].float()
+    v = x[:, nq:nq + nk] if s.values_from_keys else x[:, nq + nk:]
+    sums = torch.stack([(q * q).sum(-1), (k * k).sum(-1)], -1)
+    if reduce_sums is not None:
+        sums = reduce_sums(sums)
+    inv = torch.rsqrt(sums / torch.tensor(s.norm_dims, dtype=torch.float32) + s.eps)
+    q = (q * inv[:, :1] * s.q_norm.float()).view(T, s.heads, s.dim)
+    k = (k * inv[:, 1:] * s.k_norm.float()).view(T, s.kv_heads, s.dim)
+    if s.rot_dims:
+        q = ref.apply_rope_interleaved(q, meta.positions, s.cos_sin, s.rot_dims)
+        k = ref.apply_rope_interleaved(k, meta.positions, s.cos_sin, s.rot_dims)
+    keep = meta.slot_mapping >= 0
+    slot = meta.slot_mapping[keep]
+    bs = k_cache.shape[1]
+    k_cache[slot // bs, slot % bs] = k[keep].to(k_cache.dtype)
+    v_cache[slot // bs, slot % bs] = v.reshape(T, s.kv_heads, s.vdim)[keep].to(v_cache.dtype)
+    return q.to(qkv.dtype)
+
+
+def qkv_prep(s: PrepSpec, qkv: torch.Tensor, meta, k_cache: torch.Tensor, v_cache: torch.Tensor,
+             state: Optional[torch.Tensor] = None, reduce_sums=None) -> torch.Tensor:
+    """qkv [T, columns ...] -> q [T, heads, dim]; keys and values go to their cache slots (slot < 0: not stored).
+    ``state`` [slots, taps - 1, columns] holds the last convolution inputs of every sequence and is updated.
+    ``reduce_sums`` (tensor parallelism) completes the sums of squares [T, 2] of q and k over the ranks."""
+    if not qkv.is_cuda:
+        return _prep_ref(s, qkv, meta, k_cache, v_cache, state, reduce_sums)
+    T, dev, dt = qkv.shape[0], qkv.device, qkv.dtype
+    taps = 0 if s.conv is None else s.conv.shape[1]
+    same = [k_cache, v_cache, s.q_norm, s.k_norm] + [t for t in (s.conv, state) if t is not None]
+    if dt not in (torch.bfloat16, torch.float32) or any(t.dtype != dt for t in same) or qkv.stride(1) != 1:
+        raise TypeError("qkv_prep takes bf16 or fp32 rows with weights, state and caches of the same type")
+    if k_cache.stride(3) != 1 or v_cache.stride(3) != 1 or qkv.shape[1] < s.columns:
+        raise ValueError("qkv_prep: cache rows must be dense and the projection wide enough")
+    if taps > 1 and (state is None or tuple(state.shape[1:]) != (taps - 1, s.columns) or not state.is_contiguous()):
+        raise ValueError("qkv_prep: convolution state of another shape")
+    q = torch.empty((T, s.heads, s.dim), dtype=dt, device=dev)
+    B = meta.num_reqs
+    a = _PrepArgs(
+        qkv=qkv.data_ptr(), conv_w=_native.ptr(s.conv), state=_native.ptr(state), cu=meta.query_start_loc.data_ptr(),
+        slots=_native.ptr(meta.state_slots), has_init=_native.ptr(meta.has_initial_state), q_norm=s.q_norm.data_ptr(),
+        k_norm=s.k_norm.data_ptr(), positions=meta.positions.data_ptr(),
+        cos_sin=_native.ptr(s.cos_sin) if s.rot_dims else None, slot_mapping=meta.slot_mapping.data_ptr(),
+        q_out=q.data_ptr(), k_cache=k_cache.data_ptr(), v_cache=v_cache.data_ptr(), qkv_stride=qkv.stride(0),
+        state_rows=0 if state is None else state.shape[0], cache_slots=k_cache.shape[0] * k_cache.shape[1],
+        k_block=k_cache.stride(0), k_tok=k_cache.stride(1), k_head=k_cache.stride(2), v_block=v_cache.stride(0),
+        v_tok=v_cache.stride(1), v_head=v_cache.stride(2), tokens=T, num_seqs=B, taps=taps, heads=s.heads,
+        kv_heads=s.kv_heads, dim=s.dim, vdim=s.vdim, q_norm_dims=int(s.norm_dims[0]), k_norm_dims=int(s.norm_dims[1]),
+        values_from_keys=int(s.values_from_keys), rot=s.rot_dims, cos_rows=s.cos_sin.shape[0] if s.rot_dims else 0,
+        block_size=k_cache.shape[1], uniform=int(meta.max_query_len <= 1 and T == B), dtype=int(dt == torch.float32),
+        eps=s.eps)
+    if reduce_sums is None:
+        _launch("b200_qkv_prep", a, dev)
+        return q
+    sums = torch.empty((T, 2), dtype=torch.float32, device=dev)
+    a.sums, a.phase = sums.data_ptr(), 1
+    _launch("b200_qkv_prep", a, dev)
+    sums = reduce_sums(sums).contiguous()
+    a.sums, a.phase = sums.data_ptr(), 2
+    _launch("b200_qkv_prep", a, dev)
+    return q
+
+
+# ---------------------------------------------------------------- attention
+def _attention_ref(q, k_cache, v_cache, meta, o: AttnOptions, gate, out):
+    T, H, _ = q.shape
+    Hkv, Dv = v_cache.shape[2], v_cache.shape[3]
+    owner = torch.arange(H, device=q.device) // (H // Hkv)
+    qsl, sls = meta.query_start_loc_cpu, meta.seq_lens_cpu
+    for b in range(meta.num_reqs):
+        qs, qe, sl = int(qsl[b]), int(qsl[b + 1]), int(sls[b])
+        if qe <= qs:
+            continue
+        k = ref.gather_kv(k_cache, meta.block_table[b], sl).float()[:, owner]
+        v = ref.gather_kv(v_cache, meta.block_table[b], sl).float()[:, owner]
+        s = torch.einsum("qhd,khd->hqk", q[qs:qe].float(), k) * o.scale
+        if o.softcap:
+            s = o.softcap * torch.tanh(s / o.softcap)
+        dist = torch.arange(sl - (qe - qs), sl)[:, None] - torch.arange(sl)[None, :]
+        if o.bias is not None:
+            s = s + o.bias[:, dist.clamp(0, o.bias.shape[1] - 1)]
+        seen = dist >= 0
+        if o.window:
+            seen &= (dist < o.window) | (torch.arange(sl) < o.keep_first)[None, :]
+        s = s.masked_fill(~seen[None], float("-inf"))
+        if o.sink is not None:
+            s = torch.cat([s, o.sink.view(H, 1, 1).expand(H, qe - qs, 1)], -1)
+        p = torch.softmax(s, -1)[..., :sl]
+        out[qs:qe] = torch.einsum("hqk,khd->qhd", p, v).to(out.dtype)
+    if gate is not None:
+        out *= torch.sigmoid(gate.float())[:, :, None].to(out.dtype)
+    return out
+
+
+def _args(q, k_cache, v_cache, meta, o: AttnOptions, gate, out) -> _AttnArgs:
+    for t, w in ((o.bias, 2), (o.sink, 1)):
+        if t is not None and (t.dtype != torch.float32 or t.dim() != w or t.shape[0] != q.shape[1] or not t.is_contiguous()):
+            raise TypeError("bias and sink are dense fp32 tensors over the heads")
+    if any(t is not None and t.dtype != q.dtype for t in (k_cache, v_cache, gate, out)):
+        raise TypeError("queries, caches, gate and output are of one type")
+    if gate is not None and gate.stride(1) != 1:
+        gate = gate.contiguous()
+    a = _AttnArgs(
+        q=q.data_ptr(), k_cache=k_cache.data_ptr(), v_cache=v_cache.data_ptr(), out=out.data_ptr(),
+        cu=meta.query_start_loc.data_ptr(), seq_lens=meta.seq_lens.data_ptr(), block_table=meta.block_table.data_ptr(),
+        bias=_native.ptr(o.bias), sink=_native.ptr(o.sink), gate=_native.ptr(gate), q_stride=q.stride(0),
+        out_stride=out.stride(0), gate_stride=0 if gate is None else gate.stride(0), num_blocks=k_cache.shape[0],
+        tokens=q.shape[0], k_block=k_cache.stride(0), k_tok=k_cache.stride(1), k_head=k_cache.stride(2),
+        v_block=v_cache.stride(0), v_tok=v_cache.stride(1), v_head=v_cache.stride(2), num_seqs=meta.num_reqs,
+        max_blocks=meta.block_table.stride(0), block_size=k_cache.shape[1], heads=q.shape[1], kv_heads=k_cache.shape[2],
+        dim=q.shape[2], vdim=v_cache.shape[3], window=o.window, keep_first=o.keep_first if o.window else 0,
+        bias_len=0 if o.bias is None else o.bias.shape[1], num_splits=1, dtype=int(q.dtype == torch.float32),
+        scale=o.scale, softcap=o.softcap)
+    a.hold = gate                    # alive until the launch
+    return a
+
+
+def variant_attention_simple(q, k_cache, v_cache, meta, o: AttnOptions, gate=None, out=None) -> torch.Tensor:
+    """CUDA-core kernel: any sizes, bf16 or fp32."""
+    from .mla import _batch_rows
+    T, H, _ = q.shape
+    if q.stride(2) != 1 or q.stride(1) != q.shape[2] or k_cache.stride(3) != 1 or v_cache.stride(3) != 1:
+        raise ValueError("heads and cache rows must be dense")
+    if out is None:
+        out = torch.empty((T, H, v_cache.shape[3]), dtype=q.dtype, device=q.device)
+    a = _args(q, k_cache, v_cache, meta, o, gate, out)
+    row_seq, row_kv = _batch_rows(meta, T, q.device)
+    a.row_seq, a.row_kv_len = row_seq.data_ptr(), row_kv.data_ptr()
+    _launch("b200_attention_variant", a, q.device)
+    return out
+
+
+def variant_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, meta, o: AttnOptions,
+                      gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Attention of every query row of the step over its sequence's paged keys: q [T, H, D] -> [T, H, Dv].
+    ``gate`` [T, H]: head h's output is scaled by sigmoid(gate[:, h])."""
+    T, H, _ = q.shape
+    out = torch.empty((T, H, v_cache.shape[3]), dtype=q.dtype, device=q.device)
+    if T == 0:
+        return out
+    if not q.is_cuda:
+        return _attention_ref(q, k_cache, v_cache, meta, o, gate, out)
+    return variant_attention_simple(q, k_cache, v_cache, meta, o, gate, out)

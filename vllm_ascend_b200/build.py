@@ -82,6 +82,8 @@ def _compile_one(src: str, hdr_digest: str, verbose: bool) -> tuple[str, bool]:
 MODEL_SOURCES = {
     "Vofelix": ("activations", "attention_decode", "attention_mla_decode", "cache_ops", "gemm_bf16", "gemm_bf16_2cta",
                 "latent_attention", "linear_attention", "mla_preprocess", "sampler", "stream_norm"),
+    "Pegopel": ("activations", "attention_decode", "attention_decode_tc", "attention_tc", "attention_variant", "cache_ops",
+                "gemm_bf16", "gemm_bf16_2cta", "qkv_prep", "sampler", "stream_norm"),
 }
 
 

@@ -112,9 +112,23 @@ class ModelConfig:
     # ---- decoders described layer by layer (layer_plan.py) ----
     layer_plan: Optional[list] = None        # per layer {"mixer", "mlp", "over": fields of this layer}
     layer_loop: Optional[tuple] = None       # (start, stop, times): layers start..stop-1 run times in a row
+    layer_loop_refeed: bool = False          # the embedding output joins the stream again before every pass but the first
     norm_type: str = "rms"                   # "rms" | "layer" (weight and bias)
     token_side_dim: int = 0                  # per-layer token input: width of a layer's slice of the table
     attention_sink: bool = False             # a learned logit per head in the softmax denominator
+    # ---- options of paged grouped-query attention (models/variant_attention.py) ----
+    attn_conv_kernel: int = 0                # taps of a causal short convolution on projected q, k and v (0: none)
+    attn_values_from_keys: bool = False      # the values are the projected keys (before norm and rotation)
+    attn_sink_value: Optional[float] = None  # the same fixed logit for every head instead of a learned one
+    attn_softcap: Optional[float] = None     # scores become cap * tanh(score / cap)
+    attn_keep_first: int = 0                 # first tokens of a sequence that a sliding window keeps
+    attn_distance_max: int = 0               # > 0: learned bias by bucketed distance, buckets logarithmic up to this
+    attn_distance_buckets: int = 32          # rows of that table (a checkpoint's own table decides)
+    attn_head_gate: bool = False             # each head's output is scaled by a sigmoid of the layer's input
+    rotary_dims: Optional[int] = None        # rotated dimensions of a head (0: none) where the layer names them
+    # ---- residual streams and learned positions of plan-built decoders ----
+    residual_streams: int = 0                # > 0: that many streams with static mixing per sub-layer
+    learned_positions: int = 0               # rows of a position table added to the embeddings (0: none)
     # ---- numerics / quantization ----
     dtype: str = "bfloat16"
     quantization: Optional[str] = None   # None | "fp8" (128x128 block) | "w8a8_dynamic"
@@ -145,6 +159,11 @@ class ModelConfig:
     @property
     def is_hybrid(self) -> bool:
         return self.full_attention_interval > 0
+
+    @property
+    def keeps_sequence_state(self) -> bool:
+        """Layers keep something per sequence besides pages (recurrent states, convolution inputs)."""
+        return self.is_hybrid or any(p["over"].get("attn_conv_kernel", 0) > 1 for p in self.layer_plan or ())
 
     def layer_config(self, layer_idx: int) -> "ModelConfig":
         """The configuration as layer ``layer_idx`` sees it: its own sizes where the model has a plan."""
@@ -488,6 +507,21 @@ PRESETS: dict[str, Any] = {
                         "scaling": {"factor": 2.0, "original": 256, "fast": 16.0, "slow": 1.0}}}},
             {"type": "delta", "mixer": {"heads": 2, "kv_heads": 2, "dim": 32, "vdim": 32, "conv": 4}, "mlp": None},
         ]}, dtype="float32", name="tiny-vofelix"),
+    "tiny-pegopel": lambda: ModelConfig.from_hf_dict({
+        "architecture": "Pegopel", "vocab": 288, "width": 80, "norm": {"eps": 1e-5}, "max_positions": 512, "streams": 3,
+        "loop": {"start": 1, "stop": 2, "times": 2}, "layers": [
+            {"type": "attention", "mlp": {"kind": "dense", "ff": 136}, "mixer": {
+                "heads": 4, "kv_heads": 2, "dim": 24, "vdim": 16, "conv": 4, "scale": 0.2, "bias_max": 60,
+                "mask": {"size": 20}}},
+            {"type": "attention_2", "mlp": {"kind": "dense", "ff": 96}, "mixer": {
+                "heads": 4, "kv_heads": 2, "dim": 32, "vdim": 32, "scale": 0.18, "softcap": 20.0,
+                "mask": {"size": 12, "keep_first": 3},
+                "rot": {"base": 10000.0, "dims": 16,
+                        "scaling": {"factor": 4.0, "original": 128, "fast": 16.0, "slow": 1.0}}}},
+            {"type": "attention", "mlp": None, "mixer": {
+                "heads": 2, "kv_heads": 2, "dim": 16, "vdim": 40, "conv": 2, "scale": 0.25, "bias_max": 40,
+                "mask": {"size": 30}}},
+        ]}, dtype="float32", name="tiny-pegopel"),
     "tiny-deepseek": lambda: _preset(
         name="tiny-deepseek", architecture="DeepseekV3ForCausalLM", vocab_size=512,
         hidden_size=128, intermediate_size=256, num_hidden_layers=3, num_attention_heads=4,

@@ -150,11 +150,13 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, long q_stride,
 __global__ void merge_splits_kernel(const float* __restrict__ partial_o,
                                     const float* __restrict__ partial_lse, int num_splits, int D,
                                     int Hq, __nv_bfloat16* __restrict__ out, long out_stride,
-                                    long out_head, float* __restrict__ lse_out) {
+                                    long out_head, float* __restrict__ lse_out,
+                                    const float* __restrict__ sink,
+                                    const __nv_bfloat16* __restrict__ gate, long gate_stride) {
   const long t = blockIdx.x;
   const int hq = blockIdx.y;
   const long base = (t * Hq + hq) * num_splits;
-  float M = -INFINITY;
+  float M = sink ? sink[hq] : -INFINITY;
   for (int s = 0; s < num_splits; s++) M = fmaxf(M, partial_lse[base + s]);
   if (lse_out && threadIdx.x == 0) {
     float L = 0.f;
@@ -162,8 +164,9 @@ __global__ void merge_splits_kernel(const float* __restrict__ partial_o,
       for (int s = 0; s < num_splits; s++) L += __expf(partial_lse[base + s] - M);
     lse_out[t * Hq + hq] = L > 0.f ? M + logf(L) : -INFINITY;
   }
+  const float g = gate ? 1.f / (1.f + __expf(-__bfloat162float(gate[t * gate_stride + hq]))) : 1.f;
   for (int d = threadIdx.x; d < D; d += blockDim.x) {
-    float acc = 0.f, L = 0.f;
+    float acc = 0.f, L = sink ? __expf(sink[hq] - M) : 0.f;
     if (M != -INFINITY) {
       for (int s = 0; s < num_splits; s++) {
         const float w = __expf(partial_lse[base + s] - M);
@@ -171,17 +174,18 @@ __global__ void merge_splits_kernel(const float* __restrict__ partial_o,
         acc += w * partial_o[(base + s) * D + d];
       }
     }
-    out[t * out_stride + hq * out_head + d] = __float2bfloat16(L > 0.f ? acc / L : 0.f);
+    out[t * out_stride + hq * out_head + d] = __float2bfloat16(L > 0.f ? g * acc / L : 0.f);
   }
 }
 
 int launch_merge_splits(const float* partial_o, const float* partial_lse, long T, int Hq,
                         int num_splits, int D, void* out, long out_stride, cudaStream_t stream,
-                        float* lse_out, long out_head) {
+                        float* lse_out, long out_head, const float* sink, const void* gate, long gate_stride) {
   if (T <= 0) return 0;
   dim3 grid((unsigned)T, (unsigned)Hq);
-  merge_splits_kernel<<<grid, D >= 128 ? 128 : 64, 0, stream>>>(
-      partial_o, partial_lse, num_splits, D, Hq, (__nv_bfloat16*)out, out_stride, out_head ? out_head : D, lse_out);
+  merge_splits_kernel<<<grid, D > 64 ? 128 : 64, 0, stream>>>(
+      partial_o, partial_lse, num_splits, D, Hq, (__nv_bfloat16*)out, out_stride, out_head ? out_head : D, lse_out,
+      sink, (const __nv_bfloat16*)gate, gate_stride);
   return B200_CHECK_LAUNCH();
 }
 

@@ -4,6 +4,10 @@
 //                      r += norm_post(y) (+ scale * embed[id])   (a sub-layer's output joins; a looped
 //                                                                 stack is fed the embedding again)
 //                      x  = norm_next(r), or r rounded to the activation type
+//   stream_mix       the same pass over S parallel streams per token (hyper-connections):
+//                      x_t = sum_s mix[s, t] x_s + out[t] post(y)          (a sub-layer's output joins), or
+//                      x_t = scale * embed[id] + pos[position] for all t   (start of the streams)
+//                      u   = sum_s in[s] x_s (no weights: their sum);  x = norm_next(u)
 //   side_gate        g = gelu_tanh(a) * side_embed[id, slice]    (per-layer token input)
 //   gated_head_norm  o = rms_norm(o) * w * silu(z) per head      (delta-rule read-out)
 // Either norm is a layer norm (weight, bias) or an RMS norm, statistics in fp32.  Activations, weights and
@@ -144,6 +148,135 @@ __global__ void stream_norm_kernel(const StreamParams p) {
   }
 }
 
+struct MixParams {
+  float* r;               // [T, S, W]
+  const void* y;          // [T, W] sub-layer output (post != NONE)
+  long y_stride;
+  int post;
+  const void *post_w, *post_b;
+  const float* mix;       // [S, S] from, to
+  const float* out;       // [S]
+  int emb;                // EMB_NONE or EMB_SET
+  const long* ids;        // [T]; null: row t of the table
+  const void* table;      // [rows, W]
+  long table_rows;
+  float emb_scale;
+  const long* positions;  // [T]
+  const void* pos_table;  // [pos_rows, W] or null
+  long pos_rows;
+  const float* in;        // [S] or null: ones
+  int next;
+  const void *next_w, *next_b;
+  void* x;                // [T, W]
+  int W, S, store;        // store: the streams are written back
+  float eps;
+  int* status;
+};
+
+// MAXS >= S streams of a column live in registers; one thread block per token
+template <typename T, int VEC, int PER, int MAXS>
+__global__ void __launch_bounds__(512) stream_mix_kernel(const MixParams p) {
+  __shared__ float red[32];
+  __shared__ float cf[MAXS * MAXS + 2 * MAXS];      // mix, out, in
+  const long t = blockIdx.x;
+  const int nvec = p.W / VEC, S = p.S;
+  for (int i = threadIdx.x; i < S * S + 2 * S; i += blockDim.x) {
+    if (i < S * S) cf[i / S * MAXS + i % S] = p.mix ? p.mix[i] : 0.f;
+    else if (i < S * S + S) cf[MAXS * MAXS + i - S * S] = p.out ? p.out[i - S * S] : 0.f;
+    else cf[MAXS * MAXS + MAXS + i - S * S - S] = p.in ? p.in[i - S * S - S] : 1.f;
+  }
+  float v[PER][VEC];
+#pragma unroll
+  for (int i = 0; i < PER; i++)
+#pragma unroll
+    for (int e = 0; e < VEC; e++) v[i][e] = 0.f;
+  const T *erow = nullptr, *prow = nullptr;
+  if (p.emb == EMB_SET) {
+    const long id = p.ids ? p.ids[t] : t;
+    if (id >= 0 && id < p.table_rows) erow = (const T*)p.table + id * p.W;
+    const long pos = p.pos_table ? p.positions[t] : 0;
+    if (p.pos_table && pos >= 0 && pos < p.pos_rows) prow = (const T*)p.pos_table + pos * p.W;
+    if (threadIdx.x == 0 && p.status && (!erow || (p.pos_table && !prow))) atomicCAS(p.status, 0, B200_BAD_INDEX);
+  } else if (p.post != NORM_NONE) {
+    const T* yrow = (const T*)p.y + t * p.y_stride;
+#pragma unroll
+    for (int i = 0; i < PER; i++) {
+      const int c = (int)threadIdx.x + i * (int)blockDim.x;
+      if (c < nvec) load_vec<T, VEC>(yrow + (long)c * VEC, v[i]);
+    }
+    if (p.post != NORM_PLAIN)
+      row_norm<T, VEC, PER>(v, p.post, (const T*)p.post_w, (const T*)p.post_b, p.W, p.eps, red);
+  }
+  __syncthreads();                                  // the coefficients are there
+  float* rrow = p.r + t * (long)S * p.W;
+#pragma unroll
+  for (int i = 0; i < PER; i++) {
+    const int c = (int)threadIdx.x + i * (int)blockDim.x;
+    if (c >= nvec) continue;
+    float* rc = rrow + (long)c * VEC;
+    float xs[MAXS][VEC], u[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; e++) u[e] = 0.f;
+    if (p.emb == EMB_SET) {
+      float ev[VEC], pv[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; e++) ev[e] = pv[e] = 0.f;
+      if (erow) load_vec<T, VEC>(erow + (long)c * VEC, ev);
+      if (prow) load_vec<T, VEC>(prow + (long)c * VEC, pv);
+#pragma unroll
+      for (int e = 0; e < VEC; e++) ev[e] = ev[e] * p.emb_scale + pv[e];
+      float w = 0.f;
+#pragma unroll
+      for (int s = 0; s < MAXS; s++)
+        if (s < S) {
+          w += cf[MAXS * MAXS + MAXS + s];
+          if (p.store) store_vec<float, VEC>(rc + (long)s * p.W, ev);
+        }
+#pragma unroll
+      for (int e = 0; e < VEC; e++) v[i][e] = w * ev[e];
+      continue;
+    }
+#pragma unroll
+    for (int s = 0; s < MAXS; s++)
+      if (s < S) load_vec<float, VEC>(rc + (long)s * p.W, xs[s]);
+#pragma unroll
+    for (int to = 0; to < MAXS; to++) {
+      if (to >= S) break;
+      float nv[VEC];
+      if (p.post != NORM_NONE) {
+        const float o = cf[MAXS * MAXS + to];
+#pragma unroll
+        for (int e = 0; e < VEC; e++) nv[e] = o * v[i][e];
+#pragma unroll
+        for (int s = 0; s < MAXS; s++)
+          if (s < S) {
+            const float m = cf[s * MAXS + to];
+#pragma unroll
+            for (int e = 0; e < VEC; e++) nv[e] = fmaf(m, xs[s][e], nv[e]);
+          }
+        if (p.store) store_vec<float, VEC>(rc + (long)to * p.W, nv);
+      } else {
+#pragma unroll
+        for (int e = 0; e < VEC; e++) nv[e] = xs[to][e];
+      }
+      const float w = cf[MAXS * MAXS + MAXS + to];
+#pragma unroll
+      for (int e = 0; e < VEC; e++) u[e] = fmaf(w, nv[e], u[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; e++) v[i][e] = u[e];
+  }
+  if (p.next == NORM_NONE) return;
+  if (p.next != NORM_PLAIN)
+    row_norm<T, VEC, PER>(v, p.next, (const T*)p.next_w, (const T*)p.next_b, p.W, p.eps, red);
+  T* xrow = (T*)p.x + t * p.W;
+#pragma unroll
+  for (int i = 0; i < PER; i++) {
+    const int c = (int)threadIdx.x + i * (int)blockDim.x;
+    if (c < nvec) store_vec<T, VEC>(xrow + (long)c * VEC, v[i]);
+  }
+}
+
 // a [T, D] -> out [T, D]; the table row holds one D-wide slice per layer
 template <typename T, int VEC>
 __global__ void side_gate_kernel(const T* __restrict__ a, long a_stride, const long* __restrict__ ids,
@@ -222,6 +355,32 @@ static int stream_norm_t(const StreamParams& p, long tokens, cudaStream_t stream
   return vec ? launch_stream<T, 4>(p, tokens, stream) : launch_stream<T, 1>(p, tokens, stream);
 }
 
+template <typename T, int VEC, int MAXS>
+static int launch_mix(const MixParams& p, long tokens, cudaStream_t stream) {
+  const int nvec = p.W / VEC;
+  int threads = (((nvec + 1) / 2 + 31) / 32) * 32;
+  if (threads > 512) threads = 512;
+  const int per = (nvec + threads - 1) / threads;
+  const dim3 grid((unsigned)tokens);
+  if (per <= 1) stream_mix_kernel<T, VEC, 1, MAXS><<<grid, threads, 0, stream>>>(p);
+  else if (per <= 2) stream_mix_kernel<T, VEC, 2, MAXS><<<grid, threads, 0, stream>>>(p);
+  else if (per <= 4) stream_mix_kernel<T, VEC, 4, MAXS><<<grid, threads, 0, stream>>>(p);
+  else if (per <= 16) stream_mix_kernel<T, VEC, 16, MAXS><<<grid, threads, 0, stream>>>(p);
+  else return 9740;
+  return B200_CHECK_LAUNCH();
+}
+
+template <typename T>
+static int stream_mix_t(const MixParams& p, long tokens, cudaStream_t stream) {
+  const bool vec = p.W % 4 == 0 && p.y_stride % 4 == 0 && aligned16(p.r) && aligned16(p.y) && aligned16(p.x) &&
+                   aligned16(p.table) && aligned16(p.pos_table) && aligned16(p.post_w) && aligned16(p.post_b) &&
+                   aligned16(p.next_w) && aligned16(p.next_b);
+  if (vec)
+    return p.S <= 2 ? launch_mix<T, 4, 2>(p, tokens, stream)
+                    : p.S <= 4 ? launch_mix<T, 4, 4>(p, tokens, stream) : launch_mix<T, 4, 16>(p, tokens, stream);
+  return p.S <= 4 ? launch_mix<T, 1, 4>(p, tokens, stream) : launch_mix<T, 1, 16>(p, tokens, stream);
+}
+
 template <typename T>
 static int side_gate_t(const void* a, long a_stride, const void* ids, const void* table, long table_stride,
                        long table_rows, long offset, void* out, long tokens, int D, int* status, cudaStream_t stream) {
@@ -270,6 +429,25 @@ B200_API int b200_stream_norm(void* r, const void* y, long y_stride, int post, c
   StreamParams p{(float*)r, y, y_stride, post, post_w, post_b, emb, (const long*)ids, table, table_rows, emb_scale,
                  next, next_w, next_b, x, W, eps, status};
   return dtype ? stream_norm_t<float>(p, tokens, stream) : stream_norm_t<__nv_bfloat16>(p, tokens, stream);
+}
+
+// r [tokens, S, W]; mix [S, S] and out [S] go with y, in [S] (null: ones) with the next norm; emb: 0 none,
+// 1 the streams are set to emb_scale * table[ids] + pos_table[positions]
+B200_API int b200_stream_mix(void* r, const void* y, long y_stride, int post, const void* post_w, const void* post_b,
+                             const void* mix, const void* out, int emb, const void* ids, const void* table,
+                             long table_rows, float emb_scale, const void* positions, const void* pos_table,
+                             long pos_rows, const void* in, int next, const void* next_w, const void* next_b, void* x,
+                             long tokens, int S, int W, int store, float eps, int dtype, int* status,
+                             cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (W < 1 || S < 1 || S > 16 || (post != NORM_NONE && (!y || !mix || !out)) || (next != NORM_NONE && !x)) return 9741;
+  if ((emb != EMB_NONE && emb != EMB_SET) || (emb == EMB_SET && (!table || post != NORM_NONE))) return 9742;
+  if ((post == NORM_LAYER || post == NORM_RMS) && !post_w) return 9743;
+  if (((next == NORM_LAYER || next == NORM_RMS) && !next_w) || (pos_table && !positions)) return 9744;
+  MixParams p{(float*)r, y, y_stride, post, post_w, post_b, (const float*)mix, (const float*)out, emb, (const long*)ids,
+              table, table_rows, emb_scale, (const long*)positions, pos_table, pos_rows, (const float*)in, next, next_w,
+              next_b, x, W, S, store, eps, status};
+  return dtype ? stream_mix_t<float>(p, tokens, stream) : stream_mix_t<__nv_bfloat16>(p, tokens, stream);
 }
 
 B200_API int b200_side_gate(const void* a, long a_stride, const void* ids, const void* table, long table_stride,

@@ -396,6 +396,8 @@ class LLM:
         if quantization:
             mcfg.quantization = quantization
         mcfg.seed = seed
+        if mcfg.learned_positions:           # there is no vector for a position beyond the table
+            max_model_len = min(max_model_len, mcfg.learned_positions)
         if device is None:
             device = "cuda" if torch.cuda.is_available() else "cpu"
         device_index = None

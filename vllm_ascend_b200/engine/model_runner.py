@@ -140,13 +140,14 @@ class ModelRunner:
             # the ranks of a DCP group shard one sequence of keys: they must hold the same KV heads
             tp_ = _ps.get_tp_group().world_size
             rep = max(1, tp_ // max(1, cfg.model.num_key_value_heads))
-            if cfg.model.is_hybrid or cfg.model.sliding_window or rep % self.dcp_size:
+            if cfg.model.keeps_sequence_state or cfg.model.sliding_window or rep % self.dcp_size:
                 raise NotImplementedError(
                     "decode context parallelism for grouped-query attention needs KV heads replicated over the "
                     f"DCP ranks (tensor_parallel_size / num_key_value_heads = {rep} must be a multiple of "
                     f"{self.dcp_size}), no sliding window and no recurrent layers")
         self.pcp = _ps.get_pcp_group()
-        if self.pcp.world_size > 1 and (cfg.model.use_mla or cfg.model.is_hybrid or cfg.model.is_multimodal):
+        if self.pcp.world_size > 1 and (cfg.model.use_mla or cfg.model.is_hybrid or cfg.model.is_multimodal
+                                           or cfg.model.layer_plan):
             raise NotImplementedError("prefill context parallelism is implemented for GQA decoder models")
         self._pcp_bcast = False          # this step's tokens come from PCP rank 0
         self._prompt_lp_out: dict = {}
@@ -209,6 +210,8 @@ class ModelRunner:
         total = 0
         for L in self.model.layers:
             a = L.self_attn
+            for shape in self._extra_state_shapes(a):
+                total += math.prod(shape) * torch.empty(0, dtype=self.kv_dtype).element_size()
             if getattr(a, "is_linear_attention", False):
                 cs, ss = a.state_shapes(self.max_seqs + 1)
                 n_c = 1
@@ -220,10 +223,15 @@ class ModelRunner:
                 total += n_c * (4 if self.kv_dtype == torch.float32 else 2) + n_s * 4
         return total
 
+    def _extra_state_shapes(self, attn) -> list:
+        """Per-sequence state (one row per batch row, plus a scratch row for padded graph entries) that an
+        attention layer keeps beside its pages."""
+        return attn.sequence_state_shapes(self.max_seqs + 1) if hasattr(attn, "sequence_state_shapes") else []
+
     def kv_bytes_per_block(self) -> int:
         itemsize = torch.tensor([], dtype=self.kv_dtype).element_size()
         if self.mcfg.layer_plan:             # every layer has sizes of its own
-            per_tok = sum(L.self_attn.dc + L.self_attn.dr for L in self.model.layers
+            per_tok = sum(sum(h * d for h, d in L.self_attn.kv_cache_heads()) for L in self.model.layers
                           if not getattr(L.self_attn, "is_linear_attention", False))
         else:
             per_tok = self._num_kv_layers() * sum(self._cache_widths())
@@ -280,6 +288,9 @@ class ModelRunner:
             if getattr(layer.self_attn, "is_linear_attention", False):
                 per_layer.append(None)              # recurrent state instead of a paged cache
                 continue
+            if c.layer_plan:                        # every layer has sizes of its own
+                per_layer.append([(num_blocks, self.block_size, h, d) for h, d in layer.self_attn.kv_cache_heads()])
+                continue
             if c.use_mla:
                 nb_main = 1 if self._offload_cfg().enabled else num_blocks      # host-resident: placeholders
                 a = layer.self_attn
@@ -292,6 +303,8 @@ class ModelRunner:
             per_layer.append(shapes)
         layout = self.cfg.cache.kv_layout if self.is_cuda else "NHD"
         self.kv_arena = None
+        if self.cfg.kv_transfer_config and any(self._extra_state_shapes(L.self_attn) for L in self.model.layers):
+            raise NotImplementedError("KV transfer of layers that keep a state beside their pages")
         if self.is_cuda and self.cfg.kv_transfer_config and not self.cfg.enable_sleep_mode:
             # one exportable allocation, so a decode engine in another process of this node
             # can map the whole cache through a single CUDA IPC handle
@@ -317,7 +330,8 @@ class ModelRunner:
             self.kv_caches.append(tuple(
                 ops.alloc_kv_cache(s[0], s[1], s[2], s[3], self.kv_dtype, self.device, layout,
                                    arena=self.kv_arena)
-                for s in shapes))
+                for s in shapes) + tuple(torch.zeros(s, dtype=self.kv_dtype, device=self.device)
+                                         for s in self._extra_state_shapes(layer.self_attn)))
 
     # ------------------------------------------------------------------ persistent batch
     def _offload_cfg(self):
@@ -503,8 +517,8 @@ class ModelRunner:
             meta.extra = dict(meta.extra or {}, tok_rows=tr, positions_cpu=pc_)
         if self.mm is not None:
             self.mm.prepare(reqs, starts, q_lens, cu, pos, req_idx, T, Tp, meta)
-        if self.mcfg.is_hybrid:
-            # recurrent layers index their state by the request's batch row; padded rows use the
+        if self.mcfg.keeps_sequence_state:
+            # such layers index their state by the request's batch row; padded rows use the
             # scratch row
             hs = self._h_state
             hs[0, :B] = torch.from_numpy(rows.astype(np.int32))
@@ -515,7 +529,7 @@ class ModelRunner:
             self.state_meta[:, :Bp].copy_(hs[:, :Bp], non_blocking=True)
             meta.state_slots = self.state_meta[0, :Bp]
             meta.has_initial_state = self.state_meta[1, :Bp]
-        if self.is_cuda and not self.mcfg.use_mla:
+        if self.is_cuda and not self.mcfg.use_mla and not self.mcfg.layer_plan:
             a = self._attn_layer()
             G = a.Hq // a.Hkv
             tok_per_tile = max(1, 128 // G)
@@ -1201,7 +1215,11 @@ class ModelRunner:
             if not self.capture_sizes:
                 return
         # scratch for split-KV partials must exist before capture
-        if not self.mcfg.use_mla:
+        if self.mcfg.layer_plan:
+            for a in {id(L.self_attn): L.self_attn for L in self.model.layers}.values():
+                if hasattr(a, "reserve_decode_scratch"):
+                    a.reserve_decode_scratch(self.device, self.capture_sizes, self.max_model_len)
+        elif not self.mcfg.use_mla:
             a = self._attn_layer()
             worst = 0
             for s in self.capture_sizes:

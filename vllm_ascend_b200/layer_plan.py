@@ -6,7 +6,7 @@ it has, the mixer's sizes and constants, and whether a feed-forward follows.  It
 ``ModelConfig`` fields of that layer (``ModelConfig.layer_config(i)`` applies them), so that the mixers read
 a plain ``ModelConfig`` whether or not the model has a plan.
 
-This module turns the configuration format of the Vofelix decoder into such a plan."""
+This module turns the configuration formats of the Vofelix and Pegopel decoders into such plans."""
 from __future__ import annotations
 
 from typing import Any, Callable, Optional
@@ -42,13 +42,43 @@ _VOFELIX_MIXERS: dict[str, tuple[str, Callable[[dict], dict]]] = {
     "latent_attention": ("latent", _latent), "delta": ("delta", _delta)}
 
 
-def vofelix_fields(d: dict) -> dict[str, Any]:
-    """``ModelConfig`` fields of a Vofelix configuration."""
-    plan, kinds = [], []
+def _attention(m: dict) -> dict:
+    """Options every paged grouped-query mixer of a plan has."""
+    heads, kv = int(m["heads"]), int(m["kv_heads"])
+    if kv < 1 or heads % kv:
+        raise ValueError(f"{heads} query heads do not share {kv} key / value heads")
+    mask = m.get("mask") or {}
+    return dict(num_attention_heads=heads, num_key_value_heads=kv, head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]),
+                attention_multiplier=float(m["scale"]), sliding_window=int(mask["size"]) if mask.get("size") else None,
+                attn_keep_first=int(mask.get("keep_first") or 0), qk_norm_full=True, rotary_dims=0)
+
+
+def _biased(m: dict) -> dict:
+    return dict(_attention(m), attn_conv_kernel=int(m.get("conv") or 0), attn_distance_max=int(m["bias_max"]),
+                attention_sink=True)
+
+
+def _shared_kv(m: dict) -> dict:
+    rot = m["rot"]
+    if int(m["vdim"]) != int(m["dim"]):
+        raise ValueError("values that are the keys have the keys' size: vdim must equal dim")
+    if int(rot["dims"]) % 2 or int(rot["dims"]) > int(m["dim"]):
+        raise ValueError(f"cannot rotate {rot['dims']} of {m['dim']} dimensions")
+    return dict(_attention(m), attn_values_from_keys=True, rotary_dims=int(rot["dims"]),
+                rope_theta=float(rot["base"]), rope_scaling=_yarn(rot.get("scaling")), attn_sink_value=0.0,
+                attn_softcap=float(m["softcap"]) if m.get("softcap") else None, attn_head_gate=True)
+
+
+_PEGOPEL_MIXERS: dict[str, tuple[str, Callable[[dict], dict]]] = {
+    "attention": ("attention", _biased), "attention_2": ("attention", _shared_kv)}
+
+
+def _read_layers(d: dict, mixers: dict) -> list[dict]:
+    plan = []
     for i, layer in enumerate(d["layers"]):
-        if layer["type"] not in _VOFELIX_MIXERS:
+        if layer["type"] not in mixers:
             raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
-        mixer, read = _VOFELIX_MIXERS[layer["type"]]
+        mixer, read = mixers[layer["type"]]
         over = read(layer["mixer"])
         mlp = layer.get("mlp")
         if mlp is not None:
@@ -56,38 +86,66 @@ def vofelix_fields(d: dict) -> dict[str, Any]:
                 raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
             over["intermediate_size"] = int(mlp["ff"])
         plan.append({"mixer": mixer, "mlp": mlp is not None, "over": over})
-        kinds.append("linear_attention" if mixer == "delta" else "full_attention")
-    loop = d.get("loop")
-    if loop:
-        loop = (int(loop["start"]), int(loop["stop"]), int(loop["times"]))
-        if not (0 <= loop[0] < loop[1] <= len(plan)) or loop[2] < 1:
-            raise ValueError(f"loop {loop} does not fit {len(plan)} layers")
-    width = int(d["width"])
+    return plan
 
-    def largest(name: str, default: int) -> int:
-        return max([default] + [p["over"].get(name) or 0 for p in plan])
-    heads = largest("num_attention_heads", 0) or largest("linear_num_value_heads", 1)
+
+def _read_loop(d: dict, num_layers: int) -> Optional[tuple]:
+    loop = d.get("loop")
+    if not loop:
+        return None
+    loop = (int(loop["start"]), int(loop["stop"]), int(loop["times"]))
+    if not (0 <= loop[0] < loop[1] <= num_layers) or loop[2] < 1:
+        raise ValueError(f"loop {loop} does not fit {num_layers} layers")
+    return loop
+
+
+def _largest(plan: list, name: str, default: int) -> int:
+    return max([default] + [p["over"].get(name) or 0 for p in plan])
+
+
+def vofelix_fields(d: dict) -> dict[str, Any]:
+    """``ModelConfig`` fields of a Vofelix configuration."""
+    plan = _read_layers(d, _VOFELIX_MIXERS)
+    kinds = ["linear_attention" if p["mixer"] == "delta" else "full_attention" for p in plan]
+    width = int(d["width"])
+    heads = _largest(plan, "num_attention_heads", 0) or _largest(plan, "linear_num_value_heads", 1)
     fields: dict[str, Any] = dict(
         vocab_size=int(d["vocab"]), hidden_size=width, num_hidden_layers=len(plan), layer_plan=plan,
-        layer_loop=tuple(loop) if loop else None, layer_types=kinds,
+        layer_loop=_read_loop(d, len(plan)), layer_loop_refeed=True, layer_types=kinds,
         full_attention_interval=2 if "linear_attention" in kinds else 0,
-        num_attention_heads=heads, num_key_value_heads=heads, intermediate_size=largest("intermediate_size", width),
+        num_attention_heads=heads, num_key_value_heads=heads,
+        intermediate_size=_largest(plan, "intermediate_size", width),
         use_mla=True, hidden_act="gelu_pytorch_tanh", norm_type="layer", sandwich_norm=True, attention_sink=True,
         rms_norm_eps=float(d["norm"]["eps"]), embed_scale=float(d["embedding"]["scale"]),
         token_side_dim=int((d.get("token_side") or {}).get("dim", 0)), tie_word_embeddings=False)
     for name in ("kv_lora_rank", "qk_nope_head_dim", "qk_rope_head_dim", "v_head_dim", "head_dim",
                  "linear_num_key_heads", "linear_num_value_heads", "linear_key_head_dim", "linear_value_head_dim"):
-        fields[name] = largest(name, 0)
+        fields[name] = _largest(plan, name, 0)
     return fields
 
 
+def pegopel_fields(d: dict) -> dict[str, Any]:
+    """``ModelConfig`` fields of a Pegopel configuration."""
+    plan = _read_layers(d, _PEGOPEL_MIXERS)
+    width = int(d["width"])
+    return dict(
+        vocab_size=int(d["vocab"]), hidden_size=width, num_hidden_layers=len(plan), layer_plan=plan,
+        layer_loop=_read_loop(d, len(plan)), layer_types=["full_attention"] * len(plan),
+        num_attention_heads=_largest(plan, "num_attention_heads", 1),
+        num_key_value_heads=_largest(plan, "num_key_value_heads", 1), head_dim=_largest(plan, "head_dim", 1),
+        v_head_dim=_largest(plan, "v_head_dim", 1), intermediate_size=_largest(plan, "intermediate_size", width),
+        hidden_act="gelu_pytorch_tanh", norm_type="rms", rms_norm_eps=float(d["norm"]["eps"]),
+        residual_streams=int(d.get("streams") or 1), learned_positions=int(d["max_positions"]),
+        max_position_embeddings=int(d["max_positions"]), tie_word_embeddings=True)
+
+
 #: architecture name -> reader of its configuration format
-PLAN_FORMATS: dict[str, Callable[[dict], dict]] = {"Vofelix": vofelix_fields}
+PLAN_FORMATS: dict[str, Callable[[dict], dict]] = {"Vofelix": vofelix_fields, "Pegopel": pegopel_fields}
 
 
 def run_order(num_layers: int, loop: Optional[tuple]) -> tuple[list[int], set[int]]:
-    """Layer index of every layer run, and the runs in front of which the embedding output joins the stream
-    again (the first run of every pass through the loop but the first pass)."""
+    """Layer index of every layer run, and the first run of every pass through the loop but the first pass
+    (where ``layer_loop_refeed`` adds the embedding output to the stream again)."""
     if not loop:
         return list(range(num_layers)), set()
     start, stop, times = loop

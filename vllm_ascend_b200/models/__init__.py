@@ -33,7 +33,8 @@ def _planned_lm(cfg, device, **kw):
     return PlannedCausalLM(cfg, device, **kw)
 
 
-register_model("Vofelix", _planned_lm)
+for _arch in ("Vofelix", "Pegopel"):
+    register_model(_arch, _planned_lm)
 
 
 def _qwen_vl(cfg, device, **kw):

@@ -2,15 +2,19 @@
 
 What the plan's layers have in common:
 
-* the residual stream is fp32; a norm stands in front of and behind every sub-layer,
-  ``r += post(f(pre(r)))``, and one kernel does the token-wise work between two sub-layers
+* the residual stream is fp32; a norm stands in front of every sub-layer and, with ``sandwich_norm``, behind
+  it, ``r += post(f(pre(r)))``, and one kernel does the token-wise work between two sub-layers
   (``ops.stream.stream_norm``);
-* mixers are the framework's: latent attention (``MLAAttention`` with window and sink) and the gated delta
-  rule (``GatedDeltaNet``), each built from ``ModelConfig.layer_config(i)``;
+* with ``residual_streams`` there are several parallel streams per token, mixed by learned weights at every
+  sub-layer (``ops.stream.stream_mix``);
+* mixers are the framework's: latent attention (``MLAAttention`` with window and sink), the gated delta
+  rule (``GatedDeltaNet``) and paged attention with options (``VariantAttention``), each built from
+  ``ModelConfig.layer_config(i)``;
+* optional learned positions (``learned_positions``): a vector per position added to the embeddings;
 * optional per-layer token input (``token_side_dim``): a slice of a second embedding table, gated by the
   stream, projected, RMS-normed and added after the layer's sub-layers;
-* optional loop (``layer_loop``): some layers run several times with the same weights; before each pass but
-  the first the embedding output is added to the stream again.
+* optional loop (``layer_loop``): some layers run several times with the same weights; with
+  ``layer_loop_refeed`` the embedding output is added to the stream again before each pass but the first.
 
 ``layers`` lists the layer *runs* in execution order: a looped layer appears once per pass, so every pass
 has its own entry in the runner's cache list while the parameters are shared.
@@ -23,17 +27,23 @@ import torch
 
 from ..config import ModelConfig
 from ..layer_plan import run_order
-from ..ops.stream import PLAIN, NormSpec, side_gate, stream_norm
+from ..ops.stream import PLAIN, NormSpec, StreamMix, side_gate, stream_mix, stream_norm
 from ..parallel import state as pstate
 from .gdn import GatedDeltaNet
 from .layers import (Linear, ParallelLMHead, ParamFactory, SwiGLUMLP, TPComm, VocabParallelEmbedding, copy_exact)
 from .transformer import MLAAttention
+from .variant_attention import VariantAttention
 
 #: mixer kind of a plan -> constructor (param factory, layer config, layer index, comm, max positions)
 MIXERS = {
     "latent": lambda pf, cfg, i, comm, max_pos: MLAAttention(pf, cfg, i, comm, max_pos),
     "delta": lambda pf, cfg, i, comm, max_pos: GatedDeltaNet(pf, cfg, i, comm),
+    "attention": lambda pf, cfg, i, comm, max_pos: VariantAttention(pf, cfg, i, comm, max_pos),
 }
+
+
+#: checkpoint name -> attribute of a sub-layer's stream mixing weights
+_MIX_PARTS = {"in": "read", "out": "write", "mix": "mix"}
 
 
 def _norm(pf: ParamFactory, cfg: ModelConfig, kind: Optional[str] = None) -> NormSpec:
@@ -56,6 +66,15 @@ class TokenSide:
         return self.proj(side_gate(self.gate(x), ids, self.table, self.offset))
 
 
+def _stream_mix(pf: ParamFactory, prefix: str, streams: int) -> StreamMix:
+    """Mixing weights of a sub-layer.  Random models start near one stream per residual sum."""
+    f32 = torch.float32
+    mix = torch.eye(streams, dtype=f32, device=pf.device)
+    if streams > 1:
+        mix = 0.9 * mix + pf.normal(f"{prefix}.mix", (streams, streams), std=0.05, dtype=f32)
+    return StreamMix(pf.ones((streams,), f32) / streams, pf.ones((streams,), f32), mix.contiguous())
+
+
 class PlannedLayer:
     def __init__(self, pf: ParamFactory, cfg: ModelConfig, idx: int, comm: TPComm, max_pos: int,
                  side_table: Optional[torch.Tensor]):
@@ -65,10 +84,13 @@ class PlannedLayer:
             raise ValueError(f"layer {idx}: heads do not divide over {comm.size} tensor-parallel ranks")
         self.idx = idx
         self.self_attn = MIXERS[entry["mixer"]](pf, lcfg, idx, comm, max_pos)
-        self.norm1, self.norm1b = _norm(pf, cfg), _norm(pf, cfg)
-        self.mlp = self.norm2 = self.norm2b = None
+        sandwich, streams = cfg.sandwich_norm, cfg.residual_streams
+        self.norm1, self.norm1b = _norm(pf, cfg), _norm(pf, cfg) if sandwich else PLAIN
+        self.hc1 = _stream_mix(pf, f"model.layers.{idx}.hc1", streams) if streams else None
+        self.mlp = self.norm2 = self.norm2b = self.hc2 = None
         if entry["mlp"]:
-            self.norm2, self.norm2b = _norm(pf, cfg), _norm(pf, cfg)
+            self.norm2, self.norm2b = _norm(pf, cfg), _norm(pf, cfg) if sandwich else PLAIN
+            self.hc2 = _stream_mix(pf, f"model.layers.{idx}.hc2", streams) if streams else None
             self.mlp = SwiGLUMLP(pf, f"model.layers.{idx}.mlp", cfg.hidden_size, lcfg.intermediate_size, comm,
                                  act=cfg.hidden_act)
         self.side = TokenSide(pf, cfg, idx, side_table) if side_table is not None else None
@@ -77,7 +99,10 @@ class PlannedLayer:
         out = {"norm1": self.norm1, "norm1b": self.norm1b}
         if self.mlp is not None:
             out.update(norm2=self.norm2, norm2b=self.norm2b)
-        return out
+        return {k: n for k, n in out.items() if n is not PLAIN}
+
+    def mixes(self) -> dict[str, StreamMix]:
+        return {k: m for k, m in (("hc1", self.hc1), ("hc2", self.hc2)) if m is not None}
 
 
 class PlannedCausalLM:
@@ -111,14 +136,22 @@ class PlannedCausalLM:
         self.side_embed = None
         if cfg.token_side_dim:
             self.side_embed = pf.normal("model.side_embed", (cfg.vocab_size, cfg.num_hidden_layers * cfg.token_side_dim))
+        self.pos_embed = None
+        if cfg.learned_positions:
+            self.pos_embed = pf.normal("model.pos_embed", (cfg.learned_positions, cfg.hidden_size))
         max_pos = max(max_model_len, 16)
         self.unique_layers = [PlannedLayer(pf, cfg, i, self.comm, max_pos, self.side_embed)
                               for i in range(cfg.num_hidden_layers)]
-        order, self.fed_again = run_order(cfg.num_hidden_layers, cfg.layer_loop)
+        order, again = run_order(cfg.num_hidden_layers, cfg.layer_loop)
+        self.fed_again = again if cfg.layer_loop_refeed else set()
         self.layers = [self.unique_layers[i] for i in order]
         self.norm = _norm(pf, cfg)
-        head = VocabParallelEmbedding(pf, "lm_head", cfg.vocab_size, cfg.hidden_size, self.comm)
-        self.lm_head = ParallelLMHead(head)
+        if cfg.residual_streams and (cfg.token_side_dim or self.fed_again):
+            raise NotImplementedError("parallel streams take neither a token side input nor a second embedding feed")
+        if cfg.learned_positions and not cfg.residual_streams:
+            raise NotImplementedError("learned positions join the embeddings of decoders with residual streams")
+        self.lm_head = ParallelLMHead(self.embed_tokens if cfg.tie_word_embeddings else VocabParallelEmbedding(
+            pf, "lm_head", cfg.vocab_size, cfg.hidden_size, self.comm))
 
     # -- forward ---------------------------------------------------------
     def forward(self, input_ids: torch.Tensor, meta, kv_caches: list, intermediate=None,
@@ -132,6 +165,8 @@ class PlannedCausalLM:
             emb = dict(embed=self.embed_tokens(input_ids), embed_scale=cfg.embed_scale)
         else:
             emb = dict(embed=self.embed_tokens.weight[:cfg.vocab_size], ids=input_ids, embed_scale=cfg.embed_scale)
+        if cfg.residual_streams:
+            return self._forward_streams(T, emb, None if inputs_embeds is not None else self.pos_embed, meta, kv_caches)
         r = torch.empty((T, cfg.hidden_size), dtype=torch.float32, device=input_ids.device)
         x = stream_norm(r, None, None, self.layers[0].norm1, eps, dtype, embed_set=True, **emb)
         last = len(self.layers) - 1
@@ -152,6 +187,28 @@ class PlannedCausalLM:
         self.stream = r if self.layer_hook is not None else None
         return x
 
+    def _forward_streams(self, T: int, emb: dict, pos_table: Optional[torch.Tensor], meta, kv_caches: list):
+        """Layers on ``residual_streams`` parallel streams: a sub-layer reads a weighted sum of them, and its output
+        and the old streams make the new ones."""
+        eps, dtype, layers = self.cfg.rms_norm_eps, self.dtype, self.layers
+        r = torch.empty((T, self.cfg.residual_streams, self.cfg.hidden_size), dtype=torch.float32, device=self.device)
+        x = stream_mix(r, None, None, None, layers[0].hc1, layers[0].norm1, eps, dtype, pos_table=pos_table,
+                       positions=meta.positions[:T], **emb)
+        for run, (layer, cache) in enumerate(zip(layers, kv_caches)):
+            y, post, joined = layer.self_attn(x, meta, cache), layer.norm1b, layer.hc1
+            if layer.mlp is not None:
+                x = stream_mix(r, y, post, joined, layer.hc2, layer.norm2, eps, dtype)
+                y, post, joined = layer.mlp(x), layer.norm2b, layer.hc2
+            nxt = layers[run + 1] if run + 1 < len(layers) else None
+            if self.layer_hook is not None:
+                stream_mix(r, y, post, joined, None, None, eps, dtype)
+                self.stream = r.sum(1)
+                self.layer_hook(run)
+                y = post = joined = None
+            x = stream_mix(r, y, post, joined, nxt and nxt.hc1, nxt.norm1 if nxt else self.norm, eps, dtype,
+                           store=nxt is not None)
+        return x
+
     __call__ = forward
 
     def compute_logits(self, hidden: torch.Tensor) -> torch.Tensor:
@@ -159,6 +216,8 @@ class PlannedCausalLM:
 
     def embed_input_ids(self, input_ids: torch.Tensor) -> torch.Tensor:
         """Rows of the embedding output, as ``inputs_embeds`` takes them."""
+        if self.pos_embed is not None:
+            raise NotImplementedError("the embedding output depends on the positions as well")
         return self.embed_tokens(input_ids) * self.cfg.embed_scale
 
     # -- parameters --------------------------------------------------------
@@ -166,13 +225,21 @@ class PlannedCausalLM:
         yield "model.embed_tokens.weight", self.embed_tokens.weight
         if self.side_embed is not None:
             yield "model.side_embed.weight", self.side_embed
+        if self.pos_embed is not None:
+            yield "model.pos_embed.weight", self.pos_embed
         for L in self.unique_layers:
             p, a = f"model.layers.{L.idx}", L.self_attn
             for name, n in L.norms().items():
                 yield f"{p}.{name}.weight", n.weight
                 if n.bias is not None:
                     yield f"{p}.{name}.bias", n.bias
-            for attr in ("in_proj_qkvz", "in_proj_ba", "out_proj", "q_proj", "kv_a_proj", "kv_b_proj", "o_proj"):
+            for name, m in L.mixes().items():
+                for n in m.__slots__:
+                    yield f"{p}.{name}.{n}", getattr(m, n)
+            if isinstance(a, VariantAttention):
+                for n, t in a.named_tensors():
+                    yield f"{p}.self_attn.{n}", t
+            for attr in () if isinstance(a, VariantAttention) else ("in_proj_qkvz", "in_proj_ba", "out_proj", "q_proj", "kv_a_proj", "kv_b_proj", "o_proj"):
                 lin = getattr(a, attr, None)
                 if isinstance(lin, Linear):
                     for n, t in lin.named_tensors():
@@ -180,7 +247,7 @@ class PlannedCausalLM:
             if getattr(a, "is_linear_attention", False):
                 for n, t in a.named_tensors():
                     yield f"{p}.self_attn.{n}", t
-            else:
+            elif isinstance(a, MLAAttention):
                 yield f"{p}.self_attn.kv_a_norm.weight", a.kv_a_norm.weight
                 if a.sink is not None:
                     yield f"{p}.self_attn.sink", a.sink
@@ -195,7 +262,8 @@ class PlannedCausalLM:
         yield "model.norm.weight", self.norm.weight
         if self.norm.bias is not None:
             yield "model.norm.bias", self.norm.bias
-        yield "lm_head.weight", self.lm_head.weight
+        if not self.cfg.tie_word_embeddings:
+            yield "lm_head.weight", self.lm_head.weight
 
     def num_parameters(self) -> int:
         return sum(t.numel() for _, t in self.named_parameters())
@@ -205,13 +273,18 @@ class PlannedCausalLM:
         """Names of the tensors a checkpoint of this model has."""
         def norm(name, n):
             return {name} | ({name + ".b"} if n.bias is not None else set())
-        out = {"embed", "head"} | norm("final.norm", self.norm)
+        out = {"embed"} | norm("final.norm", self.norm)
+        if not self.cfg.tie_word_embeddings:
+            out.add("head")
+        if self.pos_embed is not None:
+            out.add("pos")
         if self.side_embed is not None:
             out.add("side.embed")
         for L in self.unique_layers:
             p = f"l{L.idx}."
             for name, n in L.norms().items():
                 out |= norm(p + name, n)
+            out |= {f"{p}{name}.{part}" for name in L.mixes() for part in _MIX_PARTS}
             out |= {p + "mix." + part for part in L.self_attn.parts()}
             if L.mlp is not None:
                 out |= {p + "mlp." + part for part in ("gate", "up", "down")}
@@ -221,6 +294,8 @@ class PlannedCausalLM:
 
     def check_loaded(self, loaded: set[str]) -> None:
         missing = sorted(self.tensor_names() - loaded)
+        if self.cfg.residual_streams == 1:           # one stream without weights is a plain residual sum
+            missing = [n for n in missing if ".hc" not in n]
         if missing:
             raise ValueError(f"checkpoint lacks {len(missing)} tensors: {', '.join(missing[:8])}")
 
@@ -236,7 +311,7 @@ class PlannedCausalLM:
                 self._load_one(name, w)
             loaded.add(name)
         for L in self.unique_layers:
-            if isinstance(L.self_attn, MLAAttention):
+            if hasattr(L.self_attn, "process_weights_after_loading"):
                 L.self_attn.process_weights_after_loading()
         return loaded
 
@@ -252,6 +327,8 @@ class PlannedCausalLM:
             rows = w[e.start:e.start + e.shard]
             e.weight[:rows.shape[0]].copy_(rows)
             return None
+        if name == "pos":
+            return copy_exact(self.pos_embed, w, name)
         if name == "side.embed":
             return copy_exact(self.side_embed, w, name)
         if name.startswith("final.norm"):
@@ -261,6 +338,8 @@ class PlannedCausalLM:
         group, _, part = rest.partition(".")
         if group == "mix":
             return L.self_attn.load_part(part, w)
+        if group in L.mixes():
+            return copy_exact(getattr(L.mixes()[group], _MIX_PARTS[part]), w, name)
         if group == "side":
             return norm(L.side.norm, "") if part == "norm" else copy_exact(getattr(L.side, part).weight, w, name)
         if group == "mlp":

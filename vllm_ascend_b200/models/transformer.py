@@ -317,6 +317,15 @@ class MLAAttention:
             return None
         raise KeyError(part)
 
+    def kv_cache_heads(self) -> list[tuple[int, int]]:
+        """(heads, width) of the paged tensors: latent, rotated key part."""
+        return [(1, self.dc), (1, self.dr)]
+
+    def reserve_decode_scratch(self, device, batch_sizes: list, max_keys: int) -> None:
+        """Split-KV scratch of decode graphs, allocated before their capture."""
+        from ..attention.mla import reserve_mla_scratch
+        reserve_mla_scratch(device, batch_sizes[-1], self.H, self.dc)
+
     def parts(self) -> list[str]:
         return ["q", "dkv", "dkv.norm", "uk", "uv", "o"] + (["sink"] if self.sink is not None else [])
 

@@ -13,6 +13,8 @@ from .. import _native
 
 P, I, L, Fl = c_void_p, c_int, c_long, c_float
 _native.register_signature("b200_stream_norm", [P, P, L, I, P, P, I, P, P, L, Fl, I, P, P, P, L, I, Fl, I, P, P])
+_native.register_signature("b200_stream_mix", [P, P, L, I, P, P, P, P, I, P, P, L, Fl, P, P, L, P, I, P, P, P, L, I, I, I,
+                                               Fl, I, P, P])
 _native.register_signature("b200_side_gate", [P, L, P, P, L, L, L, P, L, I, I, P, P])
 _native.register_signature("b200_gated_head_norm", [P, P, L, P, P, L, I, I, Fl, I, P])
 
@@ -92,6 +94,73 @@ def stream_norm(r: torch.Tensor, y: Optional[torch.Tensor], post: Optional[NormS
         _native.ptr(nxt.bias if nxt else None), _native.ptr(x), T, W, float(eps), code,
         _native.status_word(r.device).data_ptr(), _native.stream_ptr())
     _native.check(rc, "stream_norm")
+    _native.count_launch()
+    return x
+
+
+class StreamMix:
+    """How a sub-layer reads from and writes to S parallel streams (fp32): input sum_s read[s] x_s; afterwards
+    x_t = sum_s mix[s, t] x_s + write[t] y."""
+    __slots__ = ("read", "write", "mix")
+
+    def __init__(self, read: torch.Tensor, write: torch.Tensor, mix: torch.Tensor):
+        self.read, self.write, self.mix = read, write, mix
+
+
+def stream_mix(r: torch.Tensor, y: Optional[torch.Tensor], post: Optional[NormSpec], joined: Optional[StreamMix],
+               reader: Optional[StreamMix], nxt: Optional[NormSpec], eps: float, dtype: torch.dtype,
+               embed: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None, embed_scale: float = 1.0,
+               pos_table: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None,
+               store: bool = True) -> Optional[torch.Tensor]:
+    """One token-wise pass over ``r`` (fp32 [T, S, W], S parallel residual streams, updated in place):
+
+        x_t = sum_s joined.mix[s, t] x_s + joined.write[t] post(y)      when a sub-layer output ``y`` is given
+        x_t = embed_scale * embed[ids] + pos_table[positions]           when ``embed`` is given
+        return nxt(sum_s reader.read[s] x_s) as ``dtype``               (reader None: the sum; nxt None: nothing)
+
+    ``store`` False: the streams are not needed afterwards and may be left as they were."""
+    T, S, W = r.shape
+    if r.dtype != torch.float32 or not r.is_contiguous():
+        raise TypeError("the residual streams are a contiguous fp32 tensor")
+    if not r.is_cuda:
+        x = r
+        if embed is not None:
+            e = (embed if ids is None else embed[ids]).float() * embed_scale
+            if pos_table is not None:
+                if positions.numel() and (int(positions.max()) >= pos_table.shape[0] or int(positions.min()) < 0):
+                    raise IndexError("position outside the position table")
+                e = e + pos_table[positions].float()
+            x = e[:, None].expand(T, S, W)
+        elif y is not None:
+            x = torch.einsum("tsw,sz->tzw", r, joined.mix) + joined.write[:, None] * _norm_ref(y.float(), post, eps)[:, None]
+        u = x.sum(1) if reader is None else torch.einsum("s,tsw->tw", reader.read, x)
+        if store and x is not r:
+            r.copy_(x)
+        return None if nxt is None else _norm_ref(u, nxt, eps).to(dtype)
+    code = _dtype_code(dtype)
+    for t in (y, embed, pos_table, *((post.weight, post.bias) if post else ()), *((nxt.weight, nxt.bias) if nxt else ())):
+        if t is not None and t.dtype != dtype:
+            raise TypeError(f"stream_mix: {t.dtype} operand beside {dtype} activations")
+    for m in (joined, reader):
+        if m is not None and not (m.read.dtype == m.write.dtype == m.mix.dtype == torch.float32):
+            raise TypeError("stream_mix: the mixing weights are fp32")
+    if y is not None and y.stride(-1) != 1:
+        y = y.contiguous()
+    if embed is not None and not embed.is_contiguous():
+        embed = embed.contiguous()
+    x = None if nxt is None else torch.empty((T, W), dtype=dtype, device=r.device)
+    has = y is not None
+    rc = _native.lib().b200_stream_mix(
+        r.data_ptr(), _native.ptr(y), 0 if y is None else y.stride(0), _KIND[post.kind] if has else 0,
+        _native.ptr(post.weight if has else None), _native.ptr(post.bias if has else None),
+        _native.ptr(joined.mix if has else None), _native.ptr(joined.write if has else None), int(embed is not None),
+        _native.ptr(ids), _native.ptr(embed), 0 if embed is None else embed.shape[0], float(embed_scale),
+        _native.ptr(positions if pos_table is not None else None), _native.ptr(pos_table),
+        0 if pos_table is None else pos_table.shape[0], _native.ptr(reader.read if reader else None),
+        0 if nxt is None else _KIND[nxt.kind], _native.ptr(nxt.weight if nxt else None),
+        _native.ptr(nxt.bias if nxt else None), _native.ptr(x), T, S, W, int(store), float(eps), code,
+        _native.status_word(r.device).data_ptr(), _native.stream_ptr())
+    _native.check(rc, "stream_mix")
     _native.count_launch()
     return x
 

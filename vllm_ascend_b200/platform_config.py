@@ -362,11 +362,11 @@ def check_and_update_config(engine_cfg) -> B200Config:
         cc.cudagraph_mode = "NONE"        # token counts differ per replica and are padded per step
     _validate_eplb(cfg.eplb_config, mc.is_moe, pc.enable_expert_parallel)
     _validate_scheduler_ext(cfg.scheduler_config, engine_cfg, dp_size)
-    if mc.is_hybrid and engine_cfg.speculative_config:
-        # a rejected draft token has already advanced the recurrent state and cannot be taken back
-        raise ValueError("speculative decoding is not supported for models with recurrent (linear-attention) layers")
-    if mc.is_hybrid and engine_cfg.cache.enable_prefix_caching:
-        # a recurrent state is not addressable by block: a cached prefix could not restore it
+    if mc.keeps_sequence_state and engine_cfg.speculative_config:
+        # a rejected draft token has already advanced the state and cannot be taken back
+        raise ValueError("speculative decoding is not supported for models whose layers keep a state per sequence")
+    if mc.keeps_sequence_state and engine_cfg.cache.enable_prefix_caching:
+        # such a state is not addressable by block: a cached prefix could not restore it
         engine_cfg.cache.enable_prefix_caching = False
     if cfg.weight_offload_config.enabled:
         cc.cudagraph_mode = "NONE"        # offloaded weights rotate through device buffers

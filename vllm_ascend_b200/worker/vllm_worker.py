@@ -188,8 +188,8 @@ class B200VllmWorker(_WorkerBase):
         these; the cache tensors themselves are allocated by this package's runner."""
         from vllm.v1.kv_cache_interface import FullAttentionSpec
         m, r = self.cfg.model, self.runner
-        if m.is_hybrid:
-            raise NotImplementedError("hybrid linear-attention models run on the standalone engine "
+        if m.keeps_sequence_state or m.layer_plan:
+            raise NotImplementedError("hybrid and plan-built models run on the standalone engine "
                                       "(vllm_ascend_b200.LLM), not yet under a host vLLM")
         bs = self.cfg.cache.block_size
         specs = {}
