@@ -29,14 +29,15 @@ def softmax_with_sink(s, sink):
     return e / (e.sum(-1, keepdim=True) + torch.exp(sink[:, None] - top))
 
 
-def attend(q, k, v, scale, size=None, keep_first=0, softcap=None, bias=None, largest=None, sink=None):
-    """q [n, H, d], k [n, G, d], v [n, G, vd] of one whole sequence -> [n, H, vd].  ``bias`` [rows, H]."""
+def attend(q, k, v, scale, size=None, keep_first=0, softcap=None, bias=None, largest=None, sink=None, rows=None):
+    """q [n, H, d], k [n, G, d], v [n, G, vd] of one whole sequence -> [n, H, vd].  ``bias`` [buckets, H];
+    ``rows``: positions to compute (all)."""
     n, H, _ = q.shape
     owner = [h // (H // k.shape[1]) for h in range(H)]          # key / value head of a query head
     k, v = k[:, owner], v[:, owner]
     row = None if bias is None else torch.tensor([distance_bucket(m, bias.shape[0], largest) for m in range(n)])
     out = torch.zeros(n, H, v.shape[2], dtype=q.dtype)
-    for i in range(n):
+    for i in range(n) if rows is None else rows:
         js = torch.tensor([j for j in range(n) if visible(i, j, size, keep_first)])
         s = torch.einsum("hd,jhd->hj", q[i], k[js]) * scale
         if softcap:

@@ -258,6 +258,69 @@ def variant_attention_simple(q, k_cache, v_cache, meta, o: AttnOptions, gate=Non
     return out
 
 
+def _tc_ok(q, k_cache, v_cache, out) -> bool:
+    """True when the tcgen05 kernels take these tensors (TMA: 16-byte strides and bases)."""
+    D, Dv, bs = q.shape[2], v_cache.shape[3], k_cache.shape[1]
+    strides = [q.stride(0), out.stride(0), *k_cache.stride()[:3], *v_cache.stride()[:3]]
+    return (q.dtype == torch.bfloat16 and D % 8 == 0 and Dv % 8 == 0 and 8 <= D <= 128 and 8 <= Dv <= 128
+            and q.shape[1] // k_cache.shape[2] <= 128 and bs >= 8 and (128 % bs == 0 or bs % 128 == 0)
+            and all(x % 8 == 0 for x in strides) and all(t.data_ptr() % 16 == 0 for t in (q, k_cache, v_cache, out))
+            and k_cache.stride(3) == v_cache.stride(3) == 1)
+
+
+def decode_splits(num_seqs: int, kv_heads: int, o: AttnOptions, max_keys: int, device) -> int:
+    """Splits of the key range of a decode batch: about one work item per SM, none below two tiles.  Depends on
+    the batch size and the capacity only, so that a captured graph and an eager step agree."""
+    from ..batch_invariant import is_batch_invariant
+    if is_batch_invariant():
+        return 1
+    keys = min(max_keys, o.window + 127 + ((o.keep_first + 127) // 128) * 128) if o.window else max_keys
+    tiles = (keys + 127) // 128
+    sms = torch.cuda.get_device_properties(device).multi_processor_count
+    return max(1, min((sms + num_seqs * kv_heads - 1) // (num_seqs * kv_heads), tiles // 2, 32))
+
+
+def reserve_decode_scratch(device, max_seqs: int, heads: int, kv_heads: int, vdim: int, o: AttnOptions, max_keys: int) -> None:
+    """Split-KV scratch of decode batches of up to ``max_seqs`` sequences, allocated before graphs are captured."""
+    from .. import ops
+    worst = 0
+    for b in range(1, max_seqs + 1):
+        n = decode_splits(b, kv_heads, o, max_keys, device)
+        if n > 1:
+            worst = max(worst, b * heads * n * (vdim + 1) * 4)
+    if worst:
+        ops.reserve_attention_scratch(device, worst)
+
+
+def variant_attention_decode(q, k_cache, v_cache, meta, o: AttnOptions, gate=None, out=None, num_seqs=None,
+                             num_splits: int = 0) -> torch.Tensor:
+    """tcgen05 decode kernel: the first ``num_seqs`` sequences of the step, one query row each."""
+    from .. import ops
+    num_seqs = meta.num_reqs if num_seqs is None else num_seqs
+    if out is None:
+        out = torch.empty((q.shape[0], q.shape[1], v_cache.shape[3]), dtype=q.dtype, device=q.device)
+    a = _args(q, k_cache, v_cache, meta, o, gate, out)
+    a.num_seqs = num_seqs
+    a.num_splits = num_splits or decode_splits(num_seqs, a.kv_heads, o, meta.block_table.shape[1] * a.block_size, q.device)
+    if a.num_splits > 1:
+        a.scratch = ops._get_scratch(q.device, num_seqs * a.heads * a.num_splits * (a.vdim + 1) * 4).data_ptr()
+    _launch("b200_attention_variant_decode", a, q.device, 2 if a.num_splits > 1 else 1)
+    return out
+
+
+def variant_attention_prefill(q, k_cache, v_cache, meta, o: AttnOptions, gate=None, out=None,
+                              first_seq: int = 0) -> torch.Tensor:
+    """tcgen05 tile kernel: every sequence of the step from ``first_seq`` on, any number of query rows each."""
+    if out is None:
+        out = torch.empty((q.shape[0], q.shape[1], v_cache.shape[3]), dtype=q.dtype, device=q.device)
+    a = _args(q, k_cache, v_cache, meta, o, gate, out)
+    a.num_seqs = meta.num_reqs - first_seq
+    a.cu, a.seq_lens = a.cu + 4 * first_seq, a.seq_lens + 4 * first_seq
+    a.block_table += 4 * first_seq * a.max_blocks
+    _launch("b200_attention_variant_prefill", a, q.device)
+    return out
+
+
 def variant_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, meta, o: AttnOptions,
                       gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of every query row of the step over its sequence's paged keys: q [T, H, D] -> [T, H, Dv].
@@ -268,4 +331,14 @@ def variant_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
         return out
     if not q.is_cuda:
         return _attention_ref(q, k_cache, v_cache, meta, o, gate, out)
-    return variant_attention_simple(q, k_cache, v_cache, meta, o, gate, out)
+    if not _tc_ok(q, k_cache, v_cache, out):
+        return variant_attention_simple(q, k_cache, v_cache, meta, o, gate, out)
+    # the leading sequences with one row stream their keys through the decode kernel
+    nd = 0
+    if H // k_cache.shape[2] <= 16:
+        nd = meta.num_reqs if meta.max_query_len <= 1 and T == meta.num_reqs else int(meta.num_decodes)
+    if nd:
+        variant_attention_decode(q, k_cache, v_cache, meta, o, gate, out, nd)
+    if nd < meta.num_reqs:
+        variant_attention_prefill(q, k_cache, v_cache, meta, o, gate, out, nd)
+    return out

@@ -27,7 +27,7 @@ struct AttnVariantArgs {
   const float* bias;          // [Hq, bias_len]
   const float* sink;          // [Hq]
   const void* gate;           // [T, Hq], row stride gate_stride
-  float* scratch;             // split partials: T * Hq * num_splits * (Dv + 1) floats
+  float* scratch;             // split partials: rows * Hq * num_splits * (Dv + 1) floats
   long q_stride, out_stride, gate_stride, num_blocks, tokens;
   long k_block, k_tok, k_head, v_block, v_tok, v_head;      // cache strides in elements
   int num_seqs, max_blocks, block_size, Hq, Hkv, D, Dv;

@@ -15,7 +15,11 @@
 // Parity: the reference's paged decode path (_npu_paged_attention,
 // vllm_ascend/attention/attention_v1.py:1555-1574) incl. split-KV partials merged
 // by log-sum-exp (npu_attention_update).  All waits are bounded.
+// With VAR the kernel also takes the options of AttnVariantArgs (kept first tokens, capped scores, distance
+// bias, sink, output gate) for one query token per sequence, head sizes up to 128 in multiples of 8 (keys and
+// values of their own: the TMA fills the rest of a tile with zeros) and any group size up to 16.
 #include "attention.h"
+#include "attention_score.cuh"
 #include "common.cuh"
 
 #include <mutex>
@@ -49,6 +53,13 @@ struct DecParams {
   int tail_loads;            // 1: the last tile of a sequence is loaded in 32-key pieces (pages >= 128 keys)
   int l2_prefetch;           // tiles the L2 prefetch of K / V runs ahead of the staged loads (0 = off)
   int* status;
+  // VAR only
+  int keep_first, bias_len, Dv;
+  float scale, softcap;
+  const float* bias;           // [Hq, bias_len]
+  const float* sink;           // [Hq]
+  const __nv_bfloat16* gate;   // [T, Hq]
+  long gate_stride;
   long long* timeline;   // optional [3 roles][64 tiles][8 stamps] of clock64, CTA 0 only
 };
 
@@ -88,7 +99,14 @@ __device__ __forceinline__ void softmax_bar() { asm volatile("bar.sync 1, 128;" 
 struct DecItem {
   int h, seq, split;
   int q_start, q_len, seq_len, ctx, t0, n;
+  int first, kept;             // place in the sequence's tile list; its tiles before the window
 };
+
+// tile number of the item's j-th tile: kept first tokens, then the window
+template <bool VAR>
+__device__ __forceinline__ int dec_tile(const DecItem& w, int j) {
+  return VAR && w.first + j < w.kept ? w.first + j : w.t0 + j;
+}
 
 // The three words of an item that live in global memory.  They are loaded one item ahead
 // (dec_load) and turned into a DecItem (dec_make, arithmetic only) when the item starts, so no
@@ -119,10 +137,12 @@ __device__ __forceinline__ DecItem dec_make(const DecParams& p, int item, const 
   int kv_lo = 0;
   if (p.window > 0) kv_lo = max(0, w.ctx - p.window + 1);
   const int tile_lo = kv_lo >> 7, tile_hi = (w.seq_len + 127) >> 7;
-  const int n_all = tile_hi - tile_lo;
+  w.kept = p.window > 0 ? min(tile_lo, (p.keep_first + 127) >> 7) : 0;
+  const int n_all = w.kept + tile_hi - tile_lo;
   const int per_split = (n_all + p.num_splits - 1) / p.num_splits;
-  w.t0 = tile_lo + w.split * per_split;
-  w.n = w.q_len > 0 ? max(0, min(tile_hi, w.t0 + per_split) - w.t0) : 0;
+  w.first = w.split * per_split;
+  w.t0 = tile_lo - w.kept + w.first;
+  w.n = w.q_len > 0 ? max(0, min(n_all, w.first + per_split) - w.first) : 0;
   return w;
 }
 
@@ -130,7 +150,7 @@ __device__ __forceinline__ DecItem dec_item(const DecParams& p, int item) {
   return dec_make(p, item, dec_load(p, item));
 }
 
-template <int D, int NVT>
+template <int D, int NVT, bool VAR>
 __global__ void __launch_bounds__(DEC_THREADS, 1)
 attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
                       const __grid_constant__ CUtensorMap tmap_k,
@@ -167,13 +187,15 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
   float* red = (float*)(tmem_ptr + 2);            // [2 tiles][4 warps][16] maxima
   float* red_sum = red + 128;                     // [4 warps][16] row sums of the epilogue
 
-  if (p.tail_loads) {
+  if (p.tail_loads || VAR) {
     // The last tile of a sequence is fetched in 32-key pieces up to its length; the rest of the
     // stage keeps what an earlier tile left there.  Those keys are masked (P = 0), so all that is
     // asked of the stale rows is that they are finite: start from zeros instead of whatever the
     // shared memory held.
+    // With VAR a group need not fill the query columns either (the query buffers follow the stages).
     uint4* z = reinterpret_cast<uint4*>(Ks);
-    for (int i = threadIdx.x; i < 2 * ST * Cfg::TILE_BYTES / 16; i += DEC_THREADS)
+    const int fill = 2 * ST * Cfg::TILE_BYTES + (VAR ? 2 * Cfg::Q_BYTES : 0);
+    for (int i = threadIdx.x; i < fill / 16; i += DEC_THREADS)
       z[i] = make_uint4(0u, 0u, 0u, 0u);
     fence_proxy_async_smem();
   }
@@ -226,7 +248,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     // across item boundaries.
     auto first_blk = [&](const DecItem& d) -> int {
       if (d.n <= 0 || lane >= parts) return 0;
-      const int key0 = (d.t0 << 7) + lane * rpl;
+      const int key0 = (dec_tile<VAR>(d, 0) << 7) + lane * rpl;
       return p.block_table[(long)d.seq * p.max_blocks + min(key0, d.seq_len - 1) / p.block_size];
     };
     DecItem w_next;
@@ -252,7 +274,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       const int b = idx & 1;
       if (!mbar_wait(&q_empty[b], ((idx >> 1) & 1u) ^ 1u, abort_word)) return false;
       if (lane == 0) {
-        mbar_expect_tx(&q_full[b], Cfg::Q_BYTES);
+        mbar_expect_tx(&q_full[b], VAR ? NH * 128 * G : Cfg::Q_BYTES);
 #pragma unroll
         for (int hf = 0; hf < NH; hf++)
           tma_load_4d(Qs + b * Cfg::Q_BYTES + hf * DEC_QHALF, &tmap_q, &q_full[b], hf * 64, 0, d.h, d.q_start);
@@ -278,13 +300,13 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       // dependent global load never sits between a freed stage and the next TMA issue.
       auto load_blk = [&](int j) -> int {
         if (j >= w.n || lane >= parts) return 0;
-        const int key0 = ((w.t0 + j) << 7) + lane * rpl;
+        const int key0 = (dec_tile<VAR>(w, j) << 7) + lane * rpl;
         return bt[min(key0, w.seq_len - 1) / p.block_size];
       };
       for (int j = 0; j < w.n; j++, gt++) {
         const int st = gt % ST;
         const uint32_t ph = (gt / ST) & 1u;
-        const int key_base = (w.t0 + j) << 7;
+        const int key_base = dec_tile<VAR>(w, j) << 7;
         const int blk_next = load_blk(j + 1);
         if (p.l2_prefetch > 0 && j + p.l2_prefetch < w.n) {
           // ask for a later tile's pages in L2 now: the bytes in flight towards shared memory are
@@ -292,7 +314,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
           const int jp = j + p.l2_prefetch;
           const int blk_pf = load_blk(jp);
           if (lane < parts && blk_pf >= 0 && blk_pf < p.num_blocks_total) {
-            const int off = (((w.t0 + jp) << 7) + lane * rpl) % p.block_size;
+            const int off = ((dec_tile<VAR>(w, jp) << 7) + lane * rpl) % p.block_size;
 #pragma unroll
             for (int hf = 0; hf < NH; hf++) {
               tma_prefetch_l2_4d(&tmap_k, hf * 64, w.h, off, blk_pf);
@@ -444,7 +466,10 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     const int qd = warp & 3;
     const int tid = qd * 32 + lane;                 // key inside the tile; d index for O^T
     const uint32_t t_lane = tmem_base + ((uint32_t)(qd * 32) << 16);
-    const float sl2 = p.scale_log2;
+    const bool zform = VAR && (p.softcap > 0.f || p.bias != nullptr);   // scores become z = log2(e) * score
+    const float sl2 = zform ? 1.f : p.scale_log2;
+    const int dv = VAR ? p.Dv : D;
+    const SoftCap cap(VAR ? p.scale : 1.f, VAR && p.softcap > 0.f ? p.softcap : 1.f);
     int* redi = reinterpret_cast<int*>(red);        // [2 tiles][4 warps][16]
     uint32_t gt = 0, it = 0;
     DecRaw raw_next = {0, 0, 0};
@@ -459,7 +484,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
             const long pidx =
                 ((long)(w.q_start + c / G) * p.Hq + (w.h * G + c % G)) * p.num_splits + w.split;
             p.partial_lse[pidx] = -INFINITY;
-            for (int d = 0; d < D; d++) p.partial_o[pidx * D + d] = 0.f;
+            for (int d = 0; d < dv; d++) p.partial_o[pidx * dv + d] = 0.f;
           }
         } else if (p.num_splits == 1 && p.lse_out && w.q_len > 0) {
           // a caller that merges partial results of several ranks needs a defined (zero-weight)
@@ -492,6 +517,15 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
         const uint32_t g = gt + (uint32_t)j;
         const int b = g & 1;
         if (warp == 2) DEC_STAMP(2, g, 0);
+        const int tile_base = dec_tile<VAR>(w, j) << 7;
+        const int key = tile_base + tid;
+        float bz[NVT];
+        if (VAR && p.bias) {            // under way while the products are computed
+          const int dist = min(max(w.ctx - key, 0), p.bias_len - 1);
+#pragma unroll
+          for (int c = 0; c < NVT; c++)
+            bz[c] = c < G ? __ldg(p.bias + (long)(w.h * G + c) * p.bias_len + dist) * kLog2e : 0.f;
+        }
         if (!mbar_wait(&s_ready[b], (g >> 1) & 1u, abort_word)) goto done;
         if (warp == 2) DEC_STAMP(2, g, 1);
         tc_fence_after();
@@ -501,8 +535,6 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(&s_free[b]);
-        const int tile_base = (w.t0 + j) << 7;
-        const int key = tile_base + tid;
         // only tiles that straddle a visibility limit need per-key masking
         const bool need_mask = (tile_base + 128 > hi_min) || (tile_base < lo_max);
         float s[NVT];
@@ -510,7 +542,12 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
 #pragma unroll
         for (int c = 0; c < NVT; c++) {
           s[c] = __uint_as_float(r[c]);
-          if (need_mask && !(key >= lo[c] && key < hi[c])) s[c] = -INFINITY;
+          if constexpr (VAR) {
+            if (p.softcap > 0.f) s[c] = cap.any(s[c]);
+            else if (zform) s[c] *= p.scale_log2;
+            if (p.bias) s[c] += bz[c];
+          }
+          if (need_mask && !((key >= lo[c] || (VAR && key < p.keep_first)) && key < hi[c])) s[c] = -INFINITY;
           int ob = __float_as_int(s[c]);
           ob ^= (ob >> 31) & 0x7fffffff;              // order-preserving float -> int
           const int wm = __reduce_max_sync(0xffffffffu, ob);
@@ -590,24 +627,30 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       tc_fence_before();
       softmax_bar();            // row sums visible; every thread holds its O^T row
       if (lane == 0) mbar_arrive(&o_free[it & 1]);
-      if (tid < D) {
+      if (tid < dv) {
 #pragma unroll
         for (int c = 0; c < NVT; c++) {
           if (c < nv) {
             const float l = red_sum[c] + red_sum[DEC_NQ + c] + red_sum[2 * DEC_NQ + c] +
                             red_sum[3 * DEC_NQ + c];
-            const float inv = l > 0.f ? 1.f / l : 0.f;
+            float inv = l > 0.f ? 1.f / l : 0.f;
             const long tok = w.q_start + c / G;
             const int hq = w.h * G + c % G;
+            if constexpr (VAR) {
+              if (p.num_splits == 1) {            // with splits the merge does both
+                if (p.sink && l > 0.f) inv = 1.f / (l + score_exp2(p.sink[hq] * kLog2e - m[c] * sl2));
+                if (p.gate) inv *= sigmoid_f(__bfloat162float(p.gate[tok * p.gate_stride + hq]));
+              }
+            }
             const float val = __uint_as_float(o[c]) * inv;
             if (p.num_splits == 1) {
-              p.out[tok * p.out_stride + (long)hq * D + tid] = __float2bfloat16(val);
+              p.out[tok * p.out_stride + (long)hq * dv + tid] = __float2bfloat16(val);
               if (tid == 0 && p.lse_out)
                 p.lse_out[tok * p.Hq + hq] =
                     (l > 0.f) ? (m[c] * sl2 * 0.6931471805599453f + logf(l)) : -INFINITY;
             } else {
               const long pidx = (tok * p.Hq + hq) * p.num_splits + w.split;
-              p.partial_o[pidx * D + tid] = val;
+              p.partial_o[pidx * dv + tid] = val;
               if (tid == 0)
                 p.partial_lse[pidx] =
                     (l > 0.f) ? (m[c] * sl2 * 0.6931471805599453f + logf(l)) : -INFINITY;
@@ -663,6 +706,47 @@ struct DecTmapCache {
 };
 static DecTmapCache g_dec_tmaps;
 static int g_dec_l2_prefetch = 0;      // tiles of L2 prefetch ahead of the staged K / V loads (0 = off)
+
+template <bool VAR, int NV>
+static int launch_decode_nv(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv,
+                            const CUtensorMap& tk32, const CUtensorMap& tv32, const DecParams& p, unsigned grid,
+                            cudaStream_t stream) {
+  using Cfg = DecCfg<128>;
+  static bool attr_set = false;
+  if (!attr_set) {
+    cudaError_t e = cudaFuncSetAttribute(attn_decode_tc_kernel<128, NV, VAR>,
+                                         cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES);
+    if (e != cudaSuccess) return (int)e;
+    attr_set = true;
+  }
+  attn_decode_tc_kernel<128, NV, VAR><<<grid, DEC_THREADS, Cfg::SMEM_BYTES, stream>>>(tq, tk, tv, tk32, tv32, p);
+  return B200_CHECK_LAUNCH();
+}
+
+// fills in the item count; ncols: columns that can be valid
+template <bool VAR>
+static int launch_decode(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tk32,
+                         const CUtensorMap& tv32, DecParams& p, int ncols, cudaStream_t stream) {
+  const long items = (long)p.Hkv * p.num_seqs * p.num_splits;
+  if (items > 0x7fffffffL) return 9125;
+  if (ncols > DEC_NQ) return 9126;
+  p.num_items = (int)items;
+  static int sm_count[64] = {};
+  int dev = 0;
+  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return 9127;
+  if (sm_count[dev] == 0) {
+    int n = 0;
+    if (cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || n <= 0)
+      return 9127;
+    sm_count[dev] = n;
+  }
+  const unsigned grid = (unsigned)(items < sm_count[dev] ? items : sm_count[dev]);
+  if (ncols <= 1) return launch_decode_nv<VAR, 1>(tq, tk, tv, tk32, tv32, p, grid, stream);
+  if (ncols <= 2) return launch_decode_nv<VAR, 2>(tq, tk, tv, tk32, tv32, p, grid, stream);
+  if (ncols <= 4) return launch_decode_nv<VAR, 4>(tq, tk, tv, tk32, tv32, p, grid, stream);
+  if (ncols <= 8) return launch_decode_nv<VAR, 8>(tq, tk, tv, tk32, tv32, p, grid, stream);
+  return launch_decode_nv<VAR, 16>(tq, tk, tv, tk32, tv32, p, grid, stream);
+}
 
 }  // namespace b200
 
@@ -748,48 +832,16 @@ B200_API int b200_attn_decode_tc_lse(const void* q, long q_stride, long T, const
   p.num_blocks_total = num_blocks;
   p.status = status;
   p.timeline = (long long*)timeline;
-  using Cfg = DecCfg<128>;
-  const long items = (long)Hkv * num_seqs * num_splits;
-  if (items > 0x7fffffffL) return 9125;
+  // columns that can be valid: query tokens per sequence x heads per group
+  if (max_q_len < 1) max_q_len = 1;
   p.num_seqs = num_seqs;
   p.tail_loads = rpl == 128 ? 1 : 0;
   p.l2_prefetch = g_dec_l2_prefetch;
-  p.num_items = (int)items;
-  static int sm_count[64] = {};
-  int dev = 0;
-  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return 9127;
-  if (sm_count[dev] == 0) {
-    int n = 0;
-    if (cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || n <= 0)
-      return 9127;
-    sm_count[dev] = n;
+  p.keep_first = 0;
+  {
+    const int lrc = launch_decode<false>(tq, tk, tv, tk32, tv32, p, max_q_len * G, stream);
+    if (lrc) return lrc;
   }
-  dim3 grid((unsigned)(items < sm_count[dev] ? items : sm_count[dev]));
-  // columns that can be valid: query tokens per sequence x heads per group
-  if (max_q_len < 1) max_q_len = 1;
-  const int ncols = max_q_len * G;
-  if (ncols > DEC_NQ) return 9126;
-#define LAUNCH_DEC_TC(NV)                                                                   \
-  do {                                                                                      \
-    static bool attr_set = false;                                                           \
-    if (!attr_set) {                                                                        \
-      cudaError_t e = cudaFuncSetAttribute(attn_decode_tc_kernel<128, NV>,                  \
-                                           cudaFuncAttributeMaxDynamicSharedMemorySize,     \
-                                           Cfg::SMEM_BYTES);                                \
-      if (e != cudaSuccess) return (int)e;                                                  \
-      attr_set = true;                                                                      \
-    }                                                                                       \
-    attn_decode_tc_kernel<128, NV><<<grid, DEC_THREADS, Cfg::SMEM_BYTES, stream>>>(tq, tk, tv, tk32,  \
-                                                                                    tv32, p); \
-  } while (0)
-  if (ncols <= 1) LAUNCH_DEC_TC(1);
-  else if (ncols <= 2) LAUNCH_DEC_TC(2);
-  else if (ncols <= 4) LAUNCH_DEC_TC(4);
-  else if (ncols <= 8) LAUNCH_DEC_TC(8);
-  else LAUNCH_DEC_TC(16);
-#undef LAUNCH_DEC_TC
-  int rc = B200_CHECK_LAUNCH();
-  if (rc) return rc;
   if (num_splits > 1)
     return launch_merge_splits(p.partial_o, p.partial_lse, T, Hq, num_splits, D, out,
                                out_stride, stream, (float*)lse_out);
@@ -808,4 +860,69 @@ B200_API int b200_attn_decode_tc(const void* q, long q_stride, long T, const voi
                                  query_start_loc, seq_lens, block_table, max_blocks, num_seqs, Hq,
                                  Hkv, D, scale, window, num_splits, max_q_len, out, out_stride,
                                  scratch, kv_layout, nullptr, status, timeline, stream);
+}
+
+// Options as in AttnVariantArgs; one query token per sequence (row b of q belongs to sequence b), bf16, D and Dv
+// multiples of 8 up to 128, at most 16 query heads per key head
+B200_API int b200_attention_variant_decode(const b200::AttnVariantArgs* a, int* status, cudaStream_t stream) {
+  using namespace b200;
+  if (a->tokens <= 0 || a->num_seqs <= 0) return 0;
+  if (a->Hkv < 1 || a->Hq % a->Hkv || a->Hq / a->Hkv > DEC_NQ || a->tokens < a->num_seqs) return 9870;
+  if (a->D < 8 || a->D > 128 || a->D % 8 || a->Dv < 8 || a->Dv > 128 || a->Dv % 8 || a->dtype != 0) return 9871;
+  const int bs = a->block_size;
+  if (bs < 8 || (bs < 128 && 128 % bs) || (bs > 128 && bs % 128)) return 9872;
+  if ((a->q_stride & 7) || (a->out_stride & 7) || (a->bias && a->bias_len < 1) || a->keep_first < 0) return 9873;
+  if (a->num_splits < 1 || (a->num_splits > 1 && !a->scratch)) return 9874;
+  const int G = a->Hq / a->Hkv, rpl = bs < 128 ? bs : 128;
+  CUtensorMap tq, tkv[2], tkv32[2];
+  {
+    uint64_t dims[4] = {(uint64_t)a->D, (uint64_t)G, (uint64_t)a->Hkv, (uint64_t)a->tokens};
+    uint64_t str[3] = {(uint64_t)a->D * 2, (uint64_t)G * a->D * 2, (uint64_t)a->q_stride * 2};
+    uint32_t box[4] = {64, (uint32_t)G, 1, 1};
+    int rc = g_dec_tmaps.get(&tq, a->q, 4, dims, str, box);
+    if (rc) return rc;
+  }
+  for (int kv = 0; kv < 2; kv++) {
+    uint64_t dims[4] = {(uint64_t)(kv ? a->Dv : a->D), (uint64_t)a->Hkv, (uint64_t)bs, (uint64_t)a->num_blocks};
+    uint64_t str[3] = {(uint64_t)(kv ? a->v_head : a->k_head) * 2, (uint64_t)(kv ? a->v_tok : a->k_tok) * 2,
+                       (uint64_t)(kv ? a->v_block : a->k_block) * 2};
+    uint32_t box[4] = {64, 1, (uint32_t)rpl, 1}, box32[4] = {64, 1, 32, 1};
+    const void* base = kv ? a->v_cache : a->k_cache;
+    int rc = g_dec_tmaps.get(&tkv[kv], base, 4, dims, str, box);
+    if (!rc && rpl == 128) rc = g_dec_tmaps.get(&tkv32[kv], base, 4, dims, str, box32);
+    else tkv32[kv] = tkv[kv];
+    if (rc) return rc;
+  }
+  DecParams p = {};
+  p.query_start_loc = a->cu;
+  p.seq_lens = a->seq_lens;
+  p.block_table = a->block_table;
+  p.max_blocks = a->max_blocks;
+  p.block_size = bs;
+  p.rows_per_load = rpl;
+  p.G = G; p.Hkv = a->Hkv; p.Hq = a->Hq;
+  p.scale_log2 = a->scale * kLog2e;
+  p.window = a->window;
+  p.num_splits = a->num_splits;
+  p.out = (__nv_bfloat16*)a->out;
+  p.out_stride = a->out_stride;
+  p.partial_o = a->scratch;
+  p.partial_lse = a->scratch ? a->scratch + (long)a->num_seqs * a->Hq * (long)a->num_splits * a->Dv : nullptr;
+  p.num_blocks_total = a->num_blocks;
+  p.status = status;
+  p.num_seqs = a->num_seqs;
+  p.tail_loads = rpl == 128 ? 1 : 0;
+  p.l2_prefetch = g_dec_l2_prefetch;
+  p.keep_first = a->window > 0 ? a->keep_first : 0;
+  p.bias_len = a->bias_len; p.Dv = a->Dv;
+  p.scale = a->scale; p.softcap = a->softcap;
+  p.bias = a->bias; p.sink = a->sink;
+  p.gate = (const __nv_bfloat16*)a->gate;
+  p.gate_stride = a->gate_stride;
+  int rc = launch_decode<true>(tq, tkv[0], tkv[1], tkv32[0], tkv32[1], p, G, stream);
+  if (rc) return rc;
+  if (a->num_splits > 1)
+    return launch_merge_splits(p.partial_o, p.partial_lse, a->num_seqs, a->Hq, a->num_splits, a->Dv, a->out,
+                               a->out_stride, stream, nullptr, 0, a->sink, a->gate, a->gate_stride);
+  return 0;
 }

@@ -19,8 +19,12 @@
 //              shared memory); rescale O in TMEM only when the running max moved by
 //              more than a threshold; final normalise + store (or split partials)
 // All waits are bounded; on timeout the CTA aborts cleanly and reports a status.
+// With VAR the kernel also takes the options of AttnVariantArgs (kept first tokens, capped scores, distance
+// bias, sink, output gate), head sizes up to D (multiples of 8, keys and values of their own: the TMA fills the
+// rest of a tile with zeros) and any group size up to 128; it then finds its (sequence, token) tile by itself.
 #include "common.cuh"
 #include "attention.h"
+#include "attention_score.cuh"
 
 #include <mutex>
 #include <string.h>
@@ -50,6 +54,13 @@ struct AttnParams {
   int* status;
   uint32_t v_lbo, v_sbo;
   float rescale_threshold;
+  // VAR only
+  int num_seqs, keep_first, bias_len, Dv;
+  float scale, softcap;
+  const float* bias;           // [Hq, bias_len]
+  const float* sink;           // [Hq]
+  const __nv_bfloat16* gate;   // [T, Hq]
+  long gate_stride;
 };
 
 __device__ __forceinline__ float att_exp2(float x) {
@@ -70,7 +81,7 @@ struct AttCfg {
   static constexpr int O_COL = 256;
 };
 
-template <int D>
+template <int D, bool VAR>
 __global__ void __launch_bounds__(ATT_THREADS, 1)
 attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
                    const __grid_constant__ CUtensorMap tmap_k,
@@ -79,9 +90,23 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
   constexpr int NH = Cfg::NH, KS = Cfg::KS;
 
   // ---------------- work decode (uniform over the CTA)
-  const int h = blockIdx.x, wi = blockIdx.y, split = blockIdx.z;
-  const int seq = p.tile_seq ? p.tile_seq[wi] : wi;
-  const int tok0 = p.tile_qoff ? p.tile_qoff[wi] : 0;
+  const int h = blockIdx.x, split = blockIdx.z;
+  int seq, tok0;
+  if constexpr (VAR) {
+    // sequence b owns the tiles from (cu[b] - cu[0]) / tok_per_tile + b on; late tiles see more keys: first
+    const int wi = gridDim.y - 1 - blockIdx.y, base = p.query_start_loc[0];
+    int lo = 0, hi = p.num_seqs - 1;
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if ((p.query_start_loc[mid] - base) / p.tok_per_tile + mid <= wi) lo = mid; else hi = mid - 1;
+    }
+    seq = lo;
+    tok0 = (wi - ((p.query_start_loc[lo] - base) / p.tok_per_tile + lo)) * p.tok_per_tile;
+  } else {
+    const int wi = blockIdx.y;
+    seq = p.tile_seq ? p.tile_seq[wi] : wi;
+    tok0 = p.tile_qoff ? p.tile_qoff[wi] : 0;
+  }
   const int q_start = p.query_start_loc[seq];
   const int q_len = p.query_start_loc[seq + 1] - q_start;
   const int seq_len = p.seq_lens[seq];
@@ -93,11 +118,15 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
   int kv_lo = 0;
   if (p.window > 0) kv_lo = max(0, ctx + tok0 - p.window + 1);
   const int tile_lo = kv_lo >> 7, tile_hi = (kv_end + 127) >> 7;
-  const int n_all = tile_hi - tile_lo;
+  // tiles of kept first tokens that lie before the window come first in the list
+  const int kept = VAR && p.window > 0 ? min(tile_lo, (p.keep_first + 127) >> 7) : 0;
+  const int n_all = kept + tile_hi - tile_lo;
   const int per_split = (n_all + p.num_splits - 1) / p.num_splits;
-  const int t0 = tile_lo + split * per_split;
-  const int t1 = min(tile_hi, t0 + per_split);
-  const int n = t1 - t0;
+  const int first = split * per_split;
+  const int n = min(n_all, first + per_split) - first;
+  const int t0 = tile_lo - kept + first;
+  const int dv = VAR ? p.Dv : D;
+  auto tile_no = [&](int j) { return VAR && first + j < kept ? first + j : t0 + j; };
 
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
@@ -109,7 +138,7 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
         const long pidx =
             ((long)(q_start + tok0 + tok) * p.Hq + (h * G + g)) * p.num_splits + split;
         p.partial_lse[pidx] = -INFINITY;
-        for (int d = 0; d < D; d++) p.partial_o[pidx * D + d] = 0.f;
+        for (int d = 0; d < dv; d++) p.partial_o[pidx * dv + d] = 0.f;
       }
     }
     return;
@@ -171,7 +200,7 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     const int rpl = p.rows_per_load;
     const int parts = 128 / rpl;
     if (lane == 0) {
-      mbar_expect_tx(q_full, Cfg::TILE_BYTES);
+      mbar_expect_tx(q_full, VAR ? NH * 128 * G * p.tok_per_tile : Cfg::TILE_BYTES);
 #pragma unroll
       for (int hf = 0; hf < NH; hf++)
         tma_load_4d(Qs + hf * ATT_HALF_BYTES, &tmap_q, q_full, hf * 64, 0, h, q_start + tok0);
@@ -180,14 +209,14 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     // dependent global load never sits between a freed stage and the next TMA issue.
     auto load_blk = [&](int j) -> int {
       if (j >= n || lane >= parts) return 0;
-      const int key0 = ((t0 + j) << 7) + lane * rpl;
+      const int key0 = (tile_no(j) << 7) + lane * rpl;
       return bt[min(key0, seq_len - 1) / p.block_size];
     };
     int blk_cur = load_blk(0);
     for (int j = 0; j < n; j++) {
       const int ks = j % KS;
       const uint32_t ph = (uint32_t)(j / KS) & 1u;
-      const int key_base = (t0 + j) << 7;
+      const int key_base = tile_no(j) << 7;
       const int blk_next = load_blk(j + 1);
       bool bad = blk_cur < 0 || blk_cur >= p.num_blocks_total;
       bad = __any_sync(0xffffffffu, bad && lane < parts);
@@ -279,7 +308,11 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     const bool row_valid = tok < ntok;
     const int q_pos = ctx + tok0 + tok;
     const uint32_t t_lane = tmem_base + ((uint32_t)(qd * 32) << 16);
-    const float sl2 = p.scale_log2;
+    const int hq = h * G + g;
+    const bool zform = VAR && (p.softcap > 0.f || p.bias != nullptr);   // scores become z = log2(e) * score
+    const float sl2 = zform ? 1.f : p.scale_log2;
+    const float* brow = VAR && p.bias && row_valid ? p.bias + (long)hq * p.bias_len : p.bias;
+    const SoftCap cap(VAR ? p.scale : 1.f, VAR && p.softcap > 0.f ? p.softcap : 1.f);
     int hi = seq_len;                      // keys [lo, hi) are visible to this row
     if (p.causal) hi = min(hi, q_pos + 1);
     int lo = 0;
@@ -291,10 +324,10 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       const int b = j & 1;
       if (!mbar_wait(&s_ready[b], ((uint32_t)j >> 1) & 1u, abort_word)) goto done;
       tc_fence_after();
-      const int tile_base = (t0 + j) << 7;
+      const int tile_base = tile_no(j) << 7;
       // mask needed when the tile is not entirely inside every row's window
       const bool need_mask = (tile_base + 128 > min(seq_len, p.causal ? ctx + tok0 + 1 : seq_len)) ||
-                             (p.window > 0);
+                             (VAR ? p.window > 0 && tile_base <= ctx + tok0 + ntok - 1 - p.window : p.window > 0);
       // ---- the whole score row lives in registers: one TMEM read, no second pass
       uint32_t sreg[128];
       tmem_ld_32x32b_x32(t_lane + b * 128, sreg);
@@ -305,11 +338,55 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_free[b]);
+      if constexpr (VAR) {
+        if (p.softcap > 0.f) {
+          float big = 0.f;
+#pragma unroll
+          for (int i = 0; i < 128; i++) big = fmaxf(big, fabsf(__uint_as_float(sreg[i])));
+          if (__all_sync(0xffffffffu, big * fabsf(cap.to_t) <= SoftCap::kSmall || !row_valid)) {
+#pragma unroll
+            for (int i = 0; i < 128; i += 2) {
+              const float2 z = unpack2(cap.small2(pack2(__uint_as_float(sreg[i]), __uint_as_float(sreg[i + 1]))));
+              sreg[i] = __float_as_uint(z.x);
+              sreg[i + 1] = __float_as_uint(z.y);
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < 128; i++) sreg[i] = __float_as_uint(cap.any(__uint_as_float(sreg[i])));
+          }
+        } else if (zform) {
+#pragma unroll
+          for (int i = 0; i < 128; i++) sreg[i] = __float_as_uint(__uint_as_float(sreg[i]) * p.scale_log2);
+        }
+        if (p.bias) {
+          const int near = ctx + tok0 - (tile_base + 127), far = ctx + tok0 + ntok - 1 - tile_base;   // distances
+          if (near >= p.bias_len - 1) {               // all in the last bucket
+            const float bz = brow[p.bias_len - 1] * kLog2e;
+#pragma unroll
+            for (int i = 0; i < 128; i++) sreg[i] = __float_as_uint(__uint_as_float(sreg[i]) + bz);
+          } else {
+            const int d0 = row_valid ? q_pos - tile_base : 0;
+            const bool clamp = near < 0 || far >= p.bias_len || !row_valid;
+            if (__any_sync(0xffffffffu, clamp)) {
+#pragma unroll
+              for (int i = 0; i < 128; i++) {
+                const float bv = __ldg(brow + min(max(d0 - i, 0), p.bias_len - 1));
+                sreg[i] = __float_as_uint(fmaf(bv, kLog2e, __uint_as_float(sreg[i])));
+              }
+            } else {
+#pragma unroll
+              for (int i = 0; i < 128; i++)
+                sreg[i] = __float_as_uint(fmaf(__ldg(brow + d0 - i), kLog2e, __uint_as_float(sreg[i])));
+            }
+          }
+        }
+      }
       if (need_mask) {
+        const int keep = VAR ? p.keep_first : 0;
 #pragma unroll
         for (int i = 0; i < 128; i++) {
           const int key = tile_base + i;
-          if (!(key >= lo && key < hi)) sreg[i] = 0xff800000u;   // -inf
+          if (!((key >= lo || (VAR && key < keep)) && key < hi)) sreg[i] = 0xff800000u;   // -inf
         }
       }
       float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
@@ -380,9 +457,14 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     // ---- epilogue
     if (!mbar_wait(&pv_done[(n - 1) & 1], (((uint32_t)n - 1) >> 1) & 1u, abort_word)) goto done;
     tc_fence_after();
-    const float inv = l > 0.f ? 1.f / l : 0.f;
     const long tokidx = (long)q_start + tok0 + tok;
-    const int hq = h * G + g;
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    if constexpr (VAR) {
+      if (p.num_splits == 1 && row_valid) {           // with splits the merge does both
+        if (p.sink && l > 0.f) inv = 1.f / (l + score_exp2(p.sink[hq] * kLog2e - m * sl2));
+        if (p.gate) inv *= sigmoid_f(__bfloat162float(p.gate[tokidx * p.gate_stride + hq]));
+      }
+    }
 #pragma unroll 1
     for (int c = 0; c < D / 32; c++) {
       uint32_t r[32];
@@ -390,9 +472,10 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       tmem_ld_wait();
       if (row_valid) {
         if (p.num_splits == 1) {
-          __nv_bfloat16* dst = p.out + tokidx * p.out_stride + (long)hq * D + c * 32;
+          __nv_bfloat16* dst = p.out + tokidx * p.out_stride + (long)hq * dv + c * 32;
 #pragma unroll
           for (int q4 = 0; q4 < 4; q4++) {
+            if (VAR && c * 32 + q4 * 8 >= dv) break;
             uint4 o;
             o.x = pack_bf16x2(__uint_as_float(r[q4 * 8 + 0]) * inv, __uint_as_float(r[q4 * 8 + 1]) * inv);
             o.y = pack_bf16x2(__uint_as_float(r[q4 * 8 + 2]) * inv, __uint_as_float(r[q4 * 8 + 3]) * inv);
@@ -402,9 +485,10 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
           }
         } else {
           const long pidx = (tokidx * p.Hq + hq) * p.num_splits + split;
-          float* dst = p.partial_o + pidx * D + c * 32;
+          float* dst = p.partial_o + pidx * dv + c * 32;
 #pragma unroll
           for (int q4 = 0; q4 < 8; q4++) {
+            if (VAR && c * 32 + q4 * 4 >= dv) break;
             float4 o = make_float4(__uint_as_float(r[q4 * 4 + 0]) * inv, __uint_as_float(r[q4 * 4 + 1]) * inv,
                                    __uint_as_float(r[q4 * 4 + 2]) * inv, __uint_as_float(r[q4 * 4 + 3]) * inv);
             reinterpret_cast<float4*>(dst)[q4] = o;
@@ -461,13 +545,13 @@ struct TmapCache {
 };
 static TmapCache g_att_tmaps;
 
-template <int D>
+template <int D, bool VAR = false>
 static int launch_attn_tc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv,
                           const AttnParams& p, int num_tiles, cudaStream_t stream) {
   using Cfg = AttCfg<D>;
   static bool attr_set = false;
   if (!attr_set) {
-    cudaError_t e = cudaFuncSetAttribute(attn_fwd_tc_kernel<D>,
+    cudaError_t e = cudaFuncSetAttribute(attn_fwd_tc_kernel<D, VAR>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          Cfg::SMEM_BYTES);
     if (e != cudaSuccess) return (int)e;
@@ -475,7 +559,7 @@ static int launch_attn_tc(const CUtensorMap& tq, const CUtensorMap& tk, const CU
   }
   if (num_tiles > 65535) return 9125;
   dim3 grid((unsigned)p.Hkv, (unsigned)num_tiles, (unsigned)p.num_splits);
-  attn_fwd_tc_kernel<D><<<grid, ATT_THREADS, Cfg::SMEM_BYTES, stream>>>(tq, tk, tv, p);
+  attn_fwd_tc_kernel<D, VAR><<<grid, ATT_THREADS, Cfg::SMEM_BYTES, stream>>>(tq, tk, tv, p);
   return B200_CHECK_LAUNCH();
 }
 
@@ -566,5 +650,70 @@ B200_API int b200_attn_fwd_tc(const void* q, long q_stride, long T, const void* 
   if (num_splits > 1)
     return launch_merge_splits(p.partial_o, p.partial_lse, T, Hq, num_splits, D, out,
                                out_stride, stream);
+  return 0;
+}
+
+// Options as in AttnVariantArgs; rows of several tokens per sequence, bf16, D and Dv multiples of 8 up to 128
+B200_API int b200_attention_variant_prefill(const b200::AttnVariantArgs* a, int* status, cudaStream_t stream) {
+  using namespace b200;
+  if (a->tokens <= 0 || a->num_seqs <= 0) return 0;
+  if (a->Hkv < 1 || a->Hq % a->Hkv || a->Hq / a->Hkv > 128) return 9860;
+  if (a->D < 8 || a->D > 128 || a->D % 8 || a->Dv < 8 || a->Dv > 128 || a->Dv % 8 || a->dtype != 0) return 9861;
+  const int bs = a->block_size;
+  if (bs < 8 || (bs < 128 && 128 % bs) || (bs > 128 && bs % 128)) return 9862;
+  if ((a->q_stride & 7) || (a->out_stride & 7) || (a->bias && a->bias_len < 1) || a->keep_first < 0) return 9863;
+  if (a->num_splits < 1 || (a->num_splits > 1 && !a->scratch)) return 9864;
+  const int G = a->Hq / a->Hkv, tok = 128 / G, rpl = bs < 128 ? bs : 128;
+  CUtensorMap tq, tk, tv;
+  {
+    uint64_t dims[4] = {(uint64_t)a->D, (uint64_t)G, (uint64_t)a->Hkv, (uint64_t)a->tokens};
+    uint64_t str[3] = {(uint64_t)a->D * 2, (uint64_t)G * a->D * 2, (uint64_t)a->q_stride * 2};
+    uint32_t box[4] = {64, (uint32_t)G, 1, (uint32_t)tok};
+    int rc = g_att_tmaps.get(&tq, a->q, 4, dims, str, box);
+    if (rc) return rc;
+  }
+  for (int kv = 0; kv < 2; kv++) {
+    uint64_t dims[4] = {(uint64_t)(kv ? a->Dv : a->D), (uint64_t)a->Hkv, (uint64_t)bs, (uint64_t)a->num_blocks};
+    uint64_t str[3] = {(uint64_t)(kv ? a->v_head : a->k_head) * 2, (uint64_t)(kv ? a->v_tok : a->k_tok) * 2,
+                       (uint64_t)(kv ? a->v_block : a->k_block) * 2};
+    uint32_t box[4] = {64, 1, (uint32_t)rpl, 1};
+    int rc = g_att_tmaps.get(kv ? &tv : &tk, kv ? a->v_cache : a->k_cache, 4, dims, str, box);
+    if (rc) return rc;
+  }
+  AttnParams p = {};
+  p.query_start_loc = a->cu;
+  p.seq_lens = a->seq_lens;
+  p.block_table = a->block_table;
+  p.max_blocks = a->max_blocks;
+  p.block_size = bs;
+  p.rows_per_load = rpl;
+  p.G = G; p.Hkv = a->Hkv; p.Hq = a->Hq;
+  p.tok_per_tile = tok;
+  p.scale_log2 = a->scale * kLog2e;
+  p.causal = 1; p.window = a->window; p.num_splits = a->num_splits;
+  p.out = (__nv_bfloat16*)a->out;
+  p.out_stride = a->out_stride;
+  p.partial_o = a->scratch;
+  p.partial_lse = a->scratch ? a->scratch + a->tokens * a->Hq * (long)a->num_splits * a->Dv : nullptr;
+  p.num_blocks_total = a->num_blocks;
+  p.status = status;
+  p.v_lbo = ATT_HALF_BYTES;
+  p.v_sbo = 1024u;
+  p.rescale_threshold = 8.f;
+  p.num_seqs = a->num_seqs;
+  p.keep_first = a->window > 0 ? a->keep_first : 0;
+  p.bias_len = a->bias_len; p.Dv = a->Dv;
+  p.scale = a->scale; p.softcap = a->softcap;
+  p.bias = a->bias; p.sink = a->sink;
+  p.gate = (const __nv_bfloat16*)a->gate;
+  p.gate_stride = a->gate_stride;
+  const long tiles = a->tokens / tok + a->num_seqs;
+  if (tiles > 65535) return 9865;
+  int rc = (a->D > 64 || a->Dv > 64) ? launch_attn_tc<128, true>(tq, tk, tv, p, (int)tiles, stream)
+                                     : launch_attn_tc<64, true>(tq, tk, tv, p, (int)tiles, stream);
+  if (rc) return rc;
+  if (a->num_splits > 1)
+    return launch_merge_splits(p.partial_o, p.partial_lse, a->tokens, a->Hq, a->num_splits, a->Dv, a->out,
+                               a->out_stride, stream, nullptr, 0, a->sink, a->gate, a->gate_stride);
   return 0;
 }

@@ -1218,7 +1218,8 @@ class ModelRunner:
         if self.mcfg.layer_plan:
             for a in {id(L.self_attn): L.self_attn for L in self.model.layers}.values():
                 if hasattr(a, "reserve_decode_scratch"):
-                    a.reserve_decode_scratch(self.device, self.capture_sizes, self.max_model_len)
+                    a.reserve_decode_scratch(self.device, sorted({*self.capture_sizes, self.max_seqs}),
+                                             self.max_blocks_per_seq * self.block_size)
         elif not self.mcfg.use_mla:
             a = self._attn_layer()
             worst = 0

@@ -11,7 +11,8 @@ from __future__ import annotations
 
 import torch
 
-from ..attention.variant import AttnOptions, PrepSpec, distance_table, qkv_prep, variant_attention
+from ..attention.variant import (AttnOptions, PrepSpec, distance_table, qkv_prep, reserve_decode_scratch,
+                                 variant_attention)
 from ..config import ModelConfig
 from ..parallel import state as pstate
 from .layers import Linear, ParamFactory, RowParallelLinear, TPComm, copy_exact, get_cos_sin_cache
@@ -102,6 +103,9 @@ class VariantAttention:
     def sequence_state_shapes(self, num_slots: int) -> list[tuple]:
         """Per-sequence state beside the pages: the last convolution inputs."""
         return [(num_slots, self.taps - 1, self.prep.columns)] if self.taps > 1 else []
+
+    def reserve_decode_scratch(self, device, batch_sizes: list, max_keys: int) -> None:
+        reserve_decode_scratch(device, batch_sizes[-1], self.Hq, self.Hkv, self.Dv, self.options, max_keys)
 
     # ------------------------------------------------------------------ forward
     def __call__(self, x: torch.Tensor, meta, kv_cache) -> torch.Tensor:
