@@ -1,6 +1,7 @@
 """Small Pegopel configurations and random weights for the tests, and comparisons with the plain definitions."""
 import json
 
+import numpy as np
 import torch
 
 import pegopel_oracle as po
@@ -112,3 +113,24 @@ def check(got, cfg, w, ids, dtype, note=None):
     r = errors(reference(cfg, w, ids, True), want)
     assert float(e.mean()) < 2.5 * float(r.mean()) and float(e.max()) < 3 * max(float(r.max()), 0.02), \
         (note, float(e.mean()), float(r.mean()), float(e.max()), float(r.max()))
+
+
+def interleave(queue, seed):
+    """Steps over requests whose pieces wait in ``queue``: up to four live at a time, some left out of a step."""
+    rng = np.random.default_rng(seed)
+    queue = {i: list(p) for i, p in queue.items()}
+    steps, live, waiting = [], [], list(queue)
+    while live or waiting:
+        while waiting and len(live) < 4:
+            live.append(waiting.pop(0))
+        step = []
+        for i in list(live):
+            if rng.random() < 0.25 and len(live) > 1:
+                continue
+            piece = queue[i].pop(0)
+            step.append((i, piece, not queue[i]))
+            if not queue[i]:
+                live.remove(i)
+        if step:
+            steps.append(step)
+    return steps

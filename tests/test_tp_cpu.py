@@ -80,7 +80,7 @@ def _run(preset, world, tp, ep=False, pp=1, dcp=1, pcp=1, fg=None, addcfg=None, 
     return json.loads(line[7:])
 
 
-@pytest.mark.parametrize("preset", ["tiny-qwen", "tiny-moe", "tiny-deepseek", "tiny-mqa", "tiny-vofelix"])
+@pytest.mark.parametrize("preset", ["tiny-qwen", "tiny-moe", "tiny-deepseek", "tiny-mqa", "tiny-vofelix", "tiny-pegopel"])
 def test_tp2_matches_tp1(preset):
     assert _run(preset, 2, 2) == _run(preset, 1, 1)
 
