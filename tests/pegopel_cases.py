@@ -96,7 +96,7 @@ _KNOWN = {}
 
 
 def reference(cfg, w, ids, rounded=False):
-    key = (json.dumps(cfg), float(w["embed"].double().sum()), tuple(ids), rounded)
+    key = (json.dumps(cfg), sum(float(t.double().sum()) for t in w.values()), tuple(ids), rounded)
     if key not in _KNOWN:
         _KNOWN[key] = po.forward(cfg, w, ids, rounded=rounded)
     return _KNOWN[key]
