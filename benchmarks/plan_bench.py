@@ -1,5 +1,5 @@
 #!/usr/bin/env python
-"""Prefill and decode throughput of plan-built decoders (Vofelix) beside the closest existing models at equal
+"""Prefill and decode throughput of plan-built decoders (Vofelix, Pegopel) beside the closest existing models at equal
 size, random weights, one GPU.
 
     python bench.py --mode layers                 # or: python benchmarks/plan_bench.py
@@ -50,6 +50,33 @@ def _vofelix(layers, side=128, loop=None):
     return ModelConfig.from_hf_dict(d, name="vofelix-bench")
 
 
+def _biased(window=1024, conv=4):
+    return {"type": "attention", "mlp": {"kind": "dense", "ff": 12288}, "mixer": {
+        "heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "conv": conv, "scale": 128 ** -0.5, "bias_max": 512,
+        "mask": {"size": window}}}
+
+
+def _gated(window=1024, keep=64):
+    return {"type": "attention_2", "mlp": {"kind": "dense", "ff": 12288}, "mixer": {
+        "heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0,
+        "mask": {"size": window, "keep_first": keep},
+        "rot": {"base": 1e4, "dims": 128, "scaling": {"factor": 2.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}}
+
+
+def _pegopel(layers, streams=1, loop=None):
+    from vllm_ascend_b200.config import ModelConfig
+    d = {"architecture": "Pegopel", "vocab": VOCAB, "width": 4096, "norm": {"eps": 1e-6}, "max_positions": 4096,
+         "streams": streams, "layers": layers}
+    if loop:
+        d["loop"] = loop
+    return ModelConfig.from_hf_dict(d, name="pegopel-bench")
+
+
+def _gqa(window):
+    return _existing(name="gqa-dense", architecture="Qwen3ForCausalLM", num_attention_heads=32, num_key_value_heads=8,
+                     head_dim=128, qk_norm=True, sliding_window=window, rope_theta=1e4)
+
+
 def _existing(**kw):
     from vllm_ascend_b200.config import ModelConfig
     return ModelConfig(vocab_size=VOCAB, hidden_size=4096, intermediate_size=12288, num_hidden_layers=LAYERS,
@@ -69,7 +96,7 @@ def _gdn():
                      linear_value_head_dim=128, linear_conv_kernel_dim=4)
 
 
-#: label -> configuration.  The plain Vofelix stacks have the mixers and feed-forward of their neighbour
+#: label -> configuration.  The plain Vofelix and Pegopel stacks have the mixers and feed-forward of their neighbour
 MODELS = {
     "latent w=0 h32": lambda: _vofelix([_latent(32, 0)] * LAYERS, side=0),
     "existing MLA h32": lambda: _mla(32),
@@ -80,6 +107,12 @@ MODELS = {
     "existing GDN": lambda: _gdn(),
     "whole design": lambda: _vofelix([_delta(None), _latent(32, 1024), _delta(None), _delta(None), _latent(32, 1024),
                                       _delta(None)], loop={"start": 1, "stop": 4, "times": 2}),
+    "biased attention w=1024": lambda: _pegopel([_biased()] * LAYERS),
+    "gated attention w=1024": lambda: _pegopel([_gated()] * LAYERS),
+    "existing GQA w=1024": lambda: _gqa(1024),
+    "biased attention, 4 streams": lambda: _pegopel([_biased()] * LAYERS, streams=4),
+    "Pegopel, 2 streams, loop": lambda: _pegopel([_gated(), _biased(), _biased(), _gated(), _biased(), _biased()], streams=2,
+                                                 loop={"start": 1, "stop": 3, "times": 2}),
 }
 
 
@@ -219,7 +252,88 @@ def bench_kernels() -> list[dict]:
                 timeit(lambda: mla.latent_attention_tc(ql, qp, lat, pe, bt, 0.07, cu=cu, seq_lens=sl, uniform=n == 1,
                                                        window=win, sink=sink, max_kv_len=ctx)),
                 reads * 1152 + T * H * (576 + 512) * 2, keys * H * (576 + 512) * 2)
+    res += _variant_kernels(rec_list=[], hbm=hbm, tf=tf)
     return res
+
+
+def _variant_kernels(rec_list, hbm, tf) -> list[dict]:
+    """The kernels of paged attention with options and of parallel streams, beside their plain counterparts."""
+    from kernel_bench import timeit
+    from vllm_ascend_b200 import ops
+    from vllm_ascend_b200.attention import variant as va
+    from vllm_ascend_b200.attention.metadata import AttentionMetadata, build_tile_worklist
+    from vllm_ascend_b200.ops import stream as st
+    bf, dev = torch.bfloat16, "cuda"
+
+    def rec(name, ms, nbytes=0, flops=0):
+        t_mem, t_fl = nbytes / hbm / 1e6, flops / tf / 1e9
+        rec_list.append({"kernel": name, "ms": round(ms, 4), "GB/s": round(nbytes / ms / 1e6),
+                         "TFLOP/s": round(flops / ms / 1e9, 1), "roofline_frac": round(max(t_mem, t_fl) / ms, 3)})
+
+    def mk(*s, dtype=bf):
+        return torch.randn(*s, device=dev, dtype=dtype)
+    W = 4096
+    for T in (256, 8192):
+        y, w, res_b = mk(T, W), mk(W), mk(T, W)
+        rec(f"[existing] add+rms_norm T={T}", timeit(lambda: ops.rms_norm(y, w, 1e-6, res_b)), T * W * 8)
+        for S in (1, 2, 4):
+            r = mk(T, S, W, dtype=torch.float32)
+            m = st.StreamMix(torch.ones(S, device=dev) / S, torch.ones(S, device=dev), torch.eye(S, device=dev))
+            n = st.NormSpec("rms", w)
+            rec(f"stream_mix S={S} T={T}", timeit(lambda: st.stream_mix(r, y, st.PLAIN, m, m, n, 1e-6, bf)),
+                T * W * (8 * S + 4))
+    Hq, G, D = 32, 8, 128
+    for B, n, ctx in ((64, 1, 2048), (256, 1, 2048), (4, 2048, 2048)):
+        bs, T = 128, B * n
+        nb = B * ctx // bs + 1
+        kc, vc = (ops.alloc_kv_cache(nb, bs, G, D, bf, dev) for _ in "kv")
+        kc.normal_()
+        vc.normal_()
+        bt = (torch.arange(B * ctx // bs, dtype=torch.int32, device=dev).view(B, -1) + 1).contiguous()
+        cu = np.arange(0, T + 1, n, dtype=np.int32)
+        sl = np.full(B, ctx, dtype=np.int32)
+        pos = torch.arange(ctx - n, ctx, device=dev).repeat(B)
+        slot = (bt[torch.arange(B, device=dev).repeat_interleave(n), pos // bs].long()) * bs + pos % bs
+        meta = AttentionMetadata(
+            num_reqs=B, num_actual_tokens=T, max_query_len=n, max_seq_len=ctx, query_start_loc=torch.from_numpy(cu).to(dev),
+            seq_lens=torch.from_numpy(sl).to(dev), block_table=bt, slot_mapping=slot, positions=pos, query_start_loc_cpu=cu,
+            seq_lens_cpu=sl, num_decodes=B if n == 1 else 0, num_decode_tokens=B if n == 1 else 0)
+        meta.state_slots = torch.arange(B, dtype=torch.int32, device=dev)
+        meta.has_initial_state = torch.ones(B, dtype=torch.int32, device=dev)
+        if n > 1:
+            ts, tq = build_tile_worklist(np.full(B, n, dtype=np.int32), 128 // (Hq // G), sl)
+            meta.tile_seq, meta.tile_qoff, meta.num_tiles = torch.from_numpy(ts).to(dev), torch.from_numpy(tq).to(dev), len(ts)
+        else:
+            meta.num_splits = ops.choose_num_splits(B, G, ctx)
+        tag = f"{B}x{n} ctx {ctx}"
+        C = (Hq + 2 * G) * D
+        qkv, qn, kn = mk(T, C), mk(Hq * D), mk(G * D)
+        cs = torch.randn(4096, D, device=dev)
+        rec(f"[existing] qknorm_rope_kvwrite {tag}", timeit(lambda: ops.qknorm_rope_kvwrite(
+            qkv, pos, cs, D, qn[:D], kn[:D], 1e-6, kc, vc, slot, Hq, G, D)), T * C * 4)
+        spec = va.PrepSpec(Hq, G, D, D, 1e-6, qn, kn, (Hq * D, G * D), conv=mk(C, 4))
+        state = mk(B, 3, C)
+        rec(f"qkv_prep conv {tag}", timeit(lambda: va.qkv_prep(spec, qkv, meta, kc, vc, state)),
+            T * C * 4 + B * C * 3 * 4)
+        spec2 = va.PrepSpec(Hq, G, D, D, 1e-6, qn, kn, (Hq * D, G * D), values_from_keys=True, rot_dims=D, cos_sin=cs)
+        rec(f"qkv_prep rotary, v = k {tag}", timeit(lambda: va.qkv_prep(spec2, qkv, meta, kc, vc)),
+            T * ((Hq + G) * D * 2 + (Hq + 2 * G) * D * 2))
+        q = mk(T, Hq, D)
+        bias = torch.randn(Hq, 460, device=dev)
+        zero, gate = torch.zeros(Hq, device=dev), mk(T, Hq)
+        sc = D ** -0.5
+        for win in (1024, 0):
+            keys = sum(min(win or ctx, ctx - n + i + 1) for i in range(n)) * B
+            nbytes = B * min(ctx, (win or ctx) + n) * G * D * 4 + T * Hq * D * 4
+            fl = keys * Hq * D * 4
+            rec(f"[existing] paged attention {tag} window {win}",
+                timeit(lambda: ops.paged_attention(q, kc, vc, meta, sc, window=win)), nbytes, fl)
+            for name, o, g in (("no options", va.AttnOptions(sc, win), None),
+                               ("bias + sink", va.AttnOptions(sc, win, bias=bias, sink=zero), None),
+                               ("cap + kept + gate", va.AttnOptions(sc, win, 64, 50.0, sink=zero), gate)):
+                rec(f"attention {name} {tag} window {win}", timeit(lambda: va.variant_attention(q, kc, vc, meta, o, g)),
+                    nbytes, fl)
+    return rec_list
 
 
 def run_models(names=None) -> dict:
@@ -229,8 +343,13 @@ def run_models(names=None) -> dict:
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--kernels", action="store_true")
+    ap.add_argument("--variant-kernels", action="store_true", help="only the kernels of attention with options")
     ap.add_argument("--only", default="", help="model labels with commas between them")
     args = ap.parse_args()
+    if args.variant_kernels:
+        for row in _variant_kernels([], *peaks()):
+            print(json.dumps(row))
+        return
     if args.kernels:
         for row in bench_kernels():
             print(json.dumps(row))

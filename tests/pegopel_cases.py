@@ -102,17 +102,21 @@ def reference(cfg, w, ids, rounded=False):
     return _KNOWN[key]
 
 
-def check(got, cfg, w, ids, dtype, note=None):
-    """fp32: every position within 1e-4.  bf16: the errors are those of rounding, i.e. neither their mean nor
-    the largest is far above what rounding the sub-layers' inputs and outputs causes in the definition."""
-    want = reference(cfg, w, ids)
-    e = errors(got, want)
+def check_all(pairs, cfg, w, dtype, note=None):
+    """``pairs`` of (logits, token ids).  fp32: every position within 1e-4.  bf16: the errors are those of rounding,
+    i.e. neither their mean over all positions nor the largest is far above what rounding the sub-layers' inputs and
+    outputs causes in the definition."""
+    e = torch.cat([errors(got, reference(cfg, w, ids)) for got, ids in pairs])
     if dtype == "float32":
         assert float(e.max()) < 1e-4, (note, float(e.max()))
         return
-    r = errors(reference(cfg, w, ids, True), want)
+    r = torch.cat([errors(reference(cfg, w, ids, True), reference(cfg, w, ids)) for _, ids in pairs])
     assert float(e.mean()) < 2.5 * float(r.mean()) and float(e.max()) < 3 * max(float(r.max()), 0.02), \
         (note, float(e.mean()), float(r.mean()), float(e.max()), float(r.max()))
+
+
+def check(got, cfg, w, ids, dtype, note=None):
+    check_all([(got, ids)], cfg, w, dtype, note)
 
 
 def interleave(queue, seed):

@@ -50,8 +50,7 @@ def test_unequal_requests_in_one_batch_with_reused_pages_and_slots(cases, name, 
     sizes = ([40, 1, 1, 2], [1], [70], [2, 1], [5, 1], [1, 64], [3])
     rp = engine(path, dtype, max_tokens=16 * 32, page=16)
     got = pc.replay(rp, pc.interleave({i: pc.cut(t, s) for (i, t), s in zip(ids.items(), sizes)}, 7))
-    for i, t in ids.items():
-        pc.check(got[i], cfg, w, t, dtype, i)
+    pc.check_all([(got[i], t) for i, t in ids.items()], cfg, w, dtype)
 
 
 @pytest.mark.parametrize("name,dtype", [("A", "float32"), ("B", "bfloat16")])
