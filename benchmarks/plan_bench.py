@@ -110,8 +110,8 @@ MODELS = {
     "biased attention w=1024": lambda: _pegopel([_biased()] * LAYERS),
     "gated attention w=1024": lambda: _pegopel([_gated()] * LAYERS),
     "existing GQA w=1024": lambda: _gqa(1024),
-    "biased attention, 4 streams": lambda: _pegopel([_biased()] * LAYERS, streams=4),
-    "Pegopel, 2 streams, loop": lambda: _pegopel([_gated(), _biased(), _biased(), _gated(), _biased(), _biased()], streams=2,
+    "biased attention 4 streams": lambda: _pegopel([_biased()] * LAYERS, streams=4),
+    "Pegopel 2 streams loop": lambda: _pegopel([_gated(), _biased(), _biased(), _gated(), _biased(), _biased()], streams=2,
                                                  loop={"start": 1, "stop": 3, "times": 2}),
 }
 

@@ -6,8 +6,8 @@
 // stores is fp32; element type bf16 or fp32 (template), all sizes are run-time values.
 //
 // A block owns up to TILE consecutive tokens of one sequence and either all q channels or all k / v channels;
-// a thread owns PER vectors of VEC channels and walks the tokens with the convolution window in registers, the
-// next row in flight while the current one is reduced.  Only a sequence's first tile reads the convolution
+// a thread owns PER vectors of VEC channels and walks the tokens GT at a time with the convolution window in
+// registers, the next rows in flight while the current ones are reduced (one barrier per GT tokens).  Only a sequence's first tile reads the convolution
 // state, and the same threads write the new one afterwards, so no two blocks touch a state row.
 // The reference fuses split, q / k norm and rotary the same way (vllm_ascend/ops/triton/linearnorm/
 // split_qkv_rmsnorm_rope.py).
@@ -42,17 +42,44 @@ struct QkvPrepArgs {
 
 struct QkvPrepParams : QkvPrepArgs {
   int tile;                   // tokens of a block
+  int first_part;             // 0: grid.y covers q, then k / v; 1: k / v only
   int* status;
 };
 
 constexpr int PREP_THREADS = 512;
 
+// N elements kept packed in registers
+template <typename T, int N>
+struct Packed {
+  union {
+    typename RawVec<N * (int)sizeof(T)>::type raw;
+    uint32_t word[(N * sizeof(T) + 3) / 4];
+  };
+  __device__ __forceinline__ void load(const T* p) {
+    raw = *reinterpret_cast<const typename RawVec<N * (int)sizeof(T)>::type*>(p);
+  }
+  __device__ __forceinline__ void zero() {
+#pragma unroll
+    for (int i = 0; i < (int)(N * sizeof(T) + 3) / 4; i++) word[i] = 0u;
+  }
+  __device__ __forceinline__ float get(int e) const {
+    if constexpr (sizeof(T) == 4) return __uint_as_float(word[e]);
+    return __uint_as_float((e & 1) ? word[e >> 1] & 0xffff0000u : word[e >> 1] << 16);
+  }
+  __device__ __forceinline__ void add(int e, T v) {          // into a zeroed place
+    if constexpr (sizeof(T) == 4) word[e] = __float_as_uint(to_f(v));
+    else word[e >> 1] |= (e & 1) ? __float_as_uint(to_f(v)) : __float_as_uint(to_f(v)) >> 16;
+  }
+};
+
 // KR: taps held in registers (0: no convolution, 4: up to four taps, -1: any number, read again per token)
 template <typename T, int VEC, int PER, int KR>
-__global__ void __launch_bounds__(PREP_THREADS) qkv_prep_kernel(const QkvPrepParams p) {
-  __shared__ float red[2][32];
+__global__ void __launch_bounds__(PREP_THREADS, KR == 0 && PER == 1 && VEC > 1 ? 2 : 1) qkv_prep_kernel(const QkvPrepParams p) {
+  // tokens reduced together
+  constexpr int GT = KR > 0 && PER == 1 ? 4 : KR == 0 && PER == 1 && VEC > 1 ? 2 : 1;
+  __shared__ float red[2][GT][32];
   extern __shared__ float row[];                    // VEC == 1: the normalised row, for the rotary partner
-  const int part = blockIdx.y;
+  const int part = p.first_part + blockIdx.y;
   const int Nq = p.heads * p.dim, Nk = p.kv_heads * p.dim, Nv = p.values_from_keys ? 0 : p.kv_heads * p.vdim;
   const int C = Nq + Nk + Nv;
   const int width = part == 0 ? Nq : Nk + Nv, col0 = part == 0 ? 0 : Nq;
@@ -95,19 +122,29 @@ __global__ void __launch_bounds__(PREP_THREADS) qkv_prep_kernel(const QkvPrepPar
     st = (T*)p.state + (long)slot * (p.taps - 1) * C + col0;
     init = p.has_init[b] != 0;
   }
-  auto input = [&](int i, int c, T* v) {            // input of local token i, reaching back into the state
-    if (i >= 0) load_raw<T, VEC>(x + (long)i * p.qkv_stride + c, v);
-    else if (init && p.taps - 1 + i >= 0) load_raw<T, VEC>(st + (long)(p.taps - 1 + i) * C + c, v);
-    else
-#pragma unroll
-      for (int e = 0; e < VEC; e++) v[e] = from_f<T>(0.f);
+  using Vec = Packed<T, VEC>;
+  auto input = [&](int i, int c, Vec& v) {          // input of local token i, reaching back into the state
+    if (i >= 0) v.load(x + (long)i * p.qkv_stride + c);
+    else if (init && p.taps - 1 + i >= 0) v.load(st + (long)(p.taps - 1 + i) * C + c);
+    else v.zero();
   };
   constexpr int KW = KR > 0 ? KR : 1;
-  T wk[PER][KW][VEC], win[PER][KW][VEC], nxt[PER][VEC];
+  Vec wk[PER][KW], win[PER][KW], rows[GT][PER], nw[PER];
+  int head[PER], dd[PER];                           // head and place in it of the thread's channels
+  const T* norm_w = (const T*)(part == 0 ? p.q_norm : p.k_norm);
 #pragma unroll
   for (int r = 0; r < PER; r++) {
     const int v = (int)threadIdx.x + r * (int)blockDim.x, c = v * VEC;
+    head[r] = dd[r] = 0;
     if (v >= nvec) continue;
+    if (c < normed) {
+      head[r] = c / p.dim;
+      dd[r] = c - head[r] * p.dim;
+      nw[r].load(norm_w + c);
+    } else {
+      head[r] = (c - normed) / p.vdim;
+      dd[r] = c - normed - head[r] * p.vdim;
+    }
     if constexpr (KR > 0) {
       const T* w = (const T*)p.conv_w + (long)(col0 + c) * p.taps;
       if (VEC > 1 && p.taps == KR) {                // KR * VEC weights in a row
@@ -116,150 +153,173 @@ __global__ void __launch_bounds__(PREP_THREADS) qkv_prep_kernel(const QkvPrepPar
 #pragma unroll
         for (int k = 0; k < KR * VEC; k += (VEC > 1 ? WV : 1)) load_raw<T, (VEC > 1 ? WV : 1)>(w + k, wr + k);
 #pragma unroll
-        for (int k = 0; k < KR * VEC; k++) wk[r][k % KR][k / KR] = wr[k];
+        for (int j = 0; j < KR; j++) wk[r][j].zero();
+#pragma unroll
+        for (int k = 0; k < KR * VEC; k++) wk[r][k % KR].add(k / KR, wr[k]);
       } else {
 #pragma unroll
         for (int j = 0; j < KR; j++) {
           const int jj = j - (KR - p.taps);         // fewer taps: the oldest places weigh nothing
+          wk[r][j].zero();
+          if (jj >= 0)
 #pragma unroll
-          for (int e = 0; e < VEC; e++) wk[r][j][e] = jj >= 0 ? w[(long)e * p.taps + jj] : from_f<T>(0.f);
+            for (int e = 0; e < VEC; e++) wk[r][j].add(e, w[(long)e * p.taps + jj]);
         }
       }
 #pragma unroll
       for (int j = 0; j < KR - 1; j++) {
         if (j >= KR - p.taps) input(i0 - (KR - 1) + j, c, win[r][j]);
-        else
-#pragma unroll
-          for (int e = 0; e < VEC; e++) win[r][j][e] = from_f<T>(0.f);
+        else win[r][j].zero();
       }
     }
-    load_raw<T, VEC>(x + (long)i0 * p.qkv_stride + c, nxt[r]);
+    if (KR >= 0)
+#pragma unroll
+      for (int f = 0; f < GT; f++)
+        if (i0 + f < i1) rows[f][r].load(x + (long)(i0 + f) * p.qkv_stride + c);
   }
   const int warps = (blockDim.x + 31) >> 5;
-  const T* nw = (const T*)(part == 0 ? p.q_norm : p.k_norm);
   const int half = p.rot >> 1;
 
-  for (int i = i0; i < i1; i++) {
-    const long t = t_seq + i;
-    float u[PER][VEC];
-    float ss = 0.f;
+  for (int ib = i0; ib < i1; ib += GT) {
+    float u[GT][PER][VEC], ss[GT];
+    long pos[GT], slot[GT];
 #pragma unroll
-    for (int r = 0; r < PER; r++) {
-      const int v = (int)threadIdx.x + r * (int)blockDim.x, c = v * VEC;
-      if (v >= nvec) continue;
-      if constexpr (KR > 0) {
+    for (int f = 0; f < GT; f++) {
+      const bool on = ib + f < i1;
+      pos[f] = on && p.rot > 0 ? p.positions[t_seq + ib + f] : 0;
+      slot[f] = on && part == 1 ? p.slot_mapping[t_seq + ib + f] : -1;
+      ss[f] = 0.f;
+      if (!on) continue;
 #pragma unroll
-        for (int e = 0; e < VEC; e++) {
-          win[r][KR - 1][e] = nxt[r][e];
-          float a = 0.f;
+      for (int r = 0; r < PER; r++) {
+        const int v = (int)threadIdx.x + r * (int)blockDim.x, c = v * VEC;
+        if (v >= nvec) continue;
+        if constexpr (KR > 0) {
+          win[r][KR - 1] = rows[f][r];
 #pragma unroll
-          for (int j = 0; j < KR; j++) a = fmaf(to_f(wk[r][j][e]), to_f(win[r][j][e]), a);
-          u[r][e] = a;
+          for (int e = 0; e < VEC; e++) {
+            float a = 0.f;
+#pragma unroll
+            for (int j = 0; j < KR; j++) a = fmaf(wk[r][j].get(e), win[r][j].get(e), a);
+            u[f][r][e] = a;
+          }
+#pragma unroll
+          for (int j = 0; j + 1 < KR; j++) win[r][j] = win[r][j + 1];
+        } else if constexpr (KR < 0) {
+          const T* w = (const T*)p.conv_w + (long)(col0 + c) * p.taps;
+#pragma unroll
+          for (int e = 0; e < VEC; e++) u[f][r][e] = 0.f;
+          for (int j = 0; j < p.taps; j++) {
+            Vec in;
+            input(ib + f - (p.taps - 1) + j, c, in);
+#pragma unroll
+            for (int e = 0; e < VEC; e++) u[f][r][e] = fmaf(to_f(w[(long)e * p.taps + j]), in.get(e), u[f][r][e]);
+          }
+        } else {
+#pragma unroll
+          for (int e = 0; e < VEC; e++) u[f][r][e] = rows[f][r].get(e);
         }
+        if (KR >= 0 && ib + GT + f < i1) rows[f][r].load(x + (long)(ib + GT + f) * p.qkv_stride + c);
+        if (c < normed)
 #pragma unroll
-        for (int j = 0; j + 1 < KR; j++)
-#pragma unroll
-          for (int e = 0; e < VEC; e++) win[r][j][e] = win[r][j + 1][e];
-      } else if constexpr (KR < 0) {
-        const T* w = (const T*)p.conv_w + (long)(col0 + c) * p.taps;
-#pragma unroll
-        for (int e = 0; e < VEC; e++) u[r][e] = 0.f;
-        for (int j = 0; j < p.taps; j++) {
-          T in[VEC];
-          input(i - (p.taps - 1) + j, c, in);
-#pragma unroll
-          for (int e = 0; e < VEC; e++) u[r][e] = fmaf(to_f(w[(long)e * p.taps + j]), to_f(in[e]), u[r][e]);
-        }
-      } else {
-#pragma unroll
-        for (int e = 0; e < VEC; e++) u[r][e] = to_f(nxt[r][e]);
+          for (int e = 0; e < VEC; e++) ss[f] = fmaf(u[f][r][e], u[f][r][e], ss[f]);
       }
-      if (KR >= 0 && i + 1 < i1) load_raw<T, VEC>(x + (long)(i + 1) * p.qkv_stride + c, nxt[r]);
-      if (c < normed)
-#pragma unroll
-        for (int e = 0; e < VEC; e++) ss = fmaf(u[r][e], u[r][e], ss);
     }
     if (p.phase == 2) {
-      ss = p.sums[t * 2 + part];
+#pragma unroll
+      for (int f = 0; f < GT; f++)
+        if (ib + f < i1) ss[f] = p.sums[(t_seq + ib + f) * 2 + part];
     } else {
-      ss = warp_reduce_sum(ss);
+#pragma unroll
+      for (int f = 0; f < GT; f++) ss[f] = warp_reduce_sum(ss[f]);
       if (warps > 1) {
-        float* rd = red[(i - i0) & 1];              // two buffers: one barrier per token
-        if ((threadIdx.x & 31) == 0) rd[threadIdx.x >> 5] = ss;
+        auto& rd = red[((ib - i0) / GT) & 1];       // two buffers: one barrier per group
+        if ((threadIdx.x & 31) == 0)
+#pragma unroll
+          for (int f = 0; f < GT; f++) rd[f][threadIdx.x >> 5] = ss[f];
         __syncthreads();
-        ss = warp_reduce_sum((threadIdx.x & 31) < warps ? rd[threadIdx.x & 31] : 0.f);
+#pragma unroll
+        for (int f = 0; f < GT; f++) ss[f] = warp_reduce_sum((threadIdx.x & 31) < warps ? rd[f][threadIdx.x & 31] : 0.f);
       }
       if (p.phase == 1) {
-        if (threadIdx.x == 0) p.sums[t * 2 + part] = ss;
+        if (threadIdx.x == 0)
+#pragma unroll
+          for (int f = 0; f < GT; f++)
+            if (ib + f < i1) p.sums[(t_seq + ib + f) * 2 + part] = ss[f];
         continue;
       }
     }
-    const float inv = 1.f / sqrtf(ss / (float)(part == 0 ? p.q_norm_dims : p.k_norm_dims) + p.eps);
-    long slot = -1;
-    T *kdst = nullptr, *vdst = nullptr;
-    if (part == 1) {
-      slot = p.slot_mapping[t];
-      if (slot >= p.cache_slots) {
+#pragma unroll
+    for (int f = 0; f < GT; f++) {
+      if (ib + f >= i1) break;
+      const long t = t_seq + ib + f;
+      const float inv = 1.f / sqrtf(ss[f] / (float)(part == 0 ? p.q_norm_dims : p.k_norm_dims) + p.eps);
+      T *kdst = nullptr, *vdst = nullptr;
+      if (slot[f] >= p.cache_slots) {
         if (threadIdx.x == 0 && p.status) atomicExch(p.status, B200_BAD_INDEX);
-        slot = -1;
-      }
-      if (slot >= 0) {
-        const long blk = slot / p.block_size, off = slot - blk * p.block_size;
+      } else if (slot[f] >= 0) {
+        const unsigned blk = (unsigned)slot[f] / (unsigned)p.block_size, off = (unsigned)slot[f] - blk * p.block_size;
         kdst = (T*)p.k_cache + blk * p.k_block + off * p.k_tok;
         vdst = (T*)p.v_cache + blk * p.v_block + off * p.v_tok;
       }
-    }
-    const float* cs = nullptr;
-    if (p.rot > 0) {
-      const long pos = p.positions[t];
-      if (pos >= 0 && pos < p.cos_rows) cs = p.cos_sin + pos * p.rot;
-      else if (threadIdx.x == 0 && p.status) atomicExch(p.status, B200_BAD_INDEX);
-    }
-    if constexpr (VEC == 1) {
-      if (cs) {
-        __syncthreads();                            // the previous token's partners have been read
+      const float* cs = nullptr;
+      if (p.rot > 0) {
+        if (pos[f] >= 0 && pos[f] < p.cos_rows) cs = p.cos_sin + pos[f] * p.rot;
+        else if (threadIdx.x == 0 && p.status) atomicExch(p.status, B200_BAD_INDEX);
+      }
+      if constexpr (VEC == 1) {
+        if (cs) {
+          __syncthreads();                          // the previous token's partners have been read
 #pragma unroll
-        for (int r = 0; r < PER; r++) {
-          const int c = (int)threadIdx.x + r * (int)blockDim.x;
-          if (c < normed) row[c] = u[r][0] * inv * to_f(nw[c]);
+          for (int r = 0; r < PER; r++) {
+            const int c = (int)threadIdx.x + r * (int)blockDim.x;
+            if (c < normed) row[c] = u[f][r][0] * inv * nw[r].get(0);
+          }
+          __syncthreads();
         }
-        __syncthreads();
       }
-    }
 #pragma unroll
-    for (int r = 0; r < PER; r++) {
-      const int v = (int)threadIdx.x + r * (int)blockDim.x, c = v * VEC;
-      if (v >= nvec) continue;
-      if (c >= normed) {                            // values
-        const int h = (c - normed) / p.vdim, d = (c - normed) - h * p.vdim;
-        if (vdst) store_vec<T, VEC>(vdst + h * p.v_head + d, u[r]);
-        continue;
-      }
-      const int h = c / p.dim, d = c - h * p.dim;
-      if (part == 1 && p.values_from_keys && vdst) store_vec<T, VEC>(vdst + h * p.v_head + d, u[r]);
-      float wv[VEC], y[VEC];
-      load_vec<T, VEC>(nw + c, wv);
+      for (int r = 0; r < PER; r++) {
+        const int v = (int)threadIdx.x + r * (int)blockDim.x, c = v * VEC;
+        if (v >= nvec) continue;
+        const int d = dd[r];
+        if (c >= normed) {                          // values
+          if (vdst) store_vec<T, VEC>(vdst + head[r] * p.v_head + d, u[f][r]);
+          continue;
+        }
+        if (part == 1 && p.values_from_keys && vdst) store_vec<T, VEC>(vdst + head[r] * p.v_head + d, u[f][r]);
+        float y[VEC];
 #pragma unroll
-      for (int e = 0; e < VEC; e++) y[e] = u[r][e] * inv * wv[e];
-      if (cs && d < p.rot) {
-        if constexpr (VEC == 1) {
-          const int k = d >> 1;
-          const float other = (d & 1) ? row[c - 1] : row[c + 1];
-          y[0] = (d & 1) ? y[0] * cs[k] + other * cs[half + k] : y[0] * cs[k] - other * cs[half + k];
-        } else {
+        for (int e = 0; e < VEC; e++) y[e] = u[f][r][e] * inv * nw[r].get(e);
+        if (cs && d < p.rot) {
+          if constexpr (VEC == 1) {
+            const int k = d >> 1;
+            const float other = (d & 1) ? row[c - 1] : row[c + 1];
+            y[0] = (d & 1) ? y[0] * cs[k] + other * cs[half + k] : y[0] * cs[k] - other * cs[half + k];
+          } else {
+            float cc[VEC / 2], sn[VEC / 2];
+            if ((p.rot & (2 * VEC - 1)) == 0) {     // whole aligned vectors of the table
+              load_vec<float, VEC / 2>(cs + (d >> 1), cc);
+              load_vec<float, VEC / 2>(cs + half + (d >> 1), sn);
+            } else {
 #pragma unroll
-          for (int e = 0; e + 1 < VEC; e += 2) {
-            if (d + e < p.rot) {
-              const int k = (d + e) >> 1;
-              const float cc = cs[k], sn = cs[half + k], a = y[e], bb = y[e + 1];
-              y[e] = a * cc - bb * sn;
-              y[e + 1] = bb * cc + a * sn;
+              for (int e = 0; e < VEC / 2; e++) {
+                const bool turned = d + 2 * e < p.rot;
+                cc[e] = turned ? cs[(d >> 1) + e] : 1.f;
+                sn[e] = turned ? cs[half + (d >> 1) + e] : 0.f;
+              }
+            }
+#pragma unroll
+            for (int e = 0; e < VEC; e += 2) {
+              const float a = y[e], bb = y[e + 1];
+              y[e] = a * cc[e / 2] - bb * sn[e / 2];
+              y[e + 1] = bb * cc[e / 2] + a * sn[e / 2];
             }
           }
         }
+        if (part == 0) store_vec<T, VEC>((T*)p.q_out + t * Nq + c, y);
+        else if (kdst) store_vec<T, VEC>(kdst + head[r] * p.k_head + d, y);
       }
-      if (part == 0) store_vec<T, VEC>((T*)p.q_out + t * Nq + c, y);
-      else if (kdst) store_vec<T, VEC>(kdst + h * p.k_head + d, y);
     }
   }
   // ---- the last taps - 1 inputs of the sequence (its first tile owns the state row)
@@ -269,11 +329,11 @@ __global__ void __launch_bounds__(PREP_THREADS) qkv_prep_kernel(const QkvPrepPar
       const int v = (int)threadIdx.x + r * (int)blockDim.x, c = v * VEC;
       if (v >= nvec) continue;
       for (int j = 0; j < p.taps - 1; j++) {
-        T in[VEC];
+        Vec in;
         input(n - (p.taps - 1) + j, c, in);         // older rows move towards the front
         float f[VEC];
 #pragma unroll
-        for (int e = 0; e < VEC; e++) f[e] = to_f(in[e]);
+        for (int e = 0; e < VEC; e++) f[e] = in.get(e);
         store_vec<T, VEC>(st + (long)j * C + c, f);
       }
     }
@@ -290,26 +350,14 @@ static int launch_prep(const QkvPrepParams& p, dim3 grid, int threads, size_t sm
 }
 
 template <typename T>
-static int prep_t(QkvPrepParams& p, cudaStream_t stream) {
+static int launch_parts(const QkvPrepParams& p, unsigned tiles, unsigned parts, int width, bool vec, cudaStream_t stream) {
   constexpr int V = 16 / (int)sizeof(T);
-  const int Nq = p.heads * p.dim, Nkv = p.kv_heads * (p.dim + (p.values_from_keys ? 0 : p.vdim));
-  const int width = Nq > Nkv ? Nq : Nkv;
-  const long s[] = {p.qkv_stride, p.k_block, p.k_tok, p.k_head, p.v_block, p.v_tok, p.v_head, p.dim, p.vdim};
-  bool vec = aligned16(p.qkv) && aligned16(p.conv_w) && aligned16(p.state) && aligned16(p.q_norm) &&
-             aligned16(p.k_norm) && aligned16(p.q_out) && aligned16(p.k_cache) && aligned16(p.v_cache);
-  for (long x : s) vec = vec && x % V == 0;
   const int nvec = width / (vec ? V : 1);
   int per = (nvec + PREP_THREADS - 1) / PREP_THREADS;
   per = vec ? (per <= 1 ? 1 : per <= 2 ? 2 : 4) : (per <= 2 ? 2 : 16);
   if ((long)per * PREP_THREADS < nvec) return 9821;
   const int threads = ((nvec + per - 1) / per + 31) / 32 * 32;
-  // tokens of a block: enough to share the convolution's history and weights, few enough to fill the GPU
-  p.tile = p.tokens >= 8192 ? 16 : p.tokens >= 2048 ? 8 : p.tokens >= 512 ? 2 : 1;
-  if (p.taps > 0 && p.tile < 4) p.tile = 4;
-  if (p.tile < p.taps - 1) p.tile = p.taps - 1;     // only a first tile reaches back into the state
-  const long tiles = p.taps == 0 ? (p.tokens + p.tile - 1) / p.tile
-                                 : p.uniform ? p.num_seqs : p.tokens / p.tile + p.num_seqs;
-  const dim3 grid((unsigned)tiles, 2);
+  const dim3 grid(tiles, parts);
   if (vec) {
     if (per == 1) return launch_prep<T, V, 1>(p, grid, threads, 0, stream);
     if (per == 2) return launch_prep<T, V, 2>(p, grid, threads, 0, stream);
@@ -320,6 +368,32 @@ static int prep_t(QkvPrepParams& p, cudaStream_t stream) {
   return launch_prep<T, 1, 16>(p, grid, threads, smem, stream);
 }
 
+template <typename T>
+static int prep_t(QkvPrepParams& p, cudaStream_t stream) {
+  constexpr int V = 16 / (int)sizeof(T);
+  const int Nq = p.heads * p.dim, Nkv = p.kv_heads * (p.dim + (p.values_from_keys ? 0 : p.vdim));
+  const long s[] = {p.qkv_stride, p.k_block, p.k_tok, p.k_head, p.v_block, p.v_tok, p.v_head, p.dim, p.vdim};
+  bool vec = aligned16(p.cos_sin) && aligned16(p.qkv) && aligned16(p.conv_w) && aligned16(p.state) &&
+             aligned16(p.q_norm) && aligned16(p.k_norm) && aligned16(p.q_out) && aligned16(p.k_cache) &&
+             aligned16(p.v_cache);
+  for (long x : s) vec = vec && x % V == 0;
+  // tokens of a block: enough to share the convolution's history and weights, few enough to fill the GPU
+  p.tile = p.tokens >= 8192 ? 16 : p.tokens >= 2048 ? 8 : p.tokens >= 512 ? 2 : 1;
+  if (p.taps > 0 && p.tile < 4) p.tile = 4;
+  if (p.tile < p.taps - 1) p.tile = p.taps - 1;     // only a first tile reaches back into the state
+  const long tiles = p.taps == 0 ? (p.tokens + p.tile - 1) / p.tile
+                                 : p.uniform ? p.num_seqs : p.tokens / p.tile + p.num_seqs;
+  p.first_part = 0;
+  // long steps: blocks of their own size for the narrower part
+  if (p.tokens >= 2048 && 2 * Nkv <= Nq) {
+    const int rc = launch_parts<T>(p, (unsigned)tiles, 1, Nq, vec, stream);
+    if (rc) return rc;
+    p.first_part = 1;
+    return launch_parts<T>(p, (unsigned)tiles, 1, Nkv, vec, stream);
+  }
+  return launch_parts<T>(p, (unsigned)tiles, 2, Nq > Nkv ? Nq : Nkv, vec, stream);
+}
+
 }  // namespace b200
 
 using namespace b200;
@@ -327,6 +401,7 @@ using namespace b200;
 B200_API int b200_qkv_prep(const QkvPrepArgs* a, int* status, cudaStream_t stream) {
   if (a->tokens <= 0) return 0;
   if (a->heads < 1 || a->kv_heads < 1 || a->dim < 1 || a->vdim < 1 || a->block_size < 1 || a->num_seqs < 1) return 9800;
+  if (a->cache_slots > 0xffffffffL) return 9807;
   if (a->rot < 0 || a->rot > a->dim || (a->rot & 1) || (a->rot > 0 && !a->cos_sin)) return 9801;
   if (a->values_from_keys && a->vdim != a->dim) return 9802;
   if (a->taps < 0 || (a->taps > 0 && !a->conv_w)) return 9803;
