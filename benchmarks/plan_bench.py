@@ -58,9 +58,9 @@ def _biased(window=1024, conv=4):
 
 def _gated(window=1024, keep=64):
     return {"type": "attention_2", "mlp": {"kind": "dense", "ff": 12288}, "mixer": {
-        "heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0,
+        "heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0,
         "mask": {"size": window, "keep_first": keep},
-        "rot": {"base": 1e4, "dims": 128, "scaling": {"factor": 2.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}}
+        "rot": {"base": 1e4, "dims": 128, "scaling": {"factor": 4.0, "original": 1024, "fast": 24.0, "slow": 2.0}}}}
 
 
 def _pegopel(layers, streams=1, loop=None):
@@ -330,7 +330,7 @@ def _variant_kernels(rec_list, hbm, tf) -> list[dict]:
                 timeit(lambda: ops.paged_attention(q, kc, vc, meta, sc, window=win)), nbytes, fl)
             for name, o, g in (("no options", va.AttnOptions(sc, win), None),
                                ("bias + sink", va.AttnOptions(sc, win, bias=bias, sink=zero), None),
-                               ("cap + kept + gate", va.AttnOptions(sc, win, 64, 50.0, sink=zero), gate)):
+                               ("cap + kept + gate", va.AttnOptions(sc, win, 64, 30.0, sink=zero), gate)):
                 rec(f"attention {name} {tag} window {win}", timeit(lambda: va.variant_attention(q, kc, vc, meta, o, g)),
                     nbytes, fl)
     return rec_list

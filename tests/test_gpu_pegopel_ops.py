@@ -167,7 +167,7 @@ OPTIONS = {          # window, kept, cap, buckets, largest, sink, gate
     "biased": (40, 0, 0.0, 16, 60, "learned", False),
     "gated": (24, 9, 3.0, 0, 0, "zero", True),
     "far": (200, 150, 0.0, 32, 400, "learned", True),
-    "cap": (0, 0, 50.0, 0, 0, "zero", False),
+    "cap": (0, 0, 40.0, 0, 0, "zero", False),
     "all": (130, 5, 2.0, 8, 20, "learned", True),
     "one": (1, 1, 2.0, 2, 4, "zero", True),
 }
