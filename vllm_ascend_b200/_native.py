@@ -47,6 +47,8 @@ _SIGNATURES = {
     "b200_merge_attn_partials": [P, P, L, I, I, I, P, L, P, P],
     "b200_attn_decode_set_l2_prefetch": [I],
     "b200_mla_preprocess": [P, L, I, I, I, I, P, L, I, P, F, P, P, L, P, P, P, L, P, P, I, P, P],
+    "b200_latent_prep": [P, L, L, I, P, P, I, I, P, F, P, P, L, P, P, P, L, I, P, P],
+    "b200_latent_query": [P, L, I, I, I, P, P, L, P, I, P, P],
     "b200_argmax": [P, I, L, I, I, P, P],
     "b200_cast_bf16_f32": [P, L, P, L, I, I, P],
     "b200_apply_penalties": [P, L, I, I, P, I, P, I, P, P, P, P],

@@ -1,7 +1,7 @@
 """Paged grouped-query attention with options: sliding window that keeps the first tokens of a sequence, capped
 scores, a learned bias by distance, an attention sink, a gate per head on the output, value heads of another
-size than the key heads.  And the pass in front of it: short convolution, q / k norm over all heads, rotary
-positions, cache write.
+size than the key heads.  And the pass in front of it: short convolution, q / k norm (over all heads or head by
+head), rotary positions, cache write.
 
 GPU tensors run the kernels of csrc/qkv_prep.cu and csrc/attention_variant.cu (fp32, odd sizes) or the tcgen05
 kernels of csrc/attention_tc.cu and csrc/attention_decode_tc.cu (bf16); CPU tensors run the PyTorch definitions
@@ -33,7 +33,7 @@ class _PrepArgs(ctypes.Structure):
         pointers="qkv conv_w state cu slots has_init q_norm k_norm positions cos_sin slot_mapping q_out k_cache v_cache sums",
         longs="qkv_stride state_rows cache_slots k_block k_tok k_head v_block v_tok v_head tokens",
         ints="num_seqs taps heads kv_heads dim vdim q_norm_dims k_norm_dims values_from_keys rot cos_rows block_size "
-             "uniform phase dtype", floats="eps")
+             "uniform phase dtype head_norm", floats="eps")
 
 
 class _AttnArgs(ctypes.Structure):
@@ -112,6 +112,7 @@ class PrepSpec:
     conv: Optional[torch.Tensor] = None      # [columns of q, k (and v), taps]
     rot_dims: int = 0
     cos_sin: Optional[torch.Tensor] = None   # fp32 [positions, rot_dims]
+    head_norm: bool = False                  # every head by itself, q_norm and k_norm are [dim]; without convolution
 
     @property
     def columns(self) -> int:
@@ -129,12 +130,15 @@ def _prep_ref(s: PrepSpec, qkv, meta, k_cache, v_cache, state, reduce_sums):
             x = la.causal_conv1d_ref(x, s.conv, None, state, meta.query_start_loc, slots, init, act=False)
     q, k = x[:, :nq].float(), x[:, nq:nq + nk].float()
     v = x[:, nq:nq + nk] if s.values_from_keys else x[:, nq + nk:]
-    sums = torch.stack([(q * q).sum(-1), (k * k).sum(-1)], -1)
-    if reduce_sums is not None:
-        sums = reduce_sums(sums)
-    inv = torch.rsqrt(sums / torch.tensor(s.norm_dims, dtype=torch.float32) + s.eps)
-    q = (q * inv[:, :1] * s.q_norm.float()).view(T, s.heads, s.dim)
-    k = (k * inv[:, 1:] * s.k_norm.float()).view(T, s.kv_heads, s.dim)
+    if s.head_norm:
+        q, k = (ref.rms_norm(t.reshape(T, -1, s.dim), w.float(), s.eps)[0] for t, w in ((q, s.q_norm), (k, s.k_norm)))
+    else:
+        sums = torch.stack([(q * q).sum(-1), (k * k).sum(-1)], -1)
+        if reduce_sums is not None:
+            sums = reduce_sums(sums)
+        inv = torch.rsqrt(sums / torch.tensor(s.norm_dims, dtype=torch.float32) + s.eps)
+        q = (q * inv[:, :1] * s.q_norm.float()).view(T, s.heads, s.dim)
+        k = (k * inv[:, 1:] * s.k_norm.float()).view(T, s.kv_heads, s.dim)
     if s.rot_dims:
         q = ref.apply_rope_interleaved(q, meta.positions, s.cos_sin, s.rot_dims)
         k = ref.apply_rope_interleaved(k, meta.positions, s.cos_sin, s.rot_dims)
@@ -162,6 +166,9 @@ def qkv_prep(s: PrepSpec, qkv: torch.Tensor, meta, k_cache: torch.Tensor, v_cach
         raise ValueError("qkv_prep: cache rows must be dense and the projection wide enough")
     if taps > 1 and (state is None or tuple(state.shape[1:]) != (taps - 1, s.columns) or not state.is_contiguous()):
         raise ValueError("qkv_prep: convolution state of another shape")
+    widths = (s.dim, s.dim) if s.head_norm else (s.heads * s.dim, s.kv_heads * s.dim)
+    if (s.q_norm.numel(), s.k_norm.numel()) != widths or (s.head_norm and (taps or reduce_sums is not None)):
+        raise ValueError("qkv_prep: norm weights of another size, or a norm per head with a convolution")
     q = torch.empty((T, s.heads, s.dim), dtype=dt, device=dev)
     B = meta.num_reqs
     a = _PrepArgs(
@@ -176,7 +183,7 @@ def qkv_prep(s: PrepSpec, qkv: torch.Tensor, meta, k_cache: torch.Tensor, v_cach
         kv_heads=s.kv_heads, dim=s.dim, vdim=s.vdim, q_norm_dims=int(s.norm_dims[0]), k_norm_dims=int(s.norm_dims[1]),
         values_from_keys=int(s.values_from_keys), rot=s.rot_dims, cos_rows=s.cos_sin.shape[0] if s.rot_dims else 0,
         block_size=k_cache.shape[1], uniform=int(meta.max_query_len <= 1 and T == B), dtype=int(dt == torch.float32),
-        eps=s.eps)
+        head_norm=int(s.head_norm), eps=s.eps)
     if reduce_sums is None:
         _launch("b200_qkv_prep", a, dev)
         return q

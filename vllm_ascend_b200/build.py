@@ -84,6 +84,9 @@ MODEL_SOURCES = {
                 "latent_attention", "linear_attention", "mla_preprocess", "sampler", "stream_norm"),
     "Pegopel": ("activations", "attention_decode", "attention_decode_tc", "attention_tc", "attention_variant", "cache_ops",
                 "gemm_bf16", "gemm_bf16_2cta", "qkv_prep", "sampler", "stream_norm"),
+    "Dubizen": ("activations", "attention_decode", "attention_decode_tc", "attention_mla_decode", "attention_tc",
+                "attention_variant", "cache_ops", "elementwise", "gemm_bf16", "gemm_bf16_2cta", "latent_attention",
+                "mla_preprocess", "moe", "qkv_prep", "sampler", "stream_norm"),
 }
 
 

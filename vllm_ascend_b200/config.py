@@ -36,6 +36,7 @@ class ModelConfig:
     qk_norm: bool = False            # Qwen3 per-head q/k RMSNorm
     qk_norm_full: bool = False       # MiniMax-M2: RMSNorm over the whole projected q (and k) vector, all heads together
     attention_bias: bool = False     # Qwen2 style qkv bias
+    attention_out_bias: bool = False # bias of the output projection (layers of models/variant_attention.py)
     sliding_window: Optional[int] = None
     hidden_act: str = "silu"
     # ---- MoE ----
@@ -52,6 +53,8 @@ class ModelConfig:
     moe_layer_end_index: int = -1            # last MoE layer (-1: the last layer); Ernie 4.5 MoE
     moe_layer_interval: int = 1              # every n-th layer inside [first_k_dense_replace, end] is MoE
     e_score_correction_bias: bool = False
+    moe_group_score: Optional[str] = None    # score of an expert group: "max" | "top2" (sum of its best two); None: top2 with a bias
+    router_fp32: bool = False                # router weights in the model dtype, logits summed and kept in fp32
     # ---- linear attention (Gated DeltaNet hybrids: every `full_attention_interval`-th layer is
     # softmax attention, the others keep a recurrent state instead of a KV cache) ----
     full_attention_interval: int = 0
@@ -109,11 +112,14 @@ class ModelConfig:
     qk_nope_head_dim: int = 0
     qk_rope_head_dim: int = 0
     v_head_dim: int = 0
+    rope_half_split: bool = False            # checkpoint rotates (i, i + dims / 2) of the rotary part; rows are re-ordered at load
+    latent_kv_from: Optional[int] = None     # this layer attends to the latents that layer stores and has none of its own
     # ---- decoders described layer by layer (layer_plan.py) ----
     layer_plan: Optional[list] = None        # per layer {"mixer", "mlp", "over": fields of this layer}
     layer_loop: Optional[tuple] = None       # (start, stop, times): layers start..stop-1 run times in a row
     layer_loop_refeed: bool = False          # the embedding output joins the stream again before every pass but the first
-    norm_type: str = "rms"                   # "rms" | "layer" (weight and bias)
+    norm_type: str = "rms"                   # "rms" | "layer" (weight and, with norm_bias, bias)
+    norm_bias: bool = True
     token_side_dim: int = 0                  # per-layer token input: width of a layer's slice of the table
     attention_sink: bool = False             # a learned logit per head in the softmax denominator
     # ---- options of paged grouped-query attention (models/variant_attention.py) ----
@@ -175,6 +181,8 @@ class ModelConfig:
         return self.is_hybrid and (layer_idx + 1) % self.full_attention_interval != 0
 
     def is_moe_layer(self, layer_idx: int) -> bool:
+        if self.layer_plan:
+            return self.layer_plan[layer_idx]["over"].get("num_experts", 0) > 0
         if not self.is_moe or layer_idx < self.first_k_dense_replace:
             return False
         if self.moe_layer_end_index >= 0 and layer_idx > self.moe_layer_end_index:
@@ -522,6 +530,19 @@ PRESETS: dict[str, Any] = {
                 "heads": 2, "kv_heads": 2, "dim": 16, "vdim": 40, "conv": 2, "scale": 0.25, "bias_max": 40,
                 "mask": {"size": 30}}},
         ]}, dtype="float32", name="tiny-pegopel"),
+    "tiny-dubizen": lambda: ModelConfig.from_hf_dict({
+        "architecture": "Dubizen", "vocab": 296, "width": 88, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "layers": [
+            {"type": "latent_attention", "mlp": {"kind": "dense", "ff": 120}, "mixer": {
+                "heads": 4, "dim": 24, "rot_dim": 16, "vdim": 20, "kv_rank": 48, "q_rank": 56, "scale": 0.16,
+                "rot": {"base": 10000.0, "dims": 16}}},
+            {"type": "attention", "mlp": {
+                "kind": "moe", "expert": {"ff": 40}, "shared": {"ff": 72},
+                "router": {"experts": 12, "top": 3, "scale": 1.5, "groups": {"count": 3, "keep": 2}}}, "mixer": {
+                "heads": 4, "kv_heads": 2, "dim": 32, "vdim": 24, "scale": 0.2, "bias_max": 50, "mask": {"size": 30}}},
+            {"type": "latent_attention", "mlp": None, "mixer": {
+                "heads": 2, "dim": 40, "rot_dim": 16, "vdim": 32, "kv_rank": 48, "q_rank": 32, "scale": 0.14, "kv_from": 0,
+                "rot": {"base": 10000.0, "dims": 16}}},
+        ]}, dtype="float32", name="tiny-dubizen"),
     "tiny-deepseek": lambda: _preset(
         name="tiny-deepseek", architecture="DeepseekV3ForCausalLM", vocab_size=512,
         hidden_size=128, intermediate_size=256, num_hidden_layers=3, num_attention_heads=4,

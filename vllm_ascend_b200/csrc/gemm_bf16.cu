@@ -552,12 +552,12 @@ B200_API int b200_gemm_bf16(const void* A, const void* W, void* C, const void* b
 }
 
 // out[M, I] = silu(A W_gate^T) * (A W_up^T) with W = [gate (I rows); up (I rows)] of row
-// stride ldw.  I must be a multiple of 128.
+// stride ldw.  I must be a multiple of 8 (columns of a last partial tile are not stored).
 B200_API int b200_gemm_swiglu_bf16(const void* A, const void* W, void* out, int M, int I, int K,
                                    int lda, int ldw, int ldo, int* status,
                                    cudaStream_t stream) {
   if (M <= 0 || I <= 0) return 0;
-  if ((K & 7) || (I % 128) || (lda & 7) || (ldw & 7) || (ldo & 7)) return 9100;
+  if ((K & 7) || (I & 7) || (lda & 7) || (ldw & 7) || (ldo & 7)) return 9100;
   GemmParams p;
   init_params(p);
   p.M = M; p.N = I; p.K = K; p.ldc = ldo;
@@ -657,7 +657,6 @@ B200_API int b200_grouped_gemm_bf16(const void* A, const void* W, void* C, const
   if (total_rows <= 0 || N <= 0 || num_groups <= 0) return 0;
   if ((K & 7) || (N & 7) || (lda & 7) || (ldw & 7) || (ldc & 7)) return 9100;
   if (num_groups > GEMM_MAX_GROUPS) return 9131;
-  if (swiglu && (N % 128)) return 9132;
   GemmParams p;
   init_params(p);
   p.M = (int)total_rows; p.N = N; p.K = K; p.ldc = ldc;

@@ -4,10 +4,13 @@
 //     moe_gating_top_k op, csrc/moe/moe_gating_top_k; signature torch_binding.cpp:2135-2150)
 //   * permute: histogram of tokens per local expert, exclusive offsets, and the gather of
 //     token rows into expert-major order (npu_moe_init_routing_v2 / npu_moe_token_permute)
-//   * combine: weighted sum of the k expert outputs of every token (npu_moe_token_unpermute)
+//   * combine: weighted sum of the k expert outputs of every token (npu_moe_token_unpermute), where the
+//     output of a shared expert joins, scaled by the sigmoid of a dot product with the layer's input
 // The grouped GEMMs in between are csrc/gemm_bf16.cu (GROUPED mode) and
-// csrc/gemm_fp8_block.cu.
+// csrc/gemm_fp8_block.cu; moe_linear is the same product on the CUDA cores, for fp32 and for sizes those
+// kernels do not take.
 #include "common.cuh"
+#include "dtypes.cuh"
 
 namespace b200 {
 
@@ -15,13 +18,13 @@ constexpr int GATE_MAX_PER_LANE = 16;   // experts <= 512
 
 // logits [T, E] fp32 -> weights [T, k] fp32, ids [T, k] int32
 // scoring: 0 softmax, 1 sigmoid.  Group-limited: experts are split into n_group groups, the
-// topk_group groups with the best group score stay eligible (group score = max, or the sum
-// of the top two when a correction bias is given).  Selection uses score + bias, the
+// topk_group groups with the best group score stay eligible (group score = max, or with top2 the sum
+// of the best two).  Selection uses score + bias, the
 // returned weight is the unbiased score.
 __global__ void moe_gating_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias,
                                        float* __restrict__ weights, int* __restrict__ ids, int T,
                                        int E, int k, int scoring, int renorm, int n_group,
-                                       int topk_group, float scale) {
+                                       int topk_group, int top2, float scale) {
   const int warps = blockDim.x >> 5;
   const int t = blockIdx.x * warps + (threadIdx.x >> 5);
   if (t >= T) return;
@@ -42,7 +45,7 @@ __global__ void moe_gating_topk_kernel(const float* __restrict__ logits, const f
 #pragma unroll
     for (int i = 0; i < GATE_MAX_PER_LANE; i++) {
       const int e = lane + 32 * i;
-      score[i] = (i < per && e < E) ? __expf(score[i] - mx) : 0.f;
+      score[i] = (i < per && e < E) ? expf(score[i] - mx) : 0.f;
       sum += score[i];
     }
     sum = warp_reduce_sum(sum);
@@ -53,7 +56,7 @@ __global__ void moe_gating_topk_kernel(const float* __restrict__ logits, const f
 #pragma unroll
     for (int i = 0; i < GATE_MAX_PER_LANE; i++) {
       const int e = lane + 32 * i;
-      score[i] = (i < per && e < E) ? 1.f / (1.f + __expf(-score[i])) : 0.f;
+      score[i] = (i < per && e < E) ? 1.f / (1.f + expf(-score[i])) : 0.f;
     }
   }
 #pragma unroll
@@ -85,7 +88,7 @@ __global__ void moe_gating_topk_kernel(const float* __restrict__ logits, const f
         b1 = n1;
         b2 = n2;
       }
-      const float gs = bias ? (b1 + b2) : b1;
+      const float gs = top2 && gsz > 1 ? b1 + b2 : b1;
       if (lane == g) my_gscore = gs;
     }
     // pick topk_group groups
@@ -197,40 +200,135 @@ __global__ void moe_gather_rows_kernel(const __nv_bfloat16* __restrict__ x,
   uint4* dst = reinterpret_cast<uint4*>(out + (size_t)row * H);
   for (int v = threadIdx.x; v < (H >> 3); v += blockDim.x) dst[v] = src[v];
 }
-// out[t] = sum_s w[t,s] * y[pos[t,s]]
-__global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const int* __restrict__ pos,
-                                   const float* __restrict__ w, int k, int H,
-                                   __nv_bfloat16* __restrict__ out, int accumulate) {
-  const int t = blockIdx.x;
-  for (int v = threadIdx.x; v < (H >> 3); v += blockDim.x) {
-    float acc[8] = {0, 0, 0, 0, 0, 0, 0, 0};
-    if (accumulate) {
-      const uint4 o = reinterpret_cast<const uint4*>(out + (size_t)t * H)[v];
-      const uint32_t ow[4] = {o.x, o.y, o.z, o.w};
+// out[t] = sum_s w[t,s] * y[pos[t,s]] (+ sigmoid(x[t] . gate) * shared[t])
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128) moe_combine_kernel(const T* __restrict__ y, const int* __restrict__ pos,
+                                                          const float* __restrict__ w, int k, int H, T* __restrict__ out,
+                                                          int accumulate, const T* __restrict__ shared,
+                                                          const T* __restrict__ x, const T* __restrict__ gate) {
+  const long t = blockIdx.x;
+  float g = 1.f;
+  if (gate) {
+    __shared__ float red[4];
+    float dot = 0.f;
+    for (int c = (int)threadIdx.x * VEC; c < H; c += (int)blockDim.x * VEC) {
+      float a[VEC], b[VEC];
+      load_vec<T, VEC>(x + t * H + c, a);
+      load_vec<T, VEC>(gate + c, b);
 #pragma unroll
-      for (int j = 0; j < 4; j++) {
-        const float2 f = unpack_bf16x2(ow[j]);
-        acc[2 * j] = f.x;
-        acc[2 * j + 1] = f.y;
-      }
+      for (int e = 0; e < VEC; e++) dot = fmaf(a[e], b[e], dot);
     }
+    dot = warp_reduce_sum(dot);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = dot;
+    __syncthreads();
+    g = 1.f / (1.f + expf(-(red[0] + red[1] + red[2] + red[3])));
+  }
+  for (int c = (int)threadIdx.x * VEC; c < H; c += (int)blockDim.x * VEC) {
+    float acc[VEC], v[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; e++) acc[e] = 0.f;
+    if (accumulate) load_vec<T, VEC>(out + t * H + c, acc);
     for (int s = 0; s < k; s++) {
       const int r = pos[t * k + s];
       if (r < 0) continue;
       const float ws = w[t * k + s];
-      const uint4 a = reinterpret_cast<const uint4*>(y + (size_t)r * H)[v];
-      const uint32_t aw[4] = {a.x, a.y, a.z, a.w};
+      load_vec<T, VEC>(y + (long)r * H + c, v);
 #pragma unroll
-      for (int j = 0; j < 4; j++) {
-        const float2 f = unpack_bf16x2(aw[j]);
-        acc[2 * j] += ws * f.x;
-        acc[2 * j + 1] += ws * f.y;
+      for (int e = 0; e < VEC; e++) acc[e] += ws * v[e];
+    }
+    if (shared) {
+      load_vec<T, VEC>(shared + t * H + c, v);
+#pragma unroll
+      for (int e = 0; e < VEC; e++) acc[e] = fmaf(g, v[e], acc[e]);
+    }
+    store_vec<T, VEC>(out + t * H + c, acc);
+  }
+}
+
+template <typename T>
+static int launch_combine(const void* y, const void* pos, const void* w, int tokens, int k, int H, void* out,
+                          int accumulate, const void* shared, const void* x, const void* gate, cudaStream_t stream) {
+  constexpr int V = 16 / (int)sizeof(T);
+  const bool vec = H % V == 0 && aligned16(y) && aligned16(out) && aligned16(shared) && aligned16(x) && aligned16(gate);
+  if (vec)
+    moe_combine_kernel<T, V><<<tokens, 128, 0, stream>>>((const T*)y, (const int*)pos, (const float*)w, k, H, (T*)out,
+                                                         accumulate, (const T*)shared, (const T*)x, (const T*)gate);
+  else
+    moe_combine_kernel<T, 1><<<tokens, 128, 0, stream>>>((const T*)y, (const int*)pos, (const float*)w, k, H, (T*)out,
+                                                         accumulate, (const T*)shared, (const T*)x, (const T*)gate);
+  return B200_CHECK_LAUNCH();
+}
+
+// ---------------------------------------------------------------- grouped product on the CUDA cores
+constexpr int ML_TILE = 32;
+
+// Rows [offsets[e], offsets[e + 1]) of a (row r is a[src[r]] with src) meet w[e]: [N, K], or with GLU [2N, K] =
+// gate rows | up rows and out = silu(a gate^T) * (a up^T).  A block computes 32 rows x 32 columns.
+template <typename T, bool GLU>
+__global__ void __launch_bounds__(256) moe_linear_kernel(const T* __restrict__ a, const int* __restrict__ src,
+                                                         const T* __restrict__ w, T* __restrict__ out,
+                                                         const int* __restrict__ offsets, int E, int rows, int N, int K) {
+  __shared__ float sa[ML_TILE][ML_TILE + 1], sw[GLU ? 2 : 1][ML_TILE][ML_TILE + 1];
+  const int tile = blockIdx.x;
+  int lo = 0, hi = E - 1;
+  while (lo < hi) {                                  // group e owns the tiles from offsets[e] / 32 + e on
+    const int mid = (lo + hi + 1) >> 1;
+    if (offsets[mid] / ML_TILE + mid <= tile) lo = mid; else hi = mid - 1;
+  }
+  const int r0 = offsets[lo] + (tile - offsets[lo] / ML_TILE - lo) * ML_TILE;
+  const int r1 = min(offsets[lo + 1], rows);
+  if (r0 < 0 || r0 >= r1) return;
+  const int n0 = blockIdx.y * ML_TILE;
+  const T* we = w + (long)lo * (GLU ? 2 : 1) * N * K;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[GLU ? 2 : 1][2][2] = {};
+  for (int k0 = 0; k0 < K; k0 += ML_TILE) {
+    for (int i = threadIdx.x; i < ML_TILE * ML_TILE; i += 256) {
+      const int r = i / ML_TILE, k = k0 + i % ML_TILE;
+      const int row = r0 + r;
+      sa[r][i % ML_TILE] = row < r1 && k < K ? to_f(a[(long)(src ? src[row] : row) * K + k]) : 0.f;
+#pragma unroll
+      for (int h = 0; h < (GLU ? 2 : 1); h++)
+        sw[h][r][i % ML_TILE] = n0 + r < N && k < K ? to_f(we[((long)h * N + n0 + r) * K + k]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll 8
+    for (int k = 0; k < ML_TILE; k++) {
+      const float a0 = sa[ty][k], a1 = sa[ty + 16][k];
+#pragma unroll
+      for (int h = 0; h < (GLU ? 2 : 1); h++) {
+        const float b0 = sw[h][tx][k], b1 = sw[h][tx + 16][k];
+        acc[h][0][0] = fmaf(a0, b0, acc[h][0][0]);
+        acc[h][0][1] = fmaf(a0, b1, acc[h][0][1]);
+        acc[h][1][0] = fmaf(a1, b0, acc[h][1][0]);
+        acc[h][1][1] = fmaf(a1, b1, acc[h][1][1]);
       }
     }
-    reinterpret_cast<uint4*>(out + (size_t)t * H)[v] =
-        make_uint4(pack_bf16x2(acc[0], acc[1]), pack_bf16x2(acc[2], acc[3]),
-                   pack_bf16x2(acc[4], acc[5]), pack_bf16x2(acc[6], acc[7]));
+    __syncthreads();
   }
+#pragma unroll
+  for (int i = 0; i < 2; i++)
+#pragma unroll
+    for (int j = 0; j < 2; j++) {
+      const int row = r0 + ty + 16 * i, n = n0 + tx + 16 * j;
+      if (row >= r1 || n >= N) continue;
+      float v = acc[0][i][j];
+      if constexpr (GLU) v = v / (1.f + expf(-v)) * acc[1][i][j];
+      out[(long)row * N + n] = from_f<T>(v);
+    }
+}
+
+template <typename T>
+static int launch_moe_linear(const void* a, const void* src, const void* w, void* out, const void* offsets, int E, int rows,
+                             int N, int K, int swiglu, cudaStream_t stream) {
+  const dim3 grid((unsigned)(rows / ML_TILE + E), (unsigned)((N + ML_TILE - 1) / ML_TILE));
+  if (swiglu)
+    moe_linear_kernel<T, true><<<grid, 256, 0, stream>>>((const T*)a, (const int*)src, (const T*)w, (T*)out,
+                                                         (const int*)offsets, E, rows, N, K);
+  else
+    moe_linear_kernel<T, false><<<grid, 256, 0, stream>>>((const T*)a, (const int*)src, (const T*)w, (T*)out,
+                                                          (const int*)offsets, E, rows, N, K);
+  return B200_CHECK_LAUNCH();
 }
 
 }  // namespace b200
@@ -239,14 +337,14 @@ using namespace b200;
 
 B200_API int b200_moe_gating_topk(const void* logits, const void* bias, void* weights, void* ids,
                                   int T, int E, int k, int scoring, int renorm, int n_group,
-                                  int topk_group, float scale, cudaStream_t stream) {
+                                  int topk_group, int top2, float scale, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (E > 32 * GATE_MAX_PER_LANE || k > 32 || k > E) return 9150;
   if (n_group > 1 && (n_group > 32 || E % n_group || topk_group > n_group)) return 9151;
   const int wpb = 4;
   moe_gating_topk_kernel<<<(T + wpb - 1) / wpb, wpb * 32, 0, stream>>>(
       (const float*)logits, (const float*)bias, (float*)weights, (int*)ids, T, E, k, scoring,
-      renorm, n_group, topk_group, scale);
+      renorm, n_group, topk_group, top2, scale);
   return B200_CHECK_LAUNCH();
 }
 
@@ -282,11 +380,21 @@ B200_API int b200_moe_gather_rows(const void* x, const void* src_token, const vo
   return B200_CHECK_LAUNCH();
 }
 
+// shared [T, H] or null; x [T, H] and gate [H] or null.  dtype: 0 bf16, 1 fp32
 B200_API int b200_moe_combine(const void* y, const void* pos, const void* w, int T, int k, int H,
-                              void* out, int accumulate, cudaStream_t stream) {
+                              void* out, int accumulate, const void* shared, const void* x, const void* gate, int dtype,
+                              cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (H & 7) return 9100;
-  moe_combine_kernel<<<T, 128, 0, stream>>>((const __nv_bfloat16*)y, (const int*)pos,
-                                            (const float*)w, k, H, (__nv_bfloat16*)out, accumulate);
-  return B200_CHECK_LAUNCH();
+  if (H < 1 || (gate && !x)) return 9100;
+  return dtype ? launch_combine<float>(y, pos, w, T, k, H, out, accumulate, shared, x, gate, stream)
+               : launch_combine<__nv_bfloat16>(y, pos, w, T, k, H, out, accumulate, shared, x, gate, stream);
+}
+
+// a [*, K], src [rows] or null, w [E, N (2N with swiglu), K], out [rows, N], offsets int32 [E + 1].  dtype: 0 bf16, 1 fp32
+B200_API int b200_moe_linear(const void* a, const void* src, const void* w, void* out, const void* offsets, int E, int rows,
+                             int N, int K, int swiglu, int dtype, cudaStream_t stream) {
+  if (rows <= 0 || E <= 0) return 0;
+  if (N < 1 || K < 1) return 9153;
+  return dtype ? launch_moe_linear<float>(a, src, w, out, offsets, E, rows, N, K, swiglu, stream)
+               : launch_moe_linear<__nv_bfloat16>(a, src, w, out, offsets, E, rows, N, K, swiglu, stream);
 }

@@ -2,6 +2,8 @@
 //   short causal convolution over time on every channel (optional, with a per-sequence state of the last
 //   taps - 1 inputs), RMS norm over all heads of q (and of k) at once, interleaved rotary positions on the
 //   first `rot` dimensions of a head, q to a dense buffer, keys and values to their cache slots.
+// The norm may also be head by head with one weight for all heads (qkv_head_kernel, no convolution): a group of
+// lanes owns one head of one token, so no barrier is needed.
 // The values may be the keys as they were before the norm.  Everything between the projection and the
 // stores is fp32; element type bf16 or fp32 (template), all sizes are run-time values.
 //
@@ -37,6 +39,7 @@ struct QkvPrepArgs {
   int uniform;                // every sequence has exactly one token
   int phase;                  // 0: all; 1: only the sums; 2: with the given sums
   int dtype;
+  int head_norm;              // every head by itself: q_norm, k_norm [dim]
   float eps;
 };
 
@@ -340,6 +343,100 @@ __global__ void __launch_bounds__(PREP_THREADS, KR == 0 && PER == 1 && VEC > 1 ?
   }
 }
 
+// a head [dim] (or value row [vdim]) of one token per LANES lanes
+template <typename T, int VEC, int LANES>
+__global__ void __launch_bounds__(256) qkv_head_kernel(const QkvPrepParams p) {
+  const int units = p.heads + p.kv_heads * (p.values_from_keys ? 1 : 2);
+  const long i = ((long)blockIdx.x * 256 + threadIdx.x) / LANES;
+  const bool on = i < p.tokens * units;              // lanes beyond the end only take part in the shuffles
+  const int lane = threadIdx.x & (LANES - 1);
+  const long t = on ? i / units : 0;
+  const int u = on ? (int)(i - t * units) : 0;
+  const int kind = u < p.heads ? 0 : u < p.heads + p.kv_heads ? 1 : 2;                      // q, k, v
+  const int g = kind == 0 ? u : kind == 1 ? u - p.heads : u - p.heads - p.kv_heads;
+  const int dim = kind == 2 ? p.vdim : p.dim;
+  const T* x = (const T*)p.qkv + t * p.qkv_stride;
+  x += kind == 0 ? (long)g * p.dim : kind == 1 ? (long)(p.heads + g) * p.dim : (long)(p.heads + p.kv_heads) * p.dim + (long)g * p.vdim;
+  float first[VEC], ss = 0.f;                        // the first chunk stays in registers
+#pragma unroll
+  for (int e = 0; e < VEC; e++) first[e] = 0.f;
+  for (int b = 0; b < dim; b += LANES * VEC) {
+    const int c = b + lane * VEC;
+    float v[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; e++) v[e] = 0.f;
+    if (c < dim) load_vec<T, VEC>(x + c, v);
+#pragma unroll
+    for (int e = 0; e < VEC; e++) {
+      ss = fmaf(v[e], v[e], ss);
+      if (b == 0) first[e] = v[e];
+    }
+  }
+#pragma unroll
+  for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float inv = kind == 2 ? 1.f : 1.f / sqrtf(ss / (float)dim + p.eps);
+  const T* w = (const T*)(kind == 0 ? p.q_norm : p.k_norm);
+  T *dst = nullptr, *raw = nullptr;
+  if (kind == 0) dst = (T*)p.q_out + (t * p.heads + g) * (long)p.dim;
+  else {
+    const long slot = p.slot_mapping[t];
+    if (slot >= p.cache_slots) {
+      if (lane == 0 && p.status) atomicExch(p.status, B200_BAD_INDEX);
+    } else if (slot >= 0) {
+      const unsigned blk = (unsigned)slot / (unsigned)p.block_size, off = (unsigned)slot - blk * p.block_size;
+      T* vrow = (T*)p.v_cache + blk * p.v_block + off * p.v_tok + g * p.v_head;
+      dst = kind == 1 ? (T*)p.k_cache + blk * p.k_block + off * p.k_tok + g * p.k_head : vrow;
+      if (kind == 1 && p.values_from_keys) raw = vrow;
+    }
+  }
+  const float* cs = nullptr;
+  if (p.rot > 0 && kind < 2) {
+    const long pos = p.positions[t];
+    if (pos >= 0 && pos < p.cos_rows) cs = p.cos_sin + pos * p.rot;
+    else if (lane == 0 && p.status) atomicExch(p.status, B200_BAD_INDEX);
+  }
+  const int half = p.rot >> 1;
+  for (int b = 0; b < dim; b += LANES * VEC) {       // same trip count for all lanes of a group
+    const int c = b + lane * VEC;
+    float v[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; e++) v[e] = first[e];
+    if (b > 0 && c < dim) load_vec<T, VEC>(x + c, v);
+    if (on && raw && c < dim) store_vec<T, VEC>(raw + c, v);
+    if (kind < 2 && c < dim) {
+      float wv[VEC];
+      load_vec<T, VEC>(w + c, wv);
+#pragma unroll
+      for (int e = 0; e < VEC; e++) v[e] *= inv * wv[e];
+    }
+    if constexpr (VEC == 1) {
+      if (p.rot > 0) {                               // the partner of a pair sits in the next lane
+        const float other = __shfl_xor_sync(0xffffffffu, v[0], 1);
+        if (cs && c < p.rot) {
+          const float cc = cs[c >> 1], sn = cs[half + (c >> 1)];
+          v[0] = (c & 1) ? v[0] * cc + other * sn : v[0] * cc - other * sn;
+        }
+      }
+    } else if (cs) {
+#pragma unroll
+      for (int e = 0; e < VEC; e += 2)
+        if (c + e < p.rot) {
+          const float cc = cs[(c + e) >> 1], sn = cs[half + ((c + e) >> 1)], a = v[e], bb = v[e + 1];
+          v[e] = a * cc - bb * sn;
+          v[e + 1] = bb * cc + a * sn;
+        }
+    }
+    if (on && dst && c < dim) store_vec<T, VEC>(dst + c, v);
+  }
+}
+
+template <typename T, int VEC, int LANES>
+static int launch_heads(const QkvPrepParams& p, cudaStream_t stream) {
+  const long lanes = p.tokens * (p.heads + p.kv_heads * (p.values_from_keys ? 1 : 2)) * LANES;
+  qkv_head_kernel<T, VEC, LANES><<<(unsigned)((lanes + 255) / 256), 256, 0, stream>>>(p);
+  return B200_CHECK_LAUNCH();
+}
+
 template <typename T, int VEC, int PER>
 static int launch_prep(const QkvPrepParams& p, dim3 grid, int threads, size_t smem, cudaStream_t stream) {
   if (smem > 48 * 1024) return 9820;
@@ -377,6 +474,12 @@ static int prep_t(QkvPrepParams& p, cudaStream_t stream) {
              aligned16(p.q_norm) && aligned16(p.k_norm) && aligned16(p.q_out) && aligned16(p.k_cache) &&
              aligned16(p.v_cache);
   for (long x : s) vec = vec && x % V == 0;
+  if (p.head_norm) {
+    if (!vec) return launch_heads<T, 1, 32>(p, stream);
+    const int need = (p.dim > p.vdim ? p.dim : p.vdim) / V;
+    return need <= 8 ? launch_heads<T, V, 8>(p, stream)
+                     : need <= 16 ? launch_heads<T, V, 16>(p, stream) : launch_heads<T, V, 32>(p, stream);
+  }
   // tokens of a block: enough to share the convolution's history and weights, few enough to fill the GPU
   p.tile = p.tokens >= 8192 ? 16 : p.tokens >= 2048 ? 8 : p.tokens >= 512 ? 2 : 1;
   if (p.taps > 0 && p.tile < 4) p.tile = 4;
@@ -408,6 +511,7 @@ B200_API int b200_qkv_prep(const QkvPrepArgs* a, int* status, cudaStream_t strea
   if (a->taps > 1 && (!a->state || !a->slots || !a->has_init || !a->cu)) return 9804;
   if (a->phase != 0 && !a->sums) return 9805;
   if (a->taps == 1 && !a->cu) return 9806;
+  if (a->head_norm && (a->taps || a->phase)) return 9808;
   QkvPrepParams p;
   static_cast<QkvPrepArgs&>(p) = *a;
   p.status = status;

@@ -1,7 +1,7 @@
 // Kernels around an fp32 residual stream (decoders that normalise a sub-layer's input and its output):
 //   stream_norm      one pass over a token's row between two sub-layers:
 //                      r  = scale * embed[id]                    (start of the stream), or
-//                      r += norm_post(y) (+ scale * embed[id])   (a sub-layer's output joins; a looped
+//                      r += m norm_post(y) (+ scale * embed[id]) (a sub-layer's output joins; a looped
 //                                                                 stack is fed the embedding again)
 //                      x  = norm_next(r), or r rounded to the activation type
 //   stream_mix       the same pass over S parallel streams per token (hyper-connections):
@@ -27,6 +27,7 @@ struct StreamParams {
   long y_stride;
   int post;
   const void *post_w, *post_b;
+  float post_scale;       // m
   int emb;
   const long* ids;        // [T]; null: row t of the table
   const void* table;      // [rows, W]
@@ -127,7 +128,7 @@ __global__ void stream_norm_kernel(const StreamParams p) {
       float rv[VEC];
       load_vec<float, VEC>(rrow + (long)c * VEC, rv);
 #pragma unroll
-      for (int e = 0; e < VEC; e++) v[i][e] += rv[e];
+      for (int e = 0; e < VEC; e++) v[i][e] = fmaf(v[i][e], p.post_scale, rv[e]);
     }
     if (erow) {
       float ev[VEC];
@@ -419,15 +420,15 @@ using namespace b200;
 // dtype: 0 bf16, 1 fp32 (y, x, norm weights, table).  Kinds: 0 none, 1 layer norm, 2 RMS norm, 3 plain
 // (post: add y as it is; next: round r to the activation type).  emb: 0 none, 1 set, 2 add.
 B200_API int b200_stream_norm(void* r, const void* y, long y_stride, int post, const void* post_w, const void* post_b,
-                              int emb, const void* ids, const void* table, long table_rows, float emb_scale, int next,
+                              float post_scale, int emb, const void* ids, const void* table, long table_rows, float emb_scale, int next,
                               const void* next_w, const void* next_b, void* x, long tokens, int W, float eps, int dtype,
                               int* status, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (W < 1 || (post != NORM_NONE && !y) || (next != NORM_NONE && !x) || (emb != EMB_NONE && !table)) return 9700;
   if ((post == NORM_LAYER || post == NORM_RMS) && !post_w) return 9701;
   if ((next == NORM_LAYER || next == NORM_RMS) && !next_w) return 9702;
-  StreamParams p{(float*)r, y, y_stride, post, post_w, post_b, emb, (const long*)ids, table, table_rows, emb_scale,
-                 next, next_w, next_b, x, W, eps, status};
+  StreamParams p{(float*)r, y, y_stride, post, post_w, post_b, post_scale, emb, (const long*)ids, table, table_rows,
+                 emb_scale, next, next_w, next_b, x, W, eps, status};
   return dtype ? stream_norm_t<float>(p, tokens, stream) : stream_norm_t<__nv_bfloat16>(p, tokens, stream);
 }
 

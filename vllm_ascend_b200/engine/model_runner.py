@@ -305,6 +305,8 @@ class ModelRunner:
         self.kv_arena = None
         if self.cfg.kv_transfer_config and any(self._extra_state_shapes(L.self_attn) for L in self.model.layers):
             raise NotImplementedError("KV transfer of layers that keep a state beside their pages")
+        if self.cfg.kv_transfer_config and any(getattr(L.self_attn, "kv_from", None) is not None for L in self.model.layers):
+            raise NotImplementedError("KV transfer of layers that read another layer's cache")
         if self.is_cuda and self.cfg.kv_transfer_config and not self.cfg.enable_sleep_mode:
             # one exportable allocation, so a decode engine in another process of this node
             # can map the whole cache through a single CUDA IPC handle
@@ -317,7 +319,13 @@ class ModelRunner:
                     state_bytes += KVArena.bytes_needed([cs], self.kv_dtype) + KVArena.bytes_needed([ss], torch.float32)
             self.kv_arena = KVArena(KVArena.bytes_needed([s for sh in per_layer if sh for s in sh],
                                                          self.kv_dtype) + state_bytes, self.device)
-        for layer, shapes in zip(self.model.layers, per_layer):
+        last_run: dict[int, int] = {}                    # layer index -> its latest run
+        for run, (layer, shapes) in enumerate(zip(self.model.layers, per_layer)):
+            source = getattr(layer.self_attn, "kv_from", None)
+            last_run[layer.idx] = run
+            if source is not None:                       # reads what that layer stores
+                self.kv_caches.append(self.kv_caches[last_run[source]])
+                continue
             if shapes is None:
                 # one state row per batch row, plus a scratch row for padded graph entries
                 cs, ss = layer.self_attn.state_shapes(self.max_seqs + 1)

@@ -6,7 +6,7 @@ it has, the mixer's sizes and constants, and whether a feed-forward follows.  It
 ``ModelConfig`` fields of that layer (``ModelConfig.layer_config(i)`` applies them), so that the mixers read
 a plain ``ModelConfig`` whether or not the model has a plan.
 
-This module turns the configuration formats of the Vofelix and Pegopel decoders into such plans."""
+This module turns the configuration formats of the Vofelix, Pegopel and Dubizen decoders into such plans."""
 from __future__ import annotations
 
 from typing import Any, Callable, Optional
@@ -73,7 +73,45 @@ _PEGOPEL_MIXERS: dict[str, tuple[str, Callable[[dict], dict]]] = {
     "attention": ("attention", _biased), "attention_2": ("attention", _shared_kv)}
 
 
-def _read_layers(d: dict, mixers: dict) -> list[dict]:
+def _normed(m: dict) -> dict:
+    return dict(_attention(m), qk_norm_full=False, qk_norm=True, attention_bias=True, attention_out_bias=True,
+                attn_distance_max=int(m["bias_max"]))
+
+
+def _latent_query(m: dict) -> dict:
+    return dict(_latent(m), attention_sink=False, q_lora_rank=int(m["q_rank"]), rope_half_split=True,
+                latent_kv_from=None if m.get("kv_from") is None else int(m["kv_from"]))
+
+
+_DUBIZEN_MIXERS: dict[str, tuple[str, Callable[[dict], dict]]] = {
+    "attention": ("attention", _normed), "latent_attention": ("latent", _latent_query)}
+
+
+# ---------------------------------------------------------------- feed-forwards
+def _gated_mlp(m: dict) -> dict:
+    return dict(intermediate_size=int(m["ff"]))
+
+
+def _plain_mlp(m: dict) -> dict:
+    return dict(intermediate_size=int(m["ff"]), mlp_gated=False, hidden_act="gelu", num_experts=0)
+
+
+def _experts(m: dict) -> dict:
+    router, shared = m["router"], m.get("shared")
+    groups = router.get("groups") or {"count": 1, "keep": 1}
+    experts, count, keep, top = int(router["experts"]), int(groups["count"]), int(groups["keep"]), int(router["top"])
+    if count < 1 or experts % count or not 1 <= keep <= count or not 1 <= top <= experts // count * keep:
+        raise ValueError(f"cannot choose {top} of {experts} experts from {keep} of {count} groups")
+    return dict(num_experts=experts, num_experts_per_tok=top, moe_intermediate_size=int(m["expert"]["ff"]),
+                n_group=count, topk_group=keep, moe_group_score="max", scoring_func="softmax", norm_topk_prob=True,
+                routed_scaling_factor=float(router.get("scale", 1.0)), e_score_correction_bias=True, router_fp32=True,
+                shared_expert_intermediate_size=int(shared["ff"]) if shared else 0, shared_expert_gate=bool(shared))
+
+
+_DENSE = {"dense": _gated_mlp}
+
+
+def _read_layers(d: dict, mixers: dict, mlps: dict = _DENSE) -> list[dict]:
     plan = []
     for i, layer in enumerate(d["layers"]):
         if layer["type"] not in mixers:
@@ -82,9 +120,10 @@ def _read_layers(d: dict, mixers: dict) -> list[dict]:
         over = read(layer["mixer"])
         mlp = layer.get("mlp")
         if mlp is not None:
-            if mlp.get("kind", "dense") != "dense":
-                raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
-            over["intermediate_size"] = int(mlp["ff"])
+            kind = mlp.get("kind", "dense")
+            if kind not in mlps:
+                raise ValueError(f"layer {i}: unknown feed-forward {kind!r}")
+            over.update(mlps[kind](mlp))
         plan.append({"mixer": mixer, "mlp": mlp is not None, "over": over})
     return plan
 
@@ -139,8 +178,35 @@ def pegopel_fields(d: dict) -> dict[str, Any]:
         max_position_embeddings=int(d["max_positions"]), tie_word_embeddings=True)
 
 
+def dubizen_fields(d: dict) -> dict[str, Any]:
+    """``ModelConfig`` fields of a Dubizen configuration."""
+    plan = _read_layers(d, _DUBIZEN_MIXERS, {"dense": _plain_mlp, "moe": _experts})
+    for i, p in enumerate(plan):
+        src = p["over"].get("latent_kv_from")
+        if src is None:
+            continue
+        other = plan[src]["over"] if 0 <= src < i else {}
+        same = ("kv_lora_rank", "qk_rope_head_dim", "rope_theta", "rope_scaling")
+        if other.get("latent_kv_from", -1) is not None or any(other[n] != p["over"][n] for n in same):
+            raise ValueError(f"layer {i}: layer {src} has no latents of this layer's form")
+    width = int(d["width"])
+    fields: dict[str, Any] = dict(
+        vocab_size=int(d["vocab"]), hidden_size=width, num_hidden_layers=len(plan), layer_plan=plan,
+        layer_types=["full_attention"] * len(plan), use_mla=any(p["mixer"] == "latent" for p in plan),
+        num_attention_heads=_largest(plan, "num_attention_heads", 1),
+        num_key_value_heads=_largest(plan, "num_key_value_heads", 1),
+        intermediate_size=_largest(plan, "intermediate_size", width), norm_type="layer", norm_bias=False, pre_norm=False,
+        sandwich_norm=True, residual_multiplier=float(d["residual_mult"]), rms_norm_eps=float(d["norm"]["eps"]),
+        tie_word_embeddings=True)
+    for name in ("head_dim", "v_head_dim", "kv_lora_rank", "qk_nope_head_dim", "qk_rope_head_dim", "num_experts",
+                 "num_experts_per_tok", "moe_intermediate_size"):
+        fields[name] = _largest(plan, name, 0)
+    return fields
+
+
 #: architecture name -> reader of its configuration format
-PLAN_FORMATS: dict[str, Callable[[dict], dict]] = {"Vofelix": vofelix_fields, "Pegopel": pegopel_fields}
+PLAN_FORMATS: dict[str, Callable[[dict], dict]] = {"Vofelix": vofelix_fields, "Pegopel": pegopel_fields,
+                                                   "Dubizen": dubizen_fields}
 
 
 def run_order(num_layers: int, loop: Optional[tuple]) -> tuple[list[int], set[int]]:

@@ -436,8 +436,7 @@ class PlainMLP:
     """Ungated MLP: act(x W_up) -> W_down, with ReLU^2 (Arcee), GELU, SiLU or ReLU."""
 
     _ACTS = {"relu2": lambda t: torch.relu(t).square(), "relu": torch.relu, "silu": torch.nn.functional.silu,
-             "gelu": torch.nn.functional.gelu,
-             "gelu_pytorch_tanh": lambda t: torch.nn.functional.gelu(t, approximate="tanh")}
+             "gelu": lambda t: ops.activation(t, "gelu"), "gelu_pytorch_tanh": lambda t: ops.activation(t, "gelu_tanh")}
 
     def __init__(self, pf: ParamFactory, prefix: str, hidden: int, inter: int, comm: TPComm, act: str = "relu2"):
         if act not in self._ACTS:
@@ -448,6 +447,30 @@ class PlainMLP:
 
     def __call__(self, x: torch.Tensor) -> torch.Tensor:
         return self.down_proj(self.fn(self.up_proj(x)))
+
+    def parts(self) -> list[str]:
+        return ["up", "down"]
+
+    def load_part(self, part: str, w: torch.Tensor) -> None:
+        """One un-fused tensor: up, down."""
+        comm = self.down_proj.comm
+        if part == "down":
+            return copy_exact(self.down_proj.weight, _shard(w, 1, comm), part)
+        return copy_exact(self.up_proj.weight, _shard(w, 0, comm), part)
+
+    def named_tensors(self):
+        yield from _named("up_proj", self.up_proj)
+        yield from _named("down_proj", self.down_proj)
+
+
+def _shard(w: torch.Tensor, dim: int, comm: TPComm) -> torch.Tensor:
+    n = w.shape[dim] // comm.size
+    return w.narrow(dim, comm.rank * n, n)
+
+
+def _named(attr: str, linear: Linear):
+    for n, t in linear.named_tensors():
+        yield f"{attr}.{n}", t
 
 
 class SwiGLUMLP:
@@ -473,3 +496,18 @@ class SwiGLUMLP:
         if wants_quant_act(self.down_proj):
             return self.down_proj(ops.silu_and_mul_quant_fp8(gu(x)))
         return self.down_proj(ops.silu_and_mul(gu(x)))
+
+    def parts(self) -> list[str]:
+        return ["gate", "up", "down"]
+
+    def load_part(self, part: str, w: torch.Tensor) -> None:
+        """One un-fused tensor: gate, up, down."""
+        comm = self.down_proj.comm
+        if part == "down":
+            return copy_exact(self.down_proj.weight, _shard(w, 1, comm), part)
+        rows, n = self.gate_up_proj.weight, self.gate_up_proj.weight.shape[0] // 2
+        return copy_exact(rows[:n] if part == "gate" else rows[n:], _shard(w, 0, comm), part)
+
+    def named_tensors(self):
+        yield from _named("gate_up_proj", self.gate_up_proj)
+        yield from _named("down_proj", self.down_proj)

@@ -2,14 +2,14 @@
 
 What the plan's layers have in common:
 
-* the residual stream is fp32; a norm stands in front of every sub-layer and, with ``sandwich_norm``, behind
-  it, ``r += post(f(pre(r)))``, and one kernel does the token-wise work between two sub-layers
-  (``ops.stream.stream_norm``);
+* the residual stream is fp32; a norm stands in front of every sub-layer (``pre_norm``) and, with
+  ``sandwich_norm``, behind it, ``r += m post(f(pre(r)))`` with m = ``residual_multiplier``, and one kernel does
+  the token-wise work between two sub-layers (``ops.stream.stream_norm``);
 * with ``residual_streams`` there are several parallel streams per token, mixed by learned weights at every
   sub-layer (``ops.stream.stream_mix``);
-* mixers are the framework's: latent attention (``MLAAttention`` with window and sink), the gated delta
-  rule (``GatedDeltaNet``) and paged attention with options (``VariantAttention``), each built from
-  ``ModelConfig.layer_config(i)``;
+* mixers are the framework's: latent attention (``MLAAttention`` with window and sink, or over another layer's
+  latents), the gated delta rule (``GatedDeltaNet``) and paged attention with options (``VariantAttention``); so
+  are the feed-forwards (gated, plain, mixture of experts); each is built from ``ModelConfig.layer_config(i)``;
 * optional learned positions (``learned_positions``): a vector per position added to the embeddings;
 * optional per-layer token input (``token_side_dim``): a slice of a second embedding table, gated by the
   stream, projected, RMS-normed and added after the layer's sub-layers;
@@ -30,8 +30,9 @@ from ..layer_plan import run_order
 from ..ops.stream import PLAIN, NormSpec, StreamMix, side_gate, stream_mix, stream_norm
 from ..parallel import state as pstate
 from .gdn import GatedDeltaNet
-from .layers import (Linear, ParallelLMHead, ParamFactory, SwiGLUMLP, TPComm, VocabParallelEmbedding, copy_exact)
-from .transformer import MLAAttention
+from .layers import (Linear, ParallelLMHead, ParamFactory, PlainMLP, SwiGLUMLP, TPComm, VocabParallelEmbedding,
+                     copy_exact)
+from .transformer import MLAAttention, SparseMoeBlock
 from .variant_attention import VariantAttention
 
 #: mixer kind of a plan -> constructor (param factory, layer config, layer index, comm, max positions)
@@ -48,7 +49,19 @@ _MIX_PARTS = {"in": "read", "out": "write", "mix": "mix"}
 
 def _norm(pf: ParamFactory, cfg: ModelConfig, kind: Optional[str] = None) -> NormSpec:
     kind = kind or cfg.norm_type
-    return NormSpec(kind, pf.ones((cfg.hidden_size,)), pf.zeros((cfg.hidden_size,)) if kind == "layer" else None)
+    bias = kind == "layer" and cfg.norm_bias
+    return NormSpec(kind, pf.ones((cfg.hidden_size,)), pf.zeros((cfg.hidden_size,)) if bias else None)
+
+
+def _feed_forward(pf: ParamFactory, lcfg: ModelConfig, idx: int, comm: TPComm, ep_group, moe_runtime):
+    prefix = f"model.layers.{idx}.mlp"
+    if lcfg.is_moe:
+        ranks = 1 if ep_group is not None and ep_group.world_size > 1 else comm.size
+        if lcfg.moe_intermediate_size % ranks or lcfg.shared_expert_intermediate_size % comm.size:
+            raise ValueError(f"layer {idx}: experts do not divide over {comm.size} tensor-parallel ranks")
+        return SparseMoeBlock(pf, lcfg, idx, comm, ep_group, moe_runtime)
+    kind = SwiGLUMLP if lcfg.mlp_gated else PlainMLP
+    return kind(pf, prefix, lcfg.hidden_size, lcfg.intermediate_size, comm, act=lcfg.hidden_act)
 
 
 class TokenSide:
@@ -77,29 +90,31 @@ def _stream_mix(pf: ParamFactory, prefix: str, streams: int) -> StreamMix:
 
 class PlannedLayer:
     def __init__(self, pf: ParamFactory, cfg: ModelConfig, idx: int, comm: TPComm, max_pos: int,
-                 side_table: Optional[torch.Tensor]):
+                 side_table: Optional[torch.Tensor], ep_group=None, moe_runtime=None):
         entry, lcfg = cfg.layer_plan[idx], cfg.layer_config(idx)
         heads = lcfg.linear_num_key_heads if entry["mixer"] == "delta" else lcfg.num_attention_heads
         if heads % comm.size or (entry["mixer"] == "delta" and lcfg.linear_num_value_heads % comm.size):
             raise ValueError(f"layer {idx}: heads do not divide over {comm.size} tensor-parallel ranks")
         self.idx = idx
         self.self_attn = MIXERS[entry["mixer"]](pf, lcfg, idx, comm, max_pos)
-        sandwich, streams = cfg.sandwich_norm, cfg.residual_streams
-        self.norm1, self.norm1b = _norm(pf, cfg), _norm(pf, cfg) if sandwich else PLAIN
+        streams = cfg.residual_streams
+        # in front of and behind a sub-layer
+        self.norm1, self.norm1b = (_norm(pf, cfg) if on else PLAIN for on in (cfg.pre_norm, cfg.sandwich_norm))
         self.hc1 = _stream_mix(pf, f"model.layers.{idx}.hc1", streams) if streams else None
         self.mlp = self.norm2 = self.norm2b = self.hc2 = None
         if entry["mlp"]:
-            self.norm2, self.norm2b = _norm(pf, cfg), _norm(pf, cfg) if sandwich else PLAIN
+            self.norm2, self.norm2b = (_norm(pf, cfg) if on else PLAIN for on in (cfg.pre_norm, cfg.sandwich_norm))
             self.hc2 = _stream_mix(pf, f"model.layers.{idx}.hc2", streams) if streams else None
-            self.mlp = SwiGLUMLP(pf, f"model.layers.{idx}.mlp", cfg.hidden_size, lcfg.intermediate_size, comm,
-                                 act=cfg.hidden_act)
+            self.mlp = _feed_forward(pf, lcfg, idx, comm, ep_group, moe_runtime)
         self.side = TokenSide(pf, cfg, idx, side_table) if side_table is not None else None
 
     def norms(self) -> dict[str, NormSpec]:
-        out = {"norm1": self.norm1, "norm1b": self.norm1b}
-        if self.mlp is not None:
-            out.update(norm2=self.norm2, norm2b=self.norm2b)
-        return {k: n for k, n in out.items() if n is not PLAIN}
+        """The layer's norms under their checkpoint names: a sub-layer's only norm has no suffix."""
+        out = {}
+        for k, pre, post in ((1, self.norm1, self.norm1b), (2, self.norm2, self.norm2b)):
+            here = [n for n in (pre, post) if n is not None and n is not PLAIN]
+            out.update(zip((f"norm{k}", f"norm{k}b"), here))
+        return out
 
     def mixes(self) -> dict[str, StreamMix]:
         return {k: m for k, m in (("hc1", self.hc1), ("hc2", self.hc2)) if m is not None}
@@ -140,7 +155,12 @@ class PlannedCausalLM:
         if cfg.learned_positions:
             self.pos_embed = pf.normal("model.pos_embed", (cfg.learned_positions, cfg.hidden_size))
         max_pos = max(max_model_len, 16)
-        self.unique_layers = [PlannedLayer(pf, cfg, i, self.comm, max_pos, self.side_embed)
+        if moe_runtime is not None:
+            sizes = {(c.num_experts, c.num_experts_per_tok, c.moe_intermediate_size)
+                     for c in map(cfg.layer_config, range(cfg.num_hidden_layers)) if c.is_moe}
+            if len(sizes) > 1:
+                raise NotImplementedError("expert parallelism takes layers whose experts are alike")
+        self.unique_layers = [PlannedLayer(pf, cfg, i, self.comm, max_pos, self.side_embed, ep_group, moe_runtime)
                               for i in range(cfg.num_hidden_layers)]
         order, again = run_order(cfg.num_hidden_layers, cfg.layer_loop)
         self.fed_again = again if cfg.layer_loop_refeed else set()
@@ -148,6 +168,8 @@ class PlannedCausalLM:
         self.norm = _norm(pf, cfg)
         if cfg.residual_streams and (cfg.token_side_dim or self.fed_again):
             raise NotImplementedError("parallel streams take neither a token side input nor a second embedding feed")
+        if cfg.residual_streams and cfg.residual_multiplier != 1.0:
+            raise NotImplementedError("parallel streams have write weights instead of a residual multiplier")
         if cfg.learned_positions and not cfg.residual_streams:
             raise NotImplementedError("learned positions join the embeddings of decoders with residual streams")
         self.lm_head = ParallelLMHead(self.embed_tokens if cfg.tie_word_embeddings else VocabParallelEmbedding(
@@ -169,21 +191,21 @@ class PlannedCausalLM:
             return self._forward_streams(T, emb, None if inputs_embeds is not None else self.pos_embed, meta, kv_caches)
         r = torch.empty((T, cfg.hidden_size), dtype=torch.float32, device=input_ids.device)
         x = stream_norm(r, None, None, self.layers[0].norm1, eps, dtype, embed_set=True, **emb)
-        last = len(self.layers) - 1
+        last, m = len(self.layers) - 1, cfg.residual_multiplier
         for run, (layer, cache) in enumerate(zip(self.layers, kv_caches)):
             y, post = layer.self_attn(x, meta, cache), layer.norm1b
             if layer.mlp is not None:
-                x = stream_norm(r, y, post, layer.norm2, eps, dtype)
+                x = stream_norm(r, y, post, layer.norm2, eps, dtype, post_scale=m)
                 y, post = layer.mlp(x), layer.norm2b
             if layer.side is not None:
-                x = stream_norm(r, y, post, PLAIN, eps, dtype)
+                x = stream_norm(r, y, post, PLAIN, eps, dtype, post_scale=m)
                 y, post = layer.side(x, input_ids), layer.side.norm
             nxt = self.layers[run + 1].norm1 if run < last else self.norm
             if self.layer_hook is not None:      # the hook sees the stream before the next pass is fed again
-                stream_norm(r, y, post, None, eps, dtype)
+                stream_norm(r, y, post, None, eps, dtype, post_scale=m)
                 self.layer_hook(run)
                 y = post = None
-            x = stream_norm(r, y, post, nxt, eps, dtype, **(emb if run + 1 in self.fed_again else {}))
+            x = stream_norm(r, y, post, nxt, eps, dtype, post_scale=m, **(emb if run + 1 in self.fed_again else {}))
         self.stream = r if self.layer_hook is not None else None
         return x
 
@@ -239,7 +261,9 @@ class PlannedCausalLM:
             if isinstance(a, VariantAttention):
                 for n, t in a.named_tensors():
                     yield f"{p}.self_attn.{n}", t
-            for attr in () if isinstance(a, VariantAttention) else ("in_proj_qkvz", "in_proj_ba", "out_proj", "q_proj", "kv_a_proj", "kv_b_proj", "o_proj"):
+            for attr in () if isinstance(a, VariantAttention) else (
+                    "in_proj_qkvz", "in_proj_ba", "out_proj", "q_proj", "q_a_proj", "q_b_proj", "kv_a_proj", "kv_b_proj",
+                    "o_proj"):
                 lin = getattr(a, attr, None)
                 if isinstance(lin, Linear):
                     for n, t in lin.named_tensors():
@@ -248,13 +272,14 @@ class PlannedCausalLM:
                 for n, t in a.named_tensors():
                     yield f"{p}.self_attn.{n}", t
             elif isinstance(a, MLAAttention):
-                yield f"{p}.self_attn.kv_a_norm.weight", a.kv_a_norm.weight
+                for attr in ("q_a_norm", "kv_a_norm"):
+                    if getattr(a, attr, None) is not None:
+                        yield f"{p}.self_attn.{attr}.weight", getattr(a, attr).weight
                 if a.sink is not None:
                     yield f"{p}.self_attn.sink", a.sink
             if L.mlp is not None:
-                for attr in ("gate_up_proj", "down_proj"):
-                    for n, t in getattr(L.mlp, attr).named_tensors():
-                        yield f"{p}.mlp.{attr}.{n}", t
+                for n, t in L.mlp.named_tensors():
+                    yield f"{p}.mlp.{n}", t
             if L.side is not None:
                 yield f"{p}.side.gate.weight", L.side.gate.weight
                 yield f"{p}.side.proj.weight", L.side.proj.weight
@@ -287,7 +312,7 @@ class PlannedCausalLM:
             out |= {f"{p}{name}.{part}" for name in L.mixes() for part in _MIX_PARTS}
             out |= {p + "mix." + part for part in L.self_attn.parts()}
             if L.mlp is not None:
-                out |= {p + "mlp." + part for part in ("gate", "up", "down")}
+                out |= {p + "mlp." + part for part in L.mlp.parts()}
             if L.side is not None:
                 out |= {p + "side." + part for part in ("gate", "proj", "norm")}
         return out
@@ -316,8 +341,6 @@ class PlannedCausalLM:
         return loaded
 
     def _load_one(self, name: str, w: torch.Tensor) -> None:
-        tp, r = self.comm.size, self.comm.rank
-
         def norm(n: NormSpec, which: str):
             copy_exact(n.bias if which == "b" else n.weight, w, name)
         if name in ("embed", "head"):
@@ -343,10 +366,5 @@ class PlannedCausalLM:
         if group == "side":
             return norm(L.side.norm, "") if part == "norm" else copy_exact(getattr(L.side, part).weight, w, name)
         if group == "mlp":
-            if part == "down":
-                n = w.shape[1] // tp
-                return copy_exact(L.mlp.down_proj.weight, w[:, r * n:(r + 1) * n], name)
-            n = w.shape[0] // tp
-            at = 0 if part == "gate" else n
-            return copy_exact(L.mlp.gate_up_proj.weight[at:at + n], w[r * n:(r + 1) * n], name)
+            return L.mlp.load_part(part, w)
         return norm(L.norms()[group], part)

@@ -35,7 +35,7 @@ class SparseMoeBlock:
         self.comm = comm
         prefix = f"model.layers.{layer_idx}.mlp"
         E, H, I = cfg.num_experts, cfg.hidden_size, cfg.moe_intermediate_size
-        self.gate_weight = pf.normal(f"{prefix}.gate", (E, H), dtype=torch.float32)
+        self.gate_weight = pf.normal(f"{prefix}.gate", (E, H), dtype=None if cfg.router_fp32 else torch.float32)
         self.e_bias = pf.zeros((E,), dtype=torch.float32) if cfg.e_score_correction_bias else None
         self.ep = ep_group if (ep_group is not None and ep_group.world_size > 1) else None
         self.runtime = moe_runtime
@@ -89,7 +89,9 @@ class SparseMoeBlock:
 
     def route(self, x: torch.Tensor):
         cfg = self.cfg
-        if x.is_cuda and x.dtype == torch.bfloat16 and cfg.scoring_func == "softmax" and not cfg.use_mla:
+        if cfg.router_fp32:
+            logits = ops.linear_fp32(x, self.gate_weight)
+        elif x.is_cuda and x.dtype == torch.bfloat16 and cfg.scoring_func == "softmax" and not cfg.use_mla:
             # softmax routers of bf16 checkpoints run their gate in the model dtype (as the
             # original implementation does): one tensor-core GEMM instead of an fp32 SIMT one
             if self._gate_bf16 is None:
@@ -99,7 +101,7 @@ class SparseMoeBlock:
             logits = torch.nn.functional.linear(x.float(), self.gate_weight)
         w, ids = fused_moe.gating_topk(logits, cfg.num_experts_per_tok, cfg.scoring_func,
                                        cfg.norm_topk_prob, cfg.n_group, cfg.topk_group,
-                                       self.e_bias, cfg.routed_scaling_factor)
+                                       self.e_bias, cfg.routed_scaling_factor, cfg.moe_group_score)
         if self.expert_load is not None:          # per logical expert, before any redirect
             self.expert_load.scatter_add_(0, ids.flatten().long(),
                                           torch.ones(ids.numel(), dtype=self.expert_load.dtype,
@@ -132,6 +134,11 @@ class SparseMoeBlock:
         elif moe_lora is not None and moe_lora.punica.any_active and self.quant is None:
             from ..lora.moe import fused_experts_lora
             y = fused_experts_lora(x, self.w13, self.w2, w, ids, self.expert_map, moe_lora)
+        elif x.is_cuda and self.ep is None and self.quant is None and self.shared is not None and not self.shared_replicated:
+            # the shared expert joins where the routed experts' rows are summed
+            y = fused_moe.fused_experts(x, self.w13, self.w2, w, ids, self.expert_map, shared=self.shared(x),
+                                        shared_gate=self.shared_gate_weight)
+            return self.comm.all_reduce(y) if self.comm.size > 1 else y
         else:
             y = fused_moe.fused_experts(x, self.w13, self.w2, w, ids, self.expert_map, self.quant)
         replicated = self.shared is not None and self.shared_replicated
@@ -163,6 +170,49 @@ class SparseMoeBlock:
         from ..platform_config import get_b200_config
         return get_b200_config().multistream_overlap_shared_expert
 
+    # -- un-fused tensors ----------------------------------------------------
+    def parts(self) -> list[str]:
+        out = [f"e{e}.{n}" for e in range(self.cfg.num_experts) for n in ("gate", "up", "down")] + ["router"]
+        if self.e_bias is not None:
+            out.append("correction")
+        if self.shared is not None:
+            out += [f"shared.{n}" for n in self.shared.parts()]
+        if self.shared_gate_weight is not None:
+            out.append("shared.sg")
+        return out
+
+    def load_part(self, part: str, w: torch.Tensor) -> None:
+        """One un-fused tensor: router, correction (selection bias), e<n>.gate / up / down, shared.gate / up / down,
+        shared.sg (gate of the shared expert)."""
+        owner, _, name = part.rpartition(".")
+        if part in ("router", "correction", "shared.sg"):
+            dst = {"router": self.gate_weight, "correction": self.e_bias, "shared.sg": self.shared_gate_weight}[part]
+            return copy_exact(dst, w, part)
+        if owner == "shared":
+            return self.shared.load_part(name, w)
+        e = int(owner[1:])
+        if self.ep is not None:
+            e -= self.expert_start
+            if not 0 <= e < self.E_local:        # another rank's expert
+                return None
+        else:
+            dim = 1 if name == "down" else 0
+            n = w.shape[dim] // self.comm.size
+            w = w.narrow(dim, self.comm.rank * n, n)
+        inter = self.w2.shape[2]
+        rows = {"gate": self.w13[e, :inter], "up": self.w13[e, inter:], "down": self.w2[e]}
+        return copy_exact(rows[name], w, part)
+
+    def named_tensors(self):
+        yield "gate.weight", self.gate_weight
+        for n, t in (("gate.e_score_correction_bias", self.e_bias), ("experts.w13", self.w13), ("experts.w2", self.w2),
+                     ("shared_expert_gate.weight", self.shared_gate_weight)):
+            if t is not None:
+                yield n, t
+        if self.shared is not None:
+            for n, t in self.shared.named_tensors():
+                yield f"shared_experts.{n}", t
+
 
 # ---------------------------------------------------------------- MLA attention
 _HEAD_OFFSETS: dict = {}       # (device, heads, tokens) -> int32 group offsets of the per-head grouped GEMM
@@ -177,7 +227,11 @@ class MLAAttention:
     q_nope·W_UK·latent + q_pe·k_pe; the value path is latent·W_UV — i.e. MQA over a
     576-wide key with the up-projections folded into q and the output
     (``W_UK_T`` / ``W_UV`` of mla_v1.py:907-971).  Options: a sliding window (``sliding_window``), a
-    learned sink per head (``attention_sink``), a score scale of its own (``attention_multiplier``).
+    learned sink per head (``attention_sink``), a score scale of its own (``attention_multiplier``), no latents of
+    its own (``latent_kv_from``: the layer is handed another layer's caches and reads them).
+
+    Rotary pairs are (2i, 2i + 1); checkpoints that pair i with i + dr / 2 (``rope_half_split``) have the rows of
+    the rotary parts re-ordered when they are loaded, which changes no score.
     """
 
     def __init__(self, pf: ParamFactory, cfg: ModelConfig, layer_idx: int, comm: TPComm,
@@ -198,9 +252,26 @@ class MLAAttention:
             self.q_proj = None
         else:
             self.q_proj = ColumnParallelLinear(pf, f"{p}.q_proj", hid, [qd], comm)
-        self.kv_a_proj = ColumnParallelLinear(pf, f"{p}.kv_a_proj_with_mqa", hid,
-                                              [self.dc + self.dr], rep)
-        self.kv_a_norm = RMSNorm(pf, self.dc, cfg.rms_norm_eps)
+        self.kv_from = cfg.latent_kv_from
+        self.kv_a_proj = self.kv_a_norm = None
+        if self.kv_from is None:
+            self.kv_a_proj = ColumnParallelLinear(pf, f"{p}.kv_a_proj_with_mqa", hid,
+                                                  [self.dc + self.dr], rep)
+            self.kv_a_norm = RMSNorm(pf, self.dc, cfg.rms_norm_eps)
+        # both down-projections as one matrix product
+        self.down_proj = None
+        if cfg.layer_plan and cfg.q_lora_rank:
+            lins = [self.q_a_proj] + ([self.kv_a_proj] if self.kv_a_proj is not None else [])
+            rows = sum(lin.weight.shape[0] for lin in lins)
+            whole = torch.cat([lin.weight for lin in lins] + [pf.zeros((-rows % 8, hid))])      # rows of 16 bytes
+            self.down_proj = Linear(whole, name=f"{p}.down_proj")
+            at = 0
+            for lin in lins:
+                lin.weight = whole[at:at + lin.weight.shape[0]]
+                at += lin.weight.shape[0]
+        if self.kv_from is not None and (self.down_proj is None or pstate.get_dcp_group().world_size > 1):
+            raise NotImplementedError("another layer's latents are read by plan-built layers with a query latent, "
+                                      "without decode context parallelism")
         # kv_b_proj [H*(dn+dv), dc] kept for checkpoint parity, used through the absorbed views
         self.kv_b_proj = ColumnParallelLinear(pf, f"{p}.kv_b_proj", self.dc,
                                               [cfg.num_attention_heads * (self.dn + self.dv)], comm)
@@ -250,6 +321,8 @@ class MLAAttention:
 
     def __call__(self, x: torch.Tensor, meta, kv_cache) -> torch.Tensor:
         T = x.shape[0]
+        if self.down_proj is not None:
+            return self._forward_fused_down(x, meta, kv_cache)
         if self.q_proj is None:
             qr = self.q_a_norm(self.q_a_proj(x))[0]
             q = self.q_b_proj(qr)
@@ -294,20 +367,54 @@ class MLAAttention:
         o = self._per_head_matmul(o_lat, self.W_UV, self.W_UV_nk)
         return self.o_proj(o.reshape(T, self.H * self.dv))
 
+    def _forward_fused_down(self, x: torch.Tensor, meta, kv_cache) -> torch.Tensor:
+        """One down-projection [query latent | key latent | rotary key]; one pass that norms both latents, rotates
+        the key and writes the caches; after the query's up-projection one pass that rotates its rotary part and lays
+        the rest out head by head."""
+        from ..attention import mla as mla_ops
+        T = x.shape[0]
+        lat_cache, pe_cache = kv_cache[0], kv_cache[1]
+        own = self.kv_a_norm
+        qr = ops.latent_prep(self.down_proj(x), self.q_a_norm.weight, None if own is None else own.weight,
+                             self.q_a_norm.eps, meta.positions, self.cos_sin, meta.slot_mapping, lat_cache, pe_cache)
+        q = self.q_b_proj(qr).view(T, self.H, self.dn + self.dr)
+        nope = ops.latent_query(q, meta.positions, self.cos_sin)
+        q_lat = self._per_head_matmul(nope, self.W_UK, self.W_UK_nk)
+        dcp = pstate.get_dcp_group()
+        if dcp.world_size > 1:
+            from ..attention.dcp import mla_attention_dcp
+            o_lat = mla_attention_dcp(q_lat, q[..., self.dn:], lat_cache, pe_cache, meta, self.scale, dcp,
+                                      getattr(meta, "dcp_interleave", 1))
+        else:
+            o_lat = torch.empty((self.H, T, self.dc), dtype=q_lat.dtype, device=q_lat.device).transpose(0, 1)
+            mla_ops.mla_paged_attention(q_lat, q[..., self.dn:], lat_cache, pe_cache, meta, self.scale,
+                                        window=self.window, sink=self.sink, out=o_lat)
+        o = self._per_head_matmul(o_lat, self.W_UV, self.W_UV_nk)
+        return self.o_proj(o.reshape(T, self.H * self.dv))
+
     def load_part(self, part: str, w: torch.Tensor) -> None:
-        """One un-fused tensor: q, dkv (joint down-projection), dkv.norm, uk / uv (key and value
-        up-projections, head by head), sink, o."""
+        """One un-fused tensor: q (or, through a latent, dq, dq.norm, uq), dkv (joint down-projection), dkv.norm,
+        uk / uv (key and value up-projections, head by head), sink, o."""
         tp, r = self.o_proj.comm.size, self.o_proj.comm.rank
+        if part not in self.parts():
+            raise KeyError(part)
+        if part == "dq":
+            return copy_exact(self.q_a_proj.weight, w, part)
+        if part in ("dq.norm", "dkv.norm"):
+            return copy_exact((self.q_a_norm if part == "dq.norm" else self.kv_a_norm).weight, w, part)
         if part == "dkv":
+            if self.cfg.rope_half_split:
+                w = torch.cat([w[:self.dc], self._pairs_side_by_side(w[self.dc:], part)])
             return copy_exact(self.kv_a_proj.weight, w, part)
-        if part == "dkv.norm":
-            return copy_exact(self.kv_a_norm.weight, w, part)
         if part == "o":
             n = w.shape[1] // tp
             return copy_exact(self.o_proj.weight, w[:, r * n:(r + 1) * n], part)
         rows = w[r * w.shape[0] // tp:(r + 1) * w.shape[0] // tp]
-        if part == "q":
-            return copy_exact(self.q_proj.weight, rows, part)
+        if part in ("q", "uq"):
+            if self.cfg.rope_half_split:
+                heads = rows.reshape(self.H, -1, w.shape[1])
+                rows = torch.cat([heads[:, :self.dn], self._pairs_side_by_side(heads[:, self.dn:], part)], 1).flatten(0, 1)
+            return copy_exact((self.q_proj if part == "q" else self.q_b_proj).weight, rows, part)
         if part == "sink" and self.sink is not None:
             return copy_exact(self.sink, rows, part)
         if part in ("uk", "uv"):
@@ -317,9 +424,15 @@ class MLAAttention:
             return None
         raise KeyError(part)
 
+    def _pairs_side_by_side(self, rows: torch.Tensor, part: str) -> torch.Tensor:
+        """Rotary rows [..., dr, K] whose pairs are (i, i + dr / 2), in the order (2i, 2i + 1)."""
+        if rows.shape[-2] != self.dr:
+            raise ValueError(f"tensor {part}: {rows.shape[-2]} rotary rows where {self.dr} are expected")
+        return rows.unflatten(-2, (2, self.dr // 2)).transpose(-3, -2).flatten(-3, -2)
+
     def kv_cache_heads(self) -> list[tuple[int, int]]:
-        """(heads, width) of the paged tensors: latent, rotated key part."""
-        return [(1, self.dc), (1, self.dr)]
+        """(heads, width) of the paged tensors: latent, rotated key part (none where another layer's are read)."""
+        return [(1, self.dc), (1, self.dr)] if self.kv_from is None else []
 
     def reserve_decode_scratch(self, device, batch_sizes: list, max_keys: int) -> None:
         """Split-KV scratch of decode graphs, allocated before their capture."""
@@ -327,7 +440,9 @@ class MLAAttention:
         reserve_mla_scratch(device, batch_sizes[-1], self.H, self.dc)
 
     def parts(self) -> list[str]:
-        return ["q", "dkv", "dkv.norm", "uk", "uv", "o"] + (["sink"] if self.sink is not None else [])
+        query = ["dq", "dq.norm", "uq"] if self.q_proj is None else ["q"]
+        return query + (["dkv", "dkv.norm"] if self.kv_from is None else []) + ["uk", "uv", "o"] \
+            + (["sink"] if self.sink is not None else [])
 
     def _per_head_matmul(self, x: torch.Tensor, w_kn: torch.Tensor, w_nk: torch.Tensor) -> torch.Tensor:
         """x [T, H, K] times one [K, N] matrix per head -> [T, H, N] (the two weight absorptions of MLA:
@@ -347,7 +462,7 @@ class MLAAttention:
         if off is None:
             off = torch.arange(0, H + 1, dtype=torch.int32, device=x.device) * T
             _HEAD_OFFSETS[key] = off
-        rows = x.transpose(0, 1).contiguous().view(H * T, K)             # head-major rows
+        rows = x.transpose(0, 1).contiguous().view(H * T, K)             # head-major rows (no copy where they are)
         out = moe_native.grouped_gemm(rows, w_nk, off, False)            # [H * T, N]
         return out.view(H, T, N).transpose(0, 1)
 

@@ -1,11 +1,11 @@
-"""Paged grouped-query attention layer whose options come from its layer's configuration: short convolutions
-on q, k and v, q / k norm over all heads, rotary positions on part of a head or none, values that are the keys,
-value heads of another size, sliding window with kept first tokens, capped scores, learned bias by distance,
-attention sink, output gate per head.
+"""Paged grouped-query attention layer whose options come from its layer's configuration: biases of the
+projections, short convolutions on q, k and v, q / k norm over all heads at once or head by head, rotary positions
+on part of a head or none, values that are the keys, value heads of another size, sliding window with kept first
+tokens, capped scores, learned bias by distance, attention sink, output gate per head.
 
 projection [q | k | v | gate] -> one pass of convolution, norms, rotary and cache write -> paged attention with the
 options -> output projection.  Heads are sharded over TP; key / value heads are replicated when there are fewer
-than ranks, and the norms' sums of squares travel in one all-reduce.
+than ranks, and the sums of squares of norms over all heads travel in one all-reduce.
 """
 from __future__ import annotations
 
@@ -48,9 +48,13 @@ class VariantAttention:
         parts = [self._init(pf, f"{p}.in_proj.{n}", (rows[n], hid), n) for n in rows]
         if at % 8:                           # rows of 16 bytes for the kernels
             parts.append(pf.zeros((8 - at % 8, hid)))
-        self.in_proj = Linear(torch.cat(parts), name=f"{p}.in_proj")
-        self.o_proj = RowParallelLinear(pf, f"{p}.o_proj", self.total_q * self.Dv, hid, comm)
-        self.q_norm, self.k_norm = pf.ones((self.Hq * self.D,)), pf.ones((self.Hkv * self.D,))
+        weight = torch.cat(parts)
+        self.in_proj = Linear(weight, pf.zeros((weight.shape[0],)) if cfg.attention_bias else None, name=f"{p}.in_proj")
+        self.o_proj = RowParallelLinear(pf, f"{p}.o_proj", self.total_q * self.Dv, hid, comm, bias=cfg.attention_out_bias)
+        self.head_norm = bool(cfg.qk_norm and not cfg.qk_norm_full)
+        if self.head_norm and self.taps:
+            raise NotImplementedError("short convolutions come with a q / k norm over all heads")
+        self.q_norm, self.k_norm = (pf.ones((self.D if self.head_norm else h * self.D,)) for h in (self.Hq, self.Hkv))
         self.conv_weight = None
         if self.taps:
             self.conv_weight = torch.cat([self._init(pf, f"{p}.conv.{n}", (rows[n], self.taps), n, std=0.5)
@@ -66,7 +70,7 @@ class VariantAttention:
                                     pf.device) if self.rot_dim else None
         self.prep = PrepSpec(self.Hq, self.Hkv, self.D, self.Dv, cfg.rms_norm_eps, self.q_norm, self.k_norm,
                              (self.total_q * self.D, self.total_kv * self.D), self.from_keys, self.conv_weight,
-                             self.rot_dim, cos_sin)
+                             self.rot_dim, cos_sin, self.head_norm)
         scale = self.D ** -0.5 if cfg.attention_multiplier is None else float(cfg.attention_multiplier)
         self.window = int(cfg.sliding_window or 0)
         fixed = None
@@ -112,7 +116,8 @@ class VariantAttention:
         k_cache, v_cache = kv_cache[0], kv_cache[1]
         state = kv_cache[2] if len(kv_cache) > 2 else None
         qkv = self.in_proj(x)
-        q = qkv_prep(self.prep, qkv, meta, k_cache, v_cache, state, self._reduce_sums if self.comm.size > 1 else None)
+        q = qkv_prep(self.prep, qkv, meta, k_cache, v_cache, state,
+                     self._reduce_sums if self.comm.size > 1 and not self.head_norm else None)
         gate = None
         if "g" in self._at:
             at, n = self._at["g"]
@@ -132,17 +137,23 @@ class VariantAttention:
             out.append("v")
         if self.taps:
             out += ["q.conv", "k.conv"] + ([] if self.from_keys else ["v.conv"])
+        if self.in_proj.bias is not None:
+            out += [f"{n}.b" for n in self._at if n != "g"]
+        if self.o_proj.bias is not None:
+            out.append("o.b")
         return out + [n for n, on in (("g", "g" in self._at), ("rel", self.rel is not None),
                                       ("sink", self.sink is not None)) if on]
 
     def load_part(self, part: str, w: torch.Tensor) -> None:
-        """One un-fused tensor: projections q, k, v, g (output gate), o; q.norm, k.norm; convolutions q.conv,
-        k.conv, v.conv; rel (bias by distance bucket, [buckets, heads]); sink."""
+        """One un-fused tensor: projections q, k, v, g (output gate), o and their biases q.b, ...; q.norm, k.norm;
+        convolutions q.conv, k.conv, v.conv; rel (bias by distance bucket, [buckets, heads]); sink."""
         tp, r = self.comm.size, self.comm.rank
         name, _, kind = part.partition(".")
         if part == "o":
             n = w.shape[1] // tp
             return copy_exact(self.o_proj.weight, w[:, r * n:(r + 1) * n], part)
+        if part == "o.b":
+            return copy_exact(self.o_proj.bias, w, part)
         if part == "rel":
             if w.dim() != 2 or w.shape[1] != self.total_q or w.shape[0] < 2:
                 raise ValueError(f"tensor rel: unexpected shape {tuple(w.shape)}")
@@ -151,11 +162,12 @@ class VariantAttention:
         if part == "sink":
             return copy_exact(self.sink, self._rows("g", w), part)
         if kind == "norm":
-            return copy_exact(self.q_norm if name == "q" else self.k_norm, self._rows(name, w), part)
+            return copy_exact(self.q_norm if name == "q" else self.k_norm, w if self.head_norm else self._rows(name, w), part)
         if part not in self.parts():
             raise KeyError(part)
         at, n = self._at[name]
-        return copy_exact((self.conv_weight if kind == "conv" else self.in_proj.weight)[at:at + n], self._rows(name, w), part)
+        whole = {"conv": self.conv_weight, "b": self.in_proj.bias, "": self.in_proj.weight}[kind]
+        return copy_exact(whole[at:at + n], self._rows(name, w), part)
 
     def named_tensors(self):
         for attr in ("in_proj", "o_proj"):

@@ -208,6 +208,13 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] =
     return out.view(*x.shape[:-1], N)
 
 
+def linear_fp32(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """x @ weight.T summed and returned in fp32, whatever the operands' type (router logits)."""
+    if x.is_cuda and x.dtype == weight.dtype == _BF16:
+        return torch.mm(x, weight.t(), out_dtype=torch.float32)
+    return torch.nn.functional.linear(x.float(), weight.float())
+
+
 def alloc_row_stats(rows: int, max_out_features: int, device) -> torch.Tensor:
     """Row-statistics buffer of the folded-norm GEMMs: fp32 [parts][rows] partial sums of squares
     (one part per 128 output columns at most) followed by the int32 part count."""
@@ -262,7 +269,7 @@ def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Ten
     (the reference fuses the same pair in its grouped-matmul+swiglu op, csrc/gmm)."""
     I = weight.shape[0] // 2
     K = x.shape[-1]
-    if not (_use_native(x) and weight.dtype == _BF16 and I % 128 == 0 and K % 8 == 0
+    if not (_use_native(x) and weight.dtype == _BF16 and I % 8 == 0 and K % 8 == 0
             and envs.VLLM_B200_GEMM != "cublas"):
         return silu_and_mul(linear(x, weight))
     x2 = x.reshape(-1, K)
@@ -272,7 +279,7 @@ def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Ten
     if out is None:
         out = torch.empty((M, I), dtype=x.dtype, device=x.device)
     min2 = envs.VLLM_B200_GEMM_2CTA_MIN_M
-    if M > 0 and (two_cta or (min2 > 0 and M >= min2)):
+    if M > 0 and I % 128 == 0 and (two_cta or (min2 > 0 and M >= min2)):
         rc = _native.lib().b200_gemm_bf16_2cta(
             x2.data_ptr(), weight.data_ptr(), out.data_ptr(), None, None, M, I, K, x2.stride(0),
             weight.stride(0), out.stride(0), 1, _native.status_word(x.device).data_ptr(),
@@ -558,6 +565,60 @@ def mla_preprocess(q: torch.Tensor, kv: torch.Tensor, norm_w: torch.Tensor, eps:
     _native.check(rc, "mla_preprocess")
     launch_counter[0] += 1
     return (latent, k_pe) if want_outputs else None
+
+
+def latent_prep(down: torch.Tensor, q_norm: torch.Tensor, kv_norm: Optional[torch.Tensor], eps: float,
+                positions: torch.Tensor, cos_sin: torch.Tensor, slot_mapping: Optional[torch.Tensor],
+                lat_cache: torch.Tensor, pe_cache: torch.Tensor) -> torch.Tensor:
+    """A joint down-projection's rows [query latent | key latent | rotary key (| padding)]: RMSNorm of the query
+    latent (returned, dense), RMSNorm of the key latent and interleaved RoPE of the rotary key to their cache slots
+    (slot < 0: not stored).  ``kv_norm`` None: the rows hold a query latent only."""
+    T, rq = down.shape[0], q_norm.shape[0]
+    dc, dr = (0, 0) if kv_norm is None else (kv_norm.shape[0], cos_sin.shape[1])
+    if down.shape[1] < rq + dc + dr or down.stride(1) != 1:
+        raise ValueError("latent_prep: the projection's rows are too short or not dense")
+    if not down.is_cuda:
+        if kv_norm is not None:
+            lat = ref.rms_norm(down[:, rq:rq + dc], kv_norm, eps)[0]
+            pe = ref.apply_rope_interleaved(down[:, rq + dc:rq + dc + dr].reshape(T, 1, dr), positions, cos_sin, dr)
+            from ..attention.mla import write_latent_cache
+            write_latent_cache(lat, pe.view(T, dr), lat_cache, pe_cache, slot_mapping)
+        return ref.rms_norm(down[:, :rq], q_norm, eps)[0]
+    same = [q_norm] + ([kv_norm, lat_cache, pe_cache] if kv_norm is not None else [])
+    if down.dtype not in (_BF16, torch.float32) or any(t.dtype != down.dtype or not t.is_contiguous() for t in same):
+        raise TypeError("latent_prep takes bf16 or fp32 rows with dense weights and caches of the same type")
+    out = torch.empty((T, rq), dtype=down.dtype, device=down.device)
+    if T == 0:
+        return out
+    rc = _native.lib().b200_latent_prep(
+        down.data_ptr(), down.stride(0), T, rq, q_norm.data_ptr(), out.data_ptr(), dc, dr, _native.ptr(kv_norm), float(eps),
+        positions.data_ptr(), cos_sin.data_ptr(), cos_sin.shape[0], _native.ptr(slot_mapping), _native.ptr(lat_cache),
+        _native.ptr(pe_cache), lat_cache.numel() // dc if dc else 0, int(down.dtype == torch.float32),
+        _native.status_word(down.device).data_ptr(), _native.stream_ptr())
+    _native.check(rc, "latent_prep")
+    launch_counter[0] += 1
+    return out
+
+
+def latent_query(q: torch.Tensor, positions: torch.Tensor, cos_sin: torch.Tensor) -> torch.Tensor:
+    """Interleaved RoPE of the last columns of every head of ``q`` [T, H, dn + dr] in place; returns the columns in
+    front of them as [T, H, dn], laid out head by head (rows of the per-head matrix products)."""
+    T, H, D = q.shape
+    dr = cos_sin.shape[1]
+    dn = D - dr
+    if not q.is_cuda:
+        q[..., dn:] = ref.apply_rope_interleaved(q[..., dn:], positions, cos_sin, dr)
+        return q[..., :dn]
+    if q.dtype not in (_BF16, torch.float32) or not q.is_contiguous():
+        raise TypeError("latent_query takes dense bf16 or fp32 queries")
+    nope = torch.empty((H, T, dn), dtype=q.dtype, device=q.device)
+    if T:
+        rc = _native.lib().b200_latent_query(
+            q.data_ptr(), T, H, dn, dr, positions.data_ptr(), cos_sin.data_ptr(), cos_sin.shape[0], nope.data_ptr(),
+            int(q.dtype == torch.float32), _native.status_word(q.device).data_ptr(), _native.stream_ptr())
+        _native.check(rc, "latent_query")
+        launch_counter[0] += 1
+    return nope.transpose(0, 1)
 
 
 # ---------------------------------------------------------------- sampling

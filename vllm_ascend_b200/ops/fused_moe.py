@@ -20,14 +20,16 @@ from . import reference as ref
 
 def gating_topk_ref(logits: torch.Tensor, k: int, scoring: str = "softmax", renorm: bool = True,
                     n_group: int = 1, topk_group: int = 1,
-                    bias: Optional[torch.Tensor] = None, scale: float = 1.0):
+                    bias: Optional[torch.Tensor] = None, scale: float = 1.0, group_score: Optional[str] = None):
+    """``group_score``: a group counts by its best expert ("max") or by the sum of its best two ("top2"); by
+    default "top2" where a bias is given."""
     x = logits.float()
     scores = torch.softmax(x, dim=-1) if scoring == "softmax" else torch.sigmoid(x)
     choice = scores + bias.float() if bias is not None else scores
     T, E = scores.shape
     if n_group > 1:
         g = choice.view(T, n_group, E // n_group)
-        if bias is not None:
+        if _top2(group_score, bias) and g.shape[-1] > 1:
             gscore = g.topk(2, dim=-1).values.sum(-1)       # noaux_tc: sum of the top-2 per group
         else:
             gscore = g.max(dim=-1).values
@@ -43,14 +45,20 @@ def gating_topk_ref(logits: torch.Tensor, k: int, scoring: str = "softmax", reno
     return (w * scale).float(), ids.to(torch.int32)
 
 
+def _top2(group_score: Optional[str], bias: Optional[torch.Tensor]) -> bool:
+    if group_score not in (None, "max", "top2"):
+        raise ValueError(f"unknown group score {group_score!r}")
+    return bias is not None if group_score is None else group_score == "top2"
+
+
 def gating_topk(logits: torch.Tensor, k: int, scoring: str = "softmax", renorm: bool = True,
                 n_group: int = 1, topk_group: int = 1, bias: Optional[torch.Tensor] = None,
-                scale: float = 1.0):
+                scale: float = 1.0, group_score: Optional[str] = None):
     if logits.is_cuda and _native.available() and hasattr(_native.lib(), "b200_moe_gating_topk") \
-            and logits.shape[1] <= 512 and k <= 16:
+            and logits.shape[1] <= 512 and k <= 32 and n_group <= 32:
         from . import moe_native
-        return moe_native.gating_topk(logits, k, scoring, renorm, n_group, topk_group, bias, scale)
-    return gating_topk_ref(logits, k, scoring, renorm, n_group, topk_group, bias, scale)
+        return moe_native.gating_topk(logits, k, scoring, renorm, n_group, topk_group, bias, scale, group_score)
+    return gating_topk_ref(logits, k, scoring, renorm, n_group, topk_group, bias, scale, group_score)
 
 
 def fused_experts_ref(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor,
@@ -75,14 +83,21 @@ def fused_experts_ref(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor,
     return out.to(x.dtype)
 
 
-def fused_experts(x, w13, w2, topk_w, topk_ids, expert_map=None, quant=None):
-    if x.is_cuda and x.dtype == torch.bfloat16 and _native.available() \
-            and hasattr(_native.lib(), "b200_grouped_gemm_bf16") and quant is None:
+def fused_experts(x, w13, w2, topk_w, topk_ids, expert_map=None, quant=None, shared=None, shared_gate=None):
+    """Weighted sum of the chosen experts' outputs; ``shared`` [T, H] (a shared expert's output) is added, scaled
+    by sigmoid(x . shared_gate) where that vector is given."""
+    if x.is_cuda and x.dtype in (torch.bfloat16, torch.float32) and w13.dtype == x.dtype and _native.available() \
+            and hasattr(_native.lib(), "b200_moe_permute") and quant is None:
         from . import moe_native
-        return moe_native.fused_experts(x, w13, w2, topk_w, topk_ids, expert_map)
+        return moe_native.fused_experts(x, w13, w2, topk_w, topk_ids, expert_map, shared, shared_gate)
     if quant is not None:
-        return quant.apply_experts(x, w13, w2, topk_w, topk_ids, expert_map)
-    return fused_experts_ref(x, w13, w2, topk_w, topk_ids, expert_map)
+        y = quant.apply_experts(x, w13, w2, topk_w, topk_ids, expert_map)
+    else:
+        y = fused_experts_ref(x, w13, w2, topk_w, topk_ids, expert_map)
+    if shared is None:
+        return y
+    g = 1.0 if shared_gate is None else torch.sigmoid(x.float() @ shared_gate.float().view(-1, 1))
+    return (y.float() + g * shared.float()).to(y.dtype)
 
 
 def hash_topk(token_ids: torch.Tensor, table: torch.Tensor):

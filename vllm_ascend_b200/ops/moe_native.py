@@ -16,10 +16,11 @@ from .. import _native
 from . import launch_counter, quant_fp8_group128, silu_and_mul
 
 P, I, L, F = c_void_p, c_int, c_long, c_float
-_native.register_signature("b200_moe_gating_topk", [P, P, P, P, I, I, I, I, I, I, I, F, P])
+_native.register_signature("b200_moe_gating_topk", [P, P, P, P, I, I, I, I, I, I, I, I, F, P])
 _native.register_signature("b200_moe_permute", [P, I, I, I, P, P, P, P, P, P])
 _native.register_signature("b200_moe_gather_rows", [P, P, P, I, I, I, P, P])
-_native.register_signature("b200_moe_combine", [P, P, P, I, I, I, P, I, P])
+_native.register_signature("b200_moe_combine", [P, P, P, I, I, I, P, I, P, P, P, I, P])
+_native.register_signature("b200_moe_linear", [P, P, P, P, P, I, I, I, I, I, I, P])
 _native.register_signature("b200_grouped_gemm_fp8_block",
                            [P, P, P, P, P, P, I, L, I, I, I, I, I, P, P])
 
@@ -29,14 +30,15 @@ def available() -> bool:
 
 
 def gating_topk(logits: torch.Tensor, k: int, scoring: str, renorm: bool, n_group: int,
-                topk_group: int, bias: Optional[torch.Tensor], scale: float):
+                topk_group: int, bias: Optional[torch.Tensor], scale: float, group_score: Optional[str] = None):
+    from .fused_moe import _top2
     T, E = logits.shape
     logits = logits.float().contiguous()
     w = torch.empty((T, k), dtype=torch.float32, device=logits.device)
     ids = torch.empty((T, k), dtype=torch.int32, device=logits.device)
     rc = _native.lib().b200_moe_gating_topk(
         logits.data_ptr(), _native.ptr(bias), w.data_ptr(), ids.data_ptr(), T, E, k,
-        0 if scoring == "softmax" else 1, int(renorm), n_group, topk_group, scale,
+        0 if scoring == "softmax" else 1, int(renorm), n_group, topk_group, int(_top2(group_score, bias)), scale,
         _native.stream_ptr())
     _native.check(rc, "moe_gating_topk")
     launch_counter[0] += 1
@@ -78,13 +80,23 @@ class Permutation:
         return out
 
     def combine(self, y: torch.Tensor, topk_w: torch.Tensor, out: Optional[torch.Tensor] = None,
-                accumulate: bool = False) -> torch.Tensor:
+                accumulate: bool = False, shared: Optional[torch.Tensor] = None, x: Optional[torch.Tensor] = None,
+                shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Weighted sum of every token's rows of ``y``, plus ``shared`` [T, H] times sigmoid(x . shared_gate)
+        (times one without a gate)."""
         H = y.shape[1]
+        for t in (shared, x if shared_gate is not None else None):
+            if t is not None and (tuple(t.shape) != (self.T, H) or t.dtype != y.dtype or not t.is_contiguous()):
+                raise TypeError("shared expert rows and layer inputs are dense [T, H] of the experts' type")
+        if shared_gate is not None and (shared_gate.numel() != H or shared_gate.dtype != y.dtype):
+            raise TypeError("the shared expert's gate is a vector of the layer's width and type")
         if out is None:
             out = torch.empty((self.T, H), dtype=y.dtype, device=y.device)
         w = topk_w.float().contiguous()
         rc = _native.lib().b200_moe_combine(y.data_ptr(), self.pos.data_ptr(), w.data_ptr(), self.T,
-                                            self.k, H, out.data_ptr(), int(accumulate),
+                                            self.k, H, out.data_ptr(), int(accumulate), _native.ptr(shared),
+                                            _native.ptr(x) if shared_gate is not None else None,
+                                            _native.ptr(shared_gate), int(y.dtype == torch.float32),
                                             _native.stream_ptr())
         _native.check(rc, "moe_combine")
         launch_counter[0] += 1
@@ -119,20 +131,39 @@ def grouped_gemm_fp8(a8, a_scale, w8, w_scale, offsets) -> torch.Tensor:
     return out
 
 
-def fused_experts(x, w13, w2, topk_w, topk_ids, expert_map=None) -> torch.Tensor:
-    """bf16 experts: permute -> grouped GEMM1 with SwiGLU epilogue -> grouped GEMM2 -> combine."""
+def grouped_linear_simple(a: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, swiglu: bool, rows: int,
+                          src: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``grouped_gemm`` on the CUDA cores for fp32 and for sizes that are no multiples of 8.  ``src``: row r of the
+    product reads row src[r] of ``a``."""
+    E, K = w.shape[0], a.shape[1]
+    N = w.shape[1] // 2 if swiglu else w.shape[1]
+    if a.dtype != w.dtype or a.dtype not in (torch.bfloat16, torch.float32) or not (a.is_contiguous() and w.is_contiguous()):
+        raise TypeError("grouped_linear_simple takes dense rows and weights, both bf16 or both fp32")
+    out = torch.empty((max(rows, 1), N), dtype=a.dtype, device=a.device)
+    rc = _native.lib().b200_moe_linear(a.data_ptr(), _native.ptr(src), w.data_ptr(), out.data_ptr(), offsets.data_ptr(), E,
+                                       rows, N, K, int(swiglu), int(a.dtype == torch.float32), _native.stream_ptr())
+    _native.check(rc, "moe_linear")
+    launch_counter[0] += 1
+    return out
+
+
+def fused_experts(x, w13, w2, topk_w, topk_ids, expert_map=None, shared=None, shared_gate=None) -> torch.Tensor:
+    """bf16 experts: permute -> grouped GEMM1 with SwiGLU epilogue -> grouped GEMM2 -> combine (where a shared
+    expert's output joins).  fp32 and odd sizes take the same steps on the CUDA cores."""
     E, two_i, H = w13.shape
     I_ = two_i // 2
     if x.shape[0] == 0:
         return x.clone()
-    if I_ % 128 or H % 8 or E > 512:
-        from .fused_moe import fused_experts_ref
-        return fused_experts_ref(x, w13, w2, topk_w, topk_ids, expert_map)
+    x = x if x.is_contiguous() else x.contiguous()
     perm = Permutation(topk_ids, expert_map, E)
-    xs = perm.gather(x)
-    h = grouped_gemm(xs, w13, perm.offsets, swiglu=True)          # [rows, I]
-    y = grouped_gemm(h, w2, perm.offsets, swiglu=False)           # [rows, H]
-    return perm.combine(y, topk_w)
+    if x.dtype != torch.bfloat16 or I_ % 8 or H % 8 or E > 512:
+        h = grouped_linear_simple(x, w13, perm.offsets, True, perm.max_rows, perm.src_token)
+        y = grouped_linear_simple(h, w2, perm.offsets, False, perm.max_rows)
+    else:
+        xs = perm.gather(x)
+        h = grouped_gemm(xs, w13, perm.offsets, swiglu=True)          # [rows, I]
+        y = grouped_gemm(h, w2, perm.offsets, swiglu=False)           # [rows, H]
+    return perm.combine(y, topk_w, shared=shared, x=x, shared_gate=shared_gate)
 
 
 def fused_experts_fp8(x, w13, w13_scale, w2, w2_scale, topk_w, topk_ids, expert_map=None):

@@ -12,7 +12,7 @@ import torch.nn.functional as F
 from .. import _native
 
 P, I, L, Fl = c_void_p, c_int, c_long, c_float
-_native.register_signature("b200_stream_norm", [P, P, L, I, P, P, I, P, P, L, Fl, I, P, P, P, L, I, Fl, I, P, P])
+_native.register_signature("b200_stream_norm", [P, P, L, I, P, P, Fl, I, P, P, L, Fl, I, P, P, P, L, I, Fl, I, P, P])
 _native.register_signature("b200_stream_mix", [P, P, L, I, P, P, P, P, I, P, P, L, Fl, P, P, L, P, I, P, P, P, L, I, I, I,
                                                Fl, I, P, P])
 _native.register_signature("b200_side_gate", [P, L, P, P, L, L, L, P, L, I, I, P, P])
@@ -55,10 +55,10 @@ def _norm_ref(v: torch.Tensor, n: NormSpec, eps: float) -> torch.Tensor:
 
 def stream_norm(r: torch.Tensor, y: Optional[torch.Tensor], post: Optional[NormSpec], nxt: Optional[NormSpec], eps: float,
                 dtype: torch.dtype, embed: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None,
-                embed_scale: float = 1.0, embed_set: bool = False) -> Optional[torch.Tensor]:
+                embed_scale: float = 1.0, embed_set: bool = False, post_scale: float = 1.0) -> Optional[torch.Tensor]:
     """One token-wise pass over the residual stream ``r`` (fp32 [T, W], updated in place):
 
-        r += post(y)                       when a sub-layer output ``y`` [T, W] is given
+        r += post_scale * post(y)          when a sub-layer output ``y`` [T, W] is given
         r += embed_scale * embed[ids]      when ``embed`` is given (``embed_set``: r is set to it instead)
         return nxt(r) as ``dtype``         (None: nothing is returned)
 
@@ -69,7 +69,7 @@ def stream_norm(r: torch.Tensor, y: Optional[torch.Tensor], post: Optional[NormS
     if not r.is_cuda:
         v = None
         if y is not None:
-            v = _norm_ref(y.float(), post, eps)
+            v = _norm_ref(y.float(), post, eps) * post_scale
         if embed is not None:
             e = (embed if ids is None else embed[ids]).float() * embed_scale
             v = e if v is None else v + e
@@ -88,9 +88,9 @@ def stream_norm(r: torch.Tensor, y: Optional[torch.Tensor], post: Optional[NormS
     emb = 0 if embed is None else (1 if embed_set else 2)
     rc = _native.lib().b200_stream_norm(
         r.data_ptr(), _native.ptr(y), 0 if y is None else y.stride(0), _KIND[post.kind] if y is not None else 0,
-        _native.ptr(post.weight if y is not None else None), _native.ptr(post.bias if y is not None else None), emb,
-        _native.ptr(ids), _native.ptr(embed), 0 if embed is None else embed.shape[0], float(embed_scale),
-        0 if nxt is None else _KIND[nxt.kind], _native.ptr(nxt.weight if nxt else None),
+        _native.ptr(post.weight if y is not None else None), _native.ptr(post.bias if y is not None else None),
+        float(post_scale), emb, _native.ptr(ids), _native.ptr(embed), 0 if embed is None else embed.shape[0],
+        float(embed_scale), 0 if nxt is None else _KIND[nxt.kind], _native.ptr(nxt.weight if nxt else None),
         _native.ptr(nxt.bias if nxt else None), _native.ptr(x), T, W, float(eps), code,
         _native.status_word(r.device).data_ptr(), _native.stream_ptr())
     _native.check(rc, "stream_norm")
