@@ -192,6 +192,7 @@ class PlannedCausalLM:
         r = torch.empty((T, cfg.hidden_size), dtype=torch.float32, device=input_ids.device)
         x = stream_norm(r, None, None, self.layers[0].norm1, eps, dtype, embed_set=True, **emb)
         last, m = len(self.layers) - 1, cfg.residual_multiplier
+        self.stream = r if self.layer_hook is not None else None
         for run, (layer, cache) in enumerate(zip(self.layers, kv_caches)):
             y, post = layer.self_attn(x, meta, cache), layer.norm1b
             if layer.mlp is not None:
@@ -206,7 +207,6 @@ class PlannedCausalLM:
                 self.layer_hook(run)
                 y = post = None
             x = stream_norm(r, y, post, nxt, eps, dtype, post_scale=m, **(emb if run + 1 in self.fed_again else {}))
-        self.stream = r if self.layer_hook is not None else None
         return x
 
     def _forward_streams(self, T: int, emb: dict, pos_table: Optional[torch.Tensor], meta, kv_caches: list):
