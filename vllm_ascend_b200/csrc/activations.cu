@@ -1,6 +1,6 @@
 // Activation family beside SiLU-mul, and the gated RMSNorm:
-//   act_and_mul : out = act(gate) * up for act in {gelu (erf), gelu (tanh), swiglu-oai}
-//   act         : out = act(x) for act in {quick_gelu, gelu, gelu_tanh}
+//   act_and_mul : out = act(gate) * up for act in {gelu (erf), gelu (tanh), swiglu-oai, silu}
+//   act         : out = act(x) for act in {quick_gelu, gelu, gelu_tanh, silu}
 //   rms_norm_gated : out = rmsnorm(x) * w * silu(z)         (gate after the norm)
 // The reference routes these through vendor ops and small Triton kernels
 // (vllm_ascend/ops/activation.py:35-86, ops/layernorm.py:110-197).
@@ -9,7 +9,7 @@
 
 namespace b200 {
 
-enum : int { ACT_GELU = 1, ACT_GELU_TANH = 2, ACT_QUICK_GELU = 3, ACT_SWIGLU_OAI = 4 };
+enum : int { ACT_GELU = 1, ACT_GELU_TANH = 2, ACT_QUICK_GELU = 3, ACT_SWIGLU_OAI = 4, ACT_SILU = 5 };
 
 __device__ __forceinline__ float act_fn(float x, int kind) {
   switch (kind) {
@@ -80,6 +80,8 @@ __global__ void act_scalar_kernel(const T* __restrict__ x, T* __restrict__ out, 
       r = g / (1.f + expf(-alpha * g)) * (u + 1.f);
     } else if (kind == ACT_QUICK_GELU) {
       r = g / (1.f + expf(-1.702f * g)) * u;
+    } else if (kind == ACT_SILU) {
+      r = silu_f<T>(g) * u;
     } else {
       r = act_fn(g, kind) * u;
     }
@@ -128,7 +130,7 @@ using namespace b200;
 B200_API int b200_activation(const void* x, void* out, long T, int I, int kind, int gated, float alpha,
                              float limit, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (kind < ACT_GELU || kind > ACT_SWIGLU_OAI || (kind == ACT_SWIGLU_OAI && !gated)) return 9600;
+  if (kind < ACT_GELU || kind > ACT_SILU || (kind == ACT_SWIGLU_OAI && !gated)) return 9600;
   const bool scalar = dtype != 0 || (I & 7);
   const long total = T * (scalar ? I : I >> 3);
   long blocks = (total + 255) / 256;

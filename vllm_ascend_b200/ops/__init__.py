@@ -92,9 +92,11 @@ def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tenso
 
 def silu_and_mul(x: torch.Tensor, limit: float = 0.0,
                  out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    I = x.shape[-1] // 2
+    if x.is_cuda and (I % 8 or x.dtype == torch.float32) and not limit and out is None:
+        return activation(x.contiguous(), "silu", gated=True)
     if not _use_native(x):
         return ref.silu_and_mul(x, limit)
-    I = x.shape[-1] // 2
     x2 = x.view(-1, 2 * I)
     T = x2.shape[0]
     if out is None:
@@ -758,11 +760,11 @@ def silu_and_mul_quant_fp8(x: torch.Tensor, limit: float = 0.0) -> QuantAct:
     return QuantAct(q, s, x.dtype)
 
 
-_ACT_KINDS = {"gelu": 1, "gelu_tanh": 2, "quick_gelu": 3, "swiglu_oai": 4}
+_ACT_KINDS = {"gelu": 1, "gelu_tanh": 2, "quick_gelu": 3, "swiglu_oai": 4, "silu": 5}
 
 
 def activation(x: torch.Tensor, kind: str, gated: bool = False, alpha: float = 1.702, limit: float = 7.0):
-    """GELU (erf / tanh), QuickGELU, and the clamped "swiglu-oai" gate; ``gated`` inputs are [gate | up]."""
+    """GELU (erf / tanh), QuickGELU, SiLU, and the clamped "swiglu-oai" gate; ``gated`` inputs are [gate | up]."""
     I = x.shape[-1] // 2 if gated else x.shape[-1]
     if not x.is_cuda or x.dtype not in (_BF16, torch.float32) or not x.is_contiguous():
         return ref.activation(x, kind, gated, alpha, limit)

@@ -380,7 +380,7 @@ def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias, eps: float) -> torch
 
 
 def activation(x: torch.Tensor, kind: str, gated: bool = False, alpha: float = 1.702, limit: float = 7.0):
-    """kind: gelu | gelu_tanh | quick_gelu | swiglu_oai.  gated: x = [gate | up]."""
+    """kind: gelu | gelu_tanh | quick_gelu | silu | swiglu_oai.  gated: x = [gate | up]."""
     if gated:
         d = x.shape[-1] // 2
         g, u = x[..., :d].float(), x[..., d:].float()
@@ -396,6 +396,8 @@ def activation(x: torch.Tensor, kind: str, gated: bool = False, alpha: float = 1
         y = F.gelu(g, approximate="tanh")
     elif kind == "quick_gelu":
         y = g * torch.sigmoid(1.702 * g)
+    elif kind == "silu":
+        y = F.silu(g)
     else:
         raise ValueError(f"unknown activation {kind!r}")
     return (y * u if u is not None else y).to(x.dtype)
