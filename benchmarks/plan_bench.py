@@ -1,9 +1,10 @@
 #!/usr/bin/env python
-"""Prefill and decode throughput of plan-built decoders (Vofelix, Pegopel) beside the closest existing models at equal
-size, random weights, one GPU.
+"""Prefill and decode throughput of plan-built decoders (Vofelix, Pegopel, Dubizen) beside the closest existing models
+at equal size, random weights, one GPU.
 
     python bench.py --mode layers                 # or: python benchmarks/plan_bench.py
-    python benchmarks/plan_bench.py --kernels     # the single kernels with their rooflines
+    python benchmarks/plan_bench.py --kernels     # the single kernels with their rooflines (--variant-kernels,
+                                                  # --expert-kernels: those of one design)
 
 Model cases time the engine's own step on the device (CUDA events, median): a prefill step of whole prompts,
 and decode-graph replays of a batch with a given context.  Weights and caches are larger than L2.  Kernel
@@ -72,21 +73,49 @@ def _pegopel(layers, streams=1, loop=None):
     return ModelConfig.from_hf_dict(d, name="pegopel-bench")
 
 
-def _gqa(window):
+def _shared_latent(mlp, kv_from=None, heads=32):
+    m = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": 1536, "scale": 192 ** -0.5,
+         "rot": {"base": 1e4, "dims": 64}}
+    return {"type": "latent_attention", "mlp": mlp, "mixer": m if kv_from is None else dict(m, kv_from=kv_from)}
+
+
+def _normed(mlp, window=1024):
+    return {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "bias_max": 512, "mask": {"size": window}}}
+
+
+_PLAIN_FF = {"kind": "dense", "ff": 12288}
+_EXPERTS = {"kind": "moe", "expert": {"ff": 1408}, "shared": {"ff": 2816},
+            "router": {"experts": 64, "top": 8, "scale": 2.5, "groups": {"count": 8, "keep": 4}}}
+
+
+def _dubizen(layers):
+    from vllm_ascend_b200.config import ModelConfig
+    return ModelConfig.from_hf_dict({"architecture": "Dubizen", "vocab": VOCAB, "width": 4096, "norm": {"eps": 1e-6},
+                                     "residual_mult": 0.5, "layers": layers}, name="dubizen-bench")
+
+
+def _gqa(window, **kw):
     return _existing(name="gqa-dense", architecture="Qwen3ForCausalLM", num_attention_heads=32, num_key_value_heads=8,
-                     head_dim=128, qk_norm=True, sliding_window=window, rope_theta=1e4)
+                     head_dim=128, qk_norm=True, sliding_window=window, rope_theta=1e4, **kw)
 
 
 def _existing(**kw):
     from vllm_ascend_b200.config import ModelConfig
-    return ModelConfig(vocab_size=VOCAB, hidden_size=4096, intermediate_size=12288, num_hidden_layers=LAYERS,
-                       hidden_act="gelu_pytorch_tanh", **kw)
+    kw.setdefault("hidden_act", "gelu_pytorch_tanh")
+    return ModelConfig(vocab_size=VOCAB, hidden_size=4096, intermediate_size=12288, num_hidden_layers=LAYERS, **kw)
 
 
-def _mla(heads):
+def _mla(heads, **kw):
     return _existing(name="mla-dense", architecture="DeepseekV2ForCausalLM", num_attention_heads=heads,
                      num_key_value_heads=heads, head_dim=192, use_mla=True, kv_lora_rank=512, qk_nope_head_dim=128,
-                     qk_rope_head_dim=64, v_head_dim=128, rope_theta=1e4)
+                     qk_rope_head_dim=64, v_head_dim=128, rope_theta=1e4, **kw)
+
+
+#: the feed-forwards of the Dubizen stacks, for existing models
+_UNGATED = dict(mlp_gated=False, hidden_act="gelu")
+_MOE = dict(num_experts=64, num_experts_per_tok=8, moe_intermediate_size=1408, n_shared_experts=2, scoring_func="softmax",
+            n_group=8, topk_group=4, routed_scaling_factor=2.5, e_score_correction_bias=True)
 
 
 def _gdn():
@@ -113,6 +142,16 @@ MODELS = {
     "biased attention 4 streams": lambda: _pegopel([_biased()] * LAYERS, streams=4),
     "Pegopel 2 streams loop": lambda: _pegopel([_gated(), _biased(), _biased(), _gated(), _biased(), _biased()], streams=2,
                                                  loop={"start": 1, "stop": 3, "times": 2}),
+    "Dubizen latent": lambda: _dubizen([_shared_latent(_PLAIN_FF)] * LAYERS),
+    "Dubizen latent, 6 of 8 shared": lambda: _dubizen([_shared_latent(_PLAIN_FF)] + [_shared_latent(_PLAIN_FF, 0)] * 3 +
+                                                      [_shared_latent(_PLAIN_FF)] + [_shared_latent(_PLAIN_FF, 4)] * 3),
+    "existing MLA, query latent": lambda: _mla(32, q_lora_rank=1536, **_UNGATED),
+    "Dubizen attention w=1024": lambda: _dubizen([_normed(_PLAIN_FF)] * LAYERS),
+    "existing GQA w=1024, plain feed-forward": lambda: _gqa(1024, **_UNGATED),
+    "Dubizen latent, experts": lambda: _dubizen([_shared_latent(_EXPERTS)] * LAYERS),
+    "existing MLA, experts": lambda: _mla(32, q_lora_rank=1536, **_MOE),
+    "Dubizen whole": lambda: _dubizen([_shared_latent(_PLAIN_FF), _shared_latent(_EXPERTS), _normed(_PLAIN_FF),
+                                       _normed(_EXPERTS), _shared_latent(_EXPERTS, 1), _shared_latent(_PLAIN_FF, 1)]),
 }
 
 
@@ -253,7 +292,91 @@ def bench_kernels() -> list[dict]:
                                                        window=win, sink=sink, max_kv_len=ctx)),
                 reads * 1152 + T * H * (576 + 512) * 2, keys * H * (576 + 512) * 2)
     res += _variant_kernels(rec_list=[], hbm=hbm, tf=tf)
+    res += _expert_kernels(rec_list=[], hbm=hbm, tf=tf)
     return res
+
+
+def _expert_kernels(rec_list, hbm, tf) -> list[dict]:
+    """The kernels of the Dubizen stacks that others do not have, beside their counterparts."""
+    from kernel_bench import timeit
+    from vllm_ascend_b200 import ops
+    from vllm_ascend_b200.attention import variant as va
+    from vllm_ascend_b200.attention.metadata import AttentionMetadata
+    from vllm_ascend_b200.ops import fused_moe, moe_native, reference as ref
+    from vllm_ascend_b200.ops import stream as st
+    bf, dev = torch.bfloat16, "cuda"
+
+    def rec(name, ms, nbytes=0, flops=0):
+        t_mem, t_fl = nbytes / hbm / 1e6, flops / tf / 1e9
+        rec_list.append({"kernel": name, "ms": round(ms, 4), "GB/s": round(nbytes / ms / 1e6),
+                         "TFLOP/s": round(flops / ms / 1e9, 1), "roofline_frac": round(max(t_mem, t_fl) / ms, 3)})
+
+    def mk(*s, dtype=bf):
+        return torch.randn(*s, device=dev, dtype=dtype)
+    W, H, dn, dr, dc, rq, G, D = 4096, 32, 128, 64, 512, 1536, 8, 128
+    cs = ref.build_cos_sin_cache(dr, 8192, 1e4, None, torch.device("cuda"))
+    for T in (64, 256, 8192):
+        r, y, w, res_b = mk(T, W, dtype=torch.float32), mk(T, W), mk(W), mk(T, W)
+        ln = st.NormSpec("layer", w)
+        rec(f"[existing] add+rms_norm T={T}", timeit(lambda: ops.rms_norm(y, w, 1e-6, res_b)), T * W * 8)
+        rec(f"stream_norm output norm T={T}", timeit(lambda: st.stream_norm(r, y, ln, st.PLAIN, 1e-6, bf, post_scale=0.5)),
+            T * W * 12)
+        q, kv, down, nw, qw = mk(T, H, dn + dr), mk(T, dc + dr), mk(T, rq + dc + dr), mk(dc), mk(rq)
+        nb = (T + 127) // 128 + 1
+        lat, pe = torch.zeros(nb, 128, 1, dc, device=dev, dtype=bf), torch.zeros(nb, 128, 1, dr, device=dev, dtype=bf)
+        pos, slots = torch.arange(T, device=dev) % 4096, torch.arange(T, device=dev) + 128
+        rec(f"[existing] mla_preprocess T={T}", timeit(lambda: ops.mla_preprocess(q, kv, nw, 1e-6, pos, cs, slots, lat, pe, dn, dr)),
+            T * (H * dr + dc + dr) * 4)
+        cq = mk(T, rq)
+        rec(f"[existing] rms_norm of the query latent T={T}", timeit(lambda: ops.rms_norm(cq, qw, 1e-6)), T * rq * 4)
+        rec(f"[existing] copy to head-major rows T={T}", timeit(lambda: q[..., :dn].transpose(0, 1).contiguous()), T * H * dn * 4)
+        rec(f"latent_prep T={T}", timeit(lambda: ops.latent_prep(down, qw, nw, 1e-6, pos, cs, slots, lat, pe)),
+            T * (rq + dc + dr) * 4)
+        rec(f"latent_query T={T}", timeit(lambda: ops.latent_query(q, pos, cs)), T * H * (dn + dr) * 4)
+        kc, vc = (ops.alloc_kv_cache(nb, 128, G, D, bf, dev) for _ in "kv")
+        C = (H + 2 * G) * D
+        qkv, hn, c128 = mk(T, C), mk(D), torch.randn(8192, D, device=dev)
+        cu = np.array([0, T], dtype=np.int32)
+        meta = AttentionMetadata(num_reqs=1, num_actual_tokens=T, max_query_len=T, max_seq_len=T,
+                                 query_start_loc=torch.from_numpy(cu).to(dev), seq_lens=None, block_table=None,
+                                 slot_mapping=slots, positions=pos, query_start_loc_cpu=cu, seq_lens_cpu=None)
+        rec(f"[existing] qknorm_rope_kvwrite T={T}", timeit(lambda: ops.qknorm_rope_kvwrite(
+            qkv, pos, c128, D, hn, hn, 1e-6, kc, vc, slots, H, G, D)), T * C * 4)
+        spec = va.PrepSpec(H, G, D, D, 1e-6, hn, hn, (H * D, G * D), head_norm=True)
+        rec(f"qkv_prep norm per head T={T}", timeit(lambda: va.qkv_prep(spec, qkv, meta, kc, vc)), T * C * 4)
+        act = mk(T, 12288)
+        rec(f"gelu T={T}", timeit(lambda: ops.activation(act, "gelu")), T * 12288 * 4)
+        E, k, I = 64, 8, 1408
+        rw, corr = mk(E, W), torch.randn(E, device=dev) * 0.1
+        rf = rw.float()
+        rec(f"[existing] router product, fp32 operands T={T}", timeit(lambda: torch.nn.functional.linear(y.float(), rf)),
+            T * W * 2 + E * W * 2, 2 * T * W * E)
+        rec(f"router product T={T}", timeit(lambda: ops.linear_fp32(y, rw)), T * W * 2 + E * W * 2 + T * E * 4, 2 * T * W * E)
+        z = ops.linear_fp32(y, rw) * 0.01
+        for name, score in (("[existing] gating, best two of a group", "top2"), ("gating, best of a group", "max")):
+            rec(f"{name} T={T}", timeit(lambda: fused_moe.gating_topk(z, k, "softmax", True, 8, 4, corr, 2.5, score)),
+                T * E * 4 + T * k * 8)
+        tw, ids = fused_moe.gating_topk(z, k, "softmax", True, 8, 4, corr, 2.5, "max")
+        w13, w2, s, sg = mk(E, 2 * I, W) * 0.02, mk(E, W, I) * 0.02, mk(T, W), mk(1, W)
+        perm = moe_native.Permutation(ids, None, E)
+        rec(f"permute T={T}", timeit(lambda: moe_native.Permutation(ids, None, E)), T * k * 16)
+        xs = perm.gather(y)
+        rec(f"gather T={T}", timeit(lambda: perm.gather(y)), T * W * 2 + T * k * W * 2)
+        used = int((perm.counts > 0).sum())
+        h = moe_native.grouped_gemm(xs, w13, perm.offsets, True)
+        rec(f"grouped product, gate and up T={T}", timeit(lambda: moe_native.grouped_gemm(xs, w13, perm.offsets, True)),
+            used * 2 * I * W * 2 + T * k * (W + I) * 2, 4 * T * k * I * W)
+        o = moe_native.grouped_gemm(h, w2, perm.offsets, False)
+        rec(f"grouped product, down T={T}", timeit(lambda: moe_native.grouped_gemm(h, w2, perm.offsets, False)),
+            used * I * W * 2 + T * k * (W + I) * 2, 2 * T * k * I * W)
+
+        def apart():
+            return perm.combine(o, tw) + s * torch.sigmoid(torch.nn.functional.linear(y.float(), sg.float())).to(bf)
+        rec(f"[existing] combine, then the gated shared expert T={T}", timeit(apart), T * W * 2 * (k + 3))
+        rec(f"combine with the gated shared expert T={T}", timeit(lambda: perm.combine(o, tw, shared=s, x=y, shared_gate=sg)),
+            T * W * 2 * (k + 3))
+        del w13, w2, xs, h, o
+    return rec_list
 
 
 def _variant_kernels(rec_list, hbm, tf) -> list[dict]:
@@ -329,6 +452,7 @@ def _variant_kernels(rec_list, hbm, tf) -> list[dict]:
             rec(f"[existing] paged attention {tag} window {win}",
                 timeit(lambda: ops.paged_attention(q, kc, vc, meta, sc, window=win)), nbytes, fl)
             for name, o, g in (("no options", va.AttnOptions(sc, win), None),
+                               ("bias", va.AttnOptions(sc, win, bias=bias), None),
                                ("bias + sink", va.AttnOptions(sc, win, bias=bias, sink=zero), None),
                                ("cap + kept + gate", va.AttnOptions(sc, win, 64, 30.0, sink=zero), gate)):
                 rec(f"attention {name} {tag} window {win}", timeit(lambda: va.variant_attention(q, kc, vc, meta, o, g)),
@@ -344,18 +468,23 @@ def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--kernels", action="store_true")
     ap.add_argument("--variant-kernels", action="store_true", help="only the kernels of attention with options")
-    ap.add_argument("--only", default="", help="model labels with commas between them")
+    ap.add_argument("--expert-kernels", action="store_true", help="only the kernels of the Dubizen stacks")
+    ap.add_argument("--only", default="", help="model labels with semicolons between them")
     args = ap.parse_args()
     if args.variant_kernels:
         for row in _variant_kernels([], *peaks()):
             print(json.dumps(row))
+        return
+    if args.expert_kernels:
+        for row in _expert_kernels([], *peaks()):
+            print(json.dumps(row), flush=True)
         return
     if args.kernels:
         for row in bench_kernels():
             print(json.dumps(row))
         return
     for k in MODELS:
-        if not args.only or k in args.only.split(","):
+        if not args.only or k in args.only.split(";"):
             print(json.dumps({k: bench_model(MODELS[k]())}), flush=True)
 
 

@@ -202,14 +202,14 @@ __global__ void moe_gather_rows_kernel(const __nv_bfloat16* __restrict__ x,
 }
 // out[t] = sum_s w[t,s] * y[pos[t,s]] (+ sigmoid(x[t] . gate) * shared[t])
 template <typename T, int VEC>
-__global__ void __launch_bounds__(128) moe_combine_kernel(const T* __restrict__ y, const int* __restrict__ pos,
+__global__ void __launch_bounds__(512) moe_combine_kernel(const T* __restrict__ y, const int* __restrict__ pos,
                                                           const float* __restrict__ w, int k, int H, T* __restrict__ out,
                                                           int accumulate, const T* __restrict__ shared,
                                                           const T* __restrict__ x, const T* __restrict__ gate) {
   const long t = blockIdx.x;
   float g = 1.f;
   if (gate) {
-    __shared__ float red[4];
+    __shared__ float red[16];
     float dot = 0.f;
     for (int c = (int)threadIdx.x * VEC; c < H; c += (int)blockDim.x * VEC) {
       float a[VEC], b[VEC];
@@ -221,13 +221,15 @@ __global__ void __launch_bounds__(128) moe_combine_kernel(const T* __restrict__ 
     dot = warp_reduce_sum(dot);
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = dot;
     __syncthreads();
-    g = 1.f / (1.f + expf(-(red[0] + red[1] + red[2] + red[3])));
+    dot = warp_reduce_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? red[threadIdx.x & 31] : 0.f);
+    g = 1.f / (1.f + expf(-dot));
   }
   for (int c = (int)threadIdx.x * VEC; c < H; c += (int)blockDim.x * VEC) {
     float acc[VEC], v[VEC];
 #pragma unroll
     for (int e = 0; e < VEC; e++) acc[e] = 0.f;
     if (accumulate) load_vec<T, VEC>(out + t * H + c, acc);
+#pragma unroll 4
     for (int s = 0; s < k; s++) {
       const int r = pos[t * k + s];
       if (r < 0) continue;
@@ -250,11 +252,14 @@ static int launch_combine(const void* y, const void* pos, const void* w, int tok
                           int accumulate, const void* shared, const void* x, const void* gate, cudaStream_t stream) {
   constexpr int V = 16 / (int)sizeof(T);
   const bool vec = H % V == 0 && aligned16(y) && aligned16(out) && aligned16(shared) && aligned16(x) && aligned16(gate);
+  int threads = (H / (vec ? V : 1) + 31) / 32 * 32;     // few tokens: a block takes its row at once
+  if (threads > (tokens < 2048 ? 512 : 128)) threads = tokens < 2048 ? 512 : 128;
+  if (threads < 32) threads = 32;
   if (vec)
-    moe_combine_kernel<T, V><<<tokens, 128, 0, stream>>>((const T*)y, (const int*)pos, (const float*)w, k, H, (T*)out,
+    moe_combine_kernel<T, V><<<tokens, threads, 0, stream>>>((const T*)y, (const int*)pos, (const float*)w, k, H, (T*)out,
                                                          accumulate, (const T*)shared, (const T*)x, (const T*)gate);
   else
-    moe_combine_kernel<T, 1><<<tokens, 128, 0, stream>>>((const T*)y, (const int*)pos, (const float*)w, k, H, (T*)out,
+    moe_combine_kernel<T, 1><<<tokens, threads, 0, stream>>>((const T*)y, (const int*)pos, (const float*)w, k, H, (T*)out,
                                                          accumulate, (const T*)shared, (const T*)x, (const T*)gate);
   return B200_CHECK_LAUNCH();
 }
