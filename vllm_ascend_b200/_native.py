@@ -25,6 +25,8 @@ _SIGNATURES = {
     "b200_gemm_bf16_2cta": [P, P, P, P, P, I, I, I, I, I, I, I, P, P],
     "b200_gemm_bf16_2cta_norm": [P, P, P, P, P, I, I, I, I, I, I, I, P, I, ctypes.c_float, P, L, I, P, P],
     "b200_gemm_swiglu_bf16": [P, P, P, I, I, I, I, I, I, P, P],
+    "b200_gemm_glu_bf16": [P, P, P, I, I, I, I, I, I, F, F, P, P],
+    "b200_gemm_glu_bf16_2cta": [P, P, P, I, I, I, I, I, I, F, F, P, P],
     "b200_grouped_gemm_bf16": [P, P, P, P, I, L, I, I, I, I, I, I, P, P],
     "b200_rms_norm": [P, P, P, P, L, I, F, I, L, L, P],
     "b200_silu_and_mul": [P, P, L, I, F, P],
@@ -116,6 +118,12 @@ def ptr(t: Optional[torch.Tensor]) -> Optional[int]:
 
 def stream_ptr(device=None) -> int:
     return torch.cuda.current_stream(device).cuda_stream
+
+
+def struct_fields(**kinds) -> list:
+    """ctypes fields of a kernel's argument struct: pointers, then 64-bit, then 32-bit members."""
+    ctype = {"pointers": ctypes.c_void_p, "longs": ctypes.c_long, "ints": ctypes.c_int, "floats": ctypes.c_float}
+    return [(name, ctype[kind]) for kind, names in kinds.items() for name in names.split()]
 
 
 class NativeError(RuntimeError):

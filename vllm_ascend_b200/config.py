@@ -55,6 +55,10 @@ class ModelConfig:
     e_score_correction_bias: bool = False
     moe_group_score: Optional[str] = None    # score of an expert group: "max" | "top2" (sum of its best two); None: top2 with a bias
     router_fp32: bool = False                # router weights in the model dtype, logits summed and kept in fp32
+    moe_weight_input: bool = False           # an expert works on weight * input instead of having its output weighted
+    # clamped gate of an expert: min(g, limit) sigmoid(1.702 .) (clamp(u, -limit, limit) + 1); None: SiLU gate
+    expert_limit: Optional[float] = None
+    shared_expert_limit: Optional[float] = None
     # ---- linear attention (Gated DeltaNet hybrids: every `full_attention_interval`-th layer is
     # softmax attention, the others keep a recurrent state instead of a KV cache) ----
     full_attention_interval: int = 0
@@ -115,11 +119,12 @@ class ModelConfig:
     rope_half_split: bool = False            # checkpoint rotates (i, i + dims / 2) of the rotary part; rows are re-ordered at load
     latent_kv_from: Optional[int] = None     # this layer attends to the latents that layer stores and has none of its own
     # ---- decoders described layer by layer (layer_plan.py) ----
-    layer_plan: Optional[list] = None        # per layer {"mixer", "mlp", "over": fields of this layer}
+    layer_plan: Optional[list] = None        # per layer {"mixer", "mlp", "over": fields of this layer[, "weights_of": layer]}
     layer_loop: Optional[tuple] = None       # (start, stop, times): layers start..stop-1 run times in a row
     layer_loop_refeed: bool = False          # the embedding output joins the stream again before every pass but the first
     norm_type: str = "rms"                   # "rms" | "layer" (weight and, with norm_bias, bias)
     norm_bias: bool = True
+    norm_groups: int = 1                     # RMS norms of the stream: that many equal parts, each by itself
     token_side_dim: int = 0                  # per-layer token input: width of a layer's slice of the table
     attention_sink: bool = False             # a learned logit per head in the softmax denominator
     # ---- options of paged grouped-query attention (models/variant_attention.py) ----
@@ -132,6 +137,11 @@ class ModelConfig:
     attn_distance_buckets: int = 32          # rows of that table (a checkpoint's own table decides)
     attn_head_gate: bool = False             # each head's output is scaled by a sigmoid of the layer's input
     rotary_dims: Optional[int] = None        # rotated dimensions of a head (0: none) where the layer names them
+    attn_map_diff: Optional[float] = None    # two softmax maps per head over the same values, the second subtracted; this constant
+    attn_talk: bool = False                  # the scores of all heads are mixed by a learned matrix before the softmax
+    attn_query_temp: Optional[tuple] = None  # (coef, every): queries times 1 + coef ln(floor((p + 1) / every) + 1) at position p
+    # ---- two mixers side by side (models/parallel_mixer.py): paged attention and mamba_config's state space ----
+    parallel_scales: Optional[tuple] = None  # factors of the two outputs
     # ---- residual streams and learned positions of plan-built decoders ----
     residual_streams: int = 0                # > 0: that many streams with static mixing per sub-layer
     learned_positions: int = 0               # rows of a position table added to the embeddings (0: none)
@@ -169,7 +179,8 @@ class ModelConfig:
     @property
     def keeps_sequence_state(self) -> bool:
         """Layers keep something per sequence besides pages (recurrent states, convolution inputs)."""
-        return self.is_hybrid or any(p["over"].get("attn_conv_kernel", 0) > 1 for p in self.layer_plan or ())
+        return self.is_hybrid or any(p["mixer"] == "parallel" or p["over"].get("attn_conv_kernel", 0) > 1
+                                     for p in self.layer_plan or ())
 
     def layer_config(self, layer_idx: int) -> "ModelConfig":
         """The configuration as layer ``layer_idx`` sees it: its own sizes where the model has a plan."""
@@ -438,6 +449,9 @@ def _preset(**kw) -> ModelConfig:
 
 
 #: Architectures named by the benchmark configs (random-init, synthetic prompts).
+_TINY_CLAMPED = {"kind": "moe", "router": {"experts": 8, "top": 2}, "expert": {"ff": 40, "limit": 3.0},
+                 "shared": {"ff": 64, "limit": 2.0}}
+
 PRESETS: dict[str, Any] = {
     "tiny-qwen": lambda: _preset(
         name="tiny-qwen", architecture="Qwen3ForCausalLM", vocab_size=1024, hidden_size=256,
@@ -543,6 +557,21 @@ PRESETS: dict[str, Any] = {
                 "heads": 2, "dim": 40, "rot_dim": 16, "vdim": 32, "kv_rank": 48, "q_rank": 32, "scale": 0.14, "kv_from": 0,
                 "rot": {"base": 10000.0, "dims": 16}}},
         ]}, dtype="float32", name="tiny-dubizen"),
+    "tiny-nevotar": lambda: ModelConfig.from_hf_dict({
+        "architecture": "Nevotar", "vocab": 312, "width": 96, "norm": {"eps": 1e-5, "groups": 3}, "layers": [
+            {"type": "parallel", "mlp": _TINY_CLAMPED, "mixer": {
+                "left": {"heads": 4, "kv_heads": 2, "dim": 24, "vdim": 16, "scale": 0.2, "mask": {"size": 30},
+                         "rot": {"base": 10000.0, "dims": 16}},
+                "right": {"heads": 6, "vdim": 16, "state": 24, "groups": 3, "conv": 4, "norm_groups": 2},
+                "left_scale": 0.7, "right_scale": 0.4}},
+            {"type": "attention", "mlp": None, "mixer": {
+                "heads": 4, "kv_heads": 2, "dim": 16, "vdim": 24, "scale": 0.25, "diff": 0.4,
+                "q_temp": {"coef": 0.2, "every": 20}}},
+            {"type": "hgrn2", "mlp": _TINY_CLAMPED, "mixer": {"heads": 4, "dim": 16, "vdim": 32}},
+            {"type": "attention", "mlp": None, "weights_of": 1, "mixer": {
+                "heads": 4, "kv_heads": 2, "dim": 16, "vdim": 24, "scale": 0.25, "diff": 0.4,
+                "q_temp": {"coef": 0.2, "every": 20}}},
+        ]}, dtype="float32", name="tiny-nevotar"),
     "tiny-deepseek": lambda: _preset(
         name="tiny-deepseek", architecture="DeepseekV3ForCausalLM", vocab_size=512,
         hidden_size=128, intermediate_size=256, num_hidden_layers=3, num_attention_heads=4,

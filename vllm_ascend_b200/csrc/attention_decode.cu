@@ -9,6 +9,7 @@
 // Scratch layout (fp32): partial_o [B, Hq, S, D] (each split normalised by its
 // own sum), partial_lse [B, Hq, S] (natural-log sum-exp, -inf for empty splits).
 #include "common.cuh"
+#include "dtypes.cuh"
 #include "attention.h"
 
 namespace b200 {
@@ -147,12 +148,13 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, long q_stride,
 }
 
 // out[t, hq, :] = sum_s softmax_s(lse)[s] * partial_o[t, hq, s, :]
+template <typename TO>
 __global__ void merge_splits_kernel(const float* __restrict__ partial_o,
                                     const float* __restrict__ partial_lse, int num_splits, int D,
-                                    int Hq, __nv_bfloat16* __restrict__ out, long out_stride,
+                                    int Hq, TO* __restrict__ out, long out_stride,
                                     long out_head, float* __restrict__ lse_out,
                                     const float* __restrict__ sink,
-                                    const __nv_bfloat16* __restrict__ gate, long gate_stride) {
+                                    const __nv_bfloat16* __restrict__ gate, long gate_stride, float out_scale) {
   const long t = blockIdx.x;
   const int hq = blockIdx.y;
   const long base = (t * Hq + hq) * num_splits;
@@ -164,7 +166,7 @@ __global__ void merge_splits_kernel(const float* __restrict__ partial_o,
       for (int s = 0; s < num_splits; s++) L += __expf(partial_lse[base + s] - M);
     lse_out[t * Hq + hq] = L > 0.f ? M + logf(L) : -INFINITY;
   }
-  const float g = gate ? 1.f / (1.f + __expf(-__bfloat162float(gate[t * gate_stride + hq]))) : 1.f;
+  const float g = out_scale * (gate ? 1.f / (1.f + __expf(-__bfloat162float(gate[t * gate_stride + hq]))) : 1.f);
   for (int d = threadIdx.x; d < D; d += blockDim.x) {
     float acc = 0.f, L = sink ? __expf(sink[hq] - M) : 0.f;
     if (M != -INFINITY) {
@@ -174,18 +176,24 @@ __global__ void merge_splits_kernel(const float* __restrict__ partial_o,
         acc += w * partial_o[(base + s) * D + d];
       }
     }
-    out[t * out_stride + hq * out_head + d] = __float2bfloat16(L > 0.f ? g * acc / L : 0.f);
+    out[t * out_stride + hq * out_head + d] = from_f<TO>(L > 0.f ? g * acc / L : 0.f);
   }
 }
 
 int launch_merge_splits(const float* partial_o, const float* partial_lse, long T, int Hq,
                         int num_splits, int D, void* out, long out_stride, cudaStream_t stream,
-                        float* lse_out, long out_head, const float* sink, const void* gate, long gate_stride) {
+                        float* lse_out, long out_head, const float* sink, const void* gate, long gate_stride,
+                        bool out_f32, float out_scale) {
   if (T <= 0) return 0;
   dim3 grid((unsigned)T, (unsigned)Hq);
-  merge_splits_kernel<<<grid, D > 64 ? 128 : 64, 0, stream>>>(
-      partial_o, partial_lse, num_splits, D, Hq, (__nv_bfloat16*)out, out_stride, out_head ? out_head : D, lse_out,
-      sink, (const __nv_bfloat16*)gate, gate_stride);
+  if (out_f32)
+    merge_splits_kernel<float><<<grid, D > 64 ? 128 : 64, 0, stream>>>(
+        partial_o, partial_lse, num_splits, D, Hq, (float*)out, out_stride, out_head ? out_head : D, lse_out,
+        sink, (const __nv_bfloat16*)gate, gate_stride, out_scale);
+  else
+    merge_splits_kernel<__nv_bfloat16><<<grid, D > 64 ? 128 : 64, 0, stream>>>(
+        partial_o, partial_lse, num_splits, D, Hq, (__nv_bfloat16*)out, out_stride, out_head ? out_head : D, lse_out,
+        sink, (const __nv_bfloat16*)gate, gate_stride, out_scale);
   return B200_CHECK_LAUNCH();
 }
 

@@ -55,7 +55,8 @@ struct DecParams {
   int* status;
   // VAR only
   int keep_first, bias_len, Dv;
-  float scale, softcap;
+  int key_heads, out_f32;      // value head h belongs to key head h * key_heads / Hkv; out is fp32
+  float scale, softcap, out_scale;
   const float* bias;           // [Hq, bias_len]
   const float* sink;           // [Hq]
   const __nv_bfloat16* gate;   // [T, Hq]
@@ -285,6 +286,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     bool q_ahead = false;                // the next non-empty item's Q load was already issued
     for (int item = blockIdx.x; item < num_items; item += gridDim.x) {
       const DecItem w = w_next;
+      const int hk = VAR ? w.h * p.key_heads / p.Hkv : w.h;
       int blk_cur = blk_first_next;
       const int item_after = item + gridDim.x;
       if (w.n <= 0) {
@@ -317,7 +319,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
             const int off = ((dec_tile<VAR>(w, jp) << 7) + lane * rpl) % p.block_size;
 #pragma unroll
             for (int hf = 0; hf < NH; hf++) {
-              tma_prefetch_l2_4d(&tmap_k, hf * 64, w.h, off, blk_pf);
+              tma_prefetch_l2_4d(&tmap_k, hf * 64, hk, off, blk_pf);
               tma_prefetch_l2_4d(&tmap_v, hf * 64, w.h, off, blk_pf);
             }
           }
@@ -350,7 +352,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
               for (int sub = 0; sub < nsub; sub++) {
 #pragma unroll
                 for (int hf = 0; hf < NH; hf++)
-                  tma_load_4d(dst + hf * DEC_HALF + sub * 32 * 128, tm, fullb, hf * 64, w.h,
+                  tma_load_4d(dst + hf * DEC_HALF + sub * 32 * 128, tm, fullb, hf * 64, kv == 0 ? hk : w.h,
                               off + sub * 32, blk);
               }
             }
@@ -366,7 +368,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
               const int off = (key_base + part * rpl) % p.block_size;
 #pragma unroll
               for (int hf = 0; hf < NH; hf++)
-                tma_load_4d(dst + hf * DEC_HALF + part * rpl * 128, tm, fullb, hf * 64, w.h, off, blk);
+                tma_load_4d(dst + hf * DEC_HALF + part * rpl * 128, tm, fullb, hf * 64, kv == 0 ? hk : w.h, off, blk);
             }
           }
           __syncwarp();
@@ -640,10 +642,13 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
               if (p.num_splits == 1) {            // with splits the merge does both
                 if (p.sink && l > 0.f) inv = 1.f / (l + score_exp2(p.sink[hq] * kLog2e - m[c] * sl2));
                 if (p.gate) inv *= sigmoid_f(__bfloat162float(p.gate[tok * p.gate_stride + hq]));
+                inv *= p.out_scale;
               }
             }
             const float val = __uint_as_float(o[c]) * inv;
-            if (p.num_splits == 1) {
+            if (VAR && p.num_splits == 1 && p.out_f32) {
+              ((float*)p.out)[tok * p.out_stride + (long)hq * dv + tid] = val;
+            } else if (p.num_splits == 1) {
               p.out[tok * p.out_stride + (long)hq * dv + tid] = __float2bfloat16(val);
               if (tid == 0 && p.lse_out)
                 p.lse_out[tok * p.Hq + hq] =
@@ -873,6 +878,7 @@ B200_API int b200_attention_variant_decode(const b200::AttnVariantArgs* a, int* 
   if (bs < 8 || (bs < 128 && 128 % bs) || (bs > 128 && bs % 128)) return 9872;
   if ((a->q_stride & 7) || (a->out_stride & 7) || (a->bias && a->bias_len < 1) || a->keep_first < 0) return 9873;
   if (a->num_splits < 1 || (a->num_splits > 1 && !a->scratch)) return 9874;
+  if (a->key_heads < 1 || a->Hkv % a->key_heads) return 9875;
   const int G = a->Hq / a->Hkv, rpl = bs < 128 ? bs : 128;
   CUtensorMap tq, tkv[2], tkv32[2];
   {
@@ -883,7 +889,8 @@ B200_API int b200_attention_variant_decode(const b200::AttnVariantArgs* a, int* 
     if (rc) return rc;
   }
   for (int kv = 0; kv < 2; kv++) {
-    uint64_t dims[4] = {(uint64_t)(kv ? a->Dv : a->D), (uint64_t)a->Hkv, (uint64_t)bs, (uint64_t)a->num_blocks};
+    uint64_t dims[4] = {(uint64_t)(kv ? a->Dv : a->D), (uint64_t)(kv ? a->Hkv : a->key_heads), (uint64_t)bs,
+                        (uint64_t)a->num_blocks};
     uint64_t str[3] = {(uint64_t)(kv ? a->v_head : a->k_head) * 2, (uint64_t)(kv ? a->v_tok : a->k_tok) * 2,
                        (uint64_t)(kv ? a->v_block : a->k_block) * 2};
     uint32_t box[4] = {64, 1, (uint32_t)rpl, 1}, box32[4] = {64, 1, 32, 1};
@@ -916,6 +923,7 @@ B200_API int b200_attention_variant_decode(const b200::AttnVariantArgs* a, int* 
   p.keep_first = a->window > 0 ? a->keep_first : 0;
   p.bias_len = a->bias_len; p.Dv = a->Dv;
   p.scale = a->scale; p.softcap = a->softcap;
+  p.key_heads = a->key_heads; p.out_f32 = a->out_f32; p.out_scale = a->out_scale;
   p.bias = a->bias; p.sink = a->sink;
   p.gate = (const __nv_bfloat16*)a->gate;
   p.gate_stride = a->gate_stride;
@@ -923,6 +931,7 @@ B200_API int b200_attention_variant_decode(const b200::AttnVariantArgs* a, int* 
   if (rc) return rc;
   if (a->num_splits > 1)
     return launch_merge_splits(p.partial_o, p.partial_lse, a->num_seqs, a->Hq, a->num_splits, a->Dv, a->out,
-                               a->out_stride, stream, nullptr, 0, a->sink, a->gate, a->gate_stride);
+                               a->out_stride, stream, nullptr, 0, a->sink, a->gate, a->gate_stride, a->out_f32,
+                               a->out_scale);
   return 0;
 }

@@ -56,7 +56,8 @@ struct AttnParams {
   float rescale_threshold;
   // VAR only
   int num_seqs, keep_first, bias_len, Dv;
-  float scale, softcap;
+  int key_heads, out_f32;      // value head h belongs to key head h * key_heads / Hkv; out is fp32
+  float scale, softcap, out_scale;
   const float* bias;           // [Hq, bias_len]
   const float* sink;           // [Hq]
   const __nv_bfloat16* gate;   // [T, Hq]
@@ -212,6 +213,7 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       const int key0 = (tile_no(j) << 7) + lane * rpl;
       return bt[min(key0, seq_len - 1) / p.block_size];
     };
+    const int hk = VAR ? h * p.key_heads / p.Hkv : h;
     int blk_cur = load_blk(0);
     for (int j = 0; j < n; j++) {
       const int ks = j % KS;
@@ -238,7 +240,7 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
             const int off = (key_base + part * rpl) % p.block_size;
 #pragma unroll
             for (int hf = 0; hf < NH; hf++)
-              tma_load_4d(dst + hf * ATT_HALF_BYTES + part * rpl * 128, tm, fullb, hf * 64, h, off, blk);
+              tma_load_4d(dst + hf * ATT_HALF_BYTES + part * rpl * 128, tm, fullb, hf * 64, kv == 0 ? hk : h, off, blk);
           }
         }
         __syncwarp();
@@ -463,6 +465,7 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       if (p.num_splits == 1 && row_valid) {           // with splits the merge does both
         if (p.sink && l > 0.f) inv = 1.f / (l + score_exp2(p.sink[hq] * kLog2e - m * sl2));
         if (p.gate) inv *= sigmoid_f(__bfloat162float(p.gate[tokidx * p.gate_stride + hq]));
+        inv *= p.out_scale;
       }
     }
 #pragma unroll 1
@@ -471,7 +474,16 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       tmem_ld_32x32b_x32(t_lane + Cfg::O_COL + c * 32, r);
       tmem_ld_wait();
       if (row_valid) {
-        if (p.num_splits == 1) {
+        if (VAR && p.num_splits == 1 && p.out_f32) {
+          float* dst = (float*)p.out + tokidx * p.out_stride + (long)hq * dv + c * 32;
+#pragma unroll
+          for (int q4 = 0; q4 < 8; q4++) {
+            if (c * 32 + q4 * 4 >= dv) break;
+            reinterpret_cast<float4*>(dst)[q4] =
+                make_float4(__uint_as_float(r[q4 * 4 + 0]) * inv, __uint_as_float(r[q4 * 4 + 1]) * inv,
+                            __uint_as_float(r[q4 * 4 + 2]) * inv, __uint_as_float(r[q4 * 4 + 3]) * inv);
+          }
+        } else if (p.num_splits == 1) {
           __nv_bfloat16* dst = p.out + tokidx * p.out_stride + (long)hq * dv + c * 32;
 #pragma unroll
           for (int q4 = 0; q4 < 4; q4++) {
@@ -663,6 +675,7 @@ B200_API int b200_attention_variant_prefill(const b200::AttnVariantArgs* a, int*
   if (bs < 8 || (bs < 128 && 128 % bs) || (bs > 128 && bs % 128)) return 9862;
   if ((a->q_stride & 7) || (a->out_stride & 7) || (a->bias && a->bias_len < 1) || a->keep_first < 0) return 9863;
   if (a->num_splits < 1 || (a->num_splits > 1 && !a->scratch)) return 9864;
+  if (a->key_heads < 1 || a->Hkv % a->key_heads) return 9866;
   const int G = a->Hq / a->Hkv, tok = 128 / G, rpl = bs < 128 ? bs : 128;
   CUtensorMap tq, tk, tv;
   {
@@ -673,7 +686,8 @@ B200_API int b200_attention_variant_prefill(const b200::AttnVariantArgs* a, int*
     if (rc) return rc;
   }
   for (int kv = 0; kv < 2; kv++) {
-    uint64_t dims[4] = {(uint64_t)(kv ? a->Dv : a->D), (uint64_t)a->Hkv, (uint64_t)bs, (uint64_t)a->num_blocks};
+    uint64_t dims[4] = {(uint64_t)(kv ? a->Dv : a->D), (uint64_t)(kv ? a->Hkv : a->key_heads), (uint64_t)bs,
+                        (uint64_t)a->num_blocks};
     uint64_t str[3] = {(uint64_t)(kv ? a->v_head : a->k_head) * 2, (uint64_t)(kv ? a->v_tok : a->k_tok) * 2,
                        (uint64_t)(kv ? a->v_block : a->k_block) * 2};
     uint32_t box[4] = {64, 1, (uint32_t)rpl, 1};
@@ -704,6 +718,7 @@ B200_API int b200_attention_variant_prefill(const b200::AttnVariantArgs* a, int*
   p.keep_first = a->window > 0 ? a->keep_first : 0;
   p.bias_len = a->bias_len; p.Dv = a->Dv;
   p.scale = a->scale; p.softcap = a->softcap;
+  p.key_heads = a->key_heads; p.out_f32 = a->out_f32; p.out_scale = a->out_scale;
   p.bias = a->bias; p.sink = a->sink;
   p.gate = (const __nv_bfloat16*)a->gate;
   p.gate_stride = a->gate_stride;
@@ -714,6 +729,7 @@ B200_API int b200_attention_variant_prefill(const b200::AttnVariantArgs* a, int*
   if (rc) return rc;
   if (a->num_splits > 1)
     return launch_merge_splits(p.partial_o, p.partial_lse, a->tokens, a->Hq, a->num_splits, a->Dv, a->out,
-                               a->out_stride, stream, nullptr, 0, a->sink, a->gate, a->gate_stride);
+                               a->out_stride, stream, nullptr, 0, a->sink, a->gate, a->gate_stride, a->out_f32,
+                               a->out_scale);
   return 0;
 }

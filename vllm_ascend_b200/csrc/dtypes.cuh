@@ -50,6 +50,15 @@ template <typename T> __device__ __forceinline__ float silu_f(float v) {
   if constexpr (sizeof(T) == 2) return v / (1.f + __expf(-v));
   return v / (1.f + expf(-v));
 }
+// gate of a gated MLP: silu(g) u, or with alpha > 0 the clamped min(g, limit) sigmoid(alpha .) (clamp(u, -limit, limit) + 1)
+__device__ __forceinline__ float glu_f(float g, float u, float alpha, float limit) {
+  if (alpha > 0.f) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+  }
+  return g / (1.f + expf(-g)) * u;
+}
 __device__ __forceinline__ float gelu_tanh_f(float z) {
   const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
   return 0.5f * z * (1.f + tanhf(u));

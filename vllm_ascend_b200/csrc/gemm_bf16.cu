@@ -76,6 +76,8 @@ struct GemmParams {
   int rows_per_owner;
   // ---- SWIGLU
   int up_row_offset;          // row of W where the "up" half starts (I), per group
+  float glu_alpha, glu_limit; // alpha > 0: clamped gate instead of SiLU
+  const float* row_scale;     // [rows] factor of the product before the gate, or null
   // ---- GROUPED
   const int* group_offsets;   // [num_groups + 1] row offsets into A / C
   int num_groups;
@@ -323,10 +325,22 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a,
           uint32_t u[32];
           tmem_ld_32x32b_x32(t_row + OUT_COLS / 2 + c0, u);
           tmem_ld_wait();
+          if (p.glu_alpha > 0.f || p.row_scale) {
+            const float f = p.row_scale && row_ok ? p.row_scale[row] : 1.f;
+            const float a = p.glu_alpha > 0.f ? p.glu_alpha : 1.f, lim = p.glu_alpha > 0.f ? p.glu_limit : INFINITY;
+            const float one = p.glu_alpha > 0.f ? 1.f : 0.f;
 #pragma unroll
-          for (int j = 0; j < 32; j++) {
-            const float g = __uint_as_float(r[j]);
-            r[j] = __float_as_uint(g / (1.f + __expf(-g)) * __uint_as_float(u[j]));
+            for (int j = 0; j < 32; j++) {
+              const float g = fminf(__uint_as_float(r[j]) * f, lim);
+              const float up = fminf(fmaxf(__uint_as_float(u[j]) * f, -lim), lim);
+              r[j] = __float_as_uint(g / (1.f + __expf(-a * g)) * (up + one));
+            }
+          } else {
+#pragma unroll
+            for (int j = 0; j < 32; j++) {
+              const float g = __uint_as_float(r[j]);
+              r[j] = __float_as_uint(g / (1.f + __expf(-g)) * __uint_as_float(u[j]));
+            }
           }
         } else {
           tmem_ld_wait();
@@ -553,9 +567,10 @@ B200_API int b200_gemm_bf16(const void* A, const void* W, void* C, const void* b
 
 // out[M, I] = silu(A W_gate^T) * (A W_up^T) with W = [gate (I rows); up (I rows)] of row
 // stride ldw.  I must be a multiple of 8 (columns of a last partial tile are not stored).
-B200_API int b200_gemm_swiglu_bf16(const void* A, const void* W, void* out, int M, int I, int K,
-                                   int lda, int ldw, int ldo, int* status,
-                                   cudaStream_t stream) {
+// glu: alpha 0 the SiLU gate; alpha > 0: min(g, limit) sigmoid(alpha .) (clamp(u, -limit, limit) + 1)
+B200_API int b200_gemm_glu_bf16(const void* A, const void* W, void* out, int M, int I, int K,
+                                int lda, int ldw, int ldo, float alpha, float limit, int* status,
+                                cudaStream_t stream) {
   if (M <= 0 || I <= 0) return 0;
   if ((K & 7) || (I & 7) || (lda & 7) || (ldw & 7) || (ldo & 7)) return 9100;
   GemmParams p;
@@ -565,7 +580,15 @@ B200_API int b200_gemm_swiglu_bf16(const void* A, const void* W, void* out, int 
   p.status = status;
   p.mode = GEMM_SWIGLU;
   p.up_row_offset = I;
+  p.glu_alpha = alpha;
+  p.glu_limit = limit;
   return launch_gemm<256>(A, W, p, lda, ldw, M, 2L * I, 0, stream);
+}
+
+B200_API int b200_gemm_swiglu_bf16(const void* A, const void* W, void* out, int M, int I, int K,
+                                   int lda, int ldw, int ldo, int* status,
+                                   cudaStream_t stream) {
+  return b200_gemm_glu_bf16(A, W, out, M, I, K, lda, ldw, ldo, 0.f, 0.f, status, stream);
 }
 
 // All-gather -> GEMM.  A [M, K] lives in this rank's gather buffer; rows
@@ -650,10 +673,9 @@ B200_API int b200_gemm_pub_bf16(const void* A, const void* W, void* C, const voi
 // Grouped GEMM (MoE): rows [offsets[e], offsets[e+1]) of A multiply W[e] ([n_per_group, K]);
 // with swiglu != 0, W[e] = [gate (I); up (I)] and C has I columns.  total_rows bounds the
 // rows of A / C; offsets is a device int32 array of num_groups + 1 entries.
-B200_API int b200_grouped_gemm_bf16(const void* A, const void* W, void* C, const void* offsets,
-                                    int num_groups, long total_rows, int N, int K, int lda,
-                                    int ldw, int ldc, int swiglu, int* status,
-                                    cudaStream_t stream) {
+static int grouped_gemm(const void* A, const void* W, void* C, const void* offsets, int num_groups, long total_rows,
+                        int N, int K, int lda, int ldw, int ldc, int swiglu, const void* row_scale, float alpha,
+                        float limit, int* status, cudaStream_t stream) {
   if (total_rows <= 0 || N <= 0 || num_groups <= 0) return 0;
   if ((K & 7) || (N & 7) || (lda & 7) || (ldw & 7) || (ldc & 7)) return 9100;
   if (num_groups > GEMM_MAX_GROUPS) return 9131;
@@ -663,6 +685,9 @@ B200_API int b200_grouped_gemm_bf16(const void* A, const void* W, void* C, const
   p.C = (__nv_bfloat16*)C;
   p.status = status;
   p.mode = GEMM_GROUPED | (swiglu ? GEMM_SWIGLU : 0);
+  p.glu_alpha = alpha;
+  p.glu_limit = limit;
+  p.row_scale = (const float*)row_scale;
   p.group_offsets = (const int*)offsets;
   p.num_groups = num_groups;
   p.w_rows_per_group = swiglu ? 2 * N : N;
@@ -671,6 +696,22 @@ B200_API int b200_grouped_gemm_bf16(const void* A, const void* W, void* C, const
   if (swiglu || N % 256 == 0)
     return launch_gemm<256>(A, W, p, lda, ldw, total_rows, w_rows, 0, stream);
   return launch_gemm<128>(A, W, p, lda, ldw, total_rows, w_rows, 0, stream);
+}
+
+B200_API int b200_grouped_gemm_bf16(const void* A, const void* W, void* C, const void* offsets,
+                                    int num_groups, long total_rows, int N, int K, int lda,
+                                    int ldw, int ldc, int swiglu, int* status,
+                                    cudaStream_t stream) {
+  return grouped_gemm(A, W, C, offsets, num_groups, total_rows, N, K, lda, ldw, ldc, swiglu, nullptr, 0.f, 0.f, status,
+                      stream);
+}
+
+// The gate / up product of experts: rows scaled by row_scale (fp32 [rows] or null), gate as in b200_gemm_glu_bf16
+B200_API int b200_grouped_gemm_glu_bf16(const void* A, const void* W, void* C, const void* offsets, int num_groups,
+                                        long total_rows, int I, int K, int lda, int ldw, int ldc, const void* row_scale,
+                                        float alpha, float limit, int* status, cudaStream_t stream) {
+  return grouped_gemm(A, W, C, offsets, num_groups, total_rows, I, K, lda, ldw, ldc, 1, row_scale, alpha, limit, status,
+                      stream);
 }
 
 // Fused-MoE expert GEMMs over the packed receive pool of this rank.

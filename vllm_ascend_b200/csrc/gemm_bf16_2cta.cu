@@ -46,6 +46,7 @@ struct Gemm2Params {
   int* status;
   int tiles_m, tiles_n;
   int swiglu;          // W = [gate; up]: tile pairs 128 gate + 128 up columns
+  float glu_alpha, glu_limit;      // alpha > 0: clamped gate instead of SiLU
   int up_row_offset;
   // ---- fused collectives (same protocol as the single-CTA kernel's AG / RS modes)
   int mode;                           // 0, G2_AG or G2_RS
@@ -338,8 +339,14 @@ gemm_bf16_2cta_kernel(const __grid_constant__ CUtensorMap tmap_a,
           tmem_ld_wait();
 #pragma unroll
           for (int j = 0; j < 32; j++) {
-            const float g = __uint_as_float(r[j]) * rstd;
-            r[j] = __float_as_uint(g / (1.f + __expf(-g)) * (__uint_as_float(u[j]) * rstd));
+            float g = __uint_as_float(r[j]) * rstd, up = __uint_as_float(u[j]) * rstd;
+            if (p.glu_alpha > 0.f) {
+              g = fminf(g, p.glu_limit);
+              up = fminf(fmaxf(up, -p.glu_limit), p.glu_limit) + 1.f;
+              r[j] = __float_as_uint(g / (1.f + __expf(-p.glu_alpha * g)) * up);
+            } else {
+              r[j] = __float_as_uint(g / (1.f + __expf(-g)) * up);
+            }
           }
         } else {
           tmem_ld_wait();
@@ -653,6 +660,24 @@ B200_API int b200_gemm_bf16_2cta(const void* A, const void* W, void* C, const vo
   p.C = (__nv_bfloat16*)C;
   p.status = status;
   p.swiglu = swiglu;
+  return launch_2cta(A, W, p, lda, ldw, M, stream);
+}
+
+// C[M, N] = glu(A Wg^T, A Wu^T) with W = [gate (N rows); up (N rows)], N a multiple of 128; alpha 0 the SiLU gate,
+// alpha > 0 the clamped one: min(g, limit) sigmoid(alpha .) (clamp(u, -limit, limit) + 1)
+B200_API int b200_gemm_glu_bf16_2cta(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw,
+                                     int ldc, float alpha, float limit, int* status, cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if ((K & 7) || (lda & 7) || (ldw & 7) || (ldc & 7)) return 9100;
+  if (N % 128) return 9132;
+  Gemm2Params p;
+  memset(&p, 0, sizeof(p));
+  p.M = M; p.N = N; p.K = K; p.ldc = ldc;
+  p.C = (__nv_bfloat16*)C;
+  p.status = status;
+  p.swiglu = 1;
+  p.glu_alpha = alpha;
+  p.glu_limit = limit;
   return launch_2cta(A, W, p, lda, ldw, M, stream);
 }
 

@@ -4,7 +4,7 @@
 //     moe_gating_top_k op, csrc/moe/moe_gating_top_k; signature torch_binding.cpp:2135-2150)
 //   * permute: histogram of tokens per local expert, exclusive offsets, and the gather of
 //     token rows into expert-major order (npu_moe_init_routing_v2 / npu_moe_token_permute)
-//   * combine: weighted sum of the k expert outputs of every token (npu_moe_token_unpermute), where the
+//   * combine: weighted sum (sum, where the inputs were weighted) of the k expert outputs of every token (npu_moe_token_unpermute), where the
 //     output of a shared expert joins, scaled by the sigmoid of a dot product with the layer's input
 // The grouped GEMMs in between are csrc/gemm_bf16.cu (GROUPED mode) and
 // csrc/gemm_fp8_block.cu; moe_linear is the same product on the CUDA cores, for fp32 and for sizes those
@@ -189,6 +189,12 @@ __global__ void moe_assign_kernel(const int* __restrict__ local_ids, int n, int 
   pos[i] = r;
   src_token[r] = i / k;
 }
+// weight of every expert-major row: out[pos[i]] = w[i]
+__global__ void moe_row_weights_kernel(const float* __restrict__ w, const int* __restrict__ pos, int n,
+                                       float* __restrict__ out) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n && pos[i] >= 0) out[pos[i]] = w[i];
+}
 // out[row] = x[src_token[row]] for row < offsets[E]
 __global__ void moe_gather_rows_kernel(const __nv_bfloat16* __restrict__ x,
                                        const int* __restrict__ src_token,
@@ -233,7 +239,7 @@ __global__ void __launch_bounds__(512) moe_combine_kernel(const T* __restrict__ 
     for (int s = 0; s < k; s++) {
       const int r = pos[t * k + s];
       if (r < 0) continue;
-      const float ws = w[t * k + s];
+      const float ws = w ? w[t * k + s] : 1.f;
       load_vec<T, VEC>(y + (long)r * H + c, v);
 #pragma unroll
       for (int e = 0; e < VEC; e++) acc[e] += ws * v[e];
@@ -268,11 +274,13 @@ static int launch_combine(const void* y, const void* pos, const void* w, int tok
 constexpr int ML_TILE = 32;
 
 // Rows [offsets[e], offsets[e + 1]) of a (row r is a[src[r]] with src) meet w[e]: [N, K], or with GLU [2N, K] =
-// gate rows | up rows and out = silu(a gate^T) * (a up^T).  A block computes 32 rows x 32 columns.
+// gate rows | up rows and out = glu(scale a gate^T, scale a up^T) with a factor per row (null: 1).  A block computes
+// 32 rows x 32 columns.
 template <typename T, bool GLU>
 __global__ void __launch_bounds__(256) moe_linear_kernel(const T* __restrict__ a, const int* __restrict__ src,
                                                          const T* __restrict__ w, T* __restrict__ out,
-                                                         const int* __restrict__ offsets, int E, int rows, int N, int K) {
+                                                         const int* __restrict__ offsets, int E, int rows, int N, int K,
+                                                         const float* __restrict__ scale, float alpha, float limit) {
   __shared__ float sa[ML_TILE][ML_TILE + 1], sw[GLU ? 2 : 1][ML_TILE][ML_TILE + 1];
   const int tile = blockIdx.x;
   int lo = 0, hi = E - 1;
@@ -318,21 +326,25 @@ __global__ void __launch_bounds__(256) moe_linear_kernel(const T* __restrict__ a
       const int row = r0 + ty + 16 * i, n = n0 + tx + 16 * j;
       if (row >= r1 || n >= N) continue;
       float v = acc[0][i][j];
-      if constexpr (GLU) v = v / (1.f + expf(-v)) * acc[1][i][j];
+      if constexpr (GLU) {
+        const float f = scale ? scale[row] : 1.f;
+        v = glu_f(v * f, acc[1][i][j] * f, alpha, limit);
+      }
       out[(long)row * N + n] = from_f<T>(v);
     }
 }
 
 template <typename T>
 static int launch_moe_linear(const void* a, const void* src, const void* w, void* out, const void* offsets, int E, int rows,
-                             int N, int K, int swiglu, cudaStream_t stream) {
+                             int N, int K, int swiglu, const void* scale, float alpha, float limit, cudaStream_t stream) {
   const dim3 grid((unsigned)(rows / ML_TILE + E), (unsigned)((N + ML_TILE - 1) / ML_TILE));
   if (swiglu)
     moe_linear_kernel<T, true><<<grid, 256, 0, stream>>>((const T*)a, (const int*)src, (const T*)w, (T*)out,
-                                                         (const int*)offsets, E, rows, N, K);
+                                                         (const int*)offsets, E, rows, N, K, (const float*)scale, alpha,
+                                                         limit);
   else
     moe_linear_kernel<T, false><<<grid, 256, 0, stream>>>((const T*)a, (const int*)src, (const T*)w, (T*)out,
-                                                          (const int*)offsets, E, rows, N, K);
+                                                          (const int*)offsets, E, rows, N, K, nullptr, 0.f, 0.f);
   return B200_CHECK_LAUNCH();
 }
 
@@ -374,6 +386,13 @@ B200_API int b200_moe_permute(const void* local_ids, int T, int k, int E, void* 
   return B200_CHECK_LAUNCH();
 }
 
+// fp32 out[pos[i]] = w[i] for the n (token, slot) pairs of b200_moe_permute
+B200_API int b200_moe_row_weights(const void* w, const void* pos, int n, void* out, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  moe_row_weights_kernel<<<(n + 255) / 256, 256, 0, stream>>>((const float*)w, (const int*)pos, n, (float*)out);
+  return B200_CHECK_LAUNCH();
+}
+
 B200_API int b200_moe_gather_rows(const void* x, const void* src_token, const void* offsets, int E,
                                   int H, int max_rows, void* out, cudaStream_t stream) {
   if (max_rows <= 0) return 0;
@@ -395,11 +414,13 @@ B200_API int b200_moe_combine(const void* y, const void* pos, const void* w, int
                : launch_combine<__nv_bfloat16>(y, pos, w, T, k, H, out, accumulate, shared, x, gate, stream);
 }
 
-// a [*, K], src [rows] or null, w [E, N (2N with swiglu), K], out [rows, N], offsets int32 [E + 1].  dtype: 0 bf16, 1 fp32
+// a [*, K], src [rows] or null, w [E, N (2N with swiglu), K], out [rows, N], offsets int32 [E + 1].  With swiglu: row_scale
+// fp32 [rows] or null, alpha 0 the SiLU gate, else the clamped one.  dtype: 0 bf16, 1 fp32
 B200_API int b200_moe_linear(const void* a, const void* src, const void* w, void* out, const void* offsets, int E, int rows,
-                             int N, int K, int swiglu, int dtype, cudaStream_t stream) {
+                             int N, int K, int swiglu, const void* row_scale, float alpha, float limit, int dtype,
+                             cudaStream_t stream) {
   if (rows <= 0 || E <= 0) return 0;
   if (N < 1 || K < 1) return 9153;
-  return dtype ? launch_moe_linear<float>(a, src, w, out, offsets, E, rows, N, K, swiglu, stream)
-               : launch_moe_linear<__nv_bfloat16>(a, src, w, out, offsets, E, rows, N, K, swiglu, stream);
+  return dtype ? launch_moe_linear<float>(a, src, w, out, offsets, E, rows, N, K, swiglu, row_scale, alpha, limit, stream)
+               : launch_moe_linear<__nv_bfloat16>(a, src, w, out, offsets, E, rows, N, K, swiglu, row_scale, alpha, limit, stream);
 }

@@ -3,7 +3,9 @@
 //   taps - 1 inputs), RMS norm over all heads of q (and of k) at once, interleaved rotary positions on the
 //   first `rot` dimensions of a head, q to a dense buffer, keys and values to their cache slots.
 // The norm may also be head by head with one weight for all heads (qkv_head_kernel, no convolution): a group of
-// lanes owns one head of one token, so no barrier is needed.
+// lanes owns one head of one token, so no barrier is needed.  Or absent, with a factor of the queries by position and
+// wide queries (qkv_spread_kernel): a cache row holds several projected keys side by side, and part c of an output
+// head's query is a weighted sum of the projected queries that go with key part c.
 // The values may be the keys as they were before the norm.  Everything between the projection and the
 // stores is fp32; element type bf16 or fp32 (template), all sizes are run-time values.
 //
@@ -30,6 +32,8 @@ struct QkvPrepArgs {
   void* q_out;                // [T, heads * dim]
   void *k_cache, *v_cache;
   float* sums;                // [T, 2] sums of squares of q and k (phases 1 and 2)
+  const float* mix;           // [out_heads, heads] or null: identity
+  const float* q_scale;       // [q_scale_rows] factor of the queries by position, or null
   long qkv_stride, state_rows, cache_slots;
   long k_block, k_tok, k_head, v_block, v_tok, v_head;      // cache strides in elements
   long tokens;
@@ -40,6 +44,10 @@ struct QkvPrepArgs {
   int phase;                  // 0: all; 1: only the sums; 2: with the given sums
   int dtype;
   int head_norm;              // every head by itself: q_norm, k_norm [dim]
+  int v_heads;
+  int key_parts;              // > 0: qkv_spread_kernel, projected keys per cache row
+  int part_run;               // projected head g goes with key part (g / part_run) % key_parts
+  int out_heads, q_scale_rows;
   float eps;
 };
 
@@ -437,6 +445,128 @@ static int launch_heads(const QkvPrepParams& p, cudaStream_t stream) {
   return B200_CHECK_LAUNCH();
 }
 
+// One block per token.  A warp at a time takes a head: norm (optional), rotary, factor; keys and values go to their
+// cache slots, queries stay in shared memory (fp32) until the wide queries are formed from them.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) qkv_spread_kernel(const QkvPrepParams p) {
+  extern __shared__ __align__(16) float sq[];        // [heads, dim]
+  const long t = blockIdx.x;
+  const int lane = threadIdx.x & 31;
+  const int units = p.heads + p.kv_heads + p.v_heads, half = p.rot >> 1;
+  const T* x = (const T*)p.qkv + t * p.qkv_stride;
+  const long slot = p.slot_mapping[t];
+  const bool stored = slot >= 0 && slot < p.cache_slots;
+  const unsigned blk = stored ? (unsigned)slot / (unsigned)p.block_size : 0;
+  const unsigned off = stored ? (unsigned)slot - blk * p.block_size : 0;
+  const long pos = p.rot > 0 || p.q_scale ? p.positions[t] : 0;
+  const bool cs_ok = pos >= 0 && pos < p.cos_rows, qs_ok = pos >= 0 && pos < p.q_scale_rows;
+  if (threadIdx.x == 0 && p.status &&
+      (slot >= p.cache_slots || (p.rot > 0 && !cs_ok) || (p.q_scale && !qs_ok)))
+    atomicExch(p.status, B200_BAD_INDEX);
+  const float* cs = p.rot > 0 && cs_ok ? p.cos_sin + pos * p.rot : nullptr;
+  const float factor = p.q_scale && qs_ok ? p.q_scale[pos] : 1.f;
+  for (int u = threadIdx.x >> 5; u < units; u += 8) {
+    const int kind = u < p.heads ? 0 : u < p.heads + p.kv_heads ? 1 : 2;                    // q, k, v
+    const int g = kind == 0 ? u : kind == 1 ? u - p.heads : u - p.heads - p.kv_heads;
+    const int dim = kind == 2 ? p.vdim : p.dim;
+    const T* src = x + (kind == 2 ? (long)(p.heads + p.kv_heads) * p.dim + (long)g * p.vdim : (long)u * p.dim);
+    float inv = 1.f;
+    if (kind < 2 && p.head_norm) {
+      float ss = 0.f;
+      for (int c = lane * VEC; c < dim; c += 32 * VEC) {
+        float v[VEC];
+        load_vec<T, VEC>(src + c, v);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) ss = fmaf(v[e], v[e], ss);
+      }
+      inv = 1.f / sqrtf(warp_reduce_sum(ss) / (float)dim + p.eps);
+    }
+    const T* w = p.head_norm ? (const T*)(kind == 0 ? p.q_norm : p.k_norm) : nullptr;
+    T* dst = nullptr;
+    if (kind == 1 && stored)
+      dst = (T*)p.k_cache + blk * p.k_block + off * p.k_tok + g / p.key_parts * p.k_head + (long)(g % p.key_parts) * p.dim;
+    else if (kind == 2 && stored)
+      dst = (T*)p.v_cache + blk * p.v_block + off * p.v_tok + g * p.v_head;
+    for (int b = 0; b < dim; b += 32 * VEC) {        // same trip count for all lanes
+      const int c = b + lane * VEC;
+      float v[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; e++) v[e] = 0.f;
+      if (c < dim) load_vec<T, VEC>(src + c, v);
+      if (kind < 2) {
+        if (w && c < dim) {
+          float wv[VEC];
+          load_vec<T, VEC>(w + c, wv);
+#pragma unroll
+          for (int e = 0; e < VEC; e++) v[e] *= inv * wv[e];
+        }
+        if constexpr (VEC == 1) {
+          if (p.rot > 0) {                           // the partner of a pair sits in the next lane
+            const float other = __shfl_xor_sync(0xffffffffu, v[0], 1);
+            if (cs && c < p.rot) {
+              const float cc = cs[c >> 1], sn = cs[half + (c >> 1)];
+              v[0] = (c & 1) ? v[0] * cc + other * sn : v[0] * cc - other * sn;
+            }
+          }
+        } else if (cs) {
+#pragma unroll
+          for (int e = 0; e < VEC; e += 2)
+            if (c + e < p.rot) {
+              const float cc = cs[(c + e) >> 1], sn = cs[half + ((c + e) >> 1)], a = v[e], bb = v[e + 1];
+              v[e] = a * cc - bb * sn;
+              v[e + 1] = bb * cc + a * sn;
+            }
+        }
+      }
+      if (c >= dim) continue;
+      if (kind == 0) {
+#pragma unroll
+        for (int e = 0; e < VEC; e++) v[e] *= factor;
+        store_vec<float, VEC>(sq + (long)g * p.dim + c, v);
+      } else if (dst) {
+        store_vec<T, VEC>(dst + c, v);
+      }
+    }
+  }
+  __syncthreads();
+  const int per = p.dim / VEC, row = p.key_parts * per, stride = p.part_run * p.key_parts;
+  T* q = (T*)p.q_out + t * p.out_heads * (long)p.key_parts * p.dim;
+  for (int i = threadIdx.x; i < p.out_heads * row; i += 256) {
+    const int oh = i / row, r = i - oh * row, c = r / per, d = (r - c * per) * VEC;
+    float acc[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; e++) acc[e] = 0.f;
+    if (p.mix) {
+      for (int g0 = c * p.part_run; g0 < p.heads; g0 += stride)
+        for (int g = g0; g < min(g0 + p.part_run, p.heads); g++) {
+          const float m = __ldg(p.mix + (long)oh * p.heads + g);
+          float v[VEC];
+          load_vec<float, VEC>(sq + (long)g * p.dim + d, v);
+#pragma unroll
+          for (int e = 0; e < VEC; e++) acc[e] = fmaf(m, v[e], acc[e]);
+        }
+    } else if (oh / p.part_run % p.key_parts == c) {
+      load_vec<float, VEC>(sq + (long)oh * p.dim + d, acc);
+    }
+    store_vec<T, VEC>(q + (long)i * VEC, acc);
+  }
+}
+
+template <typename T, int VEC>
+static int launch_spread(const QkvPrepParams& p, cudaStream_t stream) {
+  const size_t smem = (size_t)p.heads * p.dim * sizeof(float);
+  if (smem > 200 * 1024) return 9822;
+  static bool attr_set = false;
+  if (smem > 48 * 1024 && !attr_set) {
+    const cudaError_t e = cudaFuncSetAttribute(qkv_spread_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    attr_set = true;
+  }
+  if (p.tokens > 0x7fffffffL) return 9823;
+  qkv_spread_kernel<T, VEC><<<(unsigned)p.tokens, 256, smem, stream>>>(p);
+  return B200_CHECK_LAUNCH();
+}
+
 template <typename T, int VEC, int PER>
 static int launch_prep(const QkvPrepParams& p, dim3 grid, int threads, size_t smem, cudaStream_t stream) {
   if (smem > 48 * 1024) return 9820;
@@ -473,6 +603,11 @@ static int prep_t(QkvPrepParams& p, cudaStream_t stream) {
   bool vec = aligned16(p.cos_sin) && aligned16(p.qkv) && aligned16(p.conv_w) && aligned16(p.state) &&
              aligned16(p.q_norm) && aligned16(p.k_norm) && aligned16(p.q_out) && aligned16(p.k_cache) &&
              aligned16(p.v_cache);
+  if (p.key_parts > 0) {
+    bool vec4 = vec;
+    for (long x : s) vec4 = vec4 && x % 4 == 0;
+    return vec4 ? launch_spread<T, 4>(p, stream) : launch_spread<T, 1>(p, stream);
+  }
   for (long x : s) vec = vec && x % V == 0;
   if (p.head_norm) {
     if (!vec) return launch_heads<T, 1, 32>(p, stream);
@@ -512,6 +647,13 @@ B200_API int b200_qkv_prep(const QkvPrepArgs* a, int* status, cudaStream_t strea
   if (a->phase != 0 && !a->sums) return 9805;
   if (a->taps == 1 && !a->cu) return 9806;
   if (a->head_norm && (a->taps || a->phase)) return 9808;
+  if (a->key_parts > 0) {
+    if (a->taps || a->phase || a->values_from_keys || a->v_heads < 1 || a->kv_heads % a->key_parts || a->part_run < 1 ||
+        a->out_heads < 1 || (!a->mix && a->out_heads != a->heads) || (a->head_norm && (!a->q_norm || !a->k_norm)))
+      return 9809;
+  } else if (!a->q_norm || !a->k_norm) {
+    return 9810;
+  }
   QkvPrepParams p;
   static_cast<QkvPrepArgs&>(p) = *a;
   p.status = status;

@@ -10,7 +10,8 @@
 //                      u   = sum_s in[s] x_s (no weights: their sum);  x = norm_next(u)
 //   side_gate        g = gelu_tanh(a) * side_embed[id, slice]    (per-layer token input)
 //   gated_head_norm  o = rms_norm(o) * w * silu(z) per head      (delta-rule read-out)
-// Either norm is a layer norm (weight, bias) or an RMS norm, statistics in fp32.  Activations, weights and
+// Either norm is a layer norm (weight, bias) or an RMS norm (in stream_norm also of equal parts of the row, each by
+// itself), statistics in fp32.  Activations, weights and
 // tables are bf16 or fp32.  The reference fuses add + norm the same way on a 16-bit residual
 // (vllm_ascend/ops/layernorm.py:63-85).
 #include "common.cuh"
@@ -37,6 +38,7 @@ struct StreamParams {
   const void *next_w, *next_b;
   void* x;                // [T, W]
   int W;
+  int post_groups, next_groups;      // RMS norms: equal parts of the row, each by itself
   float eps;
   int* status;
 };
@@ -89,9 +91,66 @@ __device__ __forceinline__ void row_norm(float (&v)[PER][VEC], int kind, const T
   }
 }
 
+constexpr int GROUP_BATCH = 4;         // parts reduced together
+
+// RMS norm of ``groups`` equal parts of the row; a vector lies in one part
 template <typename T, int VEC, int PER>
+__device__ __forceinline__ void row_group_norm(float (&v)[PER][VEC], const T* w, int W, int groups, float eps,
+                                               float (*red)[32]) {
+  const int nvec = W / VEC, per = nvec / groups, warps = (blockDim.x + 31) >> 5;
+  for (int g0 = 0; g0 < groups; g0 += GROUP_BATCH) {
+    float ss[GROUP_BATCH];
+#pragma unroll
+    for (int k = 0; k < GROUP_BATCH; k++) ss[k] = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; i++) {
+      const int c = (int)threadIdx.x + i * (int)blockDim.x;
+      if (c >= nvec) continue;
+      const int k = c / per - g0;
+      float s = 0.f;
+#pragma unroll
+      for (int e = 0; e < VEC; e++) s = fmaf(v[i][e], v[i][e], s);
+#pragma unroll
+      for (int j = 0; j < GROUP_BATCH; j++) ss[j] += j == k ? s : 0.f;
+    }
+#pragma unroll
+    for (int k = 0; k < GROUP_BATCH; k++) ss[k] = warp_reduce_sum(ss[k]);
+    if (warps > 1) {
+      __syncthreads();                 // the previous use of red is over
+      if ((threadIdx.x & 31) == 0)
+#pragma unroll
+        for (int k = 0; k < GROUP_BATCH; k++) red[k][threadIdx.x >> 5] = ss[k];
+      __syncthreads();
+#pragma unroll
+      for (int k = 0; k < GROUP_BATCH; k++)
+        ss[k] = warp_reduce_sum((threadIdx.x & 31) < warps ? red[k][threadIdx.x & 31] : 0.f);
+    }
+    const float n = (float)(per * VEC);
+#pragma unroll
+    for (int i = 0; i < PER; i++) {
+      const int c = (int)threadIdx.x + i * (int)blockDim.x;
+      if (c >= nvec) continue;
+      const int k = c / per - g0;
+      if (k < 0 || k >= GROUP_BATCH) continue;
+      float s = 0.f, wv[VEC];
+#pragma unroll
+      for (int j = 0; j < GROUP_BATCH; j++) s = j == k ? ss[j] : s;
+      const float inv = 1.f / sqrtf(s / n + eps);
+      load_vec<T, VEC>(w + (long)c * VEC, wv);
+#pragma unroll
+      for (int e = 0; e < VEC; e++) v[i][e] = v[i][e] * inv * wv[e];
+    }
+  }
+}
+
+// GROUPED: RMS norms may come in several parts
+template <typename T, int VEC, int PER, bool GROUPED>
 __global__ void stream_norm_kernel(const StreamParams p) {
-  __shared__ float red[32];
+  __shared__ float red[GROUPED ? GROUP_BATCH : 1][32];
+  auto norm = [&](float (&v)[PER][VEC], int kind, const void* w, const void* b, int groups) {
+    if (GROUPED && groups > 1) row_group_norm<T, VEC, PER>(v, (const T*)w, p.W, groups, p.eps, red);
+    else row_norm<T, VEC, PER>(v, kind, (const T*)w, (const T*)b, p.W, p.eps, red[0]);
+  };
   const long t = blockIdx.x;
   const int nvec = p.W / VEC;
   float v[PER][VEC];
@@ -106,8 +165,7 @@ __global__ void stream_norm_kernel(const StreamParams p) {
 #pragma unroll
         for (int e = 0; e < VEC; e++) v[i][e] = 0.f;
     }
-    if (p.post != NORM_PLAIN)
-      row_norm<T, VEC, PER>(v, p.post, (const T*)p.post_w, (const T*)p.post_b, p.W, p.eps, red);
+    if (p.post != NORM_PLAIN) norm(v, p.post, p.post_w, p.post_b, p.post_groups);
   } else {
 #pragma unroll
     for (int i = 0; i < PER; i++)
@@ -139,8 +197,7 @@ __global__ void stream_norm_kernel(const StreamParams p) {
     if (p.post != NORM_NONE || p.emb != EMB_NONE) store_vec<float, VEC>(rrow + (long)c * VEC, v[i]);
   }
   if (p.next == NORM_NONE) return;
-  if (p.next != NORM_PLAIN)
-    row_norm<T, VEC, PER>(v, p.next, (const T*)p.next_w, (const T*)p.next_b, p.W, p.eps, red);
+  if (p.next != NORM_PLAIN) norm(v, p.next, p.next_w, p.next_b, p.next_groups);
   T* xrow = (T*)p.x + t * p.W;
 #pragma unroll
   for (int i = 0; i < PER; i++) {
@@ -340,11 +397,16 @@ static int launch_stream(const StreamParams& p, long tokens, cudaStream_t stream
   if (threads > 1024) threads = 1024;
   const int per = (nvec + threads - 1) / threads;
   const dim3 grid((unsigned)tokens);
-  if (per <= 1) stream_norm_kernel<T, VEC, 1><<<grid, threads, 0, stream>>>(p);
-  else if (per <= 2) stream_norm_kernel<T, VEC, 2><<<grid, threads, 0, stream>>>(p);
-  else if (per <= 4) stream_norm_kernel<T, VEC, 4><<<grid, threads, 0, stream>>>(p);
-  else if (per <= 8) stream_norm_kernel<T, VEC, 8><<<grid, threads, 0, stream>>>(p);
+  const bool grouped = p.post_groups > 1 || p.next_groups > 1;
+#define LAUNCH_STREAM(PER)                                                                    \
+  if (grouped) stream_norm_kernel<T, VEC, PER, true><<<grid, threads, 0, stream>>>(p);        \
+  else stream_norm_kernel<T, VEC, PER, false><<<grid, threads, 0, stream>>>(p)
+  if (per <= 1) { LAUNCH_STREAM(1); }
+  else if (per <= 2) { LAUNCH_STREAM(2); }
+  else if (per <= 4) { LAUNCH_STREAM(4); }
+  else if (per <= 8) { LAUNCH_STREAM(8); }
   else return 9710;
+#undef LAUNCH_STREAM
   return B200_CHECK_LAUNCH();
 }
 
@@ -352,7 +414,7 @@ template <typename T>
 static int stream_norm_t(const StreamParams& p, long tokens, cudaStream_t stream) {
   const bool vec = p.W % 4 == 0 && p.y_stride % 4 == 0 && aligned16(p.r) && aligned16(p.y) && aligned16(p.x) &&
                    aligned16(p.table) && aligned16(p.post_w) && aligned16(p.post_b) && aligned16(p.next_w) &&
-                   aligned16(p.next_b);
+                   aligned16(p.next_b) && p.W / p.post_groups % 4 == 0 && p.W / p.next_groups % 4 == 0;
   return vec ? launch_stream<T, 4>(p, tokens, stream) : launch_stream<T, 1>(p, tokens, stream);
 }
 
@@ -421,14 +483,17 @@ using namespace b200;
 // (post: add y as it is; next: round r to the activation type).  emb: 0 none, 1 set, 2 add.
 B200_API int b200_stream_norm(void* r, const void* y, long y_stride, int post, const void* post_w, const void* post_b,
                               float post_scale, int emb, const void* ids, const void* table, long table_rows, float emb_scale, int next,
-                              const void* next_w, const void* next_b, void* x, long tokens, int W, float eps, int dtype,
-                              int* status, cudaStream_t stream) {
+                              const void* next_w, const void* next_b, void* x, long tokens, int W, int post_groups, int next_groups,
+                              float eps, int dtype, int* status, cudaStream_t stream) {
   if (tokens <= 0) return 0;
+  if (post_groups < 1 || next_groups < 1 || W % post_groups || W % next_groups ||
+      (post_groups > 1 && post != NORM_RMS && post != NORM_NONE) || (next_groups > 1 && next != NORM_RMS && next != NORM_NONE))
+    return 9703;
   if (W < 1 || (post != NORM_NONE && !y) || (next != NORM_NONE && !x) || (emb != EMB_NONE && !table)) return 9700;
   if ((post == NORM_LAYER || post == NORM_RMS) && !post_w) return 9701;
   if ((next == NORM_LAYER || next == NORM_RMS) && !next_w) return 9702;
   StreamParams p{(float*)r, y, y_stride, post, post_w, post_b, post_scale, emb, (const long*)ids, table, table_rows,
-                 emb_scale, next, next_w, next_b, x, W, eps, status};
+                 emb_scale, next, next_w, next_b, x, W, post_groups, next_groups, eps, status};
   return dtype ? stream_norm_t<float>(p, tokens, stream) : stream_norm_t<__nv_bfloat16>(p, tokens, stream);
 }
 

@@ -210,8 +210,8 @@ class ModelRunner:
         total = 0
         for L in self.model.layers:
             a = L.self_attn
-            for shape in self._extra_state_shapes(a):
-                total += math.prod(shape) * torch.empty(0, dtype=self.kv_dtype).element_size()
+            for shape, dtype in self._extra_states(a):
+                total += math.prod(shape) * torch.empty(0, dtype=dtype).element_size()
             if getattr(a, "is_linear_attention", False):
                 cs, ss = a.state_shapes(self.max_seqs + 1)
                 n_c = 1
@@ -223,10 +223,11 @@ class ModelRunner:
                 total += n_c * (4 if self.kv_dtype == torch.float32 else 2) + n_s * 4
         return total
 
-    def _extra_state_shapes(self, attn) -> list:
-        """Per-sequence state (one row per batch row, plus a scratch row for padded graph entries) that an
-        attention layer keeps beside its pages."""
-        return attn.sequence_state_shapes(self.max_seqs + 1) if hasattr(attn, "sequence_state_shapes") else []
+    def _extra_states(self, attn) -> list[tuple[tuple, torch.dtype]]:
+        """(shape, type) of the per-sequence states (one row per batch row, plus a scratch row for padded graph
+        entries) that an attention layer keeps beside its pages; a layer that names no type keeps the caches'."""
+        shapes = attn.sequence_state_shapes(self.max_seqs + 1) if hasattr(attn, "sequence_state_shapes") else []
+        return [s if isinstance(s[0], tuple) else (s, self.kv_dtype) for s in shapes]
 
     def kv_bytes_per_block(self) -> int:
         itemsize = torch.tensor([], dtype=self.kv_dtype).element_size()
@@ -303,7 +304,7 @@ class ModelRunner:
             per_layer.append(shapes)
         layout = self.cfg.cache.kv_layout if self.is_cuda else "NHD"
         self.kv_arena = None
-        if self.cfg.kv_transfer_config and any(self._extra_state_shapes(L.self_attn) for L in self.model.layers):
+        if self.cfg.kv_transfer_config and any(self._extra_states(L.self_attn) for L in self.model.layers):
             raise NotImplementedError("KV transfer of layers that keep a state beside their pages")
         if self.cfg.kv_transfer_config and any(getattr(L.self_attn, "kv_from", None) is not None for L in self.model.layers):
             raise NotImplementedError("KV transfer of layers that read another layer's cache")
@@ -338,8 +339,8 @@ class ModelRunner:
             self.kv_caches.append(tuple(
                 ops.alloc_kv_cache(s[0], s[1], s[2], s[3], self.kv_dtype, self.device, layout,
                                    arena=self.kv_arena)
-                for s in shapes) + tuple(torch.zeros(s, dtype=self.kv_dtype, device=self.device)
-                                         for s in self._extra_state_shapes(layer.self_attn)))
+                for s in shapes) + tuple(torch.zeros(s, dtype=t, device=self.device)
+                                         for s, t in self._extra_states(layer.self_attn)))
 
     # ------------------------------------------------------------------ persistent batch
     def _offload_cfg(self):

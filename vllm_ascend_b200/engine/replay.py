@@ -53,6 +53,8 @@ class TraceReplayer:
         for rid in end:
             req = self.live.pop(rid, None)
             if req is not None:
+                if req.row >= 0:             # the id may come back with other tokens
+                    self.runner.row_owner[req.row] = None
                 self.scheduler.abort_request(rid)
                 self.scheduler.requests.pop(rid, None)
         return logits

@@ -4,9 +4,10 @@ Most configurations give one set of sizes for all layers.  A *plan* gives every 
 it has, the mixer's sizes and constants, and whether a feed-forward follows.  It is kept on
 ``ModelConfig.layer_plan`` as a list of ``{"mixer": kind, "mlp": bool, "over": {...}}`` where ``over`` holds
 ``ModelConfig`` fields of that layer (``ModelConfig.layer_config(i)`` applies them), so that the mixers read
-a plain ``ModelConfig`` whether or not the model has a plan.
+a plain ``ModelConfig`` whether or not the model has a plan.  ``"weights_of": j`` marks a layer that runs with
+layer j's parameters and a cache or state of its own.
 
-This module turns the configuration formats of the Vofelix, Pegopel and Dubizen decoders into such plans."""
+This module turns the configuration formats of the Vofelix, Pegopel, Dubizen and Nevotar decoders into such plans."""
 from __future__ import annotations
 
 from typing import Any, Callable, Optional
@@ -87,6 +88,41 @@ _DUBIZEN_MIXERS: dict[str, tuple[str, Callable[[dict], dict]]] = {
     "attention": ("attention", _normed), "latent_attention": ("latent", _latent_query)}
 
 
+def _rotated(rot: dict, dim: int) -> dict:
+    if int(rot["dims"]) % 2 or not 0 <= int(rot["dims"]) <= dim:
+        raise ValueError(f"cannot rotate {rot['dims']} of {dim} dimensions")
+    return dict(rotary_dims=int(rot["dims"]), rope_theta=float(rot["base"]), rope_half_split=True)
+
+
+def _map_difference(m: dict) -> dict:
+    temp = m.get("q_temp")
+    if temp and int(temp["every"]) != temp["every"]:
+        raise ValueError("the query temperature changes every whole number of positions")
+    return dict(_attention(m), qk_norm_full=False, attention_bias=True, attn_map_diff=float(m["diff"]),
+                attn_query_temp=(float(temp["coef"]), int(temp["every"])) if temp else None)
+
+
+def _attention_and_state(m: dict) -> dict:
+    left, right = m["left"], m["right"]
+    heads, groups, parts = int(right["heads"]), int(right["groups"]), int(right["norm_groups"])
+    if groups < 1 or heads % groups or parts < 1 or heads * int(right["vdim"]) % parts:
+        raise ValueError(f"{heads} state-space heads do not divide into {groups} groups and {parts} norms")
+    return dict(_attention(left), **_rotated(left["rot"], int(left["dim"])), qk_norm_full=False, qk_norm=True,
+                attention_bias=True, attn_talk=True, parallel_scales=(float(m["left_scale"]), float(m["right_scale"])),
+                mamba_config={"n_heads": heads, "d_head": int(right["vdim"]), "n_groups": groups, "d_state": int(right["state"]),
+                              "d_conv": int(right["conv"]), "norm_groups": parts})
+
+
+def _forget(m: dict) -> dict:
+    return dict(linear_num_key_heads=int(m["heads"]), linear_num_value_heads=int(m["heads"]),
+                linear_key_head_dim=int(m["dim"]), linear_value_head_dim=int(m["vdim"]))
+
+
+_NEVOTAR_MIXERS: dict[str, tuple[str, Callable[[dict], dict]]] = {
+    "attention": ("attention", _map_difference), "parallel": ("parallel", _attention_and_state),
+    "hgrn2": ("hgrn2", _forget)}
+
+
 # ---------------------------------------------------------------- feed-forwards
 def _gated_mlp(m: dict) -> dict:
     return dict(intermediate_size=int(m["ff"]))
@@ -108,6 +144,17 @@ def _experts(m: dict) -> dict:
                 shared_expert_intermediate_size=int(shared["ff"]) if shared else 0, shared_expert_gate=bool(shared))
 
 
+def _clamped_experts(m: dict) -> dict:
+    router, shared = m["router"], m.get("shared")
+    experts, top = int(router["experts"]), int(router["top"])
+    if not 1 <= top <= experts:
+        raise ValueError(f"cannot choose {top} of {experts} experts")
+    return dict(num_experts=experts, num_experts_per_tok=top, moe_intermediate_size=int(m["expert"]["ff"]),
+                expert_limit=float(m["expert"]["limit"]), scoring_func="sigmoid", norm_topk_prob=False, router_fp32=True,
+                moe_weight_input=True, shared_expert_intermediate_size=int(shared["ff"]) if shared else 0,
+                shared_expert_limit=float(shared["limit"]) if shared else None)
+
+
 _DENSE = {"dense": _gated_mlp}
 
 
@@ -126,6 +173,25 @@ def _read_layers(d: dict, mixers: dict, mlps: dict = _DENSE) -> list[dict]:
             over.update(mlps[kind](mlp))
         plan.append({"mixer": mixer, "mlp": mlp is not None, "over": over})
     return plan
+
+
+def _share_weights(d: dict, plan: list) -> None:
+    """Mark the layers that run with another layer's parameters; a chain ends at the layer that has them."""
+    source = {i: int(layer["weights_of"]) for i, layer in enumerate(d["layers"]) if layer.get("weights_of") is not None}
+    for i in source:
+        j, seen = i, {i}
+        while j in source:
+            j = source[j]
+            if not 0 <= j < len(plan) or j in seen:
+                raise ValueError(f"layer {i}: no layer has the weights it names")
+            seen.add(j)
+        if plan[i] != plan[j]:
+            raise ValueError(f"layer {i} is not of the form of layer {j}, whose weights it uses")
+    for i in source:
+        j = i
+        while j in source:
+            j = source[j]
+        plan[i]["weights_of"] = j
 
 
 def _read_loop(d: dict, num_layers: int) -> Optional[tuple]:
@@ -204,9 +270,29 @@ def dubizen_fields(d: dict) -> dict[str, Any]:
     return fields
 
 
+def nevotar_fields(d: dict) -> dict[str, Any]:
+    """``ModelConfig`` fields of a Nevotar configuration."""
+    plan = _read_layers(d, _NEVOTAR_MIXERS, {"moe": _clamped_experts})
+    _share_weights(d, plan)
+    kinds = ["linear_attention" if p["mixer"] == "hgrn2" else "full_attention" for p in plan]
+    width, groups = int(d["width"]), int(d["norm"].get("groups", 1))
+    if groups < 1 or width % groups:
+        raise ValueError(f"a width of {width} does not divide into {groups} norm groups")
+    heads = _largest(plan, "num_attention_heads", 0) or _largest(plan, "linear_num_value_heads", 1)
+    fields: dict[str, Any] = dict(
+        vocab_size=int(d["vocab"]), hidden_size=width, num_hidden_layers=len(plan), layer_plan=plan, layer_types=kinds,
+        full_attention_interval=2 if "linear_attention" in kinds else 0, num_attention_heads=heads,
+        num_key_value_heads=_largest(plan, "num_key_value_heads", 0) or heads, intermediate_size=width, norm_type="rms",
+        norm_groups=groups, rms_norm_eps=float(d["norm"]["eps"]), tie_word_embeddings=True)
+    for name in ("head_dim", "v_head_dim", "linear_num_key_heads", "linear_num_value_heads", "linear_key_head_dim",
+                 "linear_value_head_dim", "num_experts", "num_experts_per_tok", "moe_intermediate_size"):
+        fields[name] = _largest(plan, name, 0)
+    return fields
+
+
 #: architecture name -> reader of its configuration format
 PLAN_FORMATS: dict[str, Callable[[dict], dict]] = {"Vofelix": vofelix_fields, "Pegopel": pegopel_fields,
-                                                   "Dubizen": dubizen_fields}
+                                                   "Dubizen": dubizen_fields, "Nevotar": nevotar_fields}
 
 
 def run_order(num_layers: int, loop: Optional[tuple]) -> tuple[list[int], set[int]]:

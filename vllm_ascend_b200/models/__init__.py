@@ -33,7 +33,7 @@ def _planned_lm(cfg, device, **kw):
     return PlannedCausalLM(cfg, device, **kw)
 
 
-for _arch in ("Vofelix", "Pegopel", "Dubizen"):
+for _arch in ("Vofelix", "Pegopel", "Dubizen", "Nevotar"):
     register_model(_arch, _planned_lm)
 
 

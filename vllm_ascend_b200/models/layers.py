@@ -477,10 +477,11 @@ class SwiGLUMLP:
     """Gated MLP: act(x W_gate) * (x W_up) -> W_down; SiLU (fused into the GEMM epilogue) or GELU gates."""
 
     def __init__(self, pf: ParamFactory, prefix: str, hidden: int, inter: int, comm: TPComm,
-                 reduce_results: bool = True, act: str = "silu"):
+                 reduce_results: bool = True, act: str = "silu", limit: Optional[float] = None):
         if act not in _GATED_ACTS:
             raise ValueError(f"unsupported MLP activation {act!r}")
         self.act = _GATED_ACTS[act]
+        self.limit = limit               # clamped gate (with act "silu"): ``ops.linear_swiglu``
         self.gate_up_proj = ColumnParallelLinear(pf, f"{prefix}.gate_up_proj", hidden,
                                                  [inter, inter], comm)
         self.down_proj = RowParallelLinear(pf, f"{prefix}.down_proj", inter, hidden, comm,
@@ -490,6 +491,10 @@ class SwiGLUMLP:
         gu = self.gate_up_proj
         if self.act is not None:
             return self.down_proj(ops.activation(gu(x).contiguous(), self.act, gated=True))
+        if self.limit is not None:
+            if gu.quant is not None or gu._lora_on():
+                raise NotImplementedError("the clamped gate takes plain projections")
+            return self.down_proj(ops.linear_swiglu(x, gu.weight, limit=self.limit))
         if gu.quant is None and gu.bias is None and not gu.gather_output and not gu._lora_on() \
                 and _plan().enabled("gemm_swiglu"):
             return self.down_proj(ops.linear_swiglu(x, gu.weight))

@@ -6,27 +6,28 @@ Per token: one input projection to [z | x | B | C | dt]; a short causal convolut
     S_t = exp(dt_t A_h) S_{t-1} + B_t (dt_t x_t)^T          y_t = S_t^T C_t + D_h x_t
 
 with dt = softplus(dt + dt_bias) clamped to the configured limits, A_h = -exp(A_log_h), and B, C
-shared by the heads of a group; RMSNorm of y * silu(z) over the whole inner width; output projection.
-The recurrence is gated linear attention with q = C, k = B, v = dt x and log-decay dt A
-(state-space duality), so prefill chunks run in the chunk-parallel form and decode rows in one
-batched state update (``ops.linear_attn.gated_linear_attention``).  Instead of a KV cache the
-layer keeps, per sequence, the last K-1 convolution inputs and the [N x P] state per head.
+shared by the heads of a group; RMSNorm of y * silu(z) over the whole inner width or over equal parts of it
+(``norm_groups``); output projection.  The recurrence is gated linear attention with q = C, k = B, v = dt x and
+log-decay dt A (``ops.linear_recurrence.state_space``).  Instead of a KV cache the layer keeps, per sequence, the last K-1 convolution inputs and the [N x P] state per head.
 
 Heads are sharded over TP.  Groups are sharded when there are at least as many as ranks, otherwise
 each rank keeps the one group its heads belong to (its B / C columns are computed redundantly).
-The mean square of the gated norm is all-reduced.  Role of the Mamba layers the reference runs
+The mean squares of the gated norm are all-reduced where a part spans ranks.  Role of the Mamba layers the reference runs
 through vLLM's hybrid models (vllm_ascend/patch/platform/patch_mamba_config.py: state page sizing;
 vllm_ascend/ops/triton/mamba/causal_conv1d.py: the convolution; hybrid KV + state transfer in
 vllm_ascend/distributed/kv_transfer/kv_p2p/mooncake_hybrid_connector.py).
 """
 from __future__ import annotations
 
+from typing import Optional
+
 import torch
 import torch.nn.functional as F
 
 from ..config import ModelConfig
 from ..ops import linear_attn as la
-from .layers import ColumnParallelLinear, ParamFactory, RowParallelLinear, TPComm
+from ..ops.linear_recurrence import StateSpace, group_norm, state_space
+from .layers import ColumnParallelLinear, ParamFactory, RowParallelLinear, TPComm, copy_exact
 
 
 class Mamba2Mixer:
@@ -50,6 +51,9 @@ class Mamba2Mixer:
         self.conv_dim = self.I + 2 * self.G * self.N
         self.dt_limit = tuple(float(x) for x in m.get("time_step_limit", (0.0, float("inf"))))
         self.eps = cfg.rms_norm_eps
+        self.norm_groups = int(m.get("norm_groups", 1))         # of the whole model
+        if self.I_total % self.norm_groups:
+            raise ValueError(f"Mamba-2 layer: an inner width of {self.I_total} in {self.norm_groups} norm groups")
         p = f"model.layers.{layer_idx}.mamba"
         gn_virtual = self.G * self.N * tp                        # so that a rank's share is its G groups
         self.in_proj = ColumnParallelLinear(pf, f"{p}.in_proj", cfg.hidden_size,
@@ -63,40 +67,36 @@ class Mamba2Mixer:
         self.A_log = pf.normal(f"{p}.A_log", (self.H_total,), 0, r, tp, std=0.5, dtype=torch.float32)
         self.D = pf.ones((self.H,), dtype=torch.float32)
         self.norm_weight = pf.ones((self.I,))
-        self.chunk = int(m.get("chunk_size", 64)) if int(m.get("chunk_size", 64)) <= 128 else 64
+        chunk = int(m.get("chunk_size", 64))
+        self.space = StateSpace(self.A_log, self.dt_bias, self.D, self.G, self.dt_limit, chunk if chunk <= 128 else 64)
 
     def state_shapes(self, num_slots: int):
         """(conv state, recurrent state) shapes for ``num_slots`` sequences."""
         return (num_slots, self.K - 1, self.conv_dim), (num_slots, self.H, self.N, self.P)
 
     def __call__(self, x: torch.Tensor, meta, cache) -> torch.Tensor:
-        conv_state, ssm_state = cache
-        T = x.shape[0]
-        proj = self.in_proj(x)
-        I, GN = self.I, self.G * self.N
-        z = proj[:, :I]
-        xbc = proj[:, I:I + self.conv_dim]
-        dt = proj[:, I + self.conv_dim:]
+        return self.out_proj(self.mix(self.in_proj(x), meta, *cache))
+
+    def mix(self, proj: torch.Tensor, meta, conv_state: torch.Tensor, ssm_state: torch.Tensor, scale: float = 1.0,
+            out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """What lies between the two projections: rows [z | x | B | C | dt] -> ``scale`` times the normed read-out
+        [T, I]."""
+        I, C = self.I, self.conv_dim
+        z, xbc, dt = proj[:, :I], proj[:, I:I + C], proj[:, I + C:I + C + self.H]
         cu, slots, has_init = meta.query_start_loc, meta.state_slots, meta.has_initial_state
-        xbc = la.causal_conv1d(xbc.contiguous(), self.conv_weight, self.conv_bias, conv_state, cu, slots, has_init,
-                               act=True)
-        xs = xbc[:, :I].reshape(T, self.H, self.P)
-        B = xbc[:, I:I + GN].reshape(T, self.G, self.N)
-        C = xbc[:, I + GN:].reshape(T, self.G, self.N)
-        dt = F.softplus(dt.float() + self.dt_bias)
-        dt = torch.clamp(dt, self.dt_limit[0], self.dt_limit[1])
-        g = dt * (-torch.exp(self.A_log))                                   # [T, H] log-decay
-        v = xs.float() * dt.unsqueeze(-1)
-        y = la.gated_linear_attention(C, B, v, g, ssm_state, cu, slots, has_init,
-                                      cu_cpu=meta.query_start_loc_cpu, chunk=self.chunk)
-        y = y + self.D.view(1, self.H, 1) * xs.float()
-        # gated RMSNorm over the whole inner width (all ranks' heads)
-        h = y.reshape(T, I) * F.silu(z.float())
-        ss = (h * h).sum(-1, keepdim=True)
-        if self.comm.size > 1:
-            ss = self.comm.group.all_reduce(ss)
-        h = (h * torch.rsqrt(ss / self.I_total + self.eps)).to(x.dtype) * self.norm_weight
-        return self.out_proj(h)
+        uniform = meta.max_query_len <= 1
+        xbc = la.causal_conv1d(xbc, self.conv_weight, self.conv_bias, conv_state, cu, slots, has_init, act=True,
+                               uniform=uniform)
+        y = state_space(self.space, xbc, dt, ssm_state, cu, slots, has_init, meta.query_start_loc_cpu, uniform)
+        if self.norm_groups % self.comm.size == 0:               # every part of the norm lies on one rank
+            return group_norm(y, self.norm_weight, self.norm_groups // self.comm.size, self.eps, z, scale, out)
+        h = y.float() * F.silu(z.float())
+        size = self.I_total // self.norm_groups
+        part = (self.comm.rank * I + torch.arange(I, device=h.device)) // size
+        ss = torch.zeros(h.shape[0], self.norm_groups, device=h.device).index_add_(1, part, h * h)
+        inv = torch.rsqrt(self.comm.group.all_reduce(ss) / size + self.eps)
+        h = (h * inv[:, part] * self.norm_weight.float() * scale).to(proj.dtype)
+        return h if out is None else out.copy_(h)
 
     # ------------------------------------------------------------------ checkpoints
     def _rows(self, tp: int, r: int):
@@ -130,6 +130,32 @@ class Mamba2Mixer:
         else:
             return False
         return True
+
+    def parts(self) -> list[str]:
+        return ["in", "conv", "conv.b", "dt_bias", "A_log", "D", "norm", "o"]
+
+    def load_part(self, part: str, w: torch.Tensor) -> None:
+        """One un-fused tensor: in (rows z, x, B, C, dt), conv and its bias, dt_bias, A_log, D, norm, o."""
+        tp, r = self.comm.size, self.comm.rank
+        whole = {"in": (2 * self.I_total + 2 * self.G_total * self.N + self.H_total, self.cfg.hidden_size),
+                 "conv": (self.I_total + 2 * self.G_total * self.N, self.K), "dt_bias": (self.H_total,), "A_log": (self.H_total,),
+                 "D": (self.H_total,), "norm": (self.I_total,), "o": (self.cfg.hidden_size, self.I_total)}
+        whole["conv.b"] = whole["conv"][:1]
+        if part not in whole:
+            raise KeyError(part)
+        if tuple(w.shape) != whole[part]:
+            raise ValueError(f"tensor {part}: expected shape {whole[part]}, found {tuple(w.shape)}")
+        if part == "o":
+            return copy_exact(self.out_proj.weight, w[:, r * self.I:(r + 1) * self.I], part)
+        if part == "norm":
+            return copy_exact(self.norm_weight, w[r * self.I:(r + 1) * self.I], part)
+        if part in ("dt_bias", "A_log", "D"):
+            return copy_exact(getattr(self, part), w[r * self.H:(r + 1) * self.H], part)
+        rows = self._rows(tp, r)
+        if part == "in":
+            return copy_exact(self.in_proj.weight, torch.cat([w[a:a + n] for a, n in rows]), part)
+        dst = self.conv_weight if part == "conv" else self.conv_bias
+        return copy_exact(dst, torch.cat([w[a - self.I_total:a - self.I_total + n] for a, n in rows[1:4]]), part)
 
     def named_tensors(self):
         for attr in ("in_proj", "out_proj"):

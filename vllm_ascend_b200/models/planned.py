@@ -8,16 +8,19 @@ What the plan's layers have in common:
 * with ``residual_streams`` there are several parallel streams per token, mixed by learned weights at every
   sub-layer (``ops.stream.stream_mix``);
 * mixers are the framework's: latent attention (``MLAAttention`` with window and sink, or over another layer's
-  latents), the gated delta rule (``GatedDeltaNet``) and paged attention with options (``VariantAttention``); so
+  latents), the gated delta rule (``GatedDeltaNet``), paged attention with options (``VariantAttention``), HGRN2
+  (``HGRN2Mixer``) and attention beside a Mamba-2 state space (``ParallelMixer``); so
   are the feed-forwards (gated, plain, mixture of experts); each is built from ``ModelConfig.layer_config(i)``;
 * optional learned positions (``learned_positions``): a vector per position added to the embeddings;
 * optional per-layer token input (``token_side_dim``): a slice of a second embedding table, gated by the
   stream, projected, RMS-normed and added after the layer's sub-layers;
 * optional loop (``layer_loop``): some layers run several times with the same weights; with
-  ``layer_loop_refeed`` the embedding output is added to the stream again before each pass but the first.
+  ``layer_loop_refeed`` the embedding output is added to the stream again before each pass but the first;
+* layers that use another layer's parameters (``weights_of`` of a plan's entry).
 
-``layers`` lists the layer *runs* in execution order: a looped layer appears once per pass, so every pass
-has its own entry in the runner's cache list while the parameters are shared.
+``layers`` lists the layer *runs* in execution order: a looped layer appears once per pass, and the layer whose
+parameters others use once for each of them, so every run has its own entry in the runner's cache list while the
+parameters are shared.
 """
 from __future__ import annotations
 
@@ -30,8 +33,10 @@ from ..layer_plan import run_order
 from ..ops.stream import PLAIN, NormSpec, StreamMix, side_gate, stream_mix, stream_norm
 from ..parallel import state as pstate
 from .gdn import GatedDeltaNet
+from .hgrn2 import HGRN2Mixer
 from .layers import (Linear, ParallelLMHead, ParamFactory, PlainMLP, SwiGLUMLP, TPComm, VocabParallelEmbedding,
                      copy_exact)
+from .parallel_mixer import ParallelMixer
 from .transformer import MLAAttention, SparseMoeBlock
 from .variant_attention import VariantAttention
 
@@ -40,6 +45,8 @@ MIXERS = {
     "latent": lambda pf, cfg, i, comm, max_pos: MLAAttention(pf, cfg, i, comm, max_pos),
     "delta": lambda pf, cfg, i, comm, max_pos: GatedDeltaNet(pf, cfg, i, comm),
     "attention": lambda pf, cfg, i, comm, max_pos: VariantAttention(pf, cfg, i, comm, max_pos),
+    "parallel": lambda pf, cfg, i, comm, max_pos: ParallelMixer(pf, cfg, i, comm, max_pos),
+    "hgrn2": lambda pf, cfg, i, comm, max_pos: HGRN2Mixer(pf, cfg, i, comm),
 }
 
 
@@ -50,7 +57,8 @@ _MIX_PARTS = {"in": "read", "out": "write", "mix": "mix"}
 def _norm(pf: ParamFactory, cfg: ModelConfig, kind: Optional[str] = None) -> NormSpec:
     kind = kind or cfg.norm_type
     bias = kind == "layer" and cfg.norm_bias
-    return NormSpec(kind, pf.ones((cfg.hidden_size,)), pf.zeros((cfg.hidden_size,)) if bias else None)
+    return NormSpec(kind, pf.ones((cfg.hidden_size,)), pf.zeros((cfg.hidden_size,)) if bias else None,
+                    cfg.norm_groups if kind == "rms" else 1)
 
 
 def _feed_forward(pf: ParamFactory, lcfg: ModelConfig, idx: int, comm: TPComm, ep_group, moe_runtime):
@@ -92,8 +100,9 @@ class PlannedLayer:
     def __init__(self, pf: ParamFactory, cfg: ModelConfig, idx: int, comm: TPComm, max_pos: int,
                  side_table: Optional[torch.Tensor], ep_group=None, moe_runtime=None):
         entry, lcfg = cfg.layer_plan[idx], cfg.layer_config(idx)
-        heads = lcfg.linear_num_key_heads if entry["mixer"] == "delta" else lcfg.num_attention_heads
-        if heads % comm.size or (entry["mixer"] == "delta" and lcfg.linear_num_value_heads % comm.size):
+        linear = entry["mixer"] in ("delta", "hgrn2")
+        heads = lcfg.linear_num_key_heads if linear else lcfg.num_attention_heads
+        if heads % comm.size or (linear and lcfg.linear_num_value_heads % comm.size):
             raise ValueError(f"layer {idx}: heads do not divide over {comm.size} tensor-parallel ranks")
         self.idx = idx
         self.self_attn = MIXERS[entry["mixer"]](pf, lcfg, idx, comm, max_pos)
@@ -160,11 +169,14 @@ class PlannedCausalLM:
                      for c in map(cfg.layer_config, range(cfg.num_hidden_layers)) if c.is_moe}
             if len(sizes) > 1:
                 raise NotImplementedError("expert parallelism takes layers whose experts are alike")
-        self.unique_layers = [PlannedLayer(pf, cfg, i, self.comm, max_pos, self.side_embed, ep_group, moe_runtime)
-                              for i in range(cfg.num_hidden_layers)]
+        owner = [entry.get("weights_of", i) for i, entry in enumerate(cfg.layer_plan)]
+        own = {i: PlannedLayer(pf, cfg, i, self.comm, max_pos, self.side_embed, ep_group, moe_runtime)
+               for i in sorted(set(owner))}
+        self.unique_layers = list(own.values())
         order, again = run_order(cfg.num_hidden_layers, cfg.layer_loop)
         self.fed_again = again if cfg.layer_loop_refeed else set()
-        self.layers = [self.unique_layers[i] for i in order]
+        self.layers = [own[owner[i]] for i in order]
+        self._layer_of = own
         self.norm = _norm(pf, cfg)
         if cfg.residual_streams and (cfg.token_side_dim or self.fed_again):
             raise NotImplementedError("parallel streams take neither a token side input nor a second embedding feed")
@@ -258,17 +270,18 @@ class PlannedCausalLM:
             for name, m in L.mixes().items():
                 for n in m.__slots__:
                     yield f"{p}.{name}.{n}", getattr(m, n)
-            if isinstance(a, VariantAttention):
+            whole = (VariantAttention, ParallelMixer, HGRN2Mixer)      # list all of their tensors themselves
+            if isinstance(a, whole):
                 for n, t in a.named_tensors():
                     yield f"{p}.self_attn.{n}", t
-            for attr in () if isinstance(a, VariantAttention) else (
+            for attr in () if isinstance(a, whole) else (
                     "in_proj_qkvz", "in_proj_ba", "out_proj", "q_proj", "q_a_proj", "q_b_proj", "kv_a_proj", "kv_b_proj",
                     "o_proj"):
                 lin = getattr(a, attr, None)
                 if isinstance(lin, Linear):
                     for n, t in lin.named_tensors():
                         yield f"{p}.self_attn.{attr}.{n}", t
-            if getattr(a, "is_linear_attention", False):
+            if isinstance(a, GatedDeltaNet):
                 for n, t in a.named_tensors():
                     yield f"{p}.self_attn.{n}", t
             elif isinstance(a, MLAAttention):
@@ -357,7 +370,7 @@ class PlannedCausalLM:
         if name.startswith("final.norm"):
             return norm(self.norm, name[len("final.norm."):])
         layer, _, rest = name.partition(".")
-        L = self.unique_layers[int(layer[1:])]
+        L = self._layer_of[int(layer[1:])]
         group, _, part = rest.partition(".")
         if group == "mix":
             return L.self_attn.load_part(part, w)

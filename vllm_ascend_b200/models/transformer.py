@@ -61,6 +61,11 @@ class SparseMoeBlock:
             self.w2 = pf.normal(f"{prefix}.experts.w2", (E, H, I), 2, r, tp)
             self.expert_map = None
         self.quant = None
+        #: how an expert computes, as ``fused_moe.fused_experts`` takes it
+        self.expert_form = {"limit": cfg.expert_limit, "weight_input": cfg.moe_weight_input}
+        if (cfg.expert_limit is not None or cfg.moe_weight_input) and getattr(moe_runtime, "fused", None) is not None:
+            raise NotImplementedError("the fused expert-parallel kernels take SiLU gates and weighted outputs "
+                                      "(enable_fused_moe_comm=False)")
         self.shared = None
         self.shared_gate_weight = None
         shared_inter = cfg.shared_expert_intermediate_size or I * cfg.n_shared_experts
@@ -71,7 +76,8 @@ class SparseMoeBlock:
             # replicated shared-expert weights: every rank holds the whole MLP and runs part of the rows
             self.shared_replicated = bool(get_b200_config().enable_shared_expert_dp) and comm.size > 1
             s_comm = TPComm(pstate.single_rank_group()) if self.shared_replicated else comm
-            self.shared = SwiGLUMLP(pf, f"{prefix}.shared_experts", H, shared_inter, s_comm, reduce_results=False)
+            self.shared = SwiGLUMLP(pf, f"{prefix}.shared_experts", H, shared_inter, s_comm, reduce_results=False,
+                                    limit=cfg.shared_expert_limit)
             if cfg.shared_expert_gate:           # Qwen2-MoE / Qwen3-Next: sigmoid(x . w) scales the shared expert
                 self.shared_gate_weight = pf.normal(f"{prefix}.shared_expert_gate", (1, H))
             self.shared_exec = SharedExperts(self.shared, comm, self.shared_replicated, self.shared_gate_weight)
@@ -137,10 +143,10 @@ class SparseMoeBlock:
         elif x.is_cuda and self.ep is None and self.quant is None and self.shared is not None and not self.shared_replicated:
             # the shared expert joins where the routed experts' rows are summed
             y = fused_moe.fused_experts(x, self.w13, self.w2, w, ids, self.expert_map, shared=self.shared(x),
-                                        shared_gate=self.shared_gate_weight)
+                                        shared_gate=self.shared_gate_weight, **self.expert_form)
             return self.comm.all_reduce(y) if self.comm.size > 1 else y
         else:
-            y = fused_moe.fused_experts(x, self.w13, self.w2, w, ids, self.expert_map, self.quant)
+            y = fused_moe.fused_experts(x, self.w13, self.w2, w, ids, self.expert_map, self.quant, **self.expert_form)
         replicated = self.shared is not None and self.shared_replicated
         if self.ep is None:
             # TP-sharded experts (and shared experts) hold partial sums: one reduction

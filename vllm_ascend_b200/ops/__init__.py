@@ -264,16 +264,23 @@ def linear_norm_folded(x: torch.Tensor, weight: torch.Tensor, bias: Optional[tor
     return out
 
 
+#: factor inside the sigmoid of the clamped gate
+CLAMPED_GATE_ALPHA = 1.702
+
+
 def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Tensor] = None,
-                  two_cta: bool = False) -> torch.Tensor:
+                  two_cta: bool = False, limit: Optional[float] = None) -> torch.Tensor:
     """silu(x @ Wg^T) * (x @ Wu^T) with weight = [Wg; Wu] ([2I, K]) in one GEMM: the tile pairs
     128 gate columns with the matching 128 up columns and the epilogue applies SiLU-mul
-    (the reference fuses the same pair in its grouped-matmul+swiglu op, csrc/gmm)."""
+    (the reference fuses the same pair in its grouped-matmul+swiglu op, csrc/gmm).  ``limit``: the clamped gate
+    ("swiglu_oai" of ``activation``) instead of SiLU."""
     I = weight.shape[0] // 2
     K = x.shape[-1]
     if not (_use_native(x) and weight.dtype == _BF16 and I % 8 == 0 and K % 8 == 0
             and envs.VLLM_B200_GEMM != "cublas"):
-        return silu_and_mul(linear(x, weight))
+        y = linear(x, weight)
+        return silu_and_mul(y) if limit is None else activation(y.contiguous(), "swiglu_oai", True, CLAMPED_GATE_ALPHA, limit)
+    alpha, limit = (0.0, 0.0) if limit is None else (CLAMPED_GATE_ALPHA, float(limit))
     x2 = x.reshape(-1, K)
     if x2.stride(-1) != 1 or (x2.stride(0) % 8) != 0:
         x2 = x2.contiguous()
@@ -282,17 +289,15 @@ def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Ten
         out = torch.empty((M, I), dtype=x.dtype, device=x.device)
     min2 = envs.VLLM_B200_GEMM_2CTA_MIN_M
     if M > 0 and I % 128 == 0 and (two_cta or (min2 > 0 and M >= min2)):
-        rc = _native.lib().b200_gemm_bf16_2cta(
-            x2.data_ptr(), weight.data_ptr(), out.data_ptr(), None, None, M, I, K, x2.stride(0),
-            weight.stride(0), out.stride(0), 1, _native.status_word(x.device).data_ptr(),
-            _native.stream_ptr())
+        rc = _native.lib().b200_gemm_glu_bf16_2cta(
+            x2.data_ptr(), weight.data_ptr(), out.data_ptr(), M, I, K, x2.stride(0), weight.stride(0), out.stride(0),
+            alpha, limit, _native.status_word(x.device).data_ptr(), _native.stream_ptr())
         _native.check(rc, "gemm_swiglu_2cta")
         launch_counter[0] += 1
     elif M > 0:
-        rc = _native.lib().b200_gemm_swiglu_bf16(
-            x2.data_ptr(), weight.data_ptr(), out.data_ptr(), M, I, K, x2.stride(0),
-            weight.stride(0), out.stride(0), _native.status_word(x.device).data_ptr(),
-            _native.stream_ptr())
+        rc = _native.lib().b200_gemm_glu_bf16(
+            x2.data_ptr(), weight.data_ptr(), out.data_ptr(), M, I, K, x2.stride(0), weight.stride(0), out.stride(0),
+            alpha, limit, _native.status_word(x.device).data_ptr(), _native.stream_ptr())
         _native.check(rc, "gemm_swiglu")
         launch_counter[0] += 1
     return out.view(*x.shape[:-1], I)

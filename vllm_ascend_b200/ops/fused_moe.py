@@ -63,9 +63,11 @@ def gating_topk(logits: torch.Tensor, k: int, scoring: str = "softmax", renorm: 
 
 def fused_experts_ref(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor,
                       topk_w: torch.Tensor, topk_ids: torch.Tensor,
-                      expert_map: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      expert_map: Optional[torch.Tensor] = None, limit: Optional[float] = None,
+                      weight_input: bool = False) -> torch.Tensor:
     """x [T,H]; w13 [E_local, 2I, H]; w2 [E_local, H, I]; ids are global expert ids,
-    ``expert_map`` maps global -> local (-1: not on this rank)."""
+    ``expert_map`` maps global -> local (-1: not on this rank).  ``limit``: clamped gate instead of SiLU;
+    ``weight_input``: an expert works on weight * input, its output is not weighted."""
     T, H = x.shape
     out = torch.zeros(T, H, dtype=torch.float32, device=x.device)
     ids = topk_ids.long()
@@ -77,23 +79,30 @@ def fused_experts_ref(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor,
         if tok.numel() == 0:
             continue
         h = x[tok] @ w13[e].to(x.dtype).t()
-        a = ref.silu_and_mul(h)
-        y = a @ w2[e].to(x.dtype).t()
-        out.index_add_(0, tok, y.float() * topk_w[tok, slot].unsqueeze(-1).float())
+        w = topk_w[tok, slot].unsqueeze(-1).float()
+        if weight_input:
+            h, w = h.float() * w, 1.0
+        a = ref.silu_and_mul(h) if limit is None else ref.activation(h, "swiglu_oai", gated=True, limit=limit)
+        y = a.to(x.dtype) @ w2[e].to(x.dtype).t()
+        out.index_add_(0, tok, y.float() * w)
     return out.to(x.dtype)
 
 
-def fused_experts(x, w13, w2, topk_w, topk_ids, expert_map=None, quant=None, shared=None, shared_gate=None):
-    """Weighted sum of the chosen experts' outputs; ``shared`` [T, H] (a shared expert's output) is added, scaled
-    by sigmoid(x . shared_gate) where that vector is given."""
+def fused_experts(x, w13, w2, topk_w, topk_ids, expert_map=None, quant=None, shared=None, shared_gate=None,
+                  limit=None, weight_input=False):
+    """Weighted sum of the chosen experts' outputs (``weight_input``: sum of the outputs for weighted inputs);
+    ``shared`` [T, H] (a shared expert's output) is added, scaled by sigmoid(x . shared_gate) where that vector is
+    given.  ``limit``: the experts' gate is the clamped one, min(g, limit) sigmoid(1.702 .) (clamp(u) + 1)."""
     if x.is_cuda and x.dtype in (torch.bfloat16, torch.float32) and w13.dtype == x.dtype and _native.available() \
             and hasattr(_native.lib(), "b200_moe_permute") and quant is None:
         from . import moe_native
-        return moe_native.fused_experts(x, w13, w2, topk_w, topk_ids, expert_map, shared, shared_gate)
+        return moe_native.fused_experts(x, w13, w2, topk_w, topk_ids, expert_map, shared, shared_gate, limit, weight_input)
     if quant is not None:
+        if limit is not None or weight_input:
+            raise NotImplementedError("quantised experts have SiLU gates and weighted outputs")
         y = quant.apply_experts(x, w13, w2, topk_w, topk_ids, expert_map)
     else:
-        y = fused_experts_ref(x, w13, w2, topk_w, topk_ids, expert_map)
+        y = fused_experts_ref(x, w13, w2, topk_w, topk_ids, expert_map, limit, weight_input)
     if shared is None:
         return y
     g = 1.0 if shared_gate is None else torch.sigmoid(x.float() @ shared_gate.float().view(-1, 1))

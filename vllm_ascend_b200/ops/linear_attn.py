@@ -316,8 +316,9 @@ def gated_linear_attention_ref(q, k, v, g, state, cu, slots, has_init):
 
 
 def gated_linear_attention(q, k, v, g, state, cu, slots, has_init, cu_cpu, chunk=64):
-    """Same contract as ``gated_linear_attention_ref``, two batched forms chosen per sequence from
-    the host copy of ``cu``:
+    """Same contract as ``gated_linear_attention_ref``.  GPU tensors run the recurrence kernels
+    (``linear_recurrence.decayed_attention``); on the host there are two batched forms, chosen per sequence
+    from the host copy of ``cu``:
 
     * one new token (decode): every such sequence in one batched update
       S = e^g S + k v^T, o = S^T q (no per-sequence work on the host);
@@ -332,6 +333,9 @@ def gated_linear_attention(q, k, v, g, state, cu, slots, has_init, cu_cpu, chunk
     Triton lightning-attention prefill / decode pair and vLLM's Mamba-2 kernels
     (vllm_ascend/ops/triton/mamba/lightning_attn.py, vllm_ascend/ops/triton/mamba/causal_conv1d.py)."""
     import numpy as np
+    if q.is_cuda:
+        from .linear_recurrence import decayed_attention
+        return decayed_attention(q, k, v, g, state, cu, slots, has_init, uniform=max(np.diff(cu_cpu), default=0) <= 1)
     T, H, DV = v.shape
     Hk, D = q.shape[1], q.shape[2]
     rep = H // Hk

@@ -132,7 +132,8 @@ class MoERuntime:
             y = fused_experts_lora(xg, block.w13, block.w2, wg, ig, block.expert_map, lora,
                                    slots=ep.all_gather(slots.contiguous(), 0))
         else:
-            y = fused_moe.fused_experts(xg, block.w13, block.w2, wg, ig, block.expert_map, block.quant)
+            y = fused_moe.fused_experts(xg, block.w13, block.w2, wg, ig, block.expert_map, block.quant,
+                                        **block.expert_form)
         if x.is_cuda:
             y = ep.reduce_scatter(y, 0)
         else:   # gloo has no reduce-scatter
@@ -159,6 +160,11 @@ class MoERuntime:
         out_splits = recv_counts.tolist()
         recv_x = ep.all_to_all_single(send_x, out_splits, in_splits)
         recv_e = ep.all_to_all_single(send_e, out_splits, in_splits)
+        w_sorted = topk_w.reshape(-1)[order].float()
+        recv_w = None
+        if block.expert_form["weight_input"]:          # weights of the inputs travel with them
+            recv_w = ep.all_to_all_single(w_sorted, out_splits, in_splits)
+            w_sorted = torch.ones_like(w_sorted)
         # local experts on the received rows (each row is one (token, expert) pair, weight 1)
         R = recv_x.shape[0]
         recv_s = ep.all_to_all_single(slots[send_tok].contiguous(), out_splits, in_splits) if lora is not None else None
@@ -168,14 +174,13 @@ class MoERuntime:
             y = fused_experts_lora(recv_x, block.w13, block.w2, ones, recv_e.view(R, 1).to(torch.int32),
                                    block.expert_map, lora, slots=recv_s)
         elif R > 0:
-            ones = torch.ones(R, 1, dtype=topk_w.dtype, device=x.device)
-            y = fused_moe.fused_experts(recv_x, block.w13, block.w2, ones,
+            w_in = torch.ones(R, 1, dtype=topk_w.dtype, device=x.device) if recv_w is None else recv_w.view(R, 1)
+            y = fused_moe.fused_experts(recv_x, block.w13, block.w2, w_in,
                                         recv_e.view(R, 1).to(torch.int32), block.expert_map,
-                                        block.quant)
+                                        block.quant, **block.expert_form)
         else:
             y = recv_x
         back = ep.all_to_all_single(y, in_splits, out_splits)       # rows return in send order
         out = torch.zeros(T, H, dtype=torch.float32, device=x.device)
-        w_sorted = topk_w.reshape(-1)[order].float()
         out.index_add_(0, send_tok, back.float() * w_sorted.unsqueeze(-1))
         return out.to(x.dtype)

@@ -73,7 +73,7 @@ class SharedExperts:
         if m.act is not None:
             return ops.activation(gu(x).contiguous(), m.act, gated=True)
         if gu.quant is None and gu.bias is None and not gu.gather_output and not gu._lora_on():
-            return ops.linear_swiglu(x, gu.weight)
+            return ops.linear_swiglu(x, gu.weight, limit=m.limit)
         return ops.silu_and_mul(gu(x))
 
     def part2(self, x: torch.Tensor, act: torch.Tensor) -> torch.Tensor:

@@ -12,7 +12,7 @@ import torch.nn.functional as F
 from .. import _native
 
 P, I, L, Fl = c_void_p, c_int, c_long, c_float
-_native.register_signature("b200_stream_norm", [P, P, L, I, P, P, Fl, I, P, P, L, Fl, I, P, P, P, L, I, Fl, I, P, P])
+_native.register_signature("b200_stream_norm", [P, P, L, I, P, P, Fl, I, P, P, L, Fl, I, P, P, P, L, I, I, I, Fl, I, P, P])
 _native.register_signature("b200_stream_mix", [P, P, L, I, P, P, P, P, I, P, P, L, Fl, P, P, L, P, I, P, P, P, L, I, I, I,
                                                Fl, I, P, P])
 _native.register_signature("b200_side_gate", [P, L, P, P, L, L, L, P, L, I, I, P, P])
@@ -22,14 +22,16 @@ _KIND = {None: 0, "layer": 1, "rms": 2, "plain": 3}
 
 
 class NormSpec:
-    """A norm as the stream kernel takes it: kind "layer" (weight, bias), "rms" (weight) or "plain"
-    (the row as it is)."""
-    __slots__ = ("kind", "weight", "bias")
+    """A norm as the stream kernel takes it: kind "layer" (weight, bias), "rms" (weight; over ``groups`` equal parts
+    of the row, each by itself) or "plain" (the row as it is)."""
+    __slots__ = ("kind", "weight", "bias", "groups")
 
-    def __init__(self, kind: str, weight: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None):
+    def __init__(self, kind: str, weight: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None, groups: int = 1):
         if kind not in ("layer", "rms", "plain"):
             raise ValueError(f"unknown norm kind {kind!r}")
-        self.kind, self.weight, self.bias = kind, weight, bias
+        if groups < 1 or (groups > 1 and (kind != "rms" or bias is not None or weight.shape[0] % groups)):
+            raise ValueError(f"a {kind} norm of this width does not come in {groups} groups")
+        self.kind, self.weight, self.bias, self.groups = kind, weight, bias, groups
 
 
 #: the row itself, rounded to the activation type
@@ -49,6 +51,9 @@ def _norm_ref(v: torch.Tensor, n: NormSpec, eps: float) -> torch.Tensor:
         return v
     if n.kind == "layer":
         v = v - v.mean(-1, keepdim=True)
+    if n.groups > 1:
+        parts = v.unflatten(-1, (n.groups, -1))
+        return (parts * torch.rsqrt((parts * parts).mean(-1, keepdim=True) + eps)).flatten(-2) * n.weight.float()
     v = v * torch.rsqrt((v * v).mean(-1, keepdim=True) + eps) * n.weight.float()
     return v if n.bias is None else v + n.bias.float()
 
@@ -91,7 +96,8 @@ def stream_norm(r: torch.Tensor, y: Optional[torch.Tensor], post: Optional[NormS
         _native.ptr(post.weight if y is not None else None), _native.ptr(post.bias if y is not None else None),
         float(post_scale), emb, _native.ptr(ids), _native.ptr(embed), 0 if embed is None else embed.shape[0],
         float(embed_scale), 0 if nxt is None else _KIND[nxt.kind], _native.ptr(nxt.weight if nxt else None),
-        _native.ptr(nxt.bias if nxt else None), _native.ptr(x), T, W, float(eps), code,
+        _native.ptr(nxt.bias if nxt else None), _native.ptr(x), T, W, post.groups if y is not None else 1,
+        nxt.groups if nxt else 1, float(eps), code,
         _native.status_word(r.device).data_ptr(), _native.stream_ptr())
     _native.check(rc, "stream_norm")
     _native.count_launch()
@@ -137,6 +143,8 @@ def stream_mix(r: torch.Tensor, y: Optional[torch.Tensor], post: Optional[NormSp
         if store and x is not r:
             r.copy_(x)
         return None if nxt is None else _norm_ref(u, nxt, eps).to(dtype)
+    if any(n is not None and n.groups > 1 for n in (post, nxt)):
+        raise NotImplementedError("norms in groups on several streams")
     code = _dtype_code(dtype)
     for t in (y, embed, pos_table, *((post.weight, post.bias) if post else ()), *((nxt.weight, nxt.bias) if nxt else ())):
         if t is not None and t.dtype != dtype:
