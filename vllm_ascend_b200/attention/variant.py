@@ -43,7 +43,7 @@ class _AttnArgs(ctypes.Structure):
 
 _ENTRY = [c_void_p, c_void_p, c_void_p]
 for _name in ("b200_qkv_prep", "b200_attention_variant", "b200_attention_variant_prefill",
-              "b200_attention_variant_decode"):
+              "b200_attention_variant_decode", "b200_attention_wide_prefill", "b200_attention_wide_decode"):
     _native.register_signature(_name, _ENTRY)
 
 
@@ -322,14 +322,27 @@ def variant_attention_simple(q, k_cache, v_cache, meta, o: AttnOptions, gate=Non
     return out
 
 
-def _tc_ok(q, k_cache, v_cache, out) -> bool:
-    """True when the tcgen05 kernels take these tensors (TMA: 16-byte strides and bases), keys up to 128 dimensions."""
+def _tma_ok(q, k_cache, v_cache, out) -> bool:
+    """True when the tcgen05 kernels can load these tensors (TMA: 16-byte strides and bases)."""
     D, Dv, bs = q.shape[2], v_cache.shape[3], k_cache.shape[1]
     strides = [q.stride(0), out.stride(0), *k_cache.stride()[:3], *v_cache.stride()[:3]]
-    return (q.dtype == torch.bfloat16 and D % 8 == 0 and Dv % 8 == 0 and 8 <= D <= 128 and 8 <= Dv <= 128
+    return (q.dtype == torch.bfloat16 and D % 8 == 0 and Dv % 8 == 0 and D >= 8 and 8 <= Dv <= 128
             and q.shape[1] // v_cache.shape[2] <= 128 and bs >= 8 and (128 % bs == 0 or bs % 128 == 0)
             and all(x % 8 == 0 for x in strides) and all(t.data_ptr() % 16 == 0 for t in (q, k_cache, v_cache, out))
             and k_cache.stride(3) == v_cache.stride(3) == 1)
+
+
+def _kernels(q, k_cache, v_cache, out, o: AttnOptions, gate=None) -> tuple[Optional[str], Optional[str]]:
+    """(kernel for several rows per sequence, kernel for one): "tile" (keys up to 128 dimensions, all options), "wide"
+    (wider or shared key rows) or None (CUDA cores)."""
+    if not _tma_ok(q, k_cache, v_cache, out):
+        return None, None
+    D, H, Hv, Hk = q.shape[2], q.shape[1], v_cache.shape[2], k_cache.shape[2]
+    plain, columns = o.plain and gate is None, H // Hk
+    many = "tile" if D <= 128 else "wide" if D <= 512 and plain else None
+    if plain and (D > 128 or Hk < Hv) and D <= 1024 and columns <= 32 and (2 + Hv // Hk) * (16 if columns <= 16 else 32) <= 512:
+        return many, "wide"
+    return many, "tile" if D <= 128 and H // Hv <= 16 else None
 
 
 def decode_splits(num_seqs: int, kv_heads: int, o: AttnOptions, max_keys: int, device) -> int:
@@ -372,16 +385,32 @@ def variant_attention_decode(q, k_cache, v_cache, meta, o: AttnOptions, gate=Non
     return out
 
 
+def wide_attention_decode(q, k_cache, v_cache, meta, o: AttnOptions, out=None, num_seqs=None, num_splits: int = 0) -> torch.Tensor:
+    """tcgen05 decode kernel for wide or shared key rows: the first ``num_seqs`` sequences, one query row each."""
+    from .. import ops
+    num_seqs = meta.num_reqs if num_seqs is None else num_seqs
+    if out is None:
+        out = _new_out(q, v_cache, o)
+    a = _args(q, k_cache, v_cache, meta, o, None, out)
+    a.num_seqs = num_seqs
+    a.num_splits = num_splits or decode_splits(num_seqs, a.key_heads, o, meta.block_table.shape[1] * a.block_size, q.device)
+    if a.num_splits > 1:
+        a.scratch = ops._get_scratch(q.device, num_seqs * a.heads * a.num_splits * (a.vdim + 1) * 4).data_ptr()
+    _launch("b200_attention_wide_decode", a, q.device, 2 if a.num_splits > 1 else 1)
+    return out
+
+
 def variant_attention_prefill(q, k_cache, v_cache, meta, o: AttnOptions, gate=None, out=None,
-                              first_seq: int = 0) -> torch.Tensor:
-    """tcgen05 tile kernel: every sequence of the step from ``first_seq`` on, any number of query rows each."""
+                              first_seq: int = 0, wide: bool = False) -> torch.Tensor:
+    """tcgen05 tile kernel (``wide``: for keys of more than 128 dimensions): every sequence of the step from
+    ``first_seq`` on, any number of query rows each."""
     if out is None:
         out = _new_out(q, v_cache, o)
     a = _args(q, k_cache, v_cache, meta, o, gate, out)
     a.num_seqs = meta.num_reqs - first_seq
     a.cu, a.seq_lens = a.cu + 4 * first_seq, a.seq_lens + 4 * first_seq
     a.block_table += 4 * first_seq * a.max_blocks
-    _launch("b200_attention_variant_prefill", a, q.device)
+    _launch("b200_attention_wide_prefill" if wide else "b200_attention_variant_prefill", a, q.device)
     return out
 
 
@@ -396,14 +425,17 @@ def variant_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
         return out
     if not q.is_cuda:
         return _attention_ref(q, k_cache, v_cache, meta, o, gate, out)
-    if not _tc_ok(q, k_cache, v_cache, out):
-        return variant_attention_simple(q, k_cache, v_cache, meta, o, gate, out)
+    many, one = _kernels(q, k_cache, v_cache, out, o, gate)
     # the leading sequences with one row stream their keys through the decode kernel
-    nd = 0
-    if H // v_cache.shape[2] <= 16:
-        nd = meta.num_reqs if meta.max_query_len <= 1 and T == meta.num_reqs else int(meta.num_decodes)
-    if nd:
+    nd = meta.num_reqs if meta.max_query_len <= 1 and T == meta.num_reqs else int(meta.num_decodes)
+    if many is None and (one is None or nd < meta.num_reqs):          # no tensor-core kernel takes all rows
+        return variant_attention_simple(q, k_cache, v_cache, meta, o, gate, out)
+    if one == "wide" and nd:
+        wide_attention_decode(q, k_cache, v_cache, meta, o, out, nd)
+    elif one == "tile" and nd:
         variant_attention_decode(q, k_cache, v_cache, meta, o, gate, out, nd)
+    else:
+        nd = 0
     if nd < meta.num_reqs:
-        variant_attention_prefill(q, k_cache, v_cache, meta, o, gate, out, nd)
+        variant_attention_prefill(q, k_cache, v_cache, meta, o, gate, out, nd, many == "wide")
     return out

@@ -87,9 +87,9 @@ MODEL_SOURCES = {
     "Dubizen": ("activations", "attention_decode", "attention_decode_tc", "attention_mla_decode", "attention_tc",
                 "attention_variant", "cache_ops", "elementwise", "gemm_bf16", "gemm_bf16_2cta", "latent_attention",
                 "mla_preprocess", "moe", "qkv_prep", "sampler", "stream_norm"),
-    "Nevotar": ("activations", "attention_decode", "attention_decode_tc", "attention_tc", "attention_variant", "cache_ops",
-                "elementwise", "gemm_bf16", "gemm_bf16_2cta", "group_norm", "linear_attention", "linear_recurrence", "moe",
-                "qkv_prep", "sampler", "stream_norm"),
+    "Nevotar": ("activations", "attention_decode", "attention_decode_tc", "attention_tc", "attention_variant",
+                "attention_wide", "cache_ops", "elementwise", "gemm_bf16", "gemm_bf16_2cta", "group_norm", "linear_attention",
+                "linear_recurrence", "moe", "qkv_prep", "sampler", "stream_norm"),
 }
 
 

@@ -146,7 +146,8 @@ class VariantAttention:
         return [(num_slots, self.taps - 1, self.prep.columns)] if self.taps > 1 else []
 
     def reserve_decode_scratch(self, device, batch_sizes: list, max_keys: int) -> None:
-        reserve_decode_scratch(device, batch_sizes[-1], self.Hq * self.maps, self.Hkv, self.Dv, self.options, max_keys)
+        for kv_heads in {self.Hkv, self.prep.key_heads}:
+            reserve_decode_scratch(device, batch_sizes[-1], self.Hq * self.maps, kv_heads, self.Dv, self.options, max_keys)
 
     # ------------------------------------------------------------------ forward
     def __call__(self, x: torch.Tensor, meta, kv_cache) -> torch.Tensor:
