@@ -26,7 +26,7 @@ Workloads (``--mode``):
 * ``pd``: disaggregated prefill: the first half of the ranks form the prefill engine (TP), the second
   half the decode engine (expert parallel with data-parallel attention for MoE models), KV blocks
   move over NVLink (``ours`` only).
-* ``layers``: prefill and decode throughput of plan-built decoders (Vofelix, Pegopel, Dubizen) beside the closest
+* ``layers``: prefill and decode throughput of plan-built decoders (Vofelix, Pegopel, Dubizen, Nevotar) beside the closest
   existing models at equal layer sizes, one GPU (``benchmarks/plan_bench.py``, ``ours`` only); the line's value is
   the decode rate of the whole Vofelix design and ``cases`` holds the table.
 

@@ -1,10 +1,10 @@
 #!/usr/bin/env python
-"""Prefill and decode throughput of plan-built decoders (Vofelix, Pegopel, Dubizen) beside the closest existing models
-at equal size, random weights, one GPU.
+"""Prefill and decode throughput of plan-built decoders (Vofelix, Pegopel, Dubizen, Nevotar) beside the closest existing
+models at equal size, random weights, one GPU.
 
     python bench.py --mode layers                 # or: python benchmarks/plan_bench.py
     python benchmarks/plan_bench.py --kernels     # the single kernels with their rooflines (--variant-kernels,
-                                                  # --expert-kernels: those of one design)
+                                                  # --expert-kernels, --recurrence-kernels: those of one design)
 
 Model cases time the engine's own step on the device (CUDA events, median): a prefill step of whole prompts,
 and decode-graph replays of a batch with a given context.  Weights and caches are larger than L2.  Kernel
@@ -95,8 +95,35 @@ def _dubizen(layers):
                                      "residual_mult": 0.5, "layers": layers}, name="dubizen-bench")
 
 
-def _gqa(window, **kw):
-    return _existing(name="gqa-dense", architecture="Qwen3ForCausalLM", num_attention_heads=32, num_key_value_heads=8,
+_CLAMPED = {"kind": "moe", "expert": {"ff": 1408, "limit": 7.0}, "shared": {"ff": 2816, "limit": 7.0},
+            "router": {"experts": 64, "top": 8}}
+
+
+def _side(mlp, window=1024):
+    return {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window},
+                 "rot": {"base": 1e4, "dims": 128}},
+        "right": {"heads": 64, "vdim": 64, "state": 128, "groups": 4, "conv": 4, "norm_groups": 4},
+        "left_scale": 0.7, "right_scale": 0.7}}
+
+
+def _two_maps(mlp):
+    return {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": 32, "kv_heads": 8, "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.5, "q_temp": {"coef": 0.1, "every": 512}}}
+
+
+def _forget(mlp):
+    return {"type": "hgrn2", "mlp": mlp, "mixer": {"heads": 32, "dim": 128, "vdim": 128}}
+
+
+def _nevotar(layers):
+    from vllm_ascend_b200.config import ModelConfig
+    return ModelConfig.from_hf_dict({"architecture": "Nevotar", "vocab": VOCAB, "width": 4096,
+                                     "norm": {"eps": 1e-6, "groups": 4}, "layers": layers}, name="nevotar-bench")
+
+
+def _gqa(window, heads=32, kv_heads=8, **kw):
+    return _existing(name="gqa-dense", architecture="Qwen3ForCausalLM", num_attention_heads=heads, num_key_value_heads=kv_heads,
                      head_dim=128, qk_norm=True, sliding_window=window, rope_theta=1e4, **kw)
 
 
@@ -118,11 +145,15 @@ _MOE = dict(num_experts=64, num_experts_per_tok=8, moe_intermediate_size=1408, n
             n_group=8, topk_group=4, routed_scaling_factor=2.5, e_score_correction_bias=True)
 
 
-def _gdn():
+_SIGMOID_MOE = dict(_MOE, scoring_func="sigmoid", n_group=1, topk_group=1, routed_scaling_factor=1.0, e_score_correction_bias=False,
+                    norm_topk_prob=False)
+
+
+def _gdn(**kw):
     return _existing(name="gdn-hybrid", architecture="Qwen3NextForCausalLM", num_attention_heads=32,
                      num_key_value_heads=8, head_dim=128, qk_norm=True, full_attention_interval=LAYERS,
                      linear_num_key_heads=16, linear_num_value_heads=32, linear_key_head_dim=128,
-                     linear_value_head_dim=128, linear_conv_kernel_dim=4)
+                     linear_value_head_dim=128, linear_conv_kernel_dim=4, **kw)
 
 
 #: label -> configuration.  The plain Vofelix and Pegopel stacks have the mixers and feed-forward of their neighbour
@@ -152,6 +183,14 @@ MODELS = {
     "existing MLA, experts": lambda: _mla(32, q_lora_rank=1536, **_MOE),
     "Dubizen whole": lambda: _dubizen([_shared_latent(_PLAIN_FF), _shared_latent(_EXPERTS), _normed(_PLAIN_FF),
                                        _normed(_EXPERTS), _shared_latent(_EXPERTS, 1), _shared_latent(_PLAIN_FF, 1)]),
+    "Nevotar attention beside state space": lambda: _nevotar([_side(_CLAMPED)] * LAYERS),
+    "existing GQA 16/4 w=1024, experts": lambda: _gqa(1024, 16, 4, **_SIGMOID_MOE),
+    "Nevotar two maps": lambda: _nevotar([_two_maps(_CLAMPED)] * LAYERS),
+    "existing GQA, experts": lambda: _gqa(None, **_SIGMOID_MOE),
+    "Nevotar HGRN2, 7 of 8": lambda: _nevotar([_forget(_CLAMPED)] * (LAYERS - 1) + [_two_maps(_CLAMPED)]),
+    "existing GDN, experts": lambda: _gdn(**_SIGMOID_MOE),
+    "Nevotar whole": lambda: _nevotar([_side(_CLAMPED), _side(_CLAMPED), _two_maps(_CLAMPED), _forget(_CLAMPED)] +
+                                      [dict(f(_CLAMPED), weights_of=i) for i, f in enumerate((_side, _side, _two_maps, _forget))]),
 }
 
 
@@ -293,7 +332,137 @@ def bench_kernels() -> list[dict]:
                 reads * 1152 + T * H * (576 + 512) * 2, keys * H * (576 + 512) * 2)
     res += _variant_kernels(rec_list=[], hbm=hbm, tf=tf)
     res += _expert_kernels(rec_list=[], hbm=hbm, tf=tf)
+    res += _recurrence_kernels(rec_list=[], hbm=hbm, tf=tf)
     return res
+
+
+def _recurrence_kernels(rec_list, hbm, tf) -> list[dict]:
+    """The kernels of the Nevotar stacks that others do not have, beside their counterparts."""
+    from kernel_bench import timeit
+    from vllm_ascend_b200 import ops
+    from vllm_ascend_b200.attention import variant as va
+    from vllm_ascend_b200.attention.metadata import AttentionMetadata, build_tile_worklist
+    from vllm_ascend_b200.ops import linear_attn as la
+    from vllm_ascend_b200.ops import linear_recurrence as lr
+    from vllm_ascend_b200.ops import moe_native
+    from vllm_ascend_b200.ops import stream as st
+    bf, dev = torch.bfloat16, "cuda"
+
+    def rec(name, ms, nbytes=0, flops=0):
+        t_mem, t_fl = nbytes / hbm / 1e6, flops / tf / 1e9
+        rec_list.append({"kernel": name, "ms": round(ms, 4), "GB/s": round(nbytes / ms / 1e6),
+                         "TFLOP/s": round(flops / ms / 1e9, 1), "roofline_frac": round(max(t_mem, t_fl) / ms, 3)})
+
+    def mk(*s, dtype=bf):
+        return torch.randn(*s, device=dev, dtype=dtype)
+    W = 4096
+    for T in (256, 8192):
+        r, y, w, res_b, z = mk(T, W, dtype=torch.float32), mk(T, W), mk(W), mk(T, W), mk(T, W)
+        rec(f"[existing] add+rms_norm T={T}", timeit(lambda: ops.rms_norm(y, w, 1e-6, res_b)), T * W * 8)
+        for groups in (1, 4):
+            n = st.NormSpec("rms", w, None, groups)
+            rec(f"stream_norm {groups} groups T={T}", timeit(lambda: st.stream_norm(r, y, st.PLAIN, n, 1e-6, bf)), T * W * 12)
+        h128 = mk(128)
+        rec(f"[existing] gated head norm T={T}", timeit(lambda: st.gated_head_norm(y.view(T, 32, 128), z, h128, 1e-6)), T * W * 6)
+        rec(f"group_norm 4 groups, gate T={T}", timeit(lambda: lr.group_norm(y, w, 4, 1e-6, z)), T * W * 6)
+        rec(f"group_norm per head T={T}", timeit(lambda: lr.group_norm(y, h128, 32, 1e-6)), T * W * 4)
+        o = mk(T, 64, 128, dtype=torch.float32)
+        rec(f"map_difference T={T}", timeit(lambda: lr.map_difference(o, 0.5, 1e-6, 0.5, bf)), T * 64 * 128 * 4 + T * W * 2)
+        I = 2816
+        sw, x = mk(2 * I, W) * 0.02, mk(T, W)
+        rec(f"[existing] gate / up product T={T}", timeit(lambda: ops.linear_swiglu(x, sw)), 2 * I * W * 2 + T * (W + I) * 2, 4 * T * I * W)
+        rec(f"gate / up product, clamped T={T}", timeit(lambda: ops.linear_swiglu(x, sw, limit=7.0)),
+            2 * I * W * 2 + T * (W + I) * 2, 4 * T * I * W)
+        E, k, I = 64, 8, 1408
+        w13 = mk(E, 2 * I, W) * 0.02
+        ids = torch.stack([torch.randperm(E, device=dev)[:k] for _ in range(T)]).to(torch.int32)
+        tw = torch.rand(T, k, device=dev)
+        perm = moe_native.Permutation(ids, None, E)
+        xs = perm.gather(x)
+        used = int((perm.counts > 0).sum())
+        scale = perm.row_weights(tw)
+        rec(f"row weights T={T}", timeit(lambda: perm.row_weights(tw)), T * k * 12)
+        cost = (used * 2 * I * W * 2 + T * k * (W + I) * 2, 4 * T * k * I * W)
+        rec(f"[existing] grouped product, gate and up T={T}", timeit(lambda: moe_native.grouped_gemm(xs, w13, perm.offsets, True)), *cost)
+        rec(f"grouped product, clamped, weighted rows T={T}",
+            timeit(lambda: moe_native.grouped_gemm(xs, w13, perm.offsets, True, scale, 7.0)), *cost)
+        del w13, xs, o
+    for B, n in ((256, 1), (4, 2048), (1, 8192)):
+        T, tag = B * n, f"{B}x{n}"
+        cu = torch.arange(0, T + 1, n, dtype=torch.int32, device=dev)
+        slots, init = torch.arange(B, dtype=torch.int32, device=dev), torch.ones(B, dtype=torch.int32, device=dev)
+        H, Hk, D = 32, 16, 128
+        S = torch.zeros(B, H, D, D, dtype=torch.float32, device=dev)
+        q, v, g, be = mk(T, Hk, D), mk(T, H, D), -torch.rand(T, H, device=dev), torch.rand(T, H, device=dev)
+        state = B * H * D * D * 8
+        rec(f"[existing] delta rule {tag}", timeit(lambda: la.gated_delta_rule(q, q, v, g, be, S, cu, slots, init, D ** -0.5, uniform=n == 1)),
+            T * (2 * Hk + 2 * H) * D * 2 + state, 8 * T * H * D * D)
+        qfv, fb, low, nw = mk(T, 3 * H * D), mk(H * D), torch.rand(H * D, device=dev).to(bf), mk(D)
+        at = H * D
+        rec(f"HGRN2 recurrence with its norm {tag}", timeit(lambda: lr.forget_recurrence(
+            qfv[:, :at], qfv[:, at:2 * at], qfv[:, 2 * at:], fb, low, S, cu, slots, init, nw, 1e-6, uniform=n == 1)),
+            T * 4 * H * D * 2 + state, 6 * T * H * D * D)
+        del S
+        H, G, N, P = 64, 4, 128, 64
+        C = H * P + 2 * G * N
+        S = torch.zeros(B, H, N, P, dtype=torch.float32, device=dev)
+        sp = lr.StateSpace(mk(H, dtype=torch.float32), mk(H, dtype=torch.float32), mk(H, dtype=torch.float32), G)
+        xbc, dt = mk(T, C), mk(T, H)
+        rec(f"Mamba-2 recurrence {tag}", timeit(lambda: lr.state_space(sp, xbc, dt, S, cu, slots, init, uniform=n == 1)),
+            T * (C + H * P + H) * 2 + B * H * N * P * 8, 6 * T * H * N * P)
+        del S
+    for B, n, ctx in ((64, 1, 2048), (256, 1, 2048), (4, 2048, 2048)):
+        bs, T = 128, B * n
+        nb = B * ctx // bs + 1
+        bt = (torch.arange(B * ctx // bs, dtype=torch.int32, device=dev).view(B, -1) + 1).contiguous()
+        cu, sl = np.arange(0, T + 1, n, dtype=np.int32), np.full(B, ctx, dtype=np.int32)
+        pos = torch.arange(ctx - n, ctx, device=dev).repeat(B)
+        slot = (bt[torch.arange(B, device=dev).repeat_interleave(n), pos // bs].long()) * bs + pos % bs
+        tag, cs, sc = f"{B}x{n} ctx {ctx}", torch.randn(4096, 128, device=dev), 128 ** -0.5
+
+        def meta_for(group):
+            m = AttentionMetadata(
+                num_reqs=B, num_actual_tokens=T, max_query_len=n, max_seq_len=ctx, query_start_loc=torch.from_numpy(cu).to(dev),
+                seq_lens=torch.from_numpy(sl).to(dev), block_table=bt, slot_mapping=slot, positions=pos, query_start_loc_cpu=cu,
+                seq_lens_cpu=sl, num_decodes=B if n == 1 else 0, num_decode_tokens=B if n == 1 else 0)
+            if n > 1:
+                ts, tq = build_tile_worklist(np.full(B, n, dtype=np.int32), 128 // group, sl)
+                m.tile_seq, m.tile_qoff, m.num_tiles = torch.from_numpy(ts).to(dev), torch.from_numpy(tq).to(dev), len(ts)
+            else:
+                m.num_splits = ops.choose_num_splits(B, G, ctx)
+            return m
+        for kind, H, G, parts, win in (("talk", 16, 4, 4, 1024), ("maps", 32, 8, 2, 0)):
+            D = 128
+            meta = meta_for(H // G)
+            kc, vc = (ops.alloc_kv_cache(nb, bs, G, D, bf, dev) for _ in "kv")
+            kc.normal_()
+            vc.normal_()
+            keys = sum(min(win or ctx, ctx - n + i + 1) for i in range(n)) * B
+            nbytes, q = B * min(ctx, (win or ctx) + n) * G * D * 4 + T * H * D * 4, mk(T, H, D)
+            qkv, qn = mk(T, (H + 2 * G) * D), mk(D)
+            rec(f"[existing] qknorm_rope_kvwrite {H}/{G} heads {tag}", timeit(lambda: ops.qknorm_rope_kvwrite(
+                qkv, pos, cs, D, qn, qn, 1e-6, kc, vc, slot, H, G, D)), T * (H + 2 * G) * D * 4)
+            rec(f"[existing] paged attention {H}/{G} heads {tag} window {win}",
+                timeit(lambda: ops.paged_attention(q, kc, vc, meta, sc, window=win)), nbytes, keys * H * D * 4)
+            if kind == "talk":
+                wide = torch.randn(nb, bs, 1, G * D, device=dev, dtype=bf)
+                mix = torch.randn(H, H, device=dev)
+                spec = va.PrepSpec(H, G, D, D, 1e-6, qn, qn, (H * D, G * D), rot_dims=D, cos_sin=cs, head_norm=True, v_heads=G,
+                                   key_parts=G, part_run=H // G, mix=mix)
+                o, flops = va.AttnOptions(sc, win, out_scale=0.7), keys * (H * D * 4 + H * H * 2)
+                wq = T * H * G * D * 2
+            else:
+                wide = torch.randn(nb, bs, G, D, device=dev, dtype=bf)
+                table = torch.rand(4096, device=dev)
+                spec = va.PrepSpec(2 * H, 2 * G, D // 2, D, 1e-6, None, None, (0, 0), v_heads=G, key_parts=2, q_scale=table)
+                o, flops = va.AttnOptions(sc, win, out_f32=True), keys * H * (2 * D + 4 * D)
+                wq = T * H * 2 * D * 2
+            rec(f"qkv_prep {kind} {tag}", timeit(lambda: va.qkv_prep(spec, qkv, meta, wide, vc)), T * (H + 2 * G) * D * 2 + T * 2 * G * D * 2 + wq)
+            qw = va.qkv_prep(spec, qkv, meta, wide, vc)
+            rec(f"attention {kind} {tag} window {win}", timeit(lambda: va.variant_attention(qw, wide, vc, meta, o)),
+                B * min(ctx, (win or ctx) + n) * G * D * 4 + wq + T * H * D * (2 if kind == "talk" else 8), flops)
+            del kc, vc, wide, qw
+    return rec_list
 
 
 def _expert_kernels(rec_list, hbm, tf) -> list[dict]:
@@ -469,6 +638,7 @@ def main() -> None:
     ap.add_argument("--kernels", action="store_true")
     ap.add_argument("--variant-kernels", action="store_true", help="only the kernels of attention with options")
     ap.add_argument("--expert-kernels", action="store_true", help="only the kernels of the Dubizen stacks")
+    ap.add_argument("--recurrence-kernels", action="store_true", help="only the kernels of the Nevotar stacks")
     ap.add_argument("--only", default="", help="model labels with semicolons between them")
     args = ap.parse_args()
     if args.variant_kernels:
@@ -477,6 +647,10 @@ def main() -> None:
         return
     if args.expert_kernels:
         for row in _expert_kernels([], *peaks()):
+            print(json.dumps(row), flush=True)
+        return
+    if args.recurrence_kernels:
+        for row in _recurrence_kernels([], *peaks()):
             print(json.dumps(row), flush=True)
         return
     if args.kernels:

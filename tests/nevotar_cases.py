@@ -155,14 +155,14 @@ def reference(cfg, w, ids, rounded=False):
 
 def check_all(pairs, cfg, w, dtype, note=None):
     """``pairs`` of (logits, token ids).  fp32: every position within 1e-4.  bf16: neither the mean error nor the
-    largest is far above what rounding the sub-layers' inputs and outputs causes in the definition; rounding may
-    exchange two experts that are close, so the tenth with the largest errors does not count."""
+    largest is far above what rounding causes in the definition; rounding may exchange two experts that are close, and
+    a state carries the difference on, so the fifth with the largest errors does not count."""
     e = torch.cat([errors(got, reference(cfg, w, ids)) for got, ids in pairs])
     if dtype == "float32":
         assert float(e.max()) < 1e-4, (note, float(e.max()))
         return
     r = torch.cat([errors(reference(cfg, w, ids, True), reference(cfg, w, ids)) for _, ids in pairs])
-    e, r = (t.sort().values[:max(1, len(t) * 9 // 10)] for t in (e, r))
+    e, r = (t.sort().values[:max(1, len(t) * 4 // 5)] for t in (e, r))
     assert float(e.mean()) < 2.5 * float(r.mean()) and float(e.max()) < 3 * max(float(r.max()), 0.02), \
         (note, float(e.mean()), float(r.mean()), float(e.max()), float(r.max()))
 

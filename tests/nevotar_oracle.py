@@ -40,8 +40,16 @@ def difference_of_maps(q, k, v, scale, lam, diff, eps, temp=None):
     return out
 
 
+_rounding = [False]
+
+
+def cast(t):
+    """What a 16-bit engine stores between two operations (``forward`` with ``rounded``)."""
+    return t.to(torch.bfloat16).to(t.dtype) if _rounding[0] else t
+
+
 def projection(h, p, name, heads, size):
-    return (h @ p[name].T + p[name + ".b"]).view(h.shape[0], heads, size)
+    return cast(h @ p[name].T + p[name + ".b"]).view(h.shape[0], heads, size)
 
 
 def difference_attention(h, p, c, eps):
@@ -91,9 +99,9 @@ def state_space(x, B, C, dt, A_log, D):
 def mamba(h, p, c, eps):
     n, H, P, N, G = h.shape[0], c["heads"], c["vdim"], c["state"], c["groups"]
     inner, gn = H * P, G * N
-    u = h @ p["in"].T
+    u = cast(h @ p["in"].T)
     z, xbc, dt = u[:, :inner], u[:, inner:2 * inner + 2 * gn], u[:, 2 * inner + 2 * gn:]
-    xbc = conv_silu(xbc, p["conv"], p["conv.b"])
+    xbc = cast(conv_silu(xbc, p["conv"], p["conv.b"]))
     x, B, C = xbc[:, :inner], xbc[:, inner:inner + gn], xbc[:, inner + gn:]
     y, _ = state_space(x.reshape(n, H, P), B.reshape(n, G, N), C.reshape(n, G, N), softplus(dt + p["dt_bias"]), p["A_log"],
                        p["D"])
@@ -130,8 +138,9 @@ def forget_recurrence(q, f, v):
 def hgrn2(h, p, c, eps):
     n, H, d, vd = h.shape[0], c["heads"], c["dim"], c["vdim"]
     low = p["lower"]
-    f = low + (1 - low) / (1 + torch.exp(-(h @ p["f"].T + p["f.b"])))
-    o, _ = forget_recurrence(silu(h @ p["q"].T).view(n, H, d), f.view(n, H, d), (h @ p["v"].T).view(n, H, vd))
+    f = low + (1 - low) / (1 + torch.exp(-(cast(h @ p["f"].T) + p["f.b"])))
+    q, v = cast(h @ p["q"].T), cast(h @ p["v"].T)
+    o, _ = forget_recurrence(silu(q).view(n, H, d), f.view(n, H, d), v.view(n, H, vd))
     return rms_norm(o, p["norm"], eps).reshape(n, H * vd) @ p["o"].T
 
 
@@ -165,17 +174,19 @@ def mixture(x, p, c):
 
 def forward(cfg, w, ids, dtype=torch.float64, collect=None, rounded=False):
     """Logits [n, vocab] of one sequence; ``collect`` receives the stream after every layer.  ``rounded``: what
-    enters and leaves a sub-layer is rounded to bf16."""
-    def cast(t):
-        return t.to(torch.bfloat16).to(dtype) if rounded else t
-    w = {k: t.to(dtype) for k, t in w.items()}
-    x = w["embed"][torch.as_tensor(ids, dtype=torch.int64)]
-    eps, groups = cfg["norm"]["eps"], cfg["norm"]["groups"]
-    for i, L in enumerate(cfg["layers"]):
-        p = sub(w, f"l{L.get('weights_of', i)}.")
-        x = x + cast(MIXERS[L["type"]](cast(group_norm(x, p["norm1"], eps, groups)), sub(p, "mix."), L["mixer"], eps))
-        if L["mlp"] is not None:
-            x = x + cast(mixture(cast(group_norm(x, p["norm2"], eps, groups)), sub(p, "mlp."), L["mlp"]))
-        if collect is not None:
-            collect.append(x)
-    return cast(group_norm(x, w["final.norm"], eps, groups)) @ w["embed"].T
+    enters and leaves a sub-layer, and the projections inside, are rounded to bf16."""
+    _rounding[0] = rounded
+    try:
+        w = {k: t.to(dtype) for k, t in w.items()}
+        x = w["embed"][torch.as_tensor(ids, dtype=torch.int64)]
+        eps, groups = cfg["norm"]["eps"], cfg["norm"]["groups"]
+        for i, L in enumerate(cfg["layers"]):
+            p = sub(w, f"l{L.get('weights_of', i)}.")
+            x = x + cast(MIXERS[L["type"]](cast(group_norm(x, p["norm1"], eps, groups)), sub(p, "mix."), L["mixer"], eps))
+            if L["mlp"] is not None:
+                x = x + cast(mixture(cast(group_norm(x, p["norm2"], eps, groups)), sub(p, "mlp."), L["mlp"]))
+            if collect is not None:
+                collect.append(x)
+        return cast(group_norm(x, w["final.norm"], eps, groups)) @ w["embed"].T
+    finally:
+        _rounding[0] = False

@@ -232,6 +232,7 @@ def run_wide(dtype, H, Hv, Hk, d, vd, bs, q_lens, ctx, window, kernel, splits=1,
     g = gen(H * d + window)
     q, _, _, meta = make_paged_case(q_lens, ctx, H, Hk, d, bs, dtype=dtype, layout=layout, tok_per_tile=1)[:4]
     meta.num_decodes = next((i for i, n in enumerate(q_lens) if n > 1), len(q_lens))
+    meta.positions = torch.cat([torch.arange(c, c + n) for c, n in zip(ctx, q_lens)]).cuda()
     nb = int(meta.block_table.max()) + 1
     k, v = (ops.alloc_kv_cache(nb, bs, h, w, dtype, "cuda", layout) for h, w in ((Hk, d), (Hv, vd)))
     for t in (k, v):
@@ -300,7 +301,7 @@ def test_one_key_inside_and_outside_the_window(kernel):
     dtype = torch.float32 if kernel == "simple" else torch.bfloat16
     for pos in (135, 136, 137, 200, 255, 256, 300):
         q, _, _, meta = make_paged_case([1], [pos], H, 1, d, bs, dtype=dtype, tok_per_tile=1)[:4]
-        meta.num_decodes = 1
+        meta.num_decodes, meta.positions = 1, torch.tensor([pos]).cuda()
         nb = int(meta.block_table.max()) + 1
         o = va.AttnOptions(1.0, window)
         fn = {"prefill": lambda *a: va.variant_attention_prefill(*a, wide=True), "decode": va.wide_attention_decode,
