@@ -445,13 +445,36 @@ static int launch_heads(const QkvPrepParams& p, cudaStream_t stream) {
   return B200_CHECK_LAUNCH();
 }
 
-// One block per token.  A warp at a time takes a head: norm (optional), rotary, factor; keys and values go to their
-// cache slots, queries stay in shared memory (fp32) until the wide queries are formed from them.
-template <typename T, int VEC>
+// VEC floats of shared memory, 16 bytes at a time
+template <int VEC>
+__device__ __forceinline__ void smem_get(const float* p, float* v) {
+  if constexpr (VEC % 4 == 0)
+#pragma unroll
+    for (int e = 0; e < VEC; e += 4) load_vec<float, 4>(p + e, v + e);
+  else
+#pragma unroll
+    for (int e = 0; e < VEC; e++) v[e] = p[e];
+}
+template <int VEC>
+__device__ __forceinline__ void smem_put(float* p, const float* v) {
+  if constexpr (VEC % 4 == 0)
+#pragma unroll
+    for (int e = 0; e < VEC; e += 4) store_vec<float, 4>(p + e, v + e);
+  else
+#pragma unroll
+    for (int e = 0; e < VEC; e++) p[e] = v[e];
+}
+
+// One block per token.  LANES threads take a head: norm (optional), rotary, factor; keys and values go to their cache
+// slots, queries stay in shared memory (fp32) until the wide queries are formed from them: a thread then owns VEC
+// dimensions of one key part, keeps what the first CNT projected heads of that part have there, and walks the output heads.
+template <typename T, int VEC, int LANES>
 __global__ void __launch_bounds__(256) qkv_spread_kernel(const QkvPrepParams p) {
-  extern __shared__ __align__(16) float sq[];        // [heads, dim]
+  constexpr int CNT = 4;
+  extern __shared__ __align__(16) float sq[];        // [heads, dim], then [out_heads, heads] weights
+  float* sm = sq + (p.heads * p.dim + 3) / 4 * 4;
   const long t = blockIdx.x;
-  const int lane = threadIdx.x & 31;
+  const int lane = threadIdx.x % LANES;
   const int units = p.heads + p.kv_heads + p.v_heads, half = p.rot >> 1;
   const T* x = (const T*)p.qkv + t * p.qkv_stride;
   const long slot = p.slot_mapping[t];
@@ -465,64 +488,79 @@ __global__ void __launch_bounds__(256) qkv_spread_kernel(const QkvPrepParams p) 
     atomicExch(p.status, B200_BAD_INDEX);
   const float* cs = p.rot > 0 && cs_ok ? p.cos_sin + pos * p.rot : nullptr;
   const float factor = p.q_scale && qs_ok ? p.q_scale[pos] : 1.f;
-  for (int u = threadIdx.x >> 5; u < units; u += 8) {
-    const int kind = u < p.heads ? 0 : u < p.heads + p.kv_heads ? 1 : 2;                    // q, k, v
+  if (p.mix)
+    for (int i = threadIdx.x; i < p.out_heads * p.heads; i += 256) sm[i] = p.mix[i];
+  for (int u0 = 0; u0 < units; u0 += 256 / LANES) {  // same trip count for all threads
+    const int u = u0 + (int)threadIdx.x / LANES;
+    const bool on = u < units;
+    const int kind = !on || u < p.heads ? 0 : u < p.heads + p.kv_heads ? 1 : 2;             // q, k, v
     const int g = kind == 0 ? u : kind == 1 ? u - p.heads : u - p.heads - p.kv_heads;
-    const int dim = kind == 2 ? p.vdim : p.dim;
+    const int dim = !on ? 0 : kind == 2 ? p.vdim : p.dim;
     const T* src = x + (kind == 2 ? (long)(p.heads + p.kv_heads) * p.dim + (long)g * p.vdim : (long)u * p.dim);
+    float first[VEC];                                // the first vector stays in registers
+#pragma unroll
+    for (int e = 0; e < VEC; e++) first[e] = 0.f;
+    if (lane * VEC < dim) load_vec<T, VEC>(src + lane * VEC, first);
     float inv = 1.f;
-    if (kind < 2 && p.head_norm) {
+    if (p.head_norm) {
       float ss = 0.f;
-      for (int c = lane * VEC; c < dim; c += 32 * VEC) {
+#pragma unroll
+      for (int e = 0; e < VEC; e++) ss = fmaf(first[e], first[e], ss);
+      for (int c = (LANES + lane) * VEC; c < dim; c += LANES * VEC) {
         float v[VEC];
         load_vec<T, VEC>(src + c, v);
 #pragma unroll
         for (int e = 0; e < VEC; e++) ss = fmaf(v[e], v[e], ss);
       }
-      inv = 1.f / sqrtf(warp_reduce_sum(ss) / (float)dim + p.eps);
+#pragma unroll
+      for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      inv = 1.f / sqrtf(ss / (float)max(dim, 1) + p.eps);
     }
     const T* w = p.head_norm ? (const T*)(kind == 0 ? p.q_norm : p.k_norm) : nullptr;
     T* dst = nullptr;
-    if (kind == 1 && stored)
+    if (on && kind == 1 && stored)
       dst = (T*)p.k_cache + blk * p.k_block + off * p.k_tok + g / p.key_parts * p.k_head + (long)(g % p.key_parts) * p.dim;
-    else if (kind == 2 && stored)
+    else if (on && kind == 2 && stored)
       dst = (T*)p.v_cache + blk * p.v_block + off * p.v_tok + g * p.v_head;
-    for (int b = 0; b < dim; b += 32 * VEC) {        // same trip count for all lanes
+    const int longest = p.dim > p.vdim ? p.dim : p.vdim;
+    for (int b = 0; b < longest; b += LANES * VEC) { // same trip count for all lanes
       const int c = b + lane * VEC;
       float v[VEC];
 #pragma unroll
-      for (int e = 0; e < VEC; e++) v[e] = 0.f;
-      if (c < dim) load_vec<T, VEC>(src + c, v);
-      if (kind < 2) {
-        if (w && c < dim) {
-          float wv[VEC];
-          load_vec<T, VEC>(w + c, wv);
+      for (int e = 0; e < VEC; e++) v[e] = first[e];
+      if (b > 0) {
 #pragma unroll
-          for (int e = 0; e < VEC; e++) v[e] *= inv * wv[e];
-        }
-        if constexpr (VEC == 1) {
-          if (p.rot > 0) {                           // the partner of a pair sits in the next lane
-            const float other = __shfl_xor_sync(0xffffffffu, v[0], 1);
-            if (cs && c < p.rot) {
-              const float cc = cs[c >> 1], sn = cs[half + (c >> 1)];
-              v[0] = (c & 1) ? v[0] * cc + other * sn : v[0] * cc - other * sn;
-            }
+        for (int e = 0; e < VEC; e++) v[e] = 0.f;
+        if (c < dim) load_vec<T, VEC>(src + c, v);
+      }
+      if (w && kind < 2 && c < dim) {
+        float wv[VEC];
+        load_vec<T, VEC>(w + c, wv);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) v[e] *= inv * wv[e];
+      }
+      if constexpr (VEC == 1) {
+        if (p.rot > 0) {                             // the partner of a pair sits in the next lane
+          const float other = __shfl_xor_sync(0xffffffffu, v[0], 1);
+          if (cs && kind < 2 && c < p.rot) {
+            const float cc = cs[c >> 1], sn = cs[half + (c >> 1)];
+            v[0] = (c & 1) ? v[0] * cc + other * sn : v[0] * cc - other * sn;
           }
-        } else if (cs) {
-#pragma unroll
-          for (int e = 0; e < VEC; e += 2)
-            if (c + e < p.rot) {
-              const float cc = cs[(c + e) >> 1], sn = cs[half + ((c + e) >> 1)], a = v[e], bb = v[e + 1];
-              v[e] = a * cc - bb * sn;
-              v[e + 1] = bb * cc + a * sn;
-            }
         }
+      } else if (cs && kind < 2) {
+#pragma unroll
+        for (int e = 0; e < VEC; e += 2)
+          if (c + e < p.rot) {
+            const float cc = cs[(c + e) >> 1], sn = cs[half + ((c + e) >> 1)], a = v[e], bb = v[e + 1];
+            v[e] = a * cc - bb * sn;
+            v[e + 1] = bb * cc + a * sn;
+          }
       }
       if (c >= dim) continue;
       if (kind == 0) {
 #pragma unroll
         for (int e = 0; e < VEC; e++) v[e] *= factor;
-        store_vec<float, VEC>(sq + (long)g * p.dim + c, v);
+        smem_put<VEC>(sq + (long)g * p.dim + c, v);
       } else if (dst) {
         store_vec<T, VEC>(dst + c, v);
       }
@@ -530,40 +568,70 @@ __global__ void __launch_bounds__(256) qkv_spread_kernel(const QkvPrepParams p) 
   }
   __syncthreads();
   const int per = p.dim / VEC, row = p.key_parts * per, stride = p.part_run * p.key_parts;
+  const int teams = row < 256 ? 256 / row : 1;
+  const int team = row < 256 ? (int)threadIdx.x / row : 0;
+  if (team >= teams) return;
   T* q = (T*)p.q_out + t * p.out_heads * (long)p.key_parts * p.dim;
-  for (int i = threadIdx.x; i < p.out_heads * row; i += 256) {
-    const int oh = i / row, r = i - oh * row, c = r / per, d = (r - c * per) * VEC;
-    float acc[VEC];
+  for (int r = (int)threadIdx.x - team * row; r < row; r += 256) {
+    const int c = r / per, d = (r - c * per) * VEC;
+    if (!p.mix) {
+      int left = team % stride;                      // (output head) mod (heads of a round of parts)
+      for (int oh = team; oh < p.out_heads; oh += teams) {
+        float acc[VEC];
+        const bool mine = left >= c * p.part_run && left < (c + 1) * p.part_run;
 #pragma unroll
-    for (int e = 0; e < VEC; e++) acc[e] = 0.f;
-    if (p.mix) {
-      for (int g0 = c * p.part_run; g0 < p.heads; g0 += stride)
-        for (int g = g0; g < min(g0 + p.part_run, p.heads); g++) {
-          const float m = __ldg(p.mix + (long)oh * p.heads + g);
-          float v[VEC];
-          load_vec<float, VEC>(sq + (long)g * p.dim + d, v);
-#pragma unroll
-          for (int e = 0; e < VEC; e++) acc[e] = fmaf(m, v[e], acc[e]);
-        }
-    } else if (oh / p.part_run % p.key_parts == c) {
-      load_vec<float, VEC>(sq + (long)oh * p.dim + d, acc);
+        for (int e = 0; e < VEC; e++) acc[e] = 0.f;
+        if (mine) smem_get<VEC>(sq + (long)oh * p.dim + d, acc);
+        store_vec<T, VEC>(q + ((long)oh * row + r) * VEC, acc);
+        left += teams;
+        while (left >= stride) left -= stride;
+      }
+      continue;
     }
-    store_vec<T, VEC>(q + (long)i * VEC, acc);
+    const int g0 = c * p.part_run, n = p.part_run < CNT ? p.part_run : CNT;
+    float kept[CNT][VEC];
+#pragma unroll
+    for (int j = 0; j < CNT; j++) {
+#pragma unroll
+      for (int e = 0; e < VEC; e++) kept[j][e] = 0.f;
+      if (j < n && g0 + j < p.heads) smem_get<VEC>(sq + (long)(g0 + j) * p.dim + d, kept[j]);
+    }
+    for (int oh = team; oh < p.out_heads; oh += teams) {
+      const float* m = sm + oh * p.heads;
+      float acc[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; e++) acc[e] = 0.f;
+#pragma unroll
+      for (int j = 0; j < CNT; j++) {
+        const float f = j < n && g0 + j < p.heads ? m[g0 + j] : 0.f;
+#pragma unroll
+        for (int e = 0; e < VEC; e++) acc[e] = fmaf(f, kept[j][e], acc[e]);
+      }
+      for (int s0 = g0; s0 < p.heads; s0 += stride)  // what does not fit
+        for (int g = s0 + (s0 == g0 ? n : 0); g < min(s0 + p.part_run, p.heads); g++) {
+          float v[VEC];
+          smem_get<VEC>(sq + (long)g * p.dim + d, v);
+#pragma unroll
+          for (int e = 0; e < VEC; e++) acc[e] = fmaf(m[g], v[e], acc[e]);
+        }
+      store_vec<T, VEC>(q + ((long)oh * row + r) * VEC, acc);
+    }
   }
 }
 
-template <typename T, int VEC>
+template <typename T, int VEC, int LANES>
 static int launch_spread(const QkvPrepParams& p, cudaStream_t stream) {
-  const size_t smem = (size_t)p.heads * p.dim * sizeof(float);
+  const size_t smem = ((size_t)(p.heads * p.dim + 3) / 4 * 4 + (p.mix ? (size_t)p.out_heads * p.heads : 0)) * sizeof(float);
   if (smem > 200 * 1024) return 9822;
   static bool attr_set = false;
   if (smem > 48 * 1024 && !attr_set) {
-    const cudaError_t e = cudaFuncSetAttribute(qkv_spread_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    const cudaError_t e = cudaFuncSetAttribute(qkv_spread_kernel<T, VEC, LANES>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                               200 * 1024);
     if (e != cudaSuccess) return (int)e;
     attr_set = true;
   }
   if (p.tokens > 0x7fffffffL) return 9823;
-  qkv_spread_kernel<T, VEC><<<(unsigned)p.tokens, 256, smem, stream>>>(p);
+  qkv_spread_kernel<T, VEC, LANES><<<(unsigned)p.tokens, 256, smem, stream>>>(p);
   return B200_CHECK_LAUNCH();
 }
 
@@ -604,9 +672,10 @@ static int prep_t(QkvPrepParams& p, cudaStream_t stream) {
              aligned16(p.q_norm) && aligned16(p.k_norm) && aligned16(p.q_out) && aligned16(p.k_cache) &&
              aligned16(p.v_cache);
   if (p.key_parts > 0) {
-    bool vec4 = vec;
-    for (long x : s) vec4 = vec4 && x % 4 == 0;
-    return vec4 ? launch_spread<T, 4>(p, stream) : launch_spread<T, 1>(p, stream);
+    for (long x : s) vec = vec && x % V == 0;
+    if (!vec) return launch_spread<T, 1, 32>(p, stream);
+    return p.dim / V <= 8 ? launch_spread<T, V, 8>(p, stream)
+                          : p.dim / V <= 16 ? launch_spread<T, V, 16>(p, stream) : launch_spread<T, V, 32>(p, stream);
   }
   for (long x : s) vec = vec && x % V == 0;
   if (p.head_norm) {

@@ -39,6 +39,7 @@ struct StreamParams {
   void* x;                // [T, W]
   int W;
   int post_groups, next_groups;      // RMS norms: equal parts of the row, each by itself
+  int part_threads;                  // > 0: threads of each part of the next norm (and of no other norm in parts)
   float eps;
   int* status;
 };
@@ -143,24 +144,57 @@ __device__ __forceinline__ void row_group_norm(float (&v)[PER][VEC], const T* w,
   }
 }
 
-// GROUPED: RMS norms may come in several parts
+// the sum over the threads that share a part: part_threads (a multiple of 32) neighbours each
+__device__ __forceinline__ float part_sum(float v, float* red, int part_threads) {
+  v = warp_reduce_sum(v);
+  const int warps = part_threads >> 5;
+  if (warps == 1) return v;
+  __syncthreads();                     // the previous use of red is over
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  const int first = (int)threadIdx.x / part_threads * warps;
+  return warp_reduce_sum((threadIdx.x & 31) < warps ? red[first + (threadIdx.x & 31)] : 0.f);
+}
+
+// GROUPED: RMS norms may come in several parts.  With part_threads every part has threads of its own, which reduce it as
+// plain norms reduce a row.
 template <typename T, int VEC, int PER, bool GROUPED>
 __global__ void stream_norm_kernel(const StreamParams p) {
   __shared__ float red[GROUPED ? GROUP_BATCH : 1][32];
+  const int nvec = p.W / VEC, pt = GROUPED ? p.part_threads : 0;
+  const int part = GROUPED && pt ? (int)threadIdx.x / pt : 0, per = GROUPED && pt ? nvec / p.next_groups : nvec;
+  const int base = GROUPED && pt ? part * per + (int)threadIdx.x - part * pt : (int)threadIdx.x;
+  const int step = GROUPED && pt ? pt : (int)blockDim.x, end = GROUPED && pt ? (part + 1) * per : nvec;
   auto norm = [&](float (&v)[PER][VEC], int kind, const void* w, const void* b, int groups) {
-    if (GROUPED && groups > 1) row_group_norm<T, VEC, PER>(v, (const T*)w, p.W, groups, p.eps, red);
+    if (GROUPED && pt) {
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < PER; i++)
+        if (base + i * step < end)
+#pragma unroll
+          for (int e = 0; e < VEC; e++) ss = fmaf(v[i][e], v[i][e], ss);
+      const float inv = 1.f / sqrtf(part_sum(ss, red[0], pt) / (float)(per * VEC) + p.eps);
+#pragma unroll
+      for (int i = 0; i < PER; i++) {
+        const int c = base + i * step;
+        if (c >= end) continue;
+        float wv[VEC];
+        load_vec<T, VEC>((const T*)w + (long)c * VEC, wv);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) v[i][e] *= inv * wv[e];
+      }
+    } else if (GROUPED && groups > 1) row_group_norm<T, VEC, PER>(v, (const T*)w, p.W, groups, p.eps, red);
     else row_norm<T, VEC, PER>(v, kind, (const T*)w, (const T*)b, p.W, p.eps, red[0]);
   };
   const long t = blockIdx.x;
-  const int nvec = p.W / VEC;
   float v[PER][VEC];
   float* rrow = p.r + t * p.W;
   if (p.post != NORM_NONE) {
     const T* yrow = (const T*)p.y + t * p.y_stride;
 #pragma unroll
     for (int i = 0; i < PER; i++) {
-      const int c = (int)threadIdx.x + i * (int)blockDim.x;
-      if (c < nvec) load_vec<T, VEC>(yrow + (long)c * VEC, v[i]);
+      const int c = base + i * step;
+      if (c < end) load_vec<T, VEC>(yrow + (long)c * VEC, v[i]);
       else
 #pragma unroll
         for (int e = 0; e < VEC; e++) v[i][e] = 0.f;
@@ -180,8 +214,8 @@ __global__ void stream_norm_kernel(const StreamParams p) {
   }
 #pragma unroll
   for (int i = 0; i < PER; i++) {
-    const int c = (int)threadIdx.x + i * (int)blockDim.x;
-    if (c >= nvec) continue;
+    const int c = base + i * step;
+    if (c >= end) continue;
     if (p.emb != EMB_SET) {
       float rv[VEC];
       load_vec<float, VEC>(rrow + (long)c * VEC, rv);
@@ -201,8 +235,8 @@ __global__ void stream_norm_kernel(const StreamParams p) {
   T* xrow = (T*)p.x + t * p.W;
 #pragma unroll
   for (int i = 0; i < PER; i++) {
-    const int c = (int)threadIdx.x + i * (int)blockDim.x;
-    if (c < nvec) store_vec<T, VEC>(xrow + (long)c * VEC, v[i]);
+    const int c = base + i * step;
+    if (c < end) store_vec<T, VEC>(xrow + (long)c * VEC, v[i]);
   }
 }
 
@@ -391,13 +425,22 @@ __global__ void gated_head_norm_kernel(const T* __restrict__ o, const T* __restr
 }
 
 template <typename T, int VEC>
-static int launch_stream(const StreamParams& p, long tokens, cudaStream_t stream) {
+static int launch_stream(StreamParams& p, long tokens, cudaStream_t stream) {
   const int nvec = p.W / VEC;
   int threads = (((nvec + 1) / 2 + 31) / 32) * 32;
   if (threads > 1024) threads = 1024;
-  const int per = (nvec + threads - 1) / threads;
+  int per = (nvec + threads - 1) / threads;
   const dim3 grid((unsigned)tokens);
   const bool grouped = p.post_groups > 1 || p.next_groups > 1;
+  p.part_threads = 0;
+  if (p.next_groups > 1 && (p.post == NORM_NONE || p.post == NORM_PLAIN)) {
+    const int own = nvec / p.next_groups, pt = (((own + 1) / 2 + 31) / 32) * 32;
+    if (pt * p.next_groups <= 1024) {
+      p.part_threads = pt;
+      threads = pt * p.next_groups;
+      per = (own + pt - 1) / pt;
+    }
+  }
 #define LAUNCH_STREAM(PER)                                                                    \
   if (grouped) stream_norm_kernel<T, VEC, PER, true><<<grid, threads, 0, stream>>>(p);        \
   else stream_norm_kernel<T, VEC, PER, false><<<grid, threads, 0, stream>>>(p)
@@ -411,7 +454,7 @@ static int launch_stream(const StreamParams& p, long tokens, cudaStream_t stream
 }
 
 template <typename T>
-static int stream_norm_t(const StreamParams& p, long tokens, cudaStream_t stream) {
+static int stream_norm_t(StreamParams& p, long tokens, cudaStream_t stream) {
   const bool vec = p.W % 4 == 0 && p.y_stride % 4 == 0 && aligned16(p.r) && aligned16(p.y) && aligned16(p.x) &&
                    aligned16(p.table) && aligned16(p.post_w) && aligned16(p.post_b) && aligned16(p.next_w) &&
                    aligned16(p.next_b) && p.W / p.post_groups % 4 == 0 && p.W / p.next_groups % 4 == 0;
@@ -493,7 +536,7 @@ B200_API int b200_stream_norm(void* r, const void* y, long y_stride, int post, c
   if ((post == NORM_LAYER || post == NORM_RMS) && !post_w) return 9701;
   if ((next == NORM_LAYER || next == NORM_RMS) && !next_w) return 9702;
   StreamParams p{(float*)r, y, y_stride, post, post_w, post_b, post_scale, emb, (const long*)ids, table, table_rows,
-                 emb_scale, next, next_w, next_b, x, W, post_groups, next_groups, eps, status};
+                 emb_scale, next, next_w, next_b, x, W, post_groups, next_groups, 0, eps, status};
   return dtype ? stream_norm_t<float>(p, tokens, stream) : stream_norm_t<__nv_bfloat16>(p, tokens, stream);
 }
 
