@@ -80,7 +80,8 @@ def _run(preset, world, tp, ep=False, pp=1, dcp=1, pcp=1, fg=None, addcfg=None, 
     return json.loads(line[7:])
 
 
-@pytest.mark.parametrize("preset", ["tiny-qwen", "tiny-moe", "tiny-deepseek", "tiny-mqa", "tiny-vofelix", "tiny-pegopel", "tiny-dubizen"])
+@pytest.mark.parametrize("preset", ["tiny-qwen", "tiny-moe", "tiny-deepseek", "tiny-mqa", "tiny-vofelix", "tiny-pegopel", "tiny-dubizen",
+                                    "tiny-nevotar"])
 def test_tp2_matches_tp1(preset):
     assert _run(preset, 2, 2) == _run(preset, 1, 1)
 
@@ -119,7 +120,7 @@ def test_logprobs_reach_every_rank_under_pipeline_and_prefill_context_parallelis
             assert max(abs(x[1] - y[1]) for x, y in zip(da, db)) < 1e-3
 
 
-@pytest.mark.parametrize("preset", ["tiny-moe", "tiny-dubizen"])
+@pytest.mark.parametrize("preset", ["tiny-moe", "tiny-dubizen", "tiny-nevotar"])
 def test_expert_parallel_matches_single_rank(preset):
     # EP over 2 ranks (DP attention: tp=1, experts sharded over the 2 ranks)
     assert _run(preset, 2, 1, ep=True) == _run(preset, 1, 1)

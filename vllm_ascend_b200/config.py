@@ -562,7 +562,7 @@ PRESETS: dict[str, Any] = {
             {"type": "parallel", "mlp": _TINY_CLAMPED, "mixer": {
                 "left": {"heads": 4, "kv_heads": 2, "dim": 24, "vdim": 16, "scale": 0.2, "mask": {"size": 30},
                          "rot": {"base": 10000.0, "dims": 16}},
-                "right": {"heads": 6, "vdim": 16, "state": 24, "groups": 3, "conv": 4, "norm_groups": 2},
+                "right": {"heads": 6, "vdim": 16, "state": 24, "groups": 2, "conv": 4, "norm_groups": 3},
                 "left_scale": 0.7, "right_scale": 0.4}},
             {"type": "attention", "mlp": None, "mixer": {
                 "heads": 4, "kv_heads": 2, "dim": 16, "vdim": 24, "scale": 0.25, "diff": 0.4,

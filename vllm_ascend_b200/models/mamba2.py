@@ -61,7 +61,8 @@ class Mamba2Mixer:
                                             bias=bool(m.get("proj_bias", False)))
         self.out_proj = RowParallelLinear(pf, f"{p}.out_proj", self.I_total, cfg.hidden_size, comm,
                                           bias=bool(m.get("proj_bias", False)))
-        self.conv_weight = pf.normal(f"{p}.conv1d.w", (self.conv_dim, self.K), std=0.3).contiguous()
+        conv = pf.normal(f"{p}.conv1d.w", (self.I_total + 2 * self.G_total * self.N, self.K), std=0.3)
+        self.conv_weight = torch.cat([conv[a - self.I_total:a - self.I_total + n] for a, n in self._rows(tp, r)[1:4]])
         self.conv_bias = pf.zeros((self.conv_dim,)) if m.get("conv_bias", True) else None
         self.dt_bias = pf.normal(f"{p}.dt_bias", (self.H_total,), 0, r, tp, std=0.5, dtype=torch.float32)
         self.A_log = pf.normal(f"{p}.A_log", (self.H_total,), 0, r, tp, std=0.5, dtype=torch.float32)
