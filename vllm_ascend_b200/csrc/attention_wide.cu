@@ -4,7 +4,8 @@
 //
 // attn_wide_kernel: tiles of 128 query rows (token, head of one value head) x 128 keys, any number of rows per sequence.
 //   The queries' chunks of 64 dimensions stay in shared memory, the keys' chunks stream through a ring and accumulate
-//   S in TMEM (double-buffered); values, probabilities and output as in attention_tc.cu.
+//   S in TMEM (double-buffered); the probabilities go back to TMEM as the A operand of P V, which leaves the shared
+//   memory to the rings.
 // attn_wide_decode_kernel: one query row per sequence.  A work item is (sequence, key head, KV split): all heads of the
 //   key head are the columns of S^T = K Q^T, so every key and value is read once; the output has one accumulator per
 //   value head.  Persistent, the K / V rings run across items.
@@ -32,7 +33,7 @@ struct WideParams {
   int max_blocks, block_size, rows_per_load;
   int G, Hkv, Hq, key_heads, Dv, tok_per_tile;
   int num_seqs, window, num_splits, num_items;
-  int chunks, k_stages, v_stages, p_bufs;      // chunks of 64 key dimensions; ring sizes
+  int chunks, k_stages, v_stages;              // chunks of 64 key dimensions; ring sizes
   float scale_log2, out_scale;
   int out_f32;
   void* out;
@@ -77,7 +78,8 @@ template <int NV>            // value size in units of 64
 __global__ void __launch_bounds__(WIDE_THREADS, 1)
 attn_wide_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                  const __grid_constant__ CUtensorMap tmap_v, const WideParams p) {
-  constexpr int V_BYTES = NV * WIDE_CHUNK, P_BYTES = 2 * WIDE_CHUNK, O_COL = 256;
+  // TMEM columns: two S of 128, O, two P of 64 (two bf16 keys per column)
+  constexpr int V_BYTES = NV * WIDE_CHUNK, O_COL = 256, P_COL = 384;
   // ---------------- work decode (uniform over the CTA): sequence b owns the tiles from (cu[b] - cu[0]) / tok + b on
   const int h = blockIdx.x, wi = gridDim.y - 1 - blockIdx.y, base = p.cu[0];
   int seq, lo_ = 0, hi_ = p.num_seqs - 1;
@@ -95,14 +97,13 @@ attn_wide_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
   const int t0 = kv_lo >> 7, n = ((kv_end + 127) >> 7) - t0;
   if (n <= 0) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int NC = p.chunks, KST = p.k_stages, VST = p.v_stages, PB = p.p_bufs;
+  const int NC = p.chunks, KST = p.k_stages, VST = p.v_stages;
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* Qs = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   uint8_t* Ks = Qs + NC * WIDE_CHUNK;
   uint8_t* Vs = Ks + KST * WIDE_CHUNK;
-  uint8_t* Ps = Vs + VST * V_BYTES;
-  uint64_t* q_full = (uint64_t*)(Ps + PB * P_BYTES);
+  uint64_t* q_full = (uint64_t*)(Vs + VST * V_BYTES);
   uint64_t* k_full = q_full + 1;             // WIDE_RING each
   uint64_t* k_empty = k_full + WIDE_RING;
   uint64_t* v_full = k_empty + WIDE_RING;    // 2 each
@@ -143,8 +144,6 @@ attn_wide_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_ptr;
-  auto pbuf = [&](int j) { return PB == 2 ? j & 1 : 0; };
-  auto pphase = [&](int j) { return (uint32_t)(PB == 2 ? j >> 1 : j) & 1u; };
 
   if (warp == 0) {
     // ------------------------------------------------------------ producer, in the order of consumption
@@ -192,7 +191,7 @@ attn_wide_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     // ------------------------------------------------------------ MMA issuer
     constexpr uint32_t idesc_s = make_idesc_f16(128, 128, true, false, false);
     constexpr uint32_t idesc_o = make_idesc_f16(128, NV * 64, true, false, true);
-    const uint32_t q_addr = smem_u32(Qs), k_addr = smem_u32(Ks), v_addr = smem_u32(Vs), p_addr = smem_u32(Ps);
+    const uint32_t q_addr = smem_u32(Qs), k_addr = smem_u32(Ks), v_addr = smem_u32(Vs);
     if (!mbar_wait(q_full, 0, abort_word)) goto done;
     auto issue_s = [&](int j) -> bool {
       const int b = j & 1;
@@ -218,17 +217,15 @@ attn_wide_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     if (!issue_s(0)) goto done;
     for (int j = 0; j < n; j++) {
       if (j + 1 < n && !issue_s(j + 1)) goto done;
-      const int st = j % VST, pb = pbuf(j);
+      const int st = j % VST, pb = j & 1;
       if (!mbar_wait(&v_full[st], (uint32_t)(j / VST) & 1u, abort_word)) goto done;
-      if (!mbar_wait(&p_ready[pb], pphase(j), abort_word)) goto done;
+      if (!mbar_wait(&p_ready[pb], ((uint32_t)j >> 1) & 1u, abort_word)) goto done;
       tc_fence_after();
       if (lane == 0) {
 #pragma unroll
         for (int kk = 0; kk < 8; kk++) {
-          const uint64_t da = make_smem_desc(p_addr + pb * P_BYTES + (kk >> 2) * WIDE_CHUNK + (kk & 3) * 32, 16, 1024,
-                                             kLayoutSw128);
           const uint64_t db = make_smem_desc(v_addr + st * V_BYTES + kk * 2048, WIDE_CHUNK, 1024, kLayoutSw128);
-          umma_f16_ss(tmem_base + O_COL, da, db, idesc_o, j > 0 || kk > 0 ? 1u : 0u);
+          umma_f16_ts(tmem_base + O_COL, tmem_base + P_COL + pb * 64 + kk * 8, db, idesc_o, j > 0 || kk > 0 ? 1u : 0u);
         }
         umma_commit(&v_empty[st]);
         umma_commit(&pv_done[pb]);
@@ -246,7 +243,6 @@ attn_wide_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     // a negative scale turns the order of the products around
     const float sign = sl2 < 0.f ? -1.f : 1.f, asl2 = fabsf(sl2);
     float m = -INFINITY, l = 0.f;
-    uint8_t* prow = Ps + row * 128;
     for (int j = 0; j < n; j++) {
       const int b = j & 1;
       if (!mbar_wait(&s_ready[b], ((uint32_t)j >> 1) & 1u, abort_word)) goto done;
@@ -290,10 +286,10 @@ attn_wide_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
       }
       l *= alpha;
       const bool warp_need = __any_sync(0xffffffffu, need && row_valid);
-      // the P buffer was last read by PV(j - PB); O must be quiescent only for a rescale
-      if (j >= PB && !mbar_wait(&pv_done[pbuf(j)], pphase(j - PB), abort_word)) goto done;
+      // the P buffer was last read by PV(j - 2); O must be quiescent only for a rescale
+      if (j >= 2 && !mbar_wait(&pv_done[j & 1], (((uint32_t)j - 2) >> 1) & 1u, abort_word)) goto done;
       if (warp_need) {
-        if (!mbar_wait(&pv_done[pbuf(j - 1)], pphase(j - 1), abort_word)) goto done;
+        if (!mbar_wait(&pv_done[(j - 1) & 1], (((uint32_t)j - 1) >> 1) & 1u, abort_word)) goto done;
         tc_fence_after();
         const float a = need ? alpha : 1.f;
 #pragma unroll 1
@@ -307,32 +303,30 @@ attn_wide_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
         }
         tmem_st_wait();
       }
-      // ---- probabilities -> swizzled shared memory (A operand of P V)
+      // ---- probabilities, two keys to a column -> TMEM (A operand of P V)
+      tc_fence_after();
       const float nmb = m == -INFINITY ? 0.f : -m * asl2;
       float rs0 = 0.f, rs1 = 0.f;
-      uint8_t* pb = prow + pbuf(j) * P_BYTES;
 #pragma unroll
-      for (int c8 = 0; c8 < 16; c8++) {            // 16 chunks of 8 keys = one 16-byte store
-        uint32_t pk[4];
+      for (int hf = 0; hf < 2; hf++) {
+        uint32_t pk[32];
 #pragma unroll
-        for (int q2 = 0; q2 < 4; q2++) {
-          const int i = c8 * 8 + q2 * 2;
-          const float p0 = score_exp2(fmaf(__uint_as_float(sreg[i]), asl2, nmb));
-          const float p1 = score_exp2(fmaf(__uint_as_float(sreg[i + 1]), asl2, nmb));
+        for (int i = 0; i < 32; i++) {
+          const float p0 = score_exp2(fmaf(__uint_as_float(sreg[hf * 64 + 2 * i]), asl2, nmb));
+          const float p1 = score_exp2(fmaf(__uint_as_float(sreg[hf * 64 + 2 * i + 1]), asl2, nmb));
           rs0 += p0;
           rs1 += p1;
-          pk[q2] = pack_bf16x2(p0, p1);
+          pk[i] = pack_bf16x2(p0, p1);
         }
-        *reinterpret_cast<uint4*>(pb + (c8 >> 3) * WIDE_CHUNK + (((c8 & 7) ^ (row & 7)) << 4)) =
-            make_uint4(pk[0], pk[1], pk[2], pk[3]);
+        tmem_st_32x32b_x32(t_lane + P_COL + b * 64 + hf * 32, pk);
       }
       l += rs0 + rs1;
+      tmem_st_wait();
       tc_fence_before();
-      fence_proxy_async_smem();
       __syncwarp();
-      if (lane == 0) mbar_arrive(&p_ready[pbuf(j)]);
+      if (lane == 0) mbar_arrive(&p_ready[b]);
     }
-    if (!mbar_wait(&pv_done[pbuf(n - 1)], pphase(n - 1), abort_word)) goto done;
+    if (!mbar_wait(&pv_done[(n - 1) & 1], (((uint32_t)n - 1) >> 1) & 1u, abort_word)) goto done;
     tc_fence_after();
     const long at = ((long)q_start + tok0 + tok) * p.out_stride + (long)(h * G + g) * p.Dv;
     const float inv = l > 0.f ? p.out_scale / l : 0.f;
@@ -780,7 +774,7 @@ static int launch_wide(const CUtensorMap& tq, const CUtensorMap& tk, const CUten
   static bool set = false;
   const int rc = allow_smem(attn_wide_kernel<NV>, &set);
   if (rc) return rc;
-  const int bytes = (p.chunks + p.k_stages + NV * p.v_stages + 2 * p.p_bufs) * WIDE_CHUNK + 1024 + 512;
+  const int bytes = (p.chunks + p.k_stages + NV * p.v_stages) * WIDE_CHUNK + 1024 + 512;
   if (bytes > WIDE_SMEM) return 9886;
   attn_wide_kernel<NV><<<dim3((unsigned)p.Hkv, (unsigned)tiles), WIDE_THREADS, bytes, stream>>>(tq, tk, tv, p);
   return B200_CHECK_LAUNCH();
@@ -815,9 +809,8 @@ B200_API int b200_attention_wide_prefill(const b200::AttnVariantArgs* a, int* st
   if (p.G > 128 || p.chunks > 8) return 9885;
   p.tok_per_tile = 128 / p.G;
   const int NV = a->Dv > 64 ? 2 : 1, left = 14 - p.chunks;      // chunks of shared memory beside the queries
-  p.p_bufs = left - 4 >= 2 + NV ? 2 : 1;
-  p.v_stages = left - 2 * p.p_bufs >= 2 * NV + (p.p_bufs == 2 ? 4 : 2) ? 2 : 1;
-  p.k_stages = left - 2 * p.p_bufs - NV * p.v_stages;
+  p.v_stages = left >= 2 * NV + 6 ? 2 : 1;
+  p.k_stages = left - NV * p.v_stages;
   CUtensorMap tq, tk, tv;
   {
     uint64_t dims[4] = {(uint64_t)a->D, (uint64_t)p.G, (uint64_t)p.Hkv, (uint64_t)a->tokens};
