@@ -64,13 +64,29 @@ __device__ __forceinline__ void wide_finish(volatile int* abort_word, int* statu
   }
 }
 
-// one 64-dimension chunk of 128 keys from the pages of a sequence (lane i holds the block of part i); whole warp
-__device__ __forceinline__ void load_chunk(uint8_t* dst, const CUtensorMap* tm, uint64_t* bar, int x, int head, int key_base,
-                                           int blk_lane, const WideParams& p, int lane) {
-  const int rpl = p.rows_per_load, parts = 128 / rpl;
+// Place in a ring of stages and the parity of its round.  Counted instead of divided: the producer and the MMA issuer
+// are single warps whose instructions wait for one another.
+struct Ring {
+  int st = 0;
+  uint32_t ph = 0;
+  __device__ __forceinline__ void next(int stages) {
+    if (++st == stages) {
+      st = 0;
+      ph ^= 1u;
+    }
+  }
+};
+
+// A matrix descriptor moves by adding bytes / 16; built once, since the issuer would wait for every step of building one
+__device__ __forceinline__ uint64_t desc_at(uint64_t base, int bytes) { return base + (uint64_t)(uint32_t)(bytes >> 4); }
+
+// one 64-dimension chunk of 128 keys from the pages of a sequence (lane i holds the block of part i), ``off`` rows into
+// a page that is longer than 128; whole warp
+__device__ __forceinline__ void load_chunk(uint8_t* dst, const CUtensorMap* tm, uint64_t* bar, int x, int head, int off,
+                                           int blk_lane, int parts, int rpl, int lane) {
   for (int part = 0; part < parts; part++) {
     const int blk = __shfl_sync(0xffffffffu, blk_lane, part);
-    if (lane == 0) tma_load_4d(dst + part * rpl * 128, tm, bar, x, head, (key_base + part * rpl) % p.block_size, blk);
+    if (lane == 0) tma_load_4d(dst + part * rpl * 128, tm, bar, x, off, head, blk);
   }
 }
 
@@ -148,7 +164,8 @@ attn_wide_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
   if (warp == 0) {
     // ------------------------------------------------------------ producer, in the order of consumption
     const int* bt = p.block_table + (long)seq * p.max_blocks;
-    const int parts = 128 / p.rows_per_load, hk = h * p.key_heads / p.Hkv;
+    const int rpl = p.rows_per_load, parts = 128 / rpl, hk = h * p.key_heads / p.Hkv;
+    Ring kr, vr;
     if (lane == 0) {
       mbar_expect_tx(q_full, NC * 128 * G * p.tok_per_tile);
       for (int c = 0; c < NC; c++) tma_load_4d(Qs + c * WIDE_CHUNK, &tmap_q, q_full, c * 64, 0, h, q_start + tok0);
@@ -156,19 +173,20 @@ attn_wide_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     __syncwarp();
     auto block_of = [&](int j) -> int {
       if (j >= n || lane >= parts) return 0;
-      return bt[min(((t0 + j) << 7) + lane * p.rows_per_load, seq_len - 1) / p.block_size];
+      return bt[min(((t0 + j) << 7) + lane * rpl, seq_len - 1) / p.block_size];
     };
+    auto page_row = [&](int j) { return p.block_size > 128 ? ((t0 + j) << 7) % p.block_size : 0; };
     auto load_k = [&](int j, int blk) -> bool {
       if (__any_sync(0xffffffffu, (blk < 0 || blk >= p.num_blocks_total) && lane < parts)) {
         *abort_word = B200_BAD_INDEX;
         return false;
       }
-      for (int c = 0; c < NC; c++) {
-        const int g = j * NC + c, st = g % KST;
-        if (!mbar_wait(&k_empty[st], ((uint32_t)(g / KST) & 1u) ^ 1u, abort_word)) return false;
-        if (lane == 0) mbar_expect_tx(&k_full[st], WIDE_CHUNK);
+      const int off = page_row(j);
+      for (int c = 0; c < NC; c++, kr.next(KST)) {
+        if (!mbar_wait(&k_empty[kr.st], kr.ph ^ 1u, abort_word)) return false;
+        if (lane == 0) mbar_expect_tx(&k_full[kr.st], WIDE_CHUNK);
         __syncwarp();
-        load_chunk(Ks + st * WIDE_CHUNK, &tmap_k, &k_full[st], c * 64, hk, (t0 + j) << 7, blk, p, lane);
+        load_chunk(Ks + kr.st * WIDE_CHUNK, &tmap_k, &k_full[kr.st], c * 64, hk, off, blk, parts, rpl, lane);
       }
       return true;
     };
@@ -177,13 +195,14 @@ attn_wide_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     for (int j = 0; j < n; j++) {
       const int blk_after = block_of(j + 2);
       if (j + 1 < n && !load_k(j + 1, blk_next)) goto done;
-      const int st = j % VST;
-      if (!mbar_wait(&v_empty[st], ((uint32_t)(j / VST) & 1u) ^ 1u, abort_word)) goto done;
-      if (lane == 0) mbar_expect_tx(&v_full[st], V_BYTES);
+      if (!mbar_wait(&v_empty[vr.st], vr.ph ^ 1u, abort_word)) goto done;
+      if (lane == 0) mbar_expect_tx(&v_full[vr.st], V_BYTES);
       __syncwarp();
+      const int off = page_row(j);
 #pragma unroll
       for (int hf = 0; hf < NV; hf++)
-        load_chunk(Vs + st * V_BYTES + hf * WIDE_CHUNK, &tmap_v, &v_full[st], hf * 64, h, (t0 + j) << 7, blk, p, lane);
+        load_chunk(Vs + vr.st * V_BYTES + hf * WIDE_CHUNK, &tmap_v, &v_full[vr.st], hf * 64, h, off, blk, parts, rpl, lane);
+      vr.next(VST);
       blk = blk_next;
       blk_next = blk_after;
     }
@@ -191,22 +210,23 @@ attn_wide_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     // ------------------------------------------------------------ MMA issuer
     constexpr uint32_t idesc_s = make_idesc_f16(128, 128, true, false, false);
     constexpr uint32_t idesc_o = make_idesc_f16(128, NV * 64, true, false, true);
-    const uint32_t q_addr = smem_u32(Qs), k_addr = smem_u32(Ks), v_addr = smem_u32(Vs);
+    const uint64_t q_desc = make_smem_desc(smem_u32(Qs), 16, 1024, kLayoutSw128);
+    const uint64_t k_desc = make_smem_desc(smem_u32(Ks), 16, 1024, kLayoutSw128);
+    const uint64_t v_desc = make_smem_desc(smem_u32(Vs), WIDE_CHUNK, 1024, kLayoutSw128);
     if (!mbar_wait(q_full, 0, abort_word)) goto done;
+    Ring kr, vr;
     auto issue_s = [&](int j) -> bool {
       const int b = j & 1;
       if (!mbar_wait(&s_free[b], (((uint32_t)j >> 1) & 1u) ^ 1u, abort_word)) return false;
-      for (int c = 0; c < NC; c++) {
-        const int g = j * NC + c, st = g % KST;
-        if (!mbar_wait(&k_full[st], (uint32_t)(g / KST) & 1u, abort_word)) return false;
+      for (int c = 0; c < NC; c++, kr.next(KST)) {
+        const int st = kr.st;
+        if (!mbar_wait(&k_full[st], kr.ph, abort_word)) return false;
         tc_fence_after();
         if (lane == 0) {
+          const uint64_t da = desc_at(q_desc, c * WIDE_CHUNK), db = desc_at(k_desc, st * WIDE_CHUNK);
 #pragma unroll
-          for (int kk = 0; kk < 4; kk++) {
-            const uint64_t da = make_smem_desc(q_addr + c * WIDE_CHUNK + kk * 32, 16, 1024, kLayoutSw128);
-            const uint64_t db = make_smem_desc(k_addr + st * WIDE_CHUNK + kk * 32, 16, 1024, kLayoutSw128);
-            umma_f16_ss(tmem_base + b * 128, da, db, idesc_s, c > 0 || kk > 0 ? 1u : 0u);
-          }
+          for (int kk = 0; kk < 4; kk++)
+            umma_f16_ss(tmem_base + b * 128, da + 2 * kk, db + 2 * kk, idesc_s, c > 0 || kk > 0 ? 1u : 0u);
           umma_commit(&k_empty[st]);
           if (c == NC - 1) umma_commit(&s_ready[b]);
         }
@@ -217,16 +237,17 @@ attn_wide_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     if (!issue_s(0)) goto done;
     for (int j = 0; j < n; j++) {
       if (j + 1 < n && !issue_s(j + 1)) goto done;
-      const int st = j % VST, pb = j & 1;
-      if (!mbar_wait(&v_full[st], (uint32_t)(j / VST) & 1u, abort_word)) goto done;
+      const int st = vr.st, pb = j & 1;
+      if (!mbar_wait(&v_full[st], vr.ph, abort_word)) goto done;
+      vr.next(VST);
       if (!mbar_wait(&p_ready[pb], ((uint32_t)j >> 1) & 1u, abort_word)) goto done;
       tc_fence_after();
       if (lane == 0) {
+        const uint64_t db = desc_at(v_desc, st * V_BYTES);
 #pragma unroll
-        for (int kk = 0; kk < 8; kk++) {
-          const uint64_t db = make_smem_desc(v_addr + st * V_BYTES + kk * 2048, WIDE_CHUNK, 1024, kLayoutSw128);
-          umma_f16_ts(tmem_base + O_COL, tmem_base + P_COL + pb * 64 + kk * 8, db, idesc_o, j > 0 || kk > 0 ? 1u : 0u);
-        }
+        for (int kk = 0; kk < 8; kk++)
+          umma_f16_ts(tmem_base + O_COL, tmem_base + P_COL + pb * 64 + kk * 8, db + 128 * kk, idesc_o,
+                      j > 0 || kk > 0 ? 1u : 0u);
         umma_commit(&v_empty[st]);
         umma_commit(&pv_done[pb]);
       }
@@ -449,30 +470,32 @@ attn_wide_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_ptr;
-  uint32_t it = 0, gt = 0, gk = 0, gv = 0;      // non-empty items, tiles, key chunks, value tiles of this CTA so far
+  uint32_t it = 0, gt = 0;                      // non-empty items and tiles of this CTA so far
+  Ring kr, vr;
 
   if (warp == 0) {
     // ------------------------------------------------------------ producer, in the order of consumption
-    const int parts = 128 / p.rows_per_load;
+    const int rpl = p.rows_per_load, parts = 128 / rpl;
     for (int item = blockIdx.x; item < p.num_items; item += gridDim.x) {
       const WideItem w = wide_item(p, item);
       if (w.n <= 0) continue;
       const int* bt = p.block_table + (long)w.seq * p.max_blocks;
       auto block_of = [&](int j) -> int {
         if (j >= w.n || lane >= parts) return 0;
-        return bt[min(((w.t0 + j) << 7) + lane * p.rows_per_load, w.seq_len - 1) / p.block_size];
+        return bt[min(((w.t0 + j) << 7) + lane * rpl, w.seq_len - 1) / p.block_size];
       };
+      auto page_row = [&](int j) { return p.block_size > 128 ? ((w.t0 + j) << 7) % p.block_size : 0; };
       auto load_k = [&](int j, int blk) -> bool {
         if (__any_sync(0xffffffffu, (blk < 0 || blk >= p.num_blocks_total) && lane < parts)) {
           *abort_word = B200_BAD_INDEX;
           return false;
         }
-        for (int c = 0; c < NC; c++, gk++) {
-          const int st = gk % KST;
-          if (!mbar_wait(&k_empty[st], ((gk / KST) & 1u) ^ 1u, abort_word)) return false;
-          if (lane == 0) mbar_expect_tx(&k_full[st], WIDE_CHUNK);
+        const int off = page_row(j);
+        for (int c = 0; c < NC; c++, kr.next(KST)) {
+          if (!mbar_wait(&k_empty[kr.st], kr.ph ^ 1u, abort_word)) return false;
+          if (lane == 0) mbar_expect_tx(&k_full[kr.st], WIDE_CHUNK);
           __syncwarp();
-          load_chunk(Ks + st * WIDE_CHUNK, &tmap_k, &k_full[st], c * 64, w.kh, (w.t0 + j) << 7, blk, p, lane);
+          load_chunk(Ks + kr.st * WIDE_CHUNK, &tmap_k, &k_full[kr.st], c * 64, w.kh, off, blk, parts, rpl, lane);
         }
         return true;
       };
@@ -487,14 +510,14 @@ attn_wide_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
       for (int j = 0; j < w.n; j++) {
         const int blk_after = block_of(j + 2);
         if (j + 1 < w.n && !load_k(j + 1, blk_next)) goto done;
-        for (int v = 0; v < VH; v++, gv++) {
-          const int st = gv % VST;
-          if (!mbar_wait(&v_empty[st], ((gv / VST) & 1u) ^ 1u, abort_word)) goto done;
-          if (lane == 0) mbar_expect_tx(&v_full[st], V_BYTES);
+        const int off = page_row(j);
+        for (int v = 0; v < VH; v++, vr.next(VST)) {
+          if (!mbar_wait(&v_empty[vr.st], vr.ph ^ 1u, abort_word)) goto done;
+          if (lane == 0) mbar_expect_tx(&v_full[vr.st], V_BYTES);
           __syncwarp();
           for (int hf = 0; hf < 2; hf++)
-            load_chunk(Vs + st * V_BYTES + hf * WIDE_CHUNK, &tmap_v, &v_full[st], hf * 64, w.kh * VH + v, (w.t0 + j) << 7,
-                       blk, p, lane);
+            load_chunk(Vs + vr.st * V_BYTES + hf * WIDE_CHUNK, &tmap_v, &v_full[vr.st], hf * 64, w.kh * VH + v, off, blk, parts,
+                       rpl, lane);
         }
         blk = blk_next;
         blk_next = blk_after;
@@ -505,7 +528,10 @@ attn_wide_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
     // ------------------------------------------------------------ MMA issuer
     constexpr uint32_t idesc_s = make_idesc_f16(128, NQ, true, false, false);
     constexpr uint32_t idesc_o = make_idesc_f16(128, NQ, true, true, false);      // A = V, MN-major
-    const uint32_t q_addr = smem_u32(Qs), k_addr = smem_u32(Ks), v_addr = smem_u32(Vs), p_addr = smem_u32(Ps);
+    const uint64_t q_desc = make_smem_desc(smem_u32(Qs), 16, 1024, kLayoutSw128);
+    const uint64_t k_desc = make_smem_desc(smem_u32(Ks), 16, 1024, kLayoutSw128);
+    const uint64_t v_desc = make_smem_desc(smem_u32(Vs), WIDE_CHUNK, 1024, kLayoutSw128);
+    const uint64_t p_desc = make_smem_desc(smem_u32(Ps), 16, 1024, kLayoutSw128);
     for (int item = blockIdx.x; item < p.num_items; item += gridDim.x) {
       const WideItem w = wide_item(p, item);
       if (w.n <= 0) continue;
@@ -515,17 +541,15 @@ attn_wide_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
         const uint32_t g = gt + (uint32_t)j;
         const int b = g & 1;
         if (!mbar_wait(&s_free[b], ((g >> 1) & 1u) ^ 1u, abort_word)) return false;
-        for (int c = 0; c < NC; c++, gk++) {
-          const int st = gk % KST;
-          if (!mbar_wait(&k_full[st], (gk / KST) & 1u, abort_word)) return false;
+        for (int c = 0; c < NC; c++, kr.next(KST)) {
+          const int st = kr.st;
+          if (!mbar_wait(&k_full[st], kr.ph, abort_word)) return false;
           tc_fence_after();
           if (lane == 0) {
+            const uint64_t da = desc_at(k_desc, st * WIDE_CHUNK), db = desc_at(q_desc, c * QC);
 #pragma unroll
-            for (int kk = 0; kk < 4; kk++) {
-              const uint64_t da = make_smem_desc(k_addr + st * WIDE_CHUNK + kk * 32, 16, 1024, kLayoutSw128);
-              const uint64_t db = make_smem_desc(q_addr + c * QC + kk * 32, 16, 1024, kLayoutSw128);
-              umma_f16_ss(tmem_base + b * NQ, da, db, idesc_s, c > 0 || kk > 0 ? 1u : 0u);
-            }
+            for (int kk = 0; kk < 4; kk++)
+              umma_f16_ss(tmem_base + b * NQ, da + 2 * kk, db + 2 * kk, idesc_s, c > 0 || kk > 0 ? 1u : 0u);
             umma_commit(&k_empty[st]);
             if (c == NC - 1) {
               umma_commit(&s_ready[b]);
@@ -542,19 +566,17 @@ attn_wide_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
         const uint32_t g = gt + (uint32_t)j;
         const int pb = g & 1;
         if (!mbar_wait(&p_ready[pb], (g >> 1) & 1u, abort_word)) goto done;
-        for (int v = 0; v < VH; v++, gv++) {
-          const int st = gv % VST;
-          if (!mbar_wait(&v_full[st], (gv / VST) & 1u, abort_word)) goto done;
+        for (int v = 0; v < VH; v++, vr.next(VST)) {
+          const int st = vr.st;
+          if (!mbar_wait(&v_full[st], vr.ph, abort_word)) goto done;
           tc_fence_after();
           if (lane == 0) {
+            // A: 16 keys of V^T (two 64-wide d atoms a chunk apart, 8-key groups 1024 B apart)
+            const uint64_t da = desc_at(v_desc, st * V_BYTES), db = desc_at(p_desc, pb * P_BYTES);
 #pragma unroll
-            for (int kk = 0; kk < 8; kk++) {
-              // A: 16 keys of V^T (two 64-wide d atoms a chunk apart, 8-key groups 1024 B apart)
-              const uint64_t da = make_smem_desc(v_addr + st * V_BYTES + kk * 2048, WIDE_CHUNK, 1024, kLayoutSw128);
-              const uint64_t db = make_smem_desc(p_addr + pb * P_BYTES + (kk >> 2) * QC + (kk & 3) * 32, 16, 1024,
-                                                 kLayoutSw128);
-              umma_f16_ss(tmem_base + O_COL + v * NQ, da, db, idesc_o, j > 0 || kk > 0 ? 1u : 0u);
-            }
+            for (int kk = 0; kk < 8; kk++)
+              umma_f16_ss(tmem_base + O_COL + v * NQ, da + 128 * kk, db + (kk >> 2) * (QC >> 4) + 2 * (kk & 3), idesc_o,
+                          j > 0 || kk > 0 ? 1u : 0u);
             umma_commit(&v_empty[st]);
             if (v == VH - 1) umma_commit(&pv_done[pb]);
           }
@@ -730,12 +752,13 @@ static int wide_map(CUtensorMap* out, const void* base, const uint64_t* dims, co
   return 0;
 }
 
+// the rows of a box are consecutive in the map's second dimension
 static int cache_map(CUtensorMap* out, const AttnVariantArgs* a, bool values, int rows) {
-  uint64_t dims[4] = {(uint64_t)(values ? a->Dv : a->D), (uint64_t)(values ? a->Hkv : a->key_heads), (uint64_t)a->block_size,
+  uint64_t dims[4] = {(uint64_t)(values ? a->Dv : a->D), (uint64_t)a->block_size, (uint64_t)(values ? a->Hkv : a->key_heads),
                       (uint64_t)a->num_blocks};
-  uint64_t str[3] = {(uint64_t)(values ? a->v_head : a->k_head) * 2, (uint64_t)(values ? a->v_tok : a->k_tok) * 2,
+  uint64_t str[3] = {(uint64_t)(values ? a->v_tok : a->k_tok) * 2, (uint64_t)(values ? a->v_head : a->k_head) * 2,
                      (uint64_t)(values ? a->v_block : a->k_block) * 2};
-  uint32_t box[4] = {64, 1, (uint32_t)rows, 1};
+  uint32_t box[4] = {64, (uint32_t)rows, 1, 1};
   return wide_map(out, values ? a->v_cache : a->k_cache, dims, str, box);
 }
 
