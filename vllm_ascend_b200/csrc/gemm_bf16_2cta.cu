@@ -337,15 +337,18 @@ gemm_bf16_2cta_kernel(const __grid_constant__ CUtensorMap tmap_a,
           uint32_t u[32];
           tmem_ld_32x32b_x32(t_row + 128 + c0, u);
           tmem_ld_wait();
+          if (p.glu_alpha > 0.f) {
 #pragma unroll
-          for (int j = 0; j < 32; j++) {
-            float g = __uint_as_float(r[j]) * rstd, up = __uint_as_float(u[j]) * rstd;
-            if (p.glu_alpha > 0.f) {
-              g = fminf(g, p.glu_limit);
-              up = fminf(fmaxf(up, -p.glu_limit), p.glu_limit) + 1.f;
+            for (int j = 0; j < 32; j++) {
+              const float g = fminf(__uint_as_float(r[j]) * rstd, p.glu_limit);
+              const float up = fminf(fmaxf(__uint_as_float(u[j]) * rstd, -p.glu_limit), p.glu_limit) + 1.f;
               r[j] = __float_as_uint(g / (1.f + __expf(-p.glu_alpha * g)) * up);
-            } else {
-              r[j] = __float_as_uint(g / (1.f + __expf(-g)) * up);
+            }
+          } else {
+#pragma unroll
+            for (int j = 0; j < 32; j++) {
+              const float g = __uint_as_float(r[j]) * rstd;
+              r[j] = __float_as_uint(g / (1.f + __expf(-g)) * (__uint_as_float(u[j]) * rstd));
             }
           }
         } else {
